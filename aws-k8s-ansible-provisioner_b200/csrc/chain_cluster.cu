@@ -81,7 +81,7 @@ __device__ __forceinline__ void fc_cluster_sync() {
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
-// The release/acquire forms cost every thread a GPU-scope memory barrier (MEMBAR.ALL.GPU + ERRBAR in SASS).
+// The release/acquire forms make every thread that takes part order its memory accesses with the cluster's.
 // Only the warps that wrote remote shared memory need the release and only the warps that will read the
 // reduce buffer need the acquire; everyone else just takes part in the count.
 __device__ __forceinline__ void fc_cluster_sync_roles(bool releases, bool acquires) {
