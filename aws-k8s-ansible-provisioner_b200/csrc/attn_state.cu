@@ -1,11 +1,13 @@
 // attn_state.cu -- mixers whose memory is a matrix state per head instead of a cache of keys and values: a head keeps
 // S [dim][vdim] in fp32, every token updates it and reads it out, and the state of a sequence lives in a slot of the
-// engine's sequence table.  Two update rules share the kernels (StateGeom.rule):
+// engine's sequence table.  The update rules share the kernels (StateGeom.rule):
 //
 //   STATE_RULE_DECAY   S <- diag(a_t) S + k_t v_t^T;                                  o_t = S^T q_t     (gated linear attention)
 //   STATE_RULE_DELTA   S <- diag(a_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t     (gated delta rule)
 //
-// a_t is a decay per head and key channel in (0, 1); it scales the rows of S.  Query/key head of state head a is
+//   STATE_RULE_DELTA_HEAD   the same with ONE decay per head, S <- a_t S
+//
+// a_t is a decay per head and key channel (or per head) in (0, 1); it scales the rows of S.  Query/key head of state head a is
 // a / (heads / kv_heads).
 //
 // Everything here is fp32: the state, the decays (formed as exp(-rate * softplus(.)), never as a power of a rounded
@@ -102,13 +104,15 @@ __global__ void __launch_bounds__(256) lowrank_act_kernel(const float* __restric
 // A CTA takes `upc` head units of one token (query heads, key heads, value heads, in the order of the projection's columns): first every
 // thread convolves and activates channels of the CTA's range, then a warp per query / key head turns the head into a unit vector.
 // proj [T][ld] fp32 = q (kv_heads*dim) | k (kv_heads*dim) | v (heads*vdim) | beta logits (heads) | ...; out [T][C] = the finished q | k | v,
-// beta_out [T][heads].
+// beta_out [T][heads]; with a_log one decay per head, exp(-exp(a_log) softplus(logit + dt_bias)), from the logits behind beta's.
 template <int TAPS>   // 0: any number of taps
 __global__ void __launch_bounds__(256) conv_unit_finish_kernel(const float* __restrict__ proj, int ld, StateGeom g, int taps_any,
                                                                const float* __restrict__ conv_w, const float* __restrict__ ring,
                                                                const int32_t* __restrict__ row_seq, const int32_t* __restrict__ row_first,
                                                                const int32_t* __restrict__ positions, const int32_t* __restrict__ slots,
-                                                               float unit_eps, float* __restrict__ out, float* __restrict__ beta_out, int upc) {
+                                                               float unit_eps, float* __restrict__ out, float* __restrict__ beta_out, int upc,
+                                                               const float* __restrict__ a_log, const float* __restrict__ dt_bias,
+                                                               float* __restrict__ decay_out) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -157,7 +161,10 @@ __global__ void __launch_bounds__(256) conv_unit_finish_kernel(const float* __re
     for (int i = lane; i < g.dim; i += 32) h[i] *= r;
   }
   if (blockIdx.y == 0)
-    for (int a = threadIdx.x; a < g.heads; a += 256) beta_out[(size_t)t * g.heads + a] = sigmoid_f(row[C + a]);
+    for (int a = threadIdx.x; a < g.heads; a += 256) {
+      beta_out[(size_t)t * g.heads + a] = sigmoid_f(row[C + a]);
+      if (a_log) decay_out[(size_t)t * g.heads + a] = expf(-expf(a_log[a]) * softplus_f(row[C + g.heads + a] + dt_bias[a]));
+    }
 }
 
 __global__ void __launch_bounds__(128) conv_ring_store_kernel(const float* __restrict__ proj, int ld, int C, int taps, float* __restrict__ ring,
@@ -179,9 +186,7 @@ constexpr int SC_CHUNK = 8;     // tokens of one stage (two stages)
 __device__ __forceinline__ void cp_async_f32(float* smem_dst, const float* gsrc) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(gsrc) : "memory");
 }
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
 // grid (portions, heads, column tiles); block (cols / NC) * 8.  Eight lanes share NC neighbouring columns of the state and split the key
 // channels (channel i * 8 + j belongs to lane j; DPT channels per lane, dim <= 8 * DPT), so a value of q, k or the decay read from shared
@@ -202,7 +207,9 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
   constexpr int VW = DPT >= 4 ? 4 : DPT;    // channels per shared-memory load
   constexpr int DP = DPT * SC_LANES;
   constexpr int MAXC = 32 * NC;             // columns of a CTA at most
-  __shared__ __align__(16) float qs[2][CH][RS], ks[2][CH][RS], as[2][CH][RS];
+  constexpr bool HEAD = RULE == STATE_RULE_DELTA_HEAD;   // one decay per head and token: nothing staged per channel
+  __shared__ __align__(16) float qs[2][CH][RS], ks[2][CH][RS], as[HEAD ? 1 : 2][HEAD ? 1 : CH][HEAD ? 4 : RS];
+  __shared__ float ds[2][HEAD ? CH : 1];
   __shared__ __align__(16) float vs[2][CH][MAXC];
   __shared__ float bs[2][CH];
   pdl_wait();
@@ -226,17 +233,23 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
     const int at = (d % SC_LANES) * LS + d / SC_LANES;
     qs[st][tt][at] = 0.f;
     ks[st][tt][at] = 0.f;
-    as[st][tt][at] = 1.f;
+    if constexpr (!HEAD) {
+      as[st][tt][at] = 1.f;
+    }
   }
   const int vcols = min(cols, g.vdim - col0);
-  for (int i = threadIdx.x; i < 2 * CH * MAXC; i += nthreads) (&vs[0][0][0])[i] = 0.f;
+  if (vcols < cols)   // (only what no copy ever writes)
+    for (int i = threadIdx.x; i < 2 * CH * (cols - vcols); i += nthreads) {
+      const int row = i / (cols - vcols), c = vcols + i % (cols - vcols);
+      vs[row / CH][row % CH][c] = 0.f;
+    }
   __syncthreads();
   // (flat loops over a chunk's numbers keep every thread's copies in flight together; sizes that are powers of two -- the usual case --
   // index by shifts instead of divisions)
   const int dsh = (g.dim & (g.dim - 1)) == 0 ? 31 - __clz(g.dim) : -1, vsh = (vcols & (vcols - 1)) == 0 ? 31 - __clz(vcols) : -1;
   const float* qb = q + (size_t)first * ldq + kh * g.dim;
   const float* kb = k + (size_t)first * ldk + kh * g.dim;
-  const float* ab = decay + (size_t)first * ((size_t)g.heads * g.dim) + a * g.dim;
+  const float* ab = HEAD ? decay + (size_t)first * g.heads + a : decay + (size_t)first * ((size_t)g.heads * g.dim) + a * g.dim;
   const float* vb = v + (size_t)first * ldv + a * g.vdim + col0;
   const int lda = g.heads * g.dim;
   auto issue = [&](int c0, int st) {
@@ -246,15 +259,22 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
       const int row = c0 + tt;
       cp_async_f32(&qs[st][tt][at], qb + (size_t)row * ldq + d);
       cp_async_f32(&ks[st][tt][at], kb + (size_t)row * ldk + d);
-      cp_async_f32(&as[st][tt][at], ab + (size_t)row * lda + d);
+      if constexpr (!HEAD) {
+        cp_async_f32(&as[st][tt][at], ab + (size_t)row * lda + d);
+      }
     }
     for (int i = threadIdx.x; i < cn * vcols; i += nthreads) {
       const int tt = vsh >= 0 ? i >> vsh : i / vcols, c = vsh >= 0 ? i & (vcols - 1) : i % vcols;
       cp_async_f32(&vs[st][tt][c], vb + (size_t)(c0 + tt) * ldv + c);
     }
-    if (RULE == STATE_RULE_DELTA)
-      for (int i = threadIdx.x; i < cn; i += nthreads) cp_async_f32(&bs[st][i], beta + (size_t)(first + c0 + i) * g.heads + a);
-    cp_async_commit();
+    if (RULE != STATE_RULE_DECAY) {   // (a plain `if`: a discarded loop without braces took the statement behind it along)
+      for (int i = threadIdx.x; i < cn; i += nthreads) {
+        cp_async_f32(&bs[st][i], beta + (size_t)(first + c0 + i) * g.heads + a);
+        if (HEAD) {
+          cp_async_f32(&ds[st][HEAD ? i : 0], ab + (size_t)(c0 + i) * g.heads);
+        }
+      }
+    }
   };
   issue(0, 0);
   float s[DPT][NC];
@@ -278,13 +298,9 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
   int st = 0;
   for (int c0 = 0; c0 < n; c0 += CH, st ^= 1) {
     const int cn = min(CH, n - c0);
-    if (c0 + CH < n) {
-      issue(c0 + CH, st ^ 1);     // (every thread left that stage at the barrier that ended the chunk before this one)
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    __syncthreads();
+    cp_async_wait_all();                         // this chunk's copies (the only ones in flight)
+    __syncthreads();                             // ... of every thread; and every thread has left the other stage
+    if (c0 + CH < n) issue(c0 + CH, st ^ 1);     // the next chunk's copies run beside this chunk's arithmetic
     for (int tt = 0; tt < cn; ++tt) {
       float vc[NC];
       if constexpr (NC == 4) {
@@ -294,13 +310,13 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
 #pragma unroll
         for (int c = 0; c < NC; ++c) vc[c] = vs[st][tt][cl + c];
       }
-      const float* ap = &as[st][tt][j * LS];
+      const float* ap = HEAD ? nullptr : &as[st][tt][j * LS];
       const float* kp = &ks[st][tt][j * LS];
       const float* qp = &qs[st][tt][j * LS];
       float av[VW], kw[VW], qv[VW], acc[NC];
 #pragma unroll
       for (int c = 0; c < NC; ++c) acc[c] = 0.f;
-      if (RULE == STATE_RULE_DECAY) {
+      if constexpr (RULE == STATE_RULE_DECAY) {
 #pragma unroll
         for (int i = 0; i < DPT; i += VW) {
           load(ap, i, av);
@@ -311,6 +327,39 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
               s[i + x][c] = fmaf(av[x], s[i + x][c], kw[x] * vc[c]);
+              acc[c] = fmaf(s[i + x][c], qv[x], acc[c]);
+            }
+        }
+      } else if constexpr (HEAD) {
+        // S' = g S + k u^T with u = beta (v - g S^T k): the decay is a number, so it leaves the sum over the key channels and joins the update
+        const float gd = ds[st][tt], bt = bs[st][tt];
+        float kv[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) kv[c] = 0.f;
+#pragma unroll
+        for (int i = 0; i < DPT; i += VW) {
+          load(kp, i, kw);
+#pragma unroll
+          for (int x = 0; x < VW; ++x)
+#pragma unroll
+            for (int c = 0; c < NC; ++c) kv[c] = fmaf(s[i + x][c], kw[x], kv[c]);
+        }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          kv[c] += __shfl_xor_sync(0xffffffffu, kv[c], 1);
+          kv[c] += __shfl_xor_sync(0xffffffffu, kv[c], 2);
+          kv[c] += __shfl_xor_sync(0xffffffffu, kv[c], 4);
+          kv[c] = bt * fmaf(-gd, kv[c], vc[c]);     // u
+        }
+#pragma unroll
+        for (int i = 0; i < DPT; i += VW) {
+          load(kp, i, kw);
+          load(qp, i, qv);
+#pragma unroll
+          for (int x = 0; x < VW; ++x)
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+              s[i + x][c] = fmaf(kw[x], kv[c], gd * s[i + x][c]);
               acc[c] = fmaf(s[i + x][c], qv[x], acc[c]);
             }
         }
@@ -364,7 +413,6 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
           if (col0 + cl + c < g.vdim) orow[c] = acc[c] * qscale;
       }
     }
-    __syncthreads();   // the chunk has been consumed: its stage may be filled again
   }
 #pragma unroll
   for (int i = 0; i < DPT; ++i) {
@@ -437,15 +485,16 @@ int launch_lowrank_act(const float* lr, int ld, int lr_off, int rank, const floa
 
 int launch_conv_unit_finish(const float* proj, int ld, const StateGeom& g, int taps, const float* conv_w, float* ring, const int32_t* row_seq,
                             const int32_t* row_first, const int32_t* row_end, const int32_t* positions, const int32_t* slots, float unit_eps,
-                            float* out, float* beta_out, int T, cudaStream_t s) {
+                            float* out, float* beta_out, int T, cudaStream_t s, const float* a_log, const float* dt_bias, float* decay_out) {
   if (T <= 0) return 0;
+  B2_REQUIRE(a_log == nullptr || (dt_bias != nullptr && decay_out != nullptr), "conv_unit_finish: a decay per head needs its bias and its output");
   B2_REQUIRE(taps >= 1 && conv_w && (ring || taps == 1) && row_seq && row_first && row_end, "conv_unit_finish: the convolution needs its weights and state");
   const int C = 2 * g.kv_heads * g.dim + g.heads * g.vdim;
   const int units = 2 * g.kv_heads + g.heads, upc = T >= 256 ? units : std::max(1, (units + 15) / 16);   // few tokens: up to sixteen CTAs each
   const dim3 grid(T, (units + upc - 1) / upc);
 #define B2_CONV_FINISH(TAPS)                                                                                                                      \
   B2_CUDA_OK(b2_launch(conv_unit_finish_kernel<TAPS>, grid, dim3(256), 0, s, proj, ld, g, taps, conv_w, (const float*)ring, row_seq, row_first, positions, \
-                       slots, unit_eps, out, beta_out, upc))
+                       slots, unit_eps, out, beta_out, upc, a_log, dt_bias, decay_out))
   if (taps == 4) B2_CONV_FINISH(4);
   else if (taps == 3) B2_CONV_FINISH(3);
   else if (taps == 2) B2_CONV_FINISH(2);
@@ -462,7 +511,7 @@ int launch_state_scan(const float* q, int ldq, const float* k, int ldk, const fl
                       cudaStream_t s) {
   if (portions <= 0) return 0;
   B2_REQUIRE(g.heads >= 1 && g.kv_heads >= 1 && g.heads % g.kv_heads == 0 && g.dim >= 1 && g.vdim >= 1, "state_scan: bad sizes");
-  B2_REQUIRE(g.rule == STATE_RULE_DECAY || (g.rule == STATE_RULE_DELTA && beta != nullptr), "state_scan: rule %d", g.rule);
+  B2_REQUIRE(g.rule == STATE_RULE_DECAY || ((g.rule == STATE_RULE_DELTA || g.rule == STATE_RULE_DELTA_HEAD) && beta != nullptr), "state_scan: rule %d", g.rule);
   int dpt = 1;
   while (dpt * SC_LANES < g.dim) dpt *= 2;
   B2_REQUIRE(dpt <= 32, "state_scan: key width %d not built (at most 256)", g.dim);
@@ -475,6 +524,9 @@ int launch_state_scan(const float* q, int ldq, const float* k, int ldk, const fl
   if (g.rule == STATE_RULE_DECAY)
     return launch_scan_rule<STATE_RULE_DECAY>(dpt, grid, block, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,
                                               row_first, row_end, positions, slots, out, cols);
+  if (g.rule == STATE_RULE_DELTA_HEAD)
+    return launch_scan_rule<STATE_RULE_DELTA_HEAD>(dpt, grid, block, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,
+                                                   row_first, row_end, positions, slots, out, cols);
   return launch_scan_rule<STATE_RULE_DELTA>(dpt, grid, block, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,
                                             row_first, row_end, positions, slots, out, cols);
 }

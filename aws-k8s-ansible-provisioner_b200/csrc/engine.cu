@@ -114,6 +114,9 @@ struct ListLayer {
   float *bias1 = nullptr, *bias1b = nullptr, *bias2 = nullptr, *bias2b = nullptr, *latq_gain = nullptr;
   void* uq = nullptr;
   int32_t* table = nullptr;
+  // Norms behind the sublayers only (Tolanex): gain1b / gain2b.  Its delta mixer projects q | k | v | beta | decay | gate in `wqd` (off_sg = the
+  // gate's first column), with `a_log` and `a2_bias` per head; its latent mixer q (| the latent) in `wqd`; `router` holds the shared expert's
+  // gate row behind the experts' rows.
 };
 // One run of a layer.  A looped layer runs once per pass with the same weights (ListLayer) but a cache and state of its own.
 struct ListRun {
@@ -123,7 +126,8 @@ struct ListRun {
   float* state = nullptr;      // [sequence slots][2][heads][dim][vdim] fp32 (attn_state.cu)
   float* ring = nullptr;       // [sequence slots][taps][channels] fp32: the convolutions' last inputs
 };
-inline bool list_arch(int arch) { return arch == B2_ARCH_LERASUN || arch == B2_ARCH_KEDASUN || arch == B2_ARCH_BUMALIX || arch == B2_ARCH_TINEVIK; }
+inline bool list_arch(int arch) { return arch == B2_ARCH_LERASUN || arch == B2_ARCH_KEDASUN || arch == B2_ARCH_BUMALIX || arch == B2_ARCH_TINEVIK ||
+                                        arch == B2_ARCH_TOLANEX; }
 
 struct Seq {
   bool active = false;
@@ -348,6 +352,10 @@ struct b2_engine {
   cudaEvent_t l_ev[6] = {nullptr, nullptr, nullptr, nullptr, nullptr, nullptr};
   float* l_upf2 = nullptr;           // the shared expert's gate | up sums and activation (its own, so that it can run beside the routed experts)
   void* l_act2 = nullptr;
+  // sum of three embedding rows, output norms (Tolanex)
+  void *l_bigram = nullptr, *l_pos = nullptr;
+  int32_t* l_tok_ring = nullptr;     // [sequence slots][2]: the token at a position, by the position's parity (a sequence's previous token)
+  float* l_sg = nullptr;             // the shared expert's gate, one number per token row
 };
 
 namespace {
@@ -899,7 +907,7 @@ int forward_layers(b2_engine* e, const Lane& ln, int T, int ntiles) {
 // layer share one statistic (one kernel).  Mixer = latent attention in absorbed form (attn_latent.cu); feed-forward =
 // routed squared-ReLU experts as ragged groups of gemm_any.cu.  `rows` (device, nlast entries; null = every row) selects
 // the positions that get logits.  Operands are bf16, or fp32 when the engine was created with compute_f32.
-constexpr int LIST_TC_EXPERT_ROWS = 2048;
+constexpr int LIST_TC_EXPERT_ROWS = 2048;   // (token, choice) pairs of a step from which the experts' products go expert by expert to the tcgen05 kernel
 
 // C (fp32 [M][N]) = alpha * A (operand type [M][K]) . Wt^T for the layer-list families.  Prompt-sized bf16 products whose K the tcgen05
 // projection kernel can tile (gemm_tc.cu: TMA needs 16-byte rows, its k-block is 64) take that kernel, fp32 sums written directly;
@@ -927,7 +935,72 @@ int list_dense(b2_engine* e, const void* A, const void* Wt, float* C, int M, int
   AnyGemm a;
   a.A = A; a.W = Wt; a.C = C; a.M = M; a.N = N; a.K = K; a.lda = K; a.ldw = K; a.ldc = N; a.alpha = alpha;
   return launch_gemm_any(a, f, f, 1, 1, 0, ls);
-}   // (token, choice) pairs of a step from which the experts' products go expert by expert to the tcgen05 kernel
+}
+
+// The two products of a layer's routed experts around a gated activation, for the families whose experts have gate and up rows: l_x1 rows -> gate |
+// up sums (l_upf, fp32, expert order) -> act(operand is fp32?) -> l_act -> l_y (fp32, expert order).  The permutation (l_offsets,
+// l_slot_token) is in place.  Prompt-sized bf16 steps (prompt = true) run expert by expert on the tcgen05 projection kernel: rows gathered into
+// expert order, the experts' slot ranges read back (one small copy and a stream synchronisation per layer); everything else as ragged groups.
+template <typename Act>
+int list_gated_experts(b2_engine* e, const ListLayer& L, int layer, int T, bool prompt, cudaStream_t s, Act act) {
+  const b2_layer_spec& sp = L.sp;
+  const int W = e->cfg.hidden, f = e->f32 ? 1 : 0, F = sp.ff_dim, pairs = T * sp.top;
+  const bool tc_experts = prompt && list_use_tc() && !f && e->l_xperm != nullptr && pairs >= LIST_TC_EXPERT_ROWS && W % 64 == 0 && F % 64 == 0 && W >= 128 &&
+                          F >= 64 && e->skip_mask == 0;
+  if (tc_experts) {
+    B2_CUDA_OK(cudaMemcpyAsync(e->h_offsets, e->l_offsets, (size_t)(sp.experts + 1) * 4, cudaMemcpyDeviceToHost, s));
+    {
+      KL k(e, B2K_MISC);
+      B2_TRY(launch_gather_rows((const bf16*)e->l_x1, e->l_slot_token, e->l_xperm, pairs, W, s));
+    }
+    B2_CUDA_OK(cudaStreamSynchronize(s));
+    const int32_t* off = e->h_offsets;
+    B2_REQUIRE(off[0] == 0 && off[sp.experts] == pairs, "layer %d: the experts' slot ranges do not cover the step's %d pairs", layer, pairs);
+    {
+      KL k(e, B2K_GEMM_GATEUP);
+      for (int x = 0; x < sp.experts; ++x)
+        if (off[x + 1] > off[x])
+          B2_TRY(list_dense(e, e->l_xperm + (size_t)off[x] * W, (const bf16*)L.up + (size_t)x * 2 * F * W, e->l_upf + (size_t)off[x] * 2 * F,
+                            off[x + 1] - off[x], 2 * F, W, 1.f, s));
+    }
+    {
+      KL k(e, B2K_ACT);
+      B2_TRY(act(0));
+    }
+    {
+      KL k(e, B2K_GEMM_DOWN);
+      for (int x = 0; x < sp.experts; ++x)
+        if (off[x + 1] > off[x])
+          B2_TRY(list_dense(e, (const bf16*)e->l_act + (size_t)off[x] * F, (const bf16*)L.down + (size_t)x * W * F, e->l_y + (size_t)off[x] * W,
+                            off[x + 1] - off[x], W, F, 1.f, s));
+    }
+    return 0;
+  }
+  const int max_tiles = std::min(e->l_tiles_cap, (pairs + any_gemm_tile_rows() - 1) / any_gemm_tile_rows() + sp.experts);
+  if (pairs > any_gemm_ragged_rows_limit() || W > 16384 || 2 * F > 16384) {
+    KL k(e, B2K_MISC);
+    if (!k.skip()) B2_TRY(launch_ragged_tiles(e->l_offsets, sp.experts, e->l_tile_group, e->l_tile_row0, e->l_ntiles, max_tiles, s));
+  }
+  AnyGemm a;
+  a.tile_group = e->l_tile_group; a.tile_row0 = e->l_tile_row0; a.n_tiles = e->l_ntiles; a.group_offsets = e->l_offsets;
+  {
+    KL k(e, B2K_GEMM_GATEUP);  // gate | up of every (token, choice) pair in expert order, fp32 sums
+    a.A = e->l_x1; a.a_rows = e->l_slot_token; a.W = L.up; a.C = e->l_upf; a.N = 2 * F; a.K = W; a.lda = W; a.ldw = W; a.ldc = 2 * F;
+    a.w_bs = (long)2 * F * W; a.epilogue = ANY_EPI_STORE;
+    if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, 1, 1, max_tiles, s, pairs, sp.experts));
+  }
+  {
+    KL k(e, B2K_ACT);
+    if (!k.skip()) B2_TRY(act(f));
+  }
+  {
+    KL k(e, B2K_GEMM_DOWN);
+    a.A = e->l_act; a.a_rows = nullptr; a.W = L.down; a.C = e->l_y; a.N = W; a.K = F; a.lda = F; a.ldw = F; a.ldc = W;
+    a.w_bs = (long)W * F; a.epilogue = ANY_EPI_STORE;
+    if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, 1, 1, max_tiles, s, pairs, sp.experts));
+  }
+  return 0;
+}
 
 int forward_list(b2_engine* e, int T, int ntiles, int nlast) {
   const b2_config& c = e->cfg;
@@ -1239,7 +1312,6 @@ int forward_state_list(b2_engine* e, int T, int ntiles, int nlast) {
   const PrefillTile* tiles = ntiles > 0 ? e->d_tiles : nullptr;
   const int portions = ntiles > 0 ? e->step_portions : T;
   const int32_t* last_rows = ntiles > 0 ? e->d_last_rows : nullptr;
-  const bool use_tc = list_use_tc();
   bool have_norm = false;   // l_x1 already holds this layer's norm output (the layer before wrote it)
   for (size_t r = 0; r < e->runs.size(); ++r) {
     const ListRun& R = e->runs[r];
@@ -1383,63 +1455,9 @@ int forward_state_list(b2_engine* e, int T, int ntiles, int nlast) {
           B2_TRY(launch_route_slot_weights(e->l_rw, e->l_pair_slot, e->l_slot_scale, pairs, sF));
         }
       }
-      // The weight multiplies the expert's input: gate and up are linear in it, so it is applied to their fp32 sums inside the
-      // activation.  Prompt-sized bf16 steps run expert by expert on the tcgen05 projection kernel (rows gathered into expert
-      // order, slot ranges read back); everything else as ragged groups.
-      const bool tc_experts = !multi && use_tc && !f && ntiles > 0 && e->l_xperm != nullptr && pairs >= LIST_TC_EXPERT_ROWS && W % 64 == 0 && F % 64 == 0 &&
-                              W >= 128 && F >= 64 && e->skip_mask == 0;
-      if (tc_experts) {
-        B2_CUDA_OK(cudaMemcpyAsync(e->h_offsets, e->l_offsets, (size_t)(sp.experts + 1) * 4, cudaMemcpyDeviceToHost, st));
-        {
-          KL k(e, B2K_MISC);
-          B2_TRY(launch_gather_rows((const bf16*)e->l_x1, e->l_slot_token, e->l_xperm, pairs, W, st));
-        }
-        B2_CUDA_OK(cudaStreamSynchronize(st));
-        const int32_t* off = e->h_offsets;
-        B2_REQUIRE(off[0] == 0 && off[sp.experts] == pairs, "layer %d: the experts' slot ranges do not cover the step's %d pairs", R.layer, pairs);
-        {
-          KL k(e, B2K_GEMM_GATEUP);
-          for (int x = 0; x < sp.experts; ++x)
-            if (off[x + 1] > off[x])
-              B2_TRY(dense(e->l_xperm + (size_t)off[x] * W, (const bf16*)L.up + (size_t)x * 2 * F * W, e->l_upf + (size_t)off[x] * 2 * F, off[x + 1] - off[x],
-                           2 * F, W, st));
-        }
-        {
-          KL k(e, B2K_ACT);
-          B2_TRY(launch_silu_gate(e->l_upf, e->l_slot_scale, nullptr, e->l_act, 0, pairs, F, st));
-        }
-        {
-          KL k(e, B2K_GEMM_DOWN);
-          for (int x = 0; x < sp.experts; ++x)
-            if (off[x + 1] > off[x])
-              B2_TRY(dense((const bf16*)e->l_act + (size_t)off[x] * F, (const bf16*)L.down + (size_t)x * W * F, e->l_y + (size_t)off[x] * W,
-                           off[x + 1] - off[x], W, F, st));
-        }
-      } else {
-        const int max_tiles = std::min(e->l_tiles_cap, (pairs + any_gemm_tile_rows() - 1) / any_gemm_tile_rows() + sp.experts);
-        if (pairs > any_gemm_ragged_rows_limit() || W > 16384 || 2 * F > 16384) {
-          KL k(e, B2K_MISC);
-          if (!k.skip()) B2_TRY(launch_ragged_tiles(e->l_offsets, sp.experts, e->l_tile_group, e->l_tile_row0, e->l_ntiles, max_tiles, sF));
-        }
-        AnyGemm a;
-        a.tile_group = e->l_tile_group; a.tile_row0 = e->l_tile_row0; a.n_tiles = e->l_ntiles; a.group_offsets = e->l_offsets;
-        {
-          KL k(e, B2K_GEMM_GATEUP);  // gate | up of every (token, choice) pair in expert order, fp32 sums
-          a.A = e->l_x1; a.a_rows = e->l_slot_token; a.W = L.up; a.C = e->l_upf; a.N = 2 * F; a.K = W; a.lda = W; a.ldw = W; a.ldc = 2 * F;
-          a.w_bs = (long)2 * F * W; a.epilogue = ANY_EPI_STORE;
-          if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, 1, 1, max_tiles, sF, pairs, sp.experts));
-        }
-        {
-          KL k(e, B2K_ACT);
-          if (!k.skip()) B2_TRY(launch_silu_gate(e->l_upf, e->l_slot_scale, nullptr, e->l_act, f, pairs, F, sF));
-        }
-        {
-          KL k(e, B2K_GEMM_DOWN);
-          a.A = e->l_act; a.a_rows = nullptr; a.W = L.down; a.C = e->l_y; a.N = W; a.K = F; a.lda = F; a.ldw = F; a.ldc = W;
-          a.w_bs = (long)W * F; a.epilogue = ANY_EPI_STORE;
-          if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, 1, 1, max_tiles, sF, pairs, sp.experts));
-        }
-      }
+      // The weight multiplies the expert's input: gate and up are linear in it, so it is applied to their fp32 sums inside the activation.
+      B2_TRY(list_gated_experts(e, L, R.layer, T, ntiles > 0 && !multi, sF,
+                                [&](int act_f32) { return launch_silu_gate(e->l_upf, e->l_slot_scale, nullptr, e->l_act, act_f32, pairs, F, sF); }));
       yr = e->l_y;
       if (sp.shared_ff > 0) {   // (buffers of its own: in short steps it runs beside the routed experts)
         first_on(sS);
@@ -1517,7 +1535,6 @@ int forward_mixed_list(b2_engine* e, int T, int ntiles, int nlast) {
   const PrefillTile* tiles = ntiles > 0 ? e->d_tiles : nullptr;
   const int portions = ntiles > 0 ? e->step_portions : T;
   const int32_t* last_rows = ntiles > 0 ? e->d_last_rows : nullptr;
-  const bool use_tc = list_use_tc();
   bool have_norm = false;   // l_x1 already holds this run's first norm output (the run before wrote it)
   for (size_t r = 0; r < e->runs.size(); ++r) {
     const ListRun& R = e->runs[r];
@@ -1651,62 +1668,8 @@ int forward_mixed_list(b2_engine* e, int T, int ntiles, int nlast) {
           KL k(e, B2K_MISC);
           if (!k.skip()) B2_TRY(launch_route_permute(e->l_idx, T, sp.top, sp.experts, e->l_offsets, e->l_offsets_stride, e->l_slot_token, e->l_pair_slot, st));
         }
-        // Prompt-sized bf16 steps run expert by expert on the tcgen05 projection kernel (rows gathered into expert order, the experts' slot
-        // ranges read back: one small copy and a stream synchronisation per layer); everything else as ragged groups.
-        const bool tc_experts = use_tc && !f && ntiles > 0 && e->l_xperm != nullptr && pairs >= LIST_TC_EXPERT_ROWS && W % 64 == 0 && F % 64 == 0 && W >= 128 &&
-                                F >= 64 && e->skip_mask == 0;
-        if (tc_experts) {
-          B2_CUDA_OK(cudaMemcpyAsync(e->h_offsets, e->l_offsets, (size_t)(sp.experts + 1) * 4, cudaMemcpyDeviceToHost, st));
-          {
-            KL k(e, B2K_MISC);
-            B2_TRY(launch_gather_rows((const bf16*)e->l_x1, e->l_slot_token, e->l_xperm, pairs, W, st));
-          }
-          B2_CUDA_OK(cudaStreamSynchronize(st));
-          const int32_t* off = e->h_offsets;
-          B2_REQUIRE(off[0] == 0 && off[sp.experts] == pairs, "layer %d: the experts' slot ranges do not cover the step's %d pairs", R.layer, pairs);
-          {
-            KL k(e, B2K_GEMM_GATEUP);
-            for (int x = 0; x < sp.experts; ++x)
-              if (off[x + 1] > off[x])
-                B2_TRY(dense(e->l_xperm + (size_t)off[x] * W, (const bf16*)L.up + (size_t)x * 2 * F * W, e->l_upf + (size_t)off[x] * 2 * F, off[x + 1] - off[x],
-                             2 * F, W));
-          }
-          {
-            KL k(e, B2K_ACT);
-            B2_TRY(launch_clamped_gate(e->l_upf, e->l_act, 0, pairs, F, sp.ff_limit, TINEVIK_GATE_SHARP, st));
-          }
-          {
-            KL k(e, B2K_GEMM_DOWN);
-            for (int x = 0; x < sp.experts; ++x)
-              if (off[x + 1] > off[x])
-                B2_TRY(dense((const bf16*)e->l_act + (size_t)off[x] * F, (const bf16*)L.down + (size_t)x * W * F, e->l_y + (size_t)off[x] * W,
-                             off[x + 1] - off[x], W, F));
-          }
-        } else {
-          const int max_tiles = std::min(e->l_tiles_cap, (pairs + any_gemm_tile_rows() - 1) / any_gemm_tile_rows() + sp.experts);
-          if (pairs > any_gemm_ragged_rows_limit() || W > 16384 || 2 * F > 16384) {
-            KL k(e, B2K_MISC);
-            if (!k.skip()) B2_TRY(launch_ragged_tiles(e->l_offsets, sp.experts, e->l_tile_group, e->l_tile_row0, e->l_ntiles, max_tiles, st));
-          }
-          AnyGemm a;
-          a.tile_group = e->l_tile_group; a.tile_row0 = e->l_tile_row0; a.n_tiles = e->l_ntiles; a.group_offsets = e->l_offsets;
-          {
-            KL k(e, B2K_GEMM_GATEUP);  // gate | up of every (token, choice) pair in expert order, fp32 sums
-            a.A = e->l_x1; a.a_rows = e->l_slot_token; a.W = L.up; a.C = e->l_upf; a.N = 2 * F; a.K = W; a.lda = W; a.ldw = W; a.ldc = 2 * F;
-            a.w_bs = (long)2 * F * W; a.epilogue = ANY_EPI_STORE;
-            if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, 1, 1, max_tiles, st, pairs, sp.experts));
-          }
-          {
-            KL k(e, B2K_ACT);
-            if (!k.skip()) B2_TRY(launch_clamped_gate(e->l_upf, e->l_act, f, pairs, F, sp.ff_limit, TINEVIK_GATE_SHARP, st));
-          }
-          {
-            KL k(e, B2K_GEMM_DOWN);
-            a.A = e->l_act; a.a_rows = nullptr; a.W = L.down; a.C = e->l_y; a.N = W; a.K = F; a.lda = F; a.ldw = F; a.ldc = W;
-            a.w_bs = (long)W * F; a.epilogue = ANY_EPI_STORE;
-            if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, 1, 1, max_tiles, st, pairs, sp.experts));
-          }
-        }
+        B2_TRY(list_gated_experts(e, L, R.layer, T, ntiles > 0, st,
+                                  [&](int act_f32) { return launch_clamped_gate(e->l_upf, e->l_act, act_f32, pairs, F, sp.ff_limit, TINEVIK_GATE_SHARP, st); }));
         {
           KL k(e, B2K_NORM);   // h += ln2b(mean of the token's experts)
           if (!k.skip()) B2_TRY(launch_layer_norm_add(e->l_h, e->l_y, e->l_pair_slot, sp.top, 1.0f / (float)sp.top, L.gain2b, L.bias2b, T, W, c.rms_eps, st, wn, bn,
@@ -1724,6 +1687,170 @@ int forward_mixed_list(b2_engine* e, int T, int ntiles, int nlast) {
   {
     KL k(e, B2K_LMHEAD);
     if (!k.skip()) B2_TRY(list_dense(e, e->l_xl, e->l_head, e->l_logits, nlast, c.vocab, W, c.logit_scale != 0.f ? c.logit_scale : 1.f, st));
+  }
+  {
+    KL k(e, B2K_MISC);
+    bf16* lb = (e->debug_flags & 2) ? e->logits : nullptr;
+    if (!k.skip()) B2_TRY(launch_logits_finish(e->l_logits, e->d_out_tokens, lb, bucket_batch(std::max(c.max_seqs, 1)), nlast, c.vocab, e->v_pad, st));
+  }
+  return 0;
+}
+
+// Tolanex: h <- h + m rms(mixer(h)) w1, then h <- h + m rms(ff(h)) w2 on the same fp32 residual stream; the sublayers read the stream itself (l_x1 = the
+// stream in the operand type, written by whichever kernel updated the stream).  Two mixers behind ONE fused projection each: the gated delta
+// rule with a decay per head (attn_state.cu over the sequence slots) and attention over a cached latent (attn_latent.cu, absorbed form; a layer
+// may read the region another layer wrote).  Feed-forward: experts chosen by a softmax router with grouped selection, weighted on their
+// output, plus a gated shared expert.  Per-sequence state besides the cache: matrix states, convolution rings, the previous token.
+constexpr float TOLANEX_UNIT_EPS = 1e-6f;   // q and k of the delta rule: x / sqrt(sum(x^2) + 1e-6)
+
+int forward_outnorm_list(b2_engine* e, int T, int ntiles, int nlast) {
+  const b2_config& c = e->cfg;
+  const int W = c.hidden, f = e->f32 ? 1 : 0;
+  const float mult = c.residual_mult != 0.f ? c.residual_mult : 1.f;
+  cudaStream_t st = e->stream;
+  auto dbg = [&](int slot) {
+    if ((e->debug_flags & 1) && e->dbg_hidden_f32 != nullptr && T <= e->dbg_cap_tokens && slot < e->dbg_slots)
+      cudaMemcpyAsync(e->dbg_hidden_f32 + (size_t)slot * e->dbg_cap_tokens * W, e->l_h, (size_t)T * W * 4, cudaMemcpyDeviceToDevice, st);
+  };
+  // Short steps are chains of small launches: the shared expert then runs on a stream of its own beside the routed ones (parallel
+  // branches of a captured step).  Profiled and debugged steps stay on one stream.
+  const bool multi = T <= 256 && !e->profiling && !(e->debug_flags & 1) && e->skip_mask == 0 && e->l_side[0] != nullptr;
+  auto dense = [&](const void* A, const void* Wt, float* C, int M, int N, int K, cudaStream_t s_) -> int { return list_dense(e, A, Wt, C, M, N, K, 1.f, s_); };
+  {
+    KL k(e, B2K_EMBED);
+    const BigramTable bg{e->l_bigram, c.bigram_buckets, c.bigram_mul_prev, c.bigram_mul_cur, e->l_tok_ring};
+    if (!k.skip()) B2_TRY(launch_embed_sum(e->d_tokens, e->l_embed, bg, e->l_pos, c.max_positions, f, e->l_h, e->l_x1, T, W, c.vocab, e->d_row_seq, e->d_row_first,
+                                           e->d_row_end, e->d_positions, e->d_slots, st));
+  }
+  dbg(0);
+  const PrefillTile* tiles = ntiles > 0 ? e->d_tiles : nullptr;
+  const int portions = ntiles > 0 ? e->step_portions : T;
+  const int32_t* last_rows = ntiles > 0 ? e->d_last_rows : nullptr;
+  for (int l = 0; l < c.num_layers; ++l) {
+    const ListRun& R = e->runs[l];
+    ListLayer& L = e->ll[l];
+    const b2_layer_spec& sp = L.sp;
+    const int HV = sp.heads * sp.vdim;
+    {
+      KL k(e, B2K_GEMM_QKV);   // everything that reads the mixer's input: one projection
+      if (!k.skip()) B2_TRY(dense(e->l_x1, L.wqd, e->l_qd, T, L.nqd, W, st));
+    }
+    if (sp.mixer == B2_MIXER_HEAD_DELTA) {
+      const StateGeom sg{sp.heads, sp.kv_heads, sp.dim, sp.vdim, STATE_RULE_DELTA_HEAD};
+      const int nqk = sp.kv_heads * sp.dim, C = 2 * nqk + HV;
+      {
+        KL k(e, B2K_ROPE_KV);   // convolutions, unit vectors, step sizes and decays
+        if (!k.skip()) B2_TRY(launch_conv_unit_finish(e->l_qd, L.nqd, sg, sp.conv_taps, L.conv_w, R.ring, e->d_row_seq, e->d_row_first, e->d_row_end,
+                                                      e->d_positions, e->d_slots, TOLANEX_UNIT_EPS, e->l_q, e->l_beta, T, st, L.a_log, L.a2_bias, e->l_dec));
+      }
+      {
+        KL k(e, B2K_CHAIN);
+        if (!k.skip()) B2_TRY(launch_state_scan(e->l_q, C, e->l_q + nqk, C, e->l_q + 2 * nqk, C, e->l_dec, e->l_beta, sg, 1.0f, R.state, portions, last_rows,
+                                                e->d_row_seq, e->d_row_first, e->d_row_end, e->d_positions, e->d_slots, e->l_so, st));
+      }
+      {
+        KL k(e, B2K_ACT);   // per-head RMS norm of the read-out, times silu(g)
+        if (!k.skip()) B2_TRY(launch_state_out_gate(e->l_so, L.head_gain, e->l_qd + L.off_sg, L.nqd, 1, e->l_av, f, sp.heads, sp.vdim, c.rms_eps, T, st));
+      }
+    } else {   // B2_MIXER_LATENT_ATTENTION, nothing rotated, no sink
+      const bool own = sp.kv_from < 0;
+      const LatentGeom g{sp.heads, sp.dim, 0, sp.vdim, sp.kv_rank, 0, 0.f, sp.scale, c.rms_eps, 0};
+      char* cache = e->regions[R.k_region].base;
+      {
+        KL k(e, B2K_ROPE_KV);   // queries as operands; the token's normed latent into the cache
+        if (!k.skip()) B2_TRY(launch_latent_finish(e->l_qd, L.nqd, g, own ? 1 : 0, L.lat_gain, e->d_positions, e->d_slots, e->l_qnope, f, e->l_q, cache, f, T, st));
+      }
+      {
+        KL k(e, B2K_GEMM_QKV);   // the query pulled through the key up-projection, all heads in one strided batch
+        AnyGemm a;
+        a.A = e->l_qnope; a.W = L.ukT; a.C = e->l_qabs; a.M = T; a.N = sp.kv_rank; a.K = sp.dim;
+        a.lda = (long)sp.heads * sp.dim; a.ldw = sp.dim; a.ldc = (long)sp.heads * sp.kv_rank;
+        a.a_bs = sp.dim; a.w_bs = (long)sp.kv_rank * sp.dim; a.c_bs = sp.kv_rank;
+        if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, 1, sp.heads, 0, st));
+      }
+      {
+        KL k(e, ntiles > 0 ? B2K_MISC : B2K_ATTN_DECODE);
+        if (!k.skip()) B2_TRY(launch_latent_attention(e->l_qabs, e->l_q, cache, f, g, e->d_block_table, e->bt_stride, c.block_size, tiles, ntiles, e->d_positions,
+                                                      e->d_seq_lens, nullptr, e->l_olat, f, T, st, e->l_attn_scratch, e->l_attn_scratch_floats, c.max_model_len));
+      }
+      {
+        KL k(e, B2K_GEMM_O);   // values of every head from the weighted latent
+        AnyGemm a;
+        a.A = e->l_olat; a.W = L.uv; a.C = e->l_av; a.M = T; a.N = sp.vdim; a.K = sp.kv_rank;
+        a.lda = (long)sp.heads * sp.kv_rank; a.ldw = sp.kv_rank; a.ldc = (long)HV;
+        a.a_bs = sp.kv_rank; a.w_bs = (long)sp.vdim * sp.kv_rank; a.c_bs = sp.vdim;
+        if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, f, sp.heads, 0, st));
+      }
+    }
+    {
+      KL k(e, B2K_GEMM_O);
+      if (!k.skip()) B2_TRY(dense(e->l_av, L.wo, e->l_mix, T, W, HV, st));
+    }
+    {
+      KL k(e, B2K_NORM);
+      if (!k.skip()) B2_TRY(launch_out_norm_add(e->l_h, e->l_mix, nullptr, nullptr, nullptr, nullptr, 0, L.gain1b, mult, T, W, c.rms_eps, st, e->l_x1, f));
+    }
+    if (sp.ff == B2_FF_SOFTMAX_EXPERTS) {
+      RouteGeom rg{sp.experts, sp.top, sp.groups, sp.groups_keep, 1};
+      rg.softmax = 1;
+      rg.group_best = 1;
+      rg.scale = sp.router_scale;
+      const int F = sp.ff_dim, pairs = T * sp.top;
+      const bool shared = sp.shared_ff > 0;
+      cudaStream_t sS = multi && shared ? e->l_side[0] : st;
+      auto shared_expert = [&]() -> int {   // (buffers of its own: in short steps it runs beside the routed experts)
+        if (sS != st) b2_pdl_skip_next();   // behind a cross-stream edge: an ordinary, full dependency
+        {
+          KL k(e, B2K_GEMM_GATEUP);
+          if (!k.skip()) B2_TRY(dense(e->l_x1, L.sh_up, e->l_upf2, T, 2 * sp.shared_ff, W, sS));
+        }
+        {
+          KL k(e, B2K_ACT);
+          if (!k.skip()) B2_TRY(launch_silu_gate(e->l_upf2, nullptr, nullptr, e->l_act2, f, T, sp.shared_ff, sS));
+        }
+        {
+          KL k(e, B2K_GEMM_DOWN);
+          if (!k.skip()) B2_TRY(dense(e->l_act2, L.sh_down, e->l_ffd, T, W, sp.shared_ff, sS));
+        }
+        return 0;
+      };
+      if (sS != st) {
+        B2_CUDA_OK(cudaEventRecord(e->l_ev[0], st));
+        B2_CUDA_OK(cudaStreamWaitEvent(sS, e->l_ev[0], 0));
+        B2_TRY(shared_expert());
+        B2_CUDA_OK(cudaEventRecord(e->l_ev[1], sS));
+        b2_pdl_skip_next();
+      }
+      {
+        KL k(e, B2K_ACT);
+        if (!k.skip()) B2_TRY(launch_route(e->l_x1, f, L.router, nullptr, rg, e->l_idx, e->l_rw, T, W, st, shared ? e->l_sg : nullptr));
+      }
+      {
+        KL k(e, B2K_MISC);
+        if (!k.skip()) B2_TRY(launch_route_permute(e->l_idx, T, sp.top, sp.experts, e->l_offsets, e->l_offsets_stride, e->l_slot_token, e->l_pair_slot, st));
+      }
+      B2_TRY(list_gated_experts(e, L, l, T, ntiles > 0 && !multi, st,
+                                [&](int act_f32) { return launch_silu_gate(e->l_upf, nullptr, nullptr, e->l_act, act_f32, pairs, F, st); }));
+      if (sS == st && shared) B2_TRY(shared_expert());
+      if (sS != st) {
+        B2_CUDA_OK(cudaStreamWaitEvent(st, e->l_ev[1], 0));
+        b2_pdl_skip_next();
+      }
+      {
+        KL k(e, B2K_NORM);   // h += m rms(sum of the chosen experts, weighted, + gate * shared expert) w2
+        if (!k.skip()) B2_TRY(launch_out_norm_add(e->l_h, shared ? e->l_ffd : nullptr, shared ? e->l_sg : nullptr, e->l_y, e->l_rw, e->l_pair_slot, sp.top, L.gain2b,
+                                                  mult, T, W, c.rms_eps, st, e->l_x1, f));
+      }
+    }
+    dbg(l + 1);
+  }
+  {
+    KL k(e, B2K_NORM);
+    if (!k.skip()) B2_TRY(launch_unit_norm2(e->l_h, e->l_final_gain, nullptr, e->l_xl, nullptr, f, nlast, W, c.rms_eps, ntiles > 0 ? e->d_last_rows : nullptr, st));
+  }
+  {
+    KL k(e, B2K_LMHEAD);
+    if (!k.skip()) B2_TRY(dense(e->l_xl, e->l_head, e->l_logits, nlast, c.vocab, W, st));
   }
   {
     KL k(e, B2K_MISC);
@@ -1755,6 +1882,7 @@ int forward(b2_engine* e, int T, int ntiles, int nlast, int attn_split) {
   if (c.arch == B2_ARCH_KEDASUN) return forward_heads_list(e, T, ntiles, nlast);
   if (c.arch == B2_ARCH_BUMALIX) return forward_state_list(e, T, ntiles, nlast);
   if (c.arch == B2_ARCH_TINEVIK) return forward_mixed_list(e, T, ntiles, nlast);
+  if (c.arch == B2_ARCH_TOLANEX) return forward_outnorm_list(e, T, ntiles, nlast);
   if (c.arch == B2_ARCH_OPT) return forward_opt(e, T, ntiles, nlast);
   if (ntiles == 0 && e->use_chain == 2 && e->fused_ok && c.arch == B2_ARCH_QWEN3 && !(e->debug_flags & 1) &&
       e->force_gemm_impl != 0 && T > e->simt_max_tokens && T <= 64 && e->skip_mask == 0)
@@ -2121,6 +2249,15 @@ int put_f32(float* dst, const uint16_t* src, size_t n, float add) {
   return 0;
 }
 
+// A key up-projection stored [heads * dim][rank], kept per head as [rank][dim]: the layout the absorbed-query product reads
+int put_key_up(b2_engine* e, void* dst, const uint16_t* src, size_t heads, size_t dim, size_t rank) {
+  std::vector<uint16_t> tr(heads * dim * rank);
+  for (size_t a = 0; a < heads; ++a)
+    for (size_t d = 0; d < dim; ++d)
+      for (size_t j = 0; j < rank; ++j) tr[(a * rank + j) * dim + d] = src[(a * dim + d) * rank + j];
+  return put_operand(e, dst, 0, tr.data(), tr.size());
+}
+
 int list_tensor(b2_engine* e, const std::string& name, const void* host, size_t nbytes) {
   const b2_config& c = e->cfg;
   const size_t W = c.hidden;
@@ -2141,6 +2278,12 @@ int list_tensor(b2_engine* e, const std::string& name, const void* host, size_t 
   if (name == "embed.norm") { B2_TRY(want(W)); return done(put_f32(e->l_embed_gain, src, W, 1.0f)); }
   if (name == "final.norm") { B2_TRY(want(W)); return done(put_f32(e->l_final_gain, src, W, c.arch == B2_ARCH_LERASUN ? 1.0f : 0.0f)); }
   if (name == "final.norm.b" && e->l_final_bias) { B2_TRY(want(W)); return done(put_f32(e->l_final_bias, src, W, 0.0f)); }
+  if (name == "bigram" && e->l_bigram) {
+    const size_t n = ((size_t)c.bigram_buckets + 1) * W;
+    B2_TRY(want(n));
+    return done(put_operand(e, e->l_bigram, 0, src, n));
+  }
+  if (name == "pos" && e->l_pos) { B2_TRY(want((size_t)c.max_positions * W)); return done(put_operand(e, e->l_pos, 0, src, (size_t)c.max_positions * W)); }
   if (c.arch == B2_ARCH_BUMALIX && name == "loop.in") {   // (a checkpoint may carry it although the config loops over nothing: nothing then uses it)
     B2_TRY(want(W * 2 * W));
     return done(e->l_loop_in ? put_operand(e, e->l_loop_in, 0, src, W * 2 * W) : 0);
@@ -2300,11 +2443,7 @@ int list_tensor(b2_engine* e, const std::string& name, const void* host, size_t 
       if (rest == "mix.uq") { B2_TRY(want(H * dn * qr)); return done(put_operand(e, L.uq, 0, src, H * dn * qr)); }
       if (rest == "mix.uk") {  // stored [heads * dim][kv_rank]; kept per head as [kv_rank][dim], the layout the absorbed-query product reads
         B2_TRY(want(H * dn * r));
-        std::vector<uint16_t> tr(H * dn * r);
-        for (size_t a = 0; a < H; ++a)
-          for (size_t d = 0; d < dn; ++d)
-            for (size_t j = 0; j < r; ++j) tr[(a * r + j) * dn + d] = src[(a * dn + d) * r + j];
-        return done(put_operand(e, L.ukT, 0, tr.data(), tr.size()));
+        return done(put_key_up(e, L.ukT, src, H, dn, r));
       }
       if (rest == "mix.uv") { B2_TRY(want(HV * r)); return done(put_operand(e, L.uv, 0, src, HV * r)); }
     }
@@ -2321,6 +2460,55 @@ int list_tensor(b2_engine* e, const std::string& name, const void* host, size_t 
           if (which == "gate") { B2_TRY(want(ff * W)); return done(put_operand(e, L.up, (size_t)ex * 2 * ff * W, src, ff * W)); }
           if (which == "up") { B2_TRY(want(ff * W)); return done(put_operand(e, L.up, ((size_t)ex * 2 + 1) * ff * W, src, ff * W)); }
           if (which == "down") { B2_TRY(want(W * ff)); return done(put_operand(e, L.down, (size_t)ex * W * ff, src, W * ff)); }
+        }
+      }
+    }
+    b2_set_error("unknown tensor name %s", name.c_str());
+    return -22;
+  }
+  if (c.arch == B2_ARCH_TOLANEX) {
+    const size_t HV = H * dv;
+    if (rest == "norm1") { B2_TRY(want(W)); return done(put_f32(L.gain1b, src, W, 0.0f)); }
+    if (rest == "norm2" && L.gain2b) { B2_TRY(want(W)); return done(put_f32(L.gain2b, src, W, 0.0f)); }
+    if (rest == "mix.o") { B2_TRY(want(W * HV)); return done(put_operand(e, L.wo, 0, src, W * HV)); }
+    if (sp.mixer == B2_MIXER_HEAD_DELTA) {
+      const size_t nqk = (size_t)sp.kv_heads * dn, taps = sp.conv_taps, C = 2 * nqk + HV;
+      if (rest == "mix.q") { B2_TRY(want(nqk * W)); return done(put_operand(e, L.wqd, 0, src, nqk * W)); }
+      if (rest == "mix.k") { B2_TRY(want(nqk * W)); return done(put_operand(e, L.wqd, nqk * W, src, nqk * W)); }
+      if (rest == "mix.v") { B2_TRY(want(HV * W)); return done(put_operand(e, L.wqd, 2 * nqk * W, src, HV * W)); }
+      if (rest == "mix.b") { B2_TRY(want(H * W)); return done(put_operand(e, L.wqd, C * W, src, H * W)); }
+      if (rest == "mix.a") { B2_TRY(want(H * W)); return done(put_operand(e, L.wqd, (C + H) * W, src, H * W)); }
+      if (rest == "mix.g") { B2_TRY(want(HV * W)); return done(put_operand(e, L.wqd, (size_t)L.off_sg * W, src, HV * W)); }
+      if (rest == "mix.q.conv") { B2_TRY(want(nqk * taps)); return done(put_f32(L.conv_w, src, nqk * taps, 0.0f)); }
+      if (rest == "mix.k.conv") { B2_TRY(want(nqk * taps)); return done(put_f32(L.conv_w + nqk * taps, src, nqk * taps, 0.0f)); }
+      if (rest == "mix.v.conv") { B2_TRY(want(HV * taps)); return done(put_f32(L.conv_w + 2 * nqk * taps, src, HV * taps, 0.0f)); }
+      if (rest == "mix.A_log") { B2_TRY(want(H)); return done(put_f32(L.a_log, src, H, 0.0f)); }
+      if (rest == "mix.dt_bias") { B2_TRY(want(H)); return done(put_f32(L.a2_bias, src, H, 0.0f)); }
+      if (rest == "mix.norm") { B2_TRY(want(dv)); return done(put_f32(L.head_gain, src, dv, 0.0f)); }
+    } else {
+      if (rest == "mix.q") { B2_TRY(want(H * dn * W)); return done(put_operand(e, L.wqd, 0, src, H * dn * W)); }
+      if (rest == "mix.dkv" && sp.kv_from < 0) { B2_TRY(want(r * W)); return done(put_operand(e, L.wqd, H * dn * W, src, r * W)); }
+      if (rest == "mix.dkv.norm" && sp.kv_from < 0) { B2_TRY(want(r)); return done(put_f32(L.lat_gain, src, r, 0.0f)); }
+      if (rest == "mix.uk") { B2_TRY(want(H * dn * r)); return done(put_key_up(e, L.ukT, src, H, dn, r)); }
+      if (rest == "mix.uv") { B2_TRY(want(HV * r)); return done(put_operand(e, L.uv, 0, src, HV * r)); }
+    }
+    if (sp.ff == B2_FF_SOFTMAX_EXPERTS) {
+      const size_t sf = sp.shared_ff, ne = sp.experts;
+      if (rest == "mlp.router") { B2_TRY(want(ne * W)); return done(put_f32(L.router, src, ne * W, 0.0f)); }
+      if (sf > 0 && rest == "mlp.shared.sg") { B2_TRY(want(W)); return done(put_f32(L.router + ne * W, src, W, 0.0f)); }
+      if (sf > 0 && rest == "mlp.shared.gate") { B2_TRY(want(sf * W)); return done(put_operand(e, L.sh_up, 0, src, sf * W)); }
+      if (sf > 0 && rest == "mlp.shared.up") { B2_TRY(want(sf * W)); return done(put_operand(e, L.sh_up, sf * W, src, sf * W)); }
+      if (sf > 0 && rest == "mlp.shared.down") { B2_TRY(want(W * sf)); return done(put_operand(e, L.sh_down, 0, src, W * sf)); }
+      if (rest.compare(0, 5, "mlp.e") == 0) {
+        size_t d2 = rest.find('.', 5);
+        if (d2 != std::string::npos) {
+          const int ex = atoi(rest.substr(5, d2 - 5).c_str());
+          const std::string which = rest.substr(d2 + 1);
+          if (ex >= 0 && ex < sp.experts) {   // gate rows, then up rows, expert by expert: one product gives both
+            if (which == "gate") { B2_TRY(want(ff * W)); return done(put_operand(e, L.up, (size_t)ex * 2 * ff * W, src, ff * W)); }
+            if (which == "up") { B2_TRY(want(ff * W)); return done(put_operand(e, L.up, ((size_t)ex * 2 + 1) * ff * W, src, ff * W)); }
+            if (which == "down") { B2_TRY(want(W * ff)); return done(put_operand(e, L.down, (size_t)ex * W * ff, src, W * ff)); }
+          }
         }
       }
     }
@@ -2365,11 +2553,7 @@ int list_tensor(b2_engine* e, const std::string& name, const void* host, size_t 
   if (rest == "mix.dkv.norm" && sp.kv_from < 0) { B2_TRY(want(r)); return done(put_f32(L.lat_gain, src, r, 0.0f)); }
   if (rest == "mix.uk") {  // stored [heads * dim][kv_rank]; kept per head as [kv_rank][dim], the layout the absorbed-query product reads
     B2_TRY(want(H * dn * r));
-    std::vector<uint16_t> tr(H * dn * r);
-    for (size_t a = 0; a < H; ++a)
-      for (size_t d = 0; d < dn; ++d)
-        for (size_t j = 0; j < r; ++j) tr[(a * r + j) * dn + d] = src[(a * dn + d) * r + j];
-    return done(put_operand(e, L.ukT, 0, tr.data(), tr.size()));
+    return done(put_key_up(e, L.ukT, src, H, dn, r));
   }
   if (rest == "mix.uv") { B2_TRY(want(H * dv * r)); return done(put_operand(e, L.uv, 0, src, H * dv * r)); }
   if (rest == "mix.sink") { B2_TRY(want(H)); return done(put_f32(L.sink, src, H, 0.0f)); }
@@ -3098,8 +3282,221 @@ int mixed_finalize(b2_engine* e) {
   return 0;
 }
 
+// The same for the family whose sublayers read the stream itself and whose norms sit behind them (Tolanex).
+int outnorm_engine_alloc(b2_engine* e) {
+  const b2_config& c = e->cfg;
+  const size_t W = c.hidden, es = e->esz;
+  B2_REQUIRE(!e->specs.empty() && (int)e->specs.size() == c.num_layers, "Tolanex: layer_specs missing");
+  B2_REQUIRE(c.hidden >= 1 && c.vocab >= 1 && c.num_layers >= 1, "Tolanex: bad sizes");
+  B2_REQUIRE(c.bigram_buckets >= 1 && c.max_positions >= 1, "Tolanex: bad embedding tables (%d buckets, %d positions)", c.bigram_buckets, c.max_positions);
+  auto xalloc = [&](void** p, size_t elems) -> int {
+    char* q = nullptr;
+    B2_TRY(dalloc(&q, std::max<size_t>(elems, 1) * es));
+    *p = q;
+    e->weight_bytes += (int64_t)(elems * es);
+    return 0;
+  };
+  auto falloc = [&](float** p, size_t n) -> int {
+    B2_TRY(dalloc(p, std::max<size_t>(n, 1)));
+    B2_CUDA_OK(cudaMemset(*p, 0, std::max<size_t>(n, 1) * 4));
+    e->weight_bytes += (int64_t)(n * 4);
+    return 0;
+  };
+  e->weight_bytes = 0;
+  B2_TRY(xalloc(&e->l_embed, (size_t)c.vocab * W));
+  B2_TRY(xalloc(&e->l_head, (size_t)c.vocab * W));
+  B2_TRY(xalloc(&e->l_bigram, ((size_t)c.bigram_buckets + 1) * W));
+  B2_TRY(xalloc(&e->l_pos, (size_t)c.max_positions * W));
+  B2_TRY(falloc(&e->l_final_gain, W));
+  e->ll.resize(c.num_layers);
+  size_t max_q = 1, max_hv = 1, max_up = 1, max_act = 1, max_hr = 1, max_hd = 1, max_sff = 0, max_nqd = 1;
+  int max_top = 1, max_exp = 1, max_lat_heads = 1, max_rank = 1, max_state_heads = 1;
+  bool any_latent = false, any_experts = false;
+  for (int l = 0; l < c.num_layers; ++l) {
+    ListLayer& L = e->ll[l];
+    L.sp = e->specs[l];
+    const b2_layer_spec& sp = L.sp;
+    const bool delta = sp.mixer == B2_MIXER_HEAD_DELTA;
+    B2_REQUIRE(delta || sp.mixer == B2_MIXER_LATENT_ATTENTION, "layer %d: mixer kind %d not built for this family", l, sp.mixer);
+    B2_REQUIRE(sp.heads >= 1 && sp.dim >= 1 && sp.vdim >= 1, "layer %d: bad mixer sizes (heads %d, dim %d, vdim %d)", l, sp.heads, sp.dim, sp.vdim);
+    const size_t HV = (size_t)sp.heads * sp.vdim;
+    ListRun R;
+    R.layer = l;
+    if (delta) {
+      B2_REQUIRE(sp.kv_heads >= 1 && sp.heads % sp.kv_heads == 0, "layer %d: %d heads over %d key heads", l, sp.heads, sp.kv_heads);
+      B2_REQUIRE(sp.conv_taps >= 1 && sp.dim <= 256, "layer %d: the delta rule needs at least one convolution tap and a key width of at most 256", l);
+      const size_t nqk = (size_t)sp.kv_heads * sp.dim, C = 2 * nqk + HV;
+      L.off_sg = (int)(C + 2 * sp.heads);
+      L.nqd = L.n_fixed = L.off_sg + (int)HV;
+      B2_TRY(falloc(&L.conv_w, C * sp.conv_taps));
+      B2_TRY(falloc(&L.a_log, sp.heads));
+      B2_TRY(falloc(&L.a2_bias, sp.heads));
+      B2_TRY(falloc(&L.head_gain, sp.vdim));
+      max_q = std::max(max_q, C);
+      max_state_heads = std::max(max_state_heads, sp.heads);
+      const StateGeom sg{sp.heads, sp.kv_heads, sp.dim, sp.vdim, STATE_RULE_DELTA_HEAD};
+      const size_t sf = (size_t)c.max_seqs * state_floats_per_slot(sg);
+      B2_TRY(dalloc(&R.state, sf));
+      B2_CUDA_OK(cudaMemset(R.state, 0, sf * 4));
+      if (sp.conv_taps > 1) {
+        const size_t rf = (size_t)c.max_seqs * sp.conv_taps * C;
+        B2_TRY(dalloc(&R.ring, rf));
+        B2_CUDA_OK(cudaMemset(R.ring, 0, rf * 4));
+      }
+    } else {
+      B2_REQUIRE(sp.kv_rank >= 1 && sp.rot_dim == 0, "layer %d: bad latent sizes (kv_rank %d, rot_dim %d)", l, sp.kv_rank, sp.rot_dim);
+      if (sp.kv_from >= 0) {
+        B2_REQUIRE(sp.kv_from < l && e->specs[sp.kv_from].mixer == B2_MIXER_LATENT_ATTENTION && e->specs[sp.kv_from].kv_from < 0 &&
+                       e->specs[sp.kv_from].kv_rank == sp.kv_rank,
+                   "layer %d: kv_from %d must name an earlier latent layer with a latent of its own and the same kv_rank", l, sp.kv_from);
+      } else {
+        B2_TRY(falloc(&L.lat_gain, sp.kv_rank));
+      }
+      L.nq = sp.heads * sp.dim;
+      L.nqd = L.n_fixed = L.nq + (sp.kv_from < 0 ? sp.kv_rank : 0);
+      B2_TRY(xalloc(&L.ukT, (size_t)sp.heads * sp.kv_rank * sp.dim));
+      B2_TRY(xalloc(&L.uv, HV * sp.kv_rank));
+      any_latent = true;
+      max_hd = std::max(max_hd, (size_t)L.nq);
+      max_hr = std::max(max_hr, (size_t)sp.heads * sp.kv_rank);
+      max_lat_heads = std::max(max_lat_heads, sp.heads);
+      max_rank = std::max(max_rank, sp.kv_rank);
+    }
+    e->runs.push_back(R);
+    max_hv = std::max(max_hv, HV);
+    max_nqd = std::max(max_nqd, (size_t)L.nqd);
+    B2_TRY(xalloc(&L.wqd, (size_t)L.nqd * W));
+    B2_TRY(xalloc(&L.wo, W * HV));
+    B2_TRY(falloc(&L.gain1b, W));
+    if (sp.ff == B2_FF_SOFTMAX_EXPERTS) {
+      B2_REQUIRE(sp.experts >= 1 && sp.top >= 1 && sp.ff_dim >= 1 && sp.shared_ff >= 0 && sp.groups >= 1 && sp.groups <= 64 && sp.experts % sp.groups == 0 &&
+                     sp.groups_keep >= 1 && sp.groups_keep <= sp.groups && sp.top <= sp.groups_keep * (sp.experts / sp.groups),
+                 "layer %d: bad router sizes (experts %d, top %d, groups %d, keep %d, ff %d)", l, sp.experts, sp.top, sp.groups, sp.groups_keep, sp.ff_dim);
+      B2_TRY(falloc(&L.gain2b, W));
+      B2_TRY(falloc(&L.router, (size_t)(sp.experts + (sp.shared_ff > 0 ? 1 : 0)) * W));
+      B2_TRY(xalloc(&L.up, (size_t)sp.experts * 2 * sp.ff_dim * W));
+      B2_TRY(xalloc(&L.down, (size_t)sp.experts * W * sp.ff_dim));
+      if (sp.shared_ff > 0) {
+        B2_TRY(xalloc(&L.sh_up, (size_t)2 * sp.shared_ff * W));
+        B2_TRY(xalloc(&L.sh_down, W * sp.shared_ff));
+      }
+      any_experts = true;
+      max_top = std::max(max_top, sp.top);
+      max_exp = std::max(max_exp, sp.experts);
+      max_up = std::max(max_up, (size_t)sp.top * 2 * sp.ff_dim);
+      max_act = std::max(max_act, (size_t)sp.top * sp.ff_dim);
+      max_sff = std::max(max_sff, (size_t)sp.shared_ff);
+    } else {
+      B2_REQUIRE(sp.ff == B2_FF_NONE, "layer %d: feed-forward kind %d not built for this family", l, sp.ff);
+    }
+  }
+  e->l_has_state = true;   // (the previous token at least)
+  e->dbg_slots = c.num_layers + 1;
+  B2_TRY(dalloc(&e->l_tok_ring, (size_t)c.max_seqs * 2));
+  B2_CUDA_OK(cudaMemset(e->l_tok_ring, 0, (size_t)c.max_seqs * 2 * 4));
+  B2_CUDA_OK(cudaStreamCreateWithFlags(&e->l_side[0], cudaStreamNonBlocking));
+  for (int i = 0; i < 2; ++i) B2_CUDA_OK(cudaEventCreateWithFlags(&e->l_ev[i], cudaEventDisableTiming));
+  // ---- activations ----
+  e->cap_tokens = ((std::max(c.max_batch_tokens, c.max_seqs) + 255) / 256) * 256;
+  const size_t Tc = e->cap_tokens;
+  e->l_rows_cap = (int)(Tc + bucket_batch(c.max_seqs));
+  e->l_max_top = max_top;
+  e->v_pad = (c.vocab + 7) / 8 * 8;
+  auto aalloc = [&](void** p, size_t elems) -> int {
+    char* q = nullptr;
+    B2_TRY(dalloc(&q, elems * es));
+    *p = q;
+    return 0;
+  };
+  B2_TRY(dalloc(&e->l_h, Tc * W));
+  B2_TRY(dalloc(&e->l_qd, Tc * max_nqd));
+  e->l_qd_cols = max_nqd;
+  B2_TRY(dalloc(&e->l_q, Tc * max_q));
+  B2_TRY(dalloc(&e->l_dec, Tc * max_state_heads));
+  B2_TRY(dalloc(&e->l_beta, Tc * max_state_heads));
+  B2_TRY(dalloc(&e->l_so, Tc * max_hv));
+  B2_TRY(dalloc(&e->l_mix, Tc * W));
+  B2_TRY(dalloc(&e->l_logits, (size_t)e->l_rows_cap * c.vocab));
+  B2_TRY(aalloc(&e->l_x1, Tc * W));
+  B2_TRY(aalloc(&e->l_av, Tc * max_hv));
+  B2_TRY(aalloc(&e->l_xl, (size_t)e->l_rows_cap * W));
+  if (any_latent) {
+    B2_TRY(aalloc(&e->l_qnope, Tc * max_hd));
+    B2_TRY(dalloc(&e->l_qabs, Tc * max_hr));
+    B2_TRY(aalloc(&e->l_olat, Tc * max_hr));
+    if (!e->f32) {
+      e->l_attn_scratch_floats = latent_attention_scratch_floats(bucket_batch(c.max_seqs), max_lat_heads, max_rank);
+      B2_TRY(dalloc(&e->l_attn_scratch, e->l_attn_scratch_floats));
+    }
+  }
+  if (any_experts) {
+    B2_TRY(dalloc(&e->l_ffd, Tc * W));
+    B2_TRY(dalloc(&e->l_y, Tc * max_top * W));
+    B2_TRY(dalloc(&e->l_upf, Tc * max_up));
+    B2_TRY(aalloc(&e->l_act, Tc * max_act));
+    if (max_sff > 0) {
+      B2_TRY(dalloc(&e->l_upf2, Tc * 2 * max_sff));
+      B2_TRY(aalloc(&e->l_act2, Tc * max_sff));
+    }
+    B2_TRY(dalloc(&e->l_rw, Tc * max_top));
+    B2_TRY(dalloc(&e->l_sg, Tc));
+    B2_TRY(dalloc(&e->l_idx, Tc * max_top));
+    e->l_offsets_stride = max_exp + 1;
+    B2_TRY(dalloc(&e->l_offsets, (size_t)3 * (max_exp + 1)));
+    B2_CUDA_OK(cudaMemset(e->l_offsets, 0, (size_t)3 * (max_exp + 1) * 4));
+    B2_TRY(dalloc(&e->l_slot_token, Tc * max_top));
+    B2_TRY(dalloc(&e->l_pair_slot, Tc * max_top));
+    B2_CUDA_OK(cudaMemset(e->l_pair_slot, 0, Tc * max_top * 4));
+    e->l_tiles_cap = (int)(Tc * max_top / any_gemm_tile_rows() + max_exp + 1);
+    B2_TRY(dalloc(&e->l_tile_group, (size_t)e->l_tiles_cap));
+    B2_TRY(dalloc(&e->l_tile_row0, (size_t)e->l_tiles_cap));
+    B2_TRY(dalloc(&e->l_ntiles, (size_t)1));
+    B2_CUDA_OK(cudaMemset(e->l_ntiles, 0, 4));
+    if (!e->f32 && Tc * max_top >= (size_t)LIST_TC_EXPERT_ROWS && max_exp > 1) {   // prompt-sized expert products on the tcgen05 projection kernel
+      B2_TRY(dalloc(&e->l_xperm, Tc * max_top * W));
+      B2_CUDA_OK(cudaMallocHost(&e->h_offsets, (size_t)(max_exp + 1) * sizeof(int32_t)));
+    }
+  }
+  for (int32_t** p : {&e->d_row_seq, &e->d_row_first, &e->d_row_end}) {
+    B2_TRY(dalloc(p, Tc));
+    B2_CUDA_OK(cudaMemset(*p, 0, Tc * 4));
+  }
+  return 0;
+}
+
+// Names of the tensors a Tolanex checkpoint must hold.
+std::vector<std::string> outnorm_tensor_names(const b2_engine* e) {
+  std::vector<std::string> n = {"embed", "bigram", "pos", "final.norm", "head"};
+  for (size_t l = 0; l < e->ll.size(); ++l) {
+    const b2_layer_spec& sp = e->ll[l].sp;
+    const std::string p = "l" + std::to_string(l) + ".";
+    n.push_back(p + "norm1");
+    if (sp.mixer == B2_MIXER_HEAD_DELTA) {
+      for (const char* t : {"q", "k", "v", "q.conv", "k.conv", "v.conv", "b", "a", "A_log", "dt_bias", "norm", "g", "o"}) n.push_back(p + "mix." + t);
+    } else {
+      for (const char* t : {"q", "uk", "uv", "o"}) n.push_back(p + "mix." + t);
+      if (sp.kv_from < 0)
+        for (const char* t : {"dkv", "dkv.norm"}) n.push_back(p + "mix." + t);
+    }
+    if (sp.ff == B2_FF_SOFTMAX_EXPERTS) {
+      n.push_back(p + "norm2");
+      n.push_back(p + "mlp.router");
+      for (int x = 0; x < sp.experts; ++x)
+        for (const char* t : {"gate", "up", "down"}) n.push_back(p + "mlp.e" + std::to_string(x) + "." + t);
+      if (sp.shared_ff > 0)
+        for (const char* t : {"gate", "up", "down", "sg"}) n.push_back(p + "mlp.shared." + t);
+    }
+  }
+  return n;
+}
+int outnorm_finalize(b2_engine* e) {
+  for (const std::string& name : outnorm_tensor_names(e)) B2_REQUIRE(e->loaded.count(name), "weights incomplete: %s missing", name.c_str());
+  return 0;
+}
+
 // Validates the layer list and allocates weights, activations and scratch of a layer-list engine.
 int list_engine_alloc(b2_engine* e) {
+  if (e->cfg.arch == B2_ARCH_TOLANEX) return outnorm_engine_alloc(e);
   if (e->cfg.arch == B2_ARCH_TINEVIK) return mixed_engine_alloc(e);
   if (e->cfg.arch == B2_ARCH_BUMALIX) return state_engine_alloc(e);
   if (e->cfg.arch == B2_ARCH_KEDASUN) return heads_engine_alloc(e);
@@ -3485,7 +3882,7 @@ extern "C" int b2_engine_create(const b2_config* cfg, const char* safetensors_pa
   B2_REQUIRE(cfg != nullptr && out != nullptr, "b2_engine_create: null argument");
   B2_REQUIRE(cfg->abi_version == B2_ABI_VERSION, "b2_engine_create: abi_version %d != %d", cfg->abi_version, B2_ABI_VERSION);
   B2_REQUIRE(cfg->arch == B2_ARCH_QWEN3 || cfg->arch == B2_ARCH_PHI3 || cfg->arch == B2_ARCH_OPT || list_arch(cfg->arch),
-             "arch %d not built (0 = Qwen3, 1 = Phi-3, 2 = OPT, 3 = Lerasun, 4 = Kedasun, 5 = Bumalix, 6 = Tinevik)", cfg->arch);
+             "arch %d not built (0 = Qwen3, 1 = Phi-3, 2 = OPT, 3 = Lerasun, 4 = Kedasun, 5 = Bumalix, 6 = Tinevik, 7 = Tolanex)", cfg->arch);
   const bool ls = list_arch(cfg->arch);  // a layer-list family: its sizes live in layer_specs and are checked in list_engine_alloc
   B2_REQUIRE(ls || !cfg->compute_f32, "compute_f32: only the layer-list families have an fp32 path");
   B2_REQUIRE(!ls || cfg->layer_specs != nullptr, "layer-list family: layer_specs is NULL");
@@ -3751,7 +4148,9 @@ extern "C" int b2_engine_create(const b2_config* cfg, const char* safetensors_pa
       size_t page_bytes_all = blk_elems * 2 * 2 * c.num_layers;
       const bool heads_cache = c.arch == B2_ARCH_KEDASUN;  // a K region and a V region per layer, rows of kv_heads * dim / kv_heads * vdim
       const bool state_arch = c.arch == B2_ARCH_BUMALIX;   // a K and a V region per RUN of a layer that has a softmax mixer
-      const bool mixed_arch = c.arch == B2_ARCH_TINEVIK;   // per RUN: a K and a V region for a softmax mixer, one region of latents for a latent mixer
+      // per RUN: a K and a V region for a softmax mixer, one region of latents for a latent mixer that stores its own (kv_from: the named run's)
+      const bool mixed_arch = c.arch == B2_ARCH_TINEVIK || c.arch == B2_ARCH_TOLANEX;
+      auto own_latent = [](const b2_layer_spec& sp) { return sp.mixer == B2_MIXER_GATED_LATENT || (sp.mixer == B2_MIXER_LATENT_ATTENTION && sp.kv_from < 0); };
       if (state_arch) {
         page_bytes_all = 0;
         for (const ListRun& R : e->runs)
@@ -3762,7 +4161,7 @@ extern "C" int b2_engine_create(const b2_config* cfg, const char* safetensors_pa
         for (const ListRun& R : e->runs) {
           const ListLayer& L = e->ll[R.layer];
           if (L.sp.mixer == B2_MIXER_MIXED_SCORE_ATTENTION) page_bytes_all += (size_t)c.block_size * (L.nk + L.nv) * e->esz;
-          else if (L.sp.mixer == B2_MIXER_GATED_LATENT) page_bytes_all += (size_t)c.block_size * L.sp.kv_rank * e->esz;
+          else if (own_latent(L.sp)) page_bytes_all += (size_t)c.block_size * L.sp.kv_rank * e->esz;
         }
         page_bytes_all = std::max<size_t>(page_bytes_all, 16);
       } else if (ls) {
@@ -3815,11 +4214,13 @@ extern "C" int b2_engine_create(const b2_config* cfg, const char* safetensors_pa
               R.v_region = (int)e->regions.size();
               e->regions.push_back({e->l_pool + off, vb});
               off += (size_t)nb * vb;
-            } else if (L.sp.mixer == B2_MIXER_GATED_LATENT) {
+            } else if (own_latent(L.sp)) {
               const size_t pb = (size_t)c.block_size * L.sp.kv_rank * e->esz;
               R.k_region = (int)e->regions.size();
               e->regions.push_back({e->l_pool + off, pb});
               off += (size_t)nb * pb;
+            } else if (L.sp.mixer == B2_MIXER_LATENT_ATTENTION) {
+              R.k_region = e->runs[L.sp.kv_from].k_region;   // (an earlier run: its region is set)
             }
           }
         }
@@ -3898,9 +4299,9 @@ extern "C" int b2_engine_load_safetensors(b2_engine* e, const char* path) {
 extern "C" int b2_engine_finalize(b2_engine* e) {
   B2_REQUIRE(e, "b2_engine_finalize: null engine");
   const int arch = e->cfg.arch;
-  if (arch == B2_ARCH_BUMALIX || arch == B2_ARCH_TINEVIK) {
+  if (arch == B2_ARCH_BUMALIX || arch == B2_ARCH_TINEVIK || arch == B2_ARCH_TOLANEX) {
     B2_CUDA_OK(cudaSetDevice(e->device));
-    B2_TRY(arch == B2_ARCH_BUMALIX ? state_finalize(e) : mixed_finalize(e));
+    B2_TRY(arch == B2_ARCH_BUMALIX ? state_finalize(e) : arch == B2_ARCH_TINEVIK ? mixed_finalize(e) : outnorm_finalize(e));
     e->finalized = true;
     return 0;
   }
@@ -3955,7 +4356,7 @@ extern "C" void b2_engine_free(b2_engine* e) {
   if (e->ev_tok) cudaEventDestroy(e->ev_tok);
   F(e->partial2); F(e->attn_scratch2); F(e->ssq);
   if (e->l_head == e->l_embed) e->l_head = nullptr;   // (a tied head is the embedding table)
-  F(e->l_final_bias);
+  F(e->l_final_bias); F(e->l_bigram); F(e->l_pos); F(e->l_tok_ring); F(e->l_sg);
   F(e->l_embed); F(e->l_head); F(e->l_embed_gain); F(e->l_final_gain); F(e->l_pool); F(e->l_h); F(e->l_qd); F(e->l_qrot); F(e->l_qabs);
   F(e->l_xperm); F(e->l_upf); if (e->h_offsets) cudaFreeHost(e->h_offsets);
   F(e->l_q); F(e->l_vfirst); F(e->l_cross); F(e->l_qb); F(e->d_row_seq); F(e->d_row_first); F(e->d_row_end);
@@ -3994,6 +4395,8 @@ extern "C" int b2_seq_create(b2_engine* e, int32_t reserve_tokens, int32_t* seq_
   B2_REQUIRE(e && seq_id, "b2_seq_create: null argument");
   B2_REQUIRE(reserve_tokens >= 1 && reserve_tokens <= e->cfg.max_model_len, "reserve_tokens %d outside [1, max_model_len=%d]",
              reserve_tokens, e->cfg.max_model_len);
+  B2_REQUIRE(e->l_pos == nullptr || reserve_tokens <= e->cfg.max_positions, "reserve_tokens %d: the model's position table has %d rows", reserve_tokens,
+             e->cfg.max_positions);
   const int bs = e->cfg.block_size;
   const int need = (reserve_tokens + bs - 1) / bs;
   if (pages_available(e) < need) {
@@ -4029,6 +4432,8 @@ extern "C" int b2_seq_reserve(b2_engine* e, int32_t seq_id, int32_t total_tokens
   Seq& s = e->seqs[seq_id];
   B2_REQUIRE(total_tokens >= 1 && total_tokens <= e->cfg.max_model_len, "total_tokens %d outside [1, max_model_len=%d]", total_tokens,
              e->cfg.max_model_len);
+  B2_REQUIRE(e->l_pos == nullptr || total_tokens <= e->cfg.max_positions, "total_tokens %d: the model's position table has %d rows", total_tokens,
+             e->cfg.max_positions);
   const int bs = e->cfg.block_size;
   const int need = (total_tokens + bs - 1) / bs - (int)s.blocks.size();
   if (need <= 0) return 0;

@@ -287,6 +287,23 @@ int launch_layer_norm(const float* h, const float* w, const float* b, void* x, i
 // token's routed rows, y[t] = coef * sum_k y[pair_slot[t * top + k]].  With w_next the norm in front of the next sublayer as well.
 int launch_layer_norm_add(float* h, const float* y, const int32_t* pair_slot, int top, float coef, const float* w, const float* b, int T, int W, float eps,
                           cudaStream_t s, const float* w_next = nullptr, const float* b_next = nullptr, void* x_next = nullptr, int x_f32 = 0);
+// Families that norm only the sublayers' OUTPUTS (the sublayers read the stream itself):
+// h[t] = embed[ids[t]] + bigram[row] + pos_table[positions[t]], row = (previous token * mul_prev + token * mul_cur) mod buckets, or `buckets` for a
+// sequence's first token; x = h in the operand type.  The previous token of a portion's first row comes from tok_ring [sequence slots][2]
+// (entry = position mod 2), which the same launch updates with the portion's last token.  Tables fp32 or bf16 like x.
+struct BigramTable {
+  const void* table;       // [buckets + 1][W]
+  int buckets;
+  long long mul_prev, mul_cur;
+  int32_t* tok_ring;       // [sequence slots][2]
+};
+int launch_embed_sum(const int32_t* ids, const void* table, const BigramTable& bg, const void* pos_table, int pos_rows, int table_f32, float* h, void* x,
+                     int T, int W, int vocab, const int32_t* row_seq, const int32_t* row_first, const int32_t* row_end, const int32_t* positions,
+                     const int32_t* slots, cudaStream_t s);
+// h[t] += mult * rms(v) * gain, v = a_scale[t] * a[t] + sum_k weight[t][k] * y[pair_slot[t * top + k]] (a, a_scale and y may be null; weights are
+// taken in choice order); x_next = h in the operand type (null = not wanted)
+int launch_out_norm_add(float* h, const float* a, const float* a_scale, const float* y, const float* weight, const int32_t* pair_slot, int top,
+                        const float* gain, float mult, int T, int W, float eps, cudaStream_t s, void* x_next, int x_f32);
 // act[i] = softplus(p) z^2 + z / 2 for z > 0, (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 otherwise; pq (device) = p, q
 int launch_xielu(const float* z, const float* pq, void* act, int act_f32, size_t n, cudaStream_t s);
 // out[t][i] = a[t][i] * sigmoid(gate[t * gate_ld + i]), out fp32 or bf16 [T][N]
@@ -352,7 +369,11 @@ int launch_talk_gate(const float* cross, const float* talk, const float* gate, i
                      int vdim, int T, cudaStream_t s);
 
 // ---- attn_state.cu: mixers with a matrix state per head (gated linear attention, gated delta rule) ----
-enum StateRule { STATE_RULE_DECAY = 0, STATE_RULE_DELTA = 1 };
+enum StateRule {
+  STATE_RULE_DECAY = 0,
+  STATE_RULE_DELTA = 1,
+  STATE_RULE_DELTA_HEAD = 2         // the delta rule with one decay per head: `decay` is [T][heads]
+};
 struct StateGeom {
   int heads, kv_heads, dim, vdim;   // state head a reads query/key head a / (heads / kv_heads); S is [dim][vdim] per head
   int rule;                         // StateRule
@@ -368,12 +389,14 @@ int launch_lowrank_act(const float* lr, int ld, int lr_off, int rank, const floa
 // Delta rule, behind the fused projection proj [T][ld] fp32 = q (kv_heads*dim) | k (kv_heads*dim) | v (heads*vdim) | beta logits (heads) | ...:
 // causal convolution over time (conv_w [channels][taps], last column = the current token; ring [slots][taps][channels], row = position mod
 // taps) and silu on every channel, q and k heads to unit vectors x / sqrt(sum x^2 + unit_eps), q times dim^-1/2; out [T][channels], beta_out
-// [T][heads] = sigmoid.  Updates the ring.
+// [T][heads] = sigmoid.  With a_log the decay of a head follows from the logits behind beta's, decay_out [T][heads] =
+// exp(-exp(a_log) * softplus(logit + dt_bias)).  Updates the ring.
 int launch_conv_unit_finish(const float* proj, int ld, const StateGeom& g, int taps, const float* conv_w, float* ring, const int32_t* row_seq,
                             const int32_t* row_first, const int32_t* row_end, const int32_t* positions, const int32_t* slots, float unit_eps,
-                            float* out, float* beta_out, int T, cudaStream_t s);
+                            float* out, float* beta_out, int T, cudaStream_t s, const float* a_log = nullptr, const float* dt_bias = nullptr,
+                            float* decay_out = nullptr);
 // The recurrence over every portion of the step: portion i ends at row last_rows[i] (null: row i is a portion of one token); q / k rows of
-// kv_heads*dim at strides ldq / ldk, v rows of heads*vdim at stride ldv, decay [T][heads*dim], beta [T][heads] (delta rule); q is multiplied
+// kv_heads*dim at strides ldq / ldk, v rows of heads*vdim at stride ldv, decay [T][heads*dim] ([T][heads] with STATE_RULE_DELTA_HEAD), beta [T][heads] (delta rule); q is multiplied
 // by qscale.  state [slots][2][heads][dim][vdim] fp32 (state_floats_per_slot); out [T][heads*vdim] fp32.  Rows whose slot is negative are skipped.
 int launch_state_scan(const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* decay, const float* beta,
                       const StateGeom& g, float qscale, float* state, int portions, const int32_t* last_rows, const int32_t* row_seq,
@@ -412,14 +435,18 @@ int launch_latent_attention(const float* q_abs, const float* q_rot, const void* 
 // unsplit.  max_context: longest cache the engine can hold (bounds the number of splits).
 size_t latent_attention_scratch_floats(int max_rows, int max_heads, int max_rank);
 
-// ---- moe_route.cu: sigmoid router with a choice offset and grouped selection, and the token permutation by expert ----
+// ---- moe_route.cu: sigmoid or softmax router with a choice offset and grouped selection, and the token permutation by expert ----
 struct RouteGeom {
   int experts, top, groups, keep;
   int raw_weights;   // 1: the weights are the chosen experts' scores as they are; 0: divided by their sum
+  int softmax;       // 1: scores are a softmax over all experts; 0: a sigmoid per expert
+  int group_best;    // 1: a group's score is its best choice score; 0: the sum of its two best
+  float scale;       // raw_weights: the weights are multiplied by this (0 = 1)
 };
-// x [T][W] (operand type), router [experts][W] fp32, correction [experts] fp32 (null = none) -> idx [T][top], weight [T][top]
+// x [T][W] (operand type), router [experts][W] fp32, correction [experts] fp32 (null = none) -> idx [T][top], weight [T][top].
+// gate_out != null: the router has one more row, and gate_out [T] = sigmoid of its product with x
 int launch_route(const void* x, int x_f32, const float* router, const float* correction, const RouteGeom& g, int32_t* idx, float* weight,
-                 int T, int W, cudaStream_t s);
+                 int T, int W, cudaStream_t s, float* gate_out = nullptr);
 // no router: idx[t][k] = table[ids[t]][k] (table [vocab][top] int32, entries clamped into [0, experts)), weight[t][k] = 1 / top
 int launch_route_table(const int32_t* ids, const int32_t* table, int vocab, int experts, int top, int32_t* idx, float* weight, int T, cudaStream_t s);
 // counting sort of the T*top (token, choice) pairs by expert: offsets [experts + 1] (the buffer holds 3 * stride ints,

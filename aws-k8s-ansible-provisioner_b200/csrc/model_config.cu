@@ -2,7 +2,7 @@
 // one).  b2serve, the Python mirror and bin/trace_run all choose the model class through this one function, so a family
 // is added to the framework here, in b2_engine_create and nowhere else.  Host code only.
 //
-// The fourth layer-list family, Tinevik, is described above its reader (tinevik_config).
+// The fourth and fifth layer-list families, Tinevik and Tolanex, are described above their readers (tinevik_config, tolanex_config).
 // HF families are told apart by "model_type" (the keys follow HF's Qwen3Config / Phi3Config / OPTConfig); Lerasun by
 // "architecture": "Lerasun", whose config lists its layers one by one:
 //   {"architecture": "Lerasun", "vocab": V, "width": W, "logit_scale": s, "norm": {"eps": e},
@@ -499,6 +499,132 @@ int tinevik_config(const Value& j, b2_config* c, b2_layer_spec* specs, int max_s
   return 0;
 }
 
+// Tolanex: {"architecture": "Tolanex", "vocab": V, "width": W, "max_positions": P, "norm": {"eps": e}, "residual_mult": m?,
+//   "embedding": {"bigram": {"buckets", "mul_prev", "mul_cur"}},
+//   "layers": [{"type": "delta", "mixer": {"heads", "kv_heads"?, "dim", "vdim", "conv"}, "mlp": ...},
+//              {"type": "latent_attention", "mixer": {"heads", "dim", "vdim", "kv_rank", "scale", "kv_from"?},
+//               "mlp": null | {"kind": "moe", "expert": {"ff"}, "router": {"experts", "top", "groups": {"count", "keep"}?, "scale"?},
+//                              "shared": {"ff"}?}}, ...]}
+int need_i64(const Value& o, const char* key, const char* where, int64_t* out) {
+  const Value* v = o.find(key);
+  if (!v || !v->is_number()) {
+    b2_set_error("config.json: %s.%s missing or not a number", where, key);
+    return -22;
+  }
+  *out = (int64_t)v->as_int();
+  return 0;
+}
+int tolanex_config(const Value& j, b2_config* c, b2_layer_spec* specs, int max_specs) {
+  c->arch = B2_ARCH_TOLANEX;
+  CFG_TRY(need_int(j, "vocab", "config", &c->vocab));
+  CFG_TRY(need_int(j, "width", "config", &c->hidden));
+  CFG_TRY(need_int(j, "max_positions", "config", &c->max_positions));
+  const Value* norm = j.find("norm");
+  if (!norm || !norm->is_object()) {
+    b2_set_error("config.json: norm missing");
+    return -22;
+  }
+  CFG_TRY(need_float(*norm, "eps", "norm", &c->rms_eps));
+  c->norm_groups = 1;
+  c->norm_kind = 2;
+  c->embed_scale = 1.0f;
+  c->logit_scale = 1.0f;
+  c->residual_mult = 1.0f;
+  if (const Value* rm = j.find("residual_mult"))
+    if (rm->is_number()) c->residual_mult = (float)rm->as_double();
+  const Value* em = j.find("embedding");
+  const Value* bg = em && em->is_object() ? em->find("bigram") : nullptr;
+  if (!bg || !bg->is_object()) {
+    b2_set_error("config.json: embedding.bigram missing");
+    return -22;
+  }
+  CFG_TRY(need_int(*bg, "buckets", "embedding.bigram", &c->bigram_buckets));
+  CFG_TRY(need_i64(*bg, "mul_prev", "embedding.bigram", &c->bigram_mul_prev));
+  CFG_TRY(need_i64(*bg, "mul_cur", "embedding.bigram", &c->bigram_mul_cur));
+  const Value* layers = j.find("layers");
+  if (!layers || !layers->is_array() || layers->size() == 0) {
+    b2_set_error("config.json: layers missing or empty");
+    return -22;
+  }
+  c->num_layers = (int)layers->size();
+  if (c->num_layers > max_specs || specs == nullptr) {
+    b2_set_error("config.json: %d layers, room for %d layer specs", c->num_layers, max_specs);
+    return -22;
+  }
+  for (int i = 0; i < c->num_layers; ++i) {
+    const Value& L = layers->at(i);
+    b2_layer_spec& s = specs[i];
+    memset(&s, 0, sizeof s);
+    s.kv_from = -1;
+    s.weights_of = -1;
+    char where[64];
+    snprintf(where, sizeof where, "layers[%d].mixer", i);
+    const Value* type = L.find("type");
+    const Value* m = L.find("mixer");
+    if (!type || !type->is_string() || !m || !m->is_object()) {
+      b2_set_error("config.json: layers[%d] needs type and mixer", i);
+      return -22;
+    }
+    const std::string ty = type->as_string();
+    CFG_TRY(need_int(*m, "heads", where, &s.heads));
+    s.kv_heads = s.heads;
+    CFG_TRY(need_int(*m, "dim", where, &s.dim));
+    CFG_TRY(need_int(*m, "vdim", where, &s.vdim));
+    if (ty == "delta") {
+      s.mixer = B2_MIXER_HEAD_DELTA;
+      if (const Value* kh = m->find("kv_heads"))
+        if (kh->is_number()) s.kv_heads = (int)kh->as_int();
+      CFG_TRY(need_int(*m, "conv", where, &s.conv_taps));
+    } else if (ty == "latent_attention") {
+      s.mixer = B2_MIXER_LATENT_ATTENTION;
+      CFG_TRY(need_int(*m, "kv_rank", where, &s.kv_rank));
+      CFG_TRY(need_float(*m, "scale", where, &s.scale));
+      if (const Value* kf = m->find("kv_from"))
+        if (kf->is_number()) s.kv_from = (int)kf->as_int();
+    } else {
+      b2_set_error("config.json: layers[%d]: mixer type '%s' not built (delta, latent_attention)", i, ty.c_str());
+      return -22;
+    }
+    const Value* mlp = L.find("mlp");
+    s.ff = B2_FF_NONE;
+    if (mlp && mlp->is_object()) {
+      snprintf(where, sizeof where, "layers[%d].mlp", i);
+      const Value* kind = mlp->find("kind");
+      const std::string kd = kind && kind->is_string() ? kind->as_string() : "?";
+      if (kd != "moe") {
+        b2_set_error("config.json: %s.kind '%s' not built (moe)", where, kd.c_str());
+        return -22;
+      }
+      s.ff = B2_FF_SOFTMAX_EXPERTS;
+      const Value* ex = mlp->find("expert");
+      const Value* ro = mlp->find("router");
+      if (!ex || !ex->is_object() || !ro || !ro->is_object()) {
+        b2_set_error("config.json: %s needs expert and router", where);
+        return -22;
+      }
+      CFG_TRY(need_int(*ex, "ff", where, &s.ff_dim));
+      CFG_TRY(need_int(*ro, "experts", where, &s.experts));
+      CFG_TRY(need_int(*ro, "top", where, &s.top));
+      s.groups = s.groups_keep = 1;
+      if (const Value* gr = ro->find("groups"))
+        if (gr->is_object()) {
+          CFG_TRY(need_int(*gr, "count", where, &s.groups));
+          CFG_TRY(need_int(*gr, "keep", where, &s.groups_keep));
+        }
+      s.router_scale = 1.0f;
+      if (const Value* sc = ro->find("scale"))
+        if (sc->is_number()) s.router_scale = (float)sc->as_double();
+      if (const Value* sh = mlp->find("shared"))
+        if (sh->is_object()) CFG_TRY(need_int(*sh, "ff", where, &s.shared_ff));
+    }
+  }
+  c->layer_specs = specs;
+  c->tie_embeddings = 0;
+  c->num_q_heads = c->num_kv_heads = 0;
+  c->head_dim = c->intermediate = 0;
+  return 0;
+}
+
 }  // namespace
 
 extern "C" int b2_config_from_dir(const char* model_dir, b2_config* c, b2_layer_spec* specs, int32_t max_specs) {
@@ -526,12 +652,16 @@ extern "C" int b2_config_from_dir(const char* model_dir, b2_config* c, b2_layer_
   c->loop_start = c->loop_stop = c->loop_times = 0;
   c->logit_softcap = 0.f;
   c->norm_kind = 0;
+  c->residual_mult = 0.f;
+  c->bigram_buckets = 0;
+  c->bigram_mul_prev = c->bigram_mul_cur = 0;
   const Value* archv = j.find("architecture");
   if (archv && archv->is_string()) {
     if (archv->as_string() == "Lerasun") return lerasun_config(j, c, specs, max_specs);
     if (archv->as_string() == "Kedasun") return kedasun_config(j, c, specs, max_specs);
     if (archv->as_string() == "Bumalix") return bumalix_config(j, c, specs, max_specs);
     if (archv->as_string() == "Tinevik") return tinevik_config(j, c, specs, max_specs);
+    if (archv->as_string() == "Tolanex") return tolanex_config(j, c, specs, max_specs);
     b2_set_error("%s: architecture '%s' not built", path.c_str(), archv->as_string().c_str());
     return -22;
   }

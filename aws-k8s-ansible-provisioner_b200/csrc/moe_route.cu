@@ -1,11 +1,12 @@
 // moe_route.cu -- the router of a routed-experts feed-forward, and the bookkeeping that turns its choices into ragged
 // groups for gemm_any.cu.
 //
-// Router (all fp32): z = R x, s = sigmoid(z).  The CHOICE uses s + correction (a per-expert offset that steers load and
-// may make a choice score negative); the mixing WEIGHTS use s alone.  Experts are `groups` equal runs of neighbours; a
-// group's score is the sum of its two best choice scores and only the `keep` best groups may supply experts (the others
-// are out, not zero).  Of the allowed experts the `top` with the best choice scores are taken; their s, divided by their
-// sum (+ 1e-20), are the weights.  Ties go to the lower index.
+// Router (all fp32): z = R x, s = sigmoid(z) or a softmax of z over all experts (RouteGeom.softmax).  The CHOICE uses s + correction (an
+// optional per-expert offset that steers load and may make a choice score negative); the mixing WEIGHTS use s alone.  Experts are
+// `groups` equal runs of neighbours; a group's score is the sum of its two best choice scores (or its best one, group_best) and only the
+// `keep` best groups may supply experts (the others are out, not zero).  Of the allowed experts the `top` with the best choice scores
+// are taken; their s, divided by their sum (+ 1e-20) or as they are times a constant (raw_weights, scale), are the weights.  Ties go to
+// the lower index.  A router matrix may carry one more row, whose sigmoid gates a shared expert.
 //
 // route_permute is a counting sort of the (token, choice) pairs by expert: slots of expert e are [offsets[e], offsets[e+1]).
 // Which slot of its expert a pair gets depends on the order of atomic arrivals, and that is harmless: gemm_any.cu sums every
@@ -20,88 +21,125 @@ namespace {
 
 constexpr int RT_WARPS = 16;
 
-// one CTA per token: the row is staged once as fp32, warp w takes experts w, w + 16, ...; thread 0 then selects
-template <typename TX>
+// A CTA takes NTOK tokens: their rows are staged once as fp32, warp w takes router rows w, w + 16, ... (a row is read once for all tokens of
+// the CTA), then one warp per token forms the scores and selects.  A token's arithmetic does not depend on NTOK.
+template <typename TX, int NTOK>
 __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const TX* __restrict__ x, const float* __restrict__ router,
                                                               const float* __restrict__ correction, RouteGeom g, int32_t* __restrict__ idx,
-                                                              float* __restrict__ weight, int T, int W) {
-  extern __shared__ __align__(16) float sm[];  // x row [W rounded up to 4] (read as float4), s [E], choice [E]
+                                                              float* __restrict__ weight, int T, int W, float* __restrict__ gate_out) {
+  extern __shared__ __align__(16) float sm[];  // x rows [NTOK][W rounded up to 4] (read as float4), then per token: s [E + 1], choice [E], group scores [groups]
   pdl_wait();
   pdl_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t = blockIdx.x;
-  const int E = g.experts;
+  const int t0 = blockIdx.x * NTOK, tn = min(NTOK, T - t0);
+  const int E = g.experts, ER = E + (gate_out != nullptr ? 1 : 0), Wp = (W + 3) & ~3, per_tok = 2 * E + 1 + g.groups;
   float* xs = sm;
-  float* s = xs + ((W + 3) & ~3);
-  float* ch = s + E;
-  const TX* xr = x + (size_t)t * W;
-  for (int i = threadIdx.x; i < W; i += RT_WARPS * 32) xs[i] = (float)xr[i];
+  float* sc = xs + NTOK * Wp;
+  for (int i = threadIdx.x; i < NTOK * W; i += RT_WARPS * 32) {
+    const int tt = i / W, c = i - tt * W;
+    xs[tt * Wp + c] = tt < tn ? (float)x[(size_t)(t0 + tt) * W + c] : 0.f;
+  }
   __syncthreads();
   const bool vec = (W % 4 == 0);
-  for (int e = warp; e < E; e += RT_WARPS) {
+  for (int e = warp; e < ER; e += RT_WARPS) {
     const float* rr = router + (size_t)e * W;
-    float acc = 0.f;
+    float acc[NTOK];
+#pragma unroll
+    for (int tt = 0; tt < NTOK; ++tt) acc[tt] = 0.f;
     if (vec) {
 #pragma unroll 8
       for (int i = lane * 4; i < W; i += 128) {
         const float4 r4 = *reinterpret_cast<const float4*>(rr + i);
-        const float4 x4 = *reinterpret_cast<const float4*>(xs + i);
-        acc = fmaf(x4.x, r4.x, acc); acc = fmaf(x4.y, r4.y, acc); acc = fmaf(x4.z, r4.z, acc); acc = fmaf(x4.w, r4.w, acc);
+#pragma unroll
+        for (int tt = 0; tt < NTOK; ++tt) {
+          const float4 x4 = *reinterpret_cast<const float4*>(xs + tt * Wp + i);
+          acc[tt] = fmaf(x4.x, r4.x, acc[tt]); acc[tt] = fmaf(x4.y, r4.y, acc[tt]); acc[tt] = fmaf(x4.z, r4.z, acc[tt]); acc[tt] = fmaf(x4.w, r4.w, acc[tt]);
+        }
       }
     } else {
-      for (int i = lane; i < W; i += 32) acc = fmaf(xs[i], rr[i], acc);
+      for (int i = lane; i < W; i += 32) {
+        const float r = rr[i];
+#pragma unroll
+        for (int tt = 0; tt < NTOK; ++tt) acc[tt] = fmaf(xs[tt * Wp + i], r, acc[tt]);
+      }
     }
-    acc = warp_sum(acc);
-    if (lane == 0) {
-      const float sg = 1.0f / (1.0f + expf(-acc));
-      s[e] = sg;
-      ch[e] = sg + (correction ? correction[e] : 0.f);
+#pragma unroll
+    for (int tt = 0; tt < NTOK; ++tt) {
+      const float z = warp_sum(acc[tt]);
+      if (lane == 0) sc[tt * per_tok + e] = (g.softmax && e < E) ? z : 1.0f / (1.0f + expf(-z));   // (the extra row is a gate: always a sigmoid)
     }
   }
   __syncthreads();
-  if (threadIdx.x != 0) return;
-  // groups: score = sum of the two best choice scores; all but the `keep` best are out (choice = -inf).  Ranks are formed
-  // from the untouched scores first (a 64-bit mask remembers who is out), then applied.
+  if (warp >= tn) return;
+  const int t = t0 + warp;
+  float* s = sc + warp * per_tok;
+  float* ch = s + E + 1;
+  float* gs = ch + E;
+  if (gate_out != nullptr && lane == 0) gate_out[t] = s[E];
+  if (g.softmax) {
+    float m = -INFINITY, sum = 0.f;
+    for (int e = lane; e < E; e += 32) m = fmaxf(m, s[e]);
+    m = warp_max(m);
+    for (int e = lane; e < E; e += 32) {
+      const float p = expf(s[e] - m);
+      s[e] = p;
+      sum += p;
+    }
+    const float inv = 1.0f / warp_sum(sum);
+    for (int e = lane; e < E; e += 32) s[e] *= inv;   // (a lane's own entries)
+  }
+  for (int e = lane; e < E; e += 32) ch[e] = s[e] + (correction ? correction[e] : 0.f);
+  __syncwarp();
+  // groups: all but the `keep` best are out (choice = -inf).  Ranks are formed from the untouched scores first, then applied.
   const int per = E / g.groups;
   if (g.keep < g.groups) {
-    auto group_score = [&](int gi) {
+    for (int gi = lane; gi < g.groups; gi += 32) {
       float b1 = -INFINITY, b2 = -INFINITY;
       for (int e = gi * per; e < (gi + 1) * per; ++e) {
         const float v = ch[e];
         if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) { b2 = v; }
       }
-      return per >= 2 ? b1 + b2 : b1;
-    };
-    unsigned long long out_mask = 0ull;
-    for (int gi = 0; gi < g.groups; ++gi) {
-      const float my = group_score(gi);
+      gs[gi] = (per >= 2 && !g.group_best) ? b1 + b2 : b1;
+    }
+    __syncwarp();
+    for (int gi = lane; gi < g.groups; gi += 32) {
       int beat = 0;  // groups ranked ahead of gi (lower index wins a tie)
       for (int gj = 0; gj < g.groups; ++gj) {
         if (gj == gi) continue;
-        const float other = group_score(gj);
-        if (other > my || (other == my && gj < gi)) ++beat;
+        if (gs[gj] > gs[gi] || (gs[gj] == gs[gi] && gj < gi)) ++beat;
       }
-      if (beat >= g.keep) out_mask |= 1ull << gi;
-    }
-    for (int gi = 0; gi < g.groups; ++gi)
-      if ((out_mask >> gi) & 1ull)
+      if (beat >= g.keep)
         for (int e = gi * per; e < (gi + 1) * per; ++e) ch[e] = -INFINITY;
+    }
+    __syncwarp();
   }
   float sum = 0.f;
+  const float scale = g.scale != 0.f ? g.scale : 1.0f;
   for (int k = 0; k < g.top; ++k) {
-    int best = -1;
-    float bv = -INFINITY;
-    for (int e = 0; e < E; ++e)
-      if (ch[e] > bv) { best = e; bv = ch[e]; }   // -inf = out or already taken; first index wins a tie
-    if (best < 0) best = k < E ? k : 0;  // only for rows that hold no numbers (padding rows of a graph bucket): keep the index valid
-    idx[(size_t)t * g.top + k] = best;
-    weight[(size_t)t * g.top + k] = s[best];
-    sum += s[best];
-    ch[best] = -INFINITY;
+    float bv = -INFINITY;   // -inf = out or already taken
+    int best = 0x7fffffff;
+    for (int e = lane; e < E; e += 32)
+      if (ch[e] > bv) { best = e; bv = ch[e]; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {   // the first index wins a tie
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, best, o);
+      if (ov > bv || (ov == bv && oi < best)) { bv = ov; best = oi; }
+    }
+    if (best >= E) best = k < E ? k : 0;  // only for rows that hold no numbers (padding rows of a graph bucket): keep the index valid
+    const float w = s[best];
+    if (lane == 0) {
+      idx[(size_t)t * g.top + k] = best;
+      weight[(size_t)t * g.top + k] = g.raw_weights ? w * scale : w;
+      ch[best] = -INFINITY;
+    }
+    sum += w;
+    __syncwarp();
   }
-  if (g.raw_weights) return;   // the scores as they are
+  if (g.raw_weights) return;   // the scores as they are (times the scale)
   const float inv = 1.0f / (sum + 1e-20f);
-  for (int k = 0; k < g.top; ++k) weight[(size_t)t * g.top + k] *= inv;
+  if (lane == 0)
+    for (int k = 0; k < g.top; ++k) weight[(size_t)t * g.top + k] *= inv;
 }
 
 // the permutation in three steps: histogram (any number of CTAs), scan (one thread; experts are few), placement
@@ -262,19 +300,28 @@ int launch_relu2_round(const float* up, bf16* act, size_t n, cudaStream_t s) {
 }
 
 int launch_route(const void* x, int x_f32, const float* router, const float* correction, const RouteGeom& g, int32_t* idx, float* weight,
-                 int T, int W, cudaStream_t s) {
+                 int T, int W, cudaStream_t s, float* gate_out) {
   if (T <= 0) return 0;
   B2_REQUIRE(g.experts >= 1 && g.groups >= 1 && g.groups <= 64 && g.experts % g.groups == 0, "route: %d experts do not form %d equal groups", g.experts, g.groups);
   B2_REQUIRE(g.keep >= 1 && g.keep <= g.groups, "route: keep %d outside [1, %d]", g.keep, g.groups);
   B2_REQUIRE(g.top >= 1 && g.top <= g.keep * (g.experts / g.groups), "route: top %d exceeds the %d experts of the kept groups", g.top,
              g.keep * (g.experts / g.groups));
-  const size_t smem = ((size_t)2 * g.experts + ((W + 3) & ~3)) * sizeof(float);
-  B2_REQUIRE(smem <= 48 * 1024, "route: %d experts and width %d need %zu bytes of shared memory", g.experts, W, smem);
-  const dim3 grid(T);
-  if (x_f32)
-    B2_CUDA_OK(b2_launch(route_kernel<float>, grid, dim3(RT_WARPS * 32), smem, s, (const float*)x, router, correction, g, idx, weight, T, W));
-  else
-    B2_CUDA_OK(b2_launch(route_kernel<bf16>, grid, dim3(RT_WARPS * 32), smem, s, (const bf16*)x, router, correction, g, idx, weight, T, W));
+  auto bytes = [&](int ntok) { return (size_t)ntok * (2 * g.experts + 1 + g.groups + ((W + 3) & ~3)) * sizeof(float); };
+  B2_REQUIRE(bytes(1) <= 48 * 1024, "route: %d experts and width %d need %zu bytes of shared memory", g.experts, W, bytes(1));
+  // prompt-sized steps: several tokens per CTA share one pass over the router's rows
+  const int ntok = T >= 1024 && bytes(4) <= 48 * 1024 ? 4 : T >= 512 && bytes(2) <= 48 * 1024 ? 2 : 1;
+  const dim3 grid((T + ntok - 1) / ntok);
+#define B2_ROUTE(TX, N) B2_CUDA_OK(b2_launch(route_kernel<TX, N>, grid, dim3(RT_WARPS * 32), bytes(N), s, (const TX*)x, router, correction, g, idx, weight, T, W, gate_out))
+  if (x_f32) {
+    if (ntok == 4) B2_ROUTE(float, 4);
+    else if (ntok == 2) B2_ROUTE(float, 2);
+    else B2_ROUTE(float, 1);
+  } else {
+    if (ntok == 4) B2_ROUTE(bf16, 4);
+    else if (ntok == 2) B2_ROUTE(bf16, 2);
+    else B2_ROUTE(bf16, 1);
+  }
+#undef B2_ROUTE
   return 0;
 }
 

@@ -463,6 +463,187 @@ __global__ void __launch_bounds__(256) sigmoid_gate_kernel(const float* __restri
     out[(size_t)t * N + i] = (TX)(a[(size_t)t * N + i] / (1.0f + expf(-gate[(size_t)t * gate_ld + i])));
 }
 
+// ---- sublayers that read the stream itself; only their outputs are normed (Tolanex) ----
+// One CTA of 128 threads per token row.  Thread 0 finds the previous token (the row above, or the sequence's ring when the portion starts
+// here) and, in the portion's first row, leaves the portion's last token in the ring: read and write sit in one thread, so a portion
+// whose last token lands on the entry that its first row reads is safe.
+template <typename TX>
+__global__ void __launch_bounds__(128) embed_sum_kernel(const int32_t* __restrict__ ids, const TX* __restrict__ table, const TX* __restrict__ bigram,
+                                                        int buckets, long long mul_prev, long long mul_cur, int32_t* __restrict__ tok_ring,
+                                                        const TX* __restrict__ pos_table, int pos_rows, float* __restrict__ h, TX* __restrict__ x, int W,
+                                                        int vocab, const int32_t* __restrict__ row_seq, const int32_t* __restrict__ row_first,
+                                                        const int32_t* __restrict__ row_end, const int32_t* __restrict__ positions,
+                                                        const int32_t* __restrict__ slots) {
+  __shared__ int bg_row;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  const int pos = positions[t];
+  int id = ids[t];
+  id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+  if (threadIdx.x == 0) {
+    long long row = buckets;
+    const int first = row_first[t];
+    int32_t* ring = tok_ring + (size_t)row_seq[t] * 2;
+    if (slots[t] >= 0) {                       // (padding rows of a decode bucket touch nothing)
+      if (pos > 0) {
+        const long long prev = t > first ? ids[t - 1] : ring[(pos - 1) & 1];
+        row = (prev * mul_prev + (long long)id * mul_cur) % buckets;
+        if (row < 0) row += buckets;
+      }
+      if (t == first) {
+        const int last = row_end[t] - 1;
+        ring[(pos + (last - t)) & 1] = ids[last];
+      }
+    }
+    bg_row = (int)row;
+  }
+  __syncthreads();
+  const TX* er = table + (size_t)id * W;
+  const TX* br = bigram + (size_t)bg_row * W;
+  const TX* pr = pos_table + (size_t)(pos < 0 ? 0 : (pos >= pos_rows ? pos_rows - 1 : pos)) * W;
+  for (int i = threadIdx.x; i < W; i += 128) {
+    const float v = ((float)er[i] + (float)br[i]) + (float)pr[i];
+    h[(size_t)t * W + i] = v;
+    x[(size_t)t * W + i] = (TX)v;
+  }
+}
+
+// h[t] += mult * rms(v) * gain with v = a_scale[t] * a[t] + sum_k weight_k y[slot_k]; x_next[t] = h[t] in the operand type.  One CTA of NT
+// threads per row; a thread keeps R groups of four neighbouring numbers in registers (W <= 4 NT R, W a multiple of 4), every load of the row
+// in flight before the one reduction.
+constexpr int ON_MAX_TOP = 16;
+template <typename TX, int NT, int R>
+__global__ void __launch_bounds__(NT) out_norm_add_kernel(float* __restrict__ h, const float* __restrict__ a, const float* __restrict__ a_scale,
+                                                          const float* __restrict__ y, const float* __restrict__ weight,
+                                                          const int32_t* __restrict__ pair_slot, int top, const float* __restrict__ gain, float mult,
+                                                          int W, float eps, TX* __restrict__ x_next) {
+  __shared__ float red[NT / 32];
+  __shared__ float w_s[ON_MAX_TOP];
+  __shared__ int slot_s[ON_MAX_TOP];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, W4 = W >> 2;
+  const float as = a_scale ? a_scale[t] : 1.0f;
+  if (y != nullptr) {
+    if ((int)threadIdx.x < top) {
+      w_s[threadIdx.x] = weight[(size_t)t * top + threadIdx.x];
+      slot_s[threadIdx.x] = pair_slot[(size_t)t * top + threadIdx.x];
+    }
+    __syncthreads();
+  }
+  float4* hr = reinterpret_cast<float4*>(h + (size_t)t * W);
+  const float4* ar = a ? reinterpret_cast<const float4*>(a + (size_t)t * W) : nullptr;
+  const float4* gr = reinterpret_cast<const float4*>(gain);
+  float4 v[R], hv[R], gv[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int i = threadIdx.x + r * NT;
+    const bool in = i < W4;
+    hv[r] = in ? hr[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    gv[r] = in ? gr[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    v[r] = (in && ar) ? ar[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    v[r].x *= as; v[r].y *= as; v[r].z *= as; v[r].w *= as;
+  }
+  if (y != nullptr)
+    for (int k = 0; k < top; ++k) {   // choice order
+      const float w = w_s[k];
+      const float4* yr = reinterpret_cast<const float4*>(y + (size_t)slot_s[k] * W);
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        const int i = threadIdx.x + r * NT;
+        if (i < W4) {
+          const float4 q = yr[i];
+          v[r].x = fmaf(w, q.x, v[r].x); v[r].y = fmaf(w, q.y, v[r].y); v[r].z = fmaf(w, q.z, v[r].z); v[r].w = fmaf(w, q.w, v[r].w);
+        }
+      }
+    }
+  float ss = 0.f;
+#pragma unroll
+  for (int r = 0; r < R; ++r) ss += (v[r].x * v[r].x + v[r].y * v[r].y) + (v[r].z * v[r].z + v[r].w * v[r].w);
+  const float rn = mult / sqrtf(block_sum_n<NT>(ss, red) / (float)W + eps);
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int i = threadIdx.x + r * NT;
+    if (i >= W4) continue;
+    float4 o;
+    o.x = fmaf(v[r].x * rn, gv[r].x, hv[r].x);
+    o.y = fmaf(v[r].y * rn, gv[r].y, hv[r].y);
+    o.z = fmaf(v[r].z * rn, gv[r].z, hv[r].z);
+    o.w = fmaf(v[r].w * rn, gv[r].w, hv[r].w);
+    hr[i] = o;
+    if (x_next != nullptr) {
+      TX* dst = x_next + (size_t)t * W + 4 * i;
+      if constexpr (sizeof(TX) == 4) {
+        *reinterpret_cast<float4*>(dst) = o;
+      } else {
+        uint2 pk;
+        pk.x = pack_bf16x2(o.x, o.y);
+        pk.y = pack_bf16x2(o.z, o.w);
+        *reinterpret_cast<uint2*>(dst) = pk;
+      }
+    }
+  }
+}
+
+// the same for any width and any number of choices: the row staged in shared memory, one number at a time
+template <typename TX>
+__global__ void __launch_bounds__(256) out_norm_add_any_kernel(float* __restrict__ h, const float* __restrict__ a, const float* __restrict__ a_scale,
+                                                               const float* __restrict__ y, const float* __restrict__ weight,
+                                                               const int32_t* __restrict__ pair_slot, int top, const float* __restrict__ gain,
+                                                               float mult, int W, float eps, TX* __restrict__ x_next) {
+  extern __shared__ float lrow[];
+  __shared__ float red[8];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  const float as = a_scale ? a_scale[t] : 1.0f;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < W; i += 256) {
+    float v = a ? a[(size_t)t * W + i] * as : 0.f;
+    if (y != nullptr)
+      for (int k = 0; k < top; ++k) v = fmaf(weight[(size_t)t * top + k], y[(size_t)pair_slot[(size_t)t * top + k] * W + i], v);
+    lrow[i] = v;
+    ss = fmaf(v, v, ss);
+  }
+  const float rn = mult / sqrtf(block_sum_n<256>(ss, red) / (float)W + eps);
+  for (int i = threadIdx.x; i < W; i += 256) {
+    const float o = fmaf(lrow[i] * rn, gain[i], h[(size_t)t * W + i]);
+    h[(size_t)t * W + i] = o;
+    if (x_next != nullptr) x_next[(size_t)t * W + i] = (TX)o;
+  }
+}
+
+template <typename TX>
+int out_norm_add_typed(float* h, const float* a, const float* a_scale, const float* y, const float* weight, const int32_t* pair_slot, int top,
+                       const float* gain, float mult, int T, int W, float eps, cudaStream_t s, TX* x_next) {
+#define B2_OUT_NORM(NT, R)                                                                                                                        \
+  do {                                                                                                                                            \
+    B2_CUDA_OK(b2_launch(out_norm_add_kernel<TX, NT, R>, dim3(T), dim3(NT), 0, s, h, a, a_scale, y, weight, pair_slot, top, gain, mult, W, eps, x_next)); \
+    return 0;                                                                                                                                     \
+  } while (0)
+  if (W % 4 == 0 && W <= 8192 && (y == nullptr || top <= ON_MAX_TOP)) {
+    if (T < 1024) {   // few tokens: wide CTAs, a row is one or two rounds of loads
+      if (W <= 512) B2_OUT_NORM(128, 1);
+      if (W <= 2048) B2_OUT_NORM(512, 1);
+      if (W <= 4096) B2_OUT_NORM(512, 2);
+      B2_OUT_NORM(512, 4);
+    }
+    if (W <= 512) B2_OUT_NORM(128, 1);
+    if (W <= 1024) B2_OUT_NORM(128, 2);
+    if (W <= 2048) B2_OUT_NORM(256, 2);
+    if (W <= 4096) B2_OUT_NORM(256, 4);
+    B2_OUT_NORM(512, 4);
+  }
+#undef B2_OUT_NORM
+  const size_t smem = (size_t)W * 4;
+  B2_REQUIRE(smem <= 160 * 1024, "out_norm_add: a row of %d numbers does not fit in shared memory", W);
+  static B2PerDeviceOnce once;
+  if (smem > 48 * 1024) b2_prefer_max_smem(out_norm_add_any_kernel<TX>, once);
+  B2_CUDA_OK(b2_launch(out_norm_add_any_kernel<TX>, dim3(T), dim3(256), smem, s, h, a, a_scale, y, weight, pair_slot, top, gain, mult, W, eps, x_next));
+  return 0;
+}
+
 }  // namespace
 
 constexpr int GN_EARLY_ROWS = 1024;
@@ -614,6 +795,29 @@ int launch_layer_norm_add(float* h, const float* y, const int32_t* pair_slot, in
     B2_CUDA_OK(b2_launch(layer_norm_add_kernel<bf16>, dim3(T), dim3(128), smem, s, h, y, pair_slot, top, coef, w, b, W, eps, w_next, b_next, (bf16*)x_next));
   }
   return 0;
+}
+
+int launch_embed_sum(const int32_t* ids, const void* table, const BigramTable& bg, const void* pos_table, int pos_rows, int table_f32, float* h, void* x,
+                     int T, int W, int vocab, const int32_t* row_seq, const int32_t* row_first, const int32_t* row_end, const int32_t* positions,
+                     const int32_t* slots, cudaStream_t s) {
+  if (T <= 0) return 0;
+  B2_REQUIRE(bg.buckets >= 1 && bg.tok_ring && pos_rows >= 1 && row_seq && row_first && row_end, "embed_sum: bad tables");
+#define B2_EMBED_SUM(TX)                                                                                                                              \
+  B2_CUDA_OK(b2_launch(embed_sum_kernel<TX>, dim3(T), dim3(128), 0, s, ids, (const TX*)table, (const TX*)bg.table, bg.buckets, bg.mul_prev, bg.mul_cur,   \
+                       bg.tok_ring, (const TX*)pos_table, pos_rows, h, (TX*)x, W, vocab, row_seq, row_first, row_end, positions, slots))
+  if (table_f32) B2_EMBED_SUM(float);
+  else B2_EMBED_SUM(bf16);
+#undef B2_EMBED_SUM
+  return 0;
+}
+
+int launch_out_norm_add(float* h, const float* a, const float* a_scale, const float* y, const float* weight, const int32_t* pair_slot, int top,
+                        const float* gain, float mult, int T, int W, float eps, cudaStream_t s, void* x_next, int x_f32) {
+  if (T <= 0) return 0;
+  B2_REQUIRE(a != nullptr || y != nullptr, "out_norm_add: nothing to add");
+  B2_REQUIRE(y == nullptr || (weight != nullptr && pair_slot != nullptr && top >= 1), "out_norm_add: routed rows need their weights and slots");
+  if (x_f32) return out_norm_add_typed<float>(h, a, a_scale, y, weight, pair_slot, top, gain, mult, T, W, eps, s, (float*)x_next);
+  return out_norm_add_typed<bf16>(h, a, a_scale, y, weight, pair_slot, top, gain, mult, T, W, eps, s, (bf16*)x_next);
 }
 
 int launch_xielu(const float* z, const float* pq, void* act, int act_f32, size_t n, cudaStream_t s) {

@@ -131,6 +131,11 @@ static std::string read_file(const std::string& p) {
 static bool is_dir(const std::string& p) { struct stat st; return stat(p.c_str(), &st) == 0 && S_ISDIR(st.st_mode); }
 static bool is_file(const std::string& p) { struct stat st; return stat(p.c_str(), &st) == 0 && S_ISREG(st.st_mode); }
 
+// families whose config lists the layers one by one (they have an fp32 path)
+static bool has_layer_list(const b2_config& c) {
+  return c.arch == B2_ARCH_LERASUN || c.arch == B2_ARCH_KEDASUN || c.arch == B2_ARCH_BUMALIX || c.arch == B2_ARCH_TINEVIK || c.arch == B2_ARCH_TOLANEX;
+}
+
 static void fill_config(const Options& o, b2_config& c) {
   memset(&c, 0, sizeof c);
   c.abi_version = B2_ABI_VERSION;
@@ -143,8 +148,9 @@ static void fill_config(const Options& o, b2_config& c) {
     fprintf(stderr, "b2serve: %s\n", b2_last_error());
     exit(1);
   }
-  c.compute_f32 = (o.f32 && (c.arch == B2_ARCH_LERASUN || c.arch == B2_ARCH_KEDASUN || c.arch == B2_ARCH_BUMALIX || c.arch == B2_ARCH_TINEVIK)) ? 1 : 0;  // the other families have no fp32 path: the flag is accepted and ignored
+  c.compute_f32 = (o.f32 && has_layer_list(c)) ? 1 : 0;  // the other families have no fp32 path: the flag is accepted and ignored
   c.max_model_len = o.max_model_len;
+  if (has_layer_list(c) && c.max_positions > 0) c.max_model_len = std::min(c.max_model_len, c.max_positions);   // (rows of a learned position table)
   c.block_size = o.block_size;
   c.num_blocks = o.num_blocks;
   c.gpu_mem_fraction = o.gpu_mem_util;
@@ -162,7 +168,7 @@ static uint16_t f2bf(float f) {
 
 // HF default init statistics: N(0, 0.02) for Linear/Embedding, ones for norm gains.
 static int load_dummy_weights(b2_engine* e, const b2_config& c, uint64_t seed) {
-  if (c.arch == B2_ARCH_LERASUN || c.arch == B2_ARCH_KEDASUN || c.arch == B2_ARCH_BUMALIX || c.arch == B2_ARCH_TINEVIK) {
+  if (has_layer_list(c)) {
     fprintf(stderr, "b2serve: random-init weights are built for the HF families; a layer-list model directory needs its model.safetensors\n");
     return -22;
   }

@@ -37,9 +37,9 @@ class EngineConfig:
     max_seqs: int = 64
     max_batch_tokens: int = 8192
     use_cuda_graphs: bool = True
-    arch: str = "qwen3"          # "qwen3" | "phi3" | "opt" | "lerasun" | "kedasun" | "bumalix" | "tinevik" (include/b2_engine.h, enum b2_arch)
+    arch: str = "qwen3"          # "qwen3" | "phi3" | "opt" | "lerasun" | "kedasun" | "bumalix" | "tinevik" | "tolanex" (include/b2_engine.h, enum b2_arch)
     rotary_dim: int = 0          # 0 = head_dim
-    max_positions: int = 0       # OPT: learned position table rows - 2 (0 = max_model_len)
+    max_positions: int = 0       # OPT: learned position table rows - 2 (0 = max_model_len); Tolanex: rows
     sliding_window: int = 0      # Phi-3: attend to the last N keys only (0 = all)
     layers: list | None = None   # layer-list families (arch "lerasun", "kedasun", "bumalix"): the "layers" entries of the model's config.json
     compute_f32: bool = False    # families with an fp32 path: operands, weights and cache in fp32
@@ -48,7 +48,9 @@ class EngineConfig:
     norm_groups: int = 0         # Kedasun: pieces of every norm (0 = 1)
     loop: tuple = (0, 0, 0)      # Bumalix: layers [start, stop) run `times` times in a row (times 0 = no loop)
     logit_softcap: float = 0.0   # logits <- cap * tanh(logits / cap) (0 = none)
-    norm_kind: int = 0           # 1: layer norms with gain and bias around every sublayer (Tinevik)
+    norm_kind: int = 0           # 1: layer norms with gain and bias around every sublayer (Tinevik); 2: RMS norms behind the sublayers only (Tolanex)
+    residual_mult: float = 0.0   # Tolanex: factor on a sublayer's normed output (0 = 1)
+    bigram: tuple = (0, 0, 0)    # Tolanex: (buckets, mul_prev, mul_cur) of the bigram table
 
     @staticmethod
     def lerasun(model_cfg: dict, **runtime) -> "EngineConfig":
@@ -84,6 +86,17 @@ class EngineConfig:
                             rms_eps=model_cfg["norm"]["eps"], embed_scale=(model_cfg.get("embedding") or {}).get("scale", 1.0),
                             logit_scale=model_cfg.get("logit_scale", 1.0), arch="tinevik", layers=model_cfg["layers"], tie_embeddings=True,
                             num_q_heads=0, num_kv_heads=0, head_dim=0, intermediate=0, norm_kind=1, **runtime)
+
+    @staticmethod
+    def tolanex(model_cfg: dict, **runtime) -> "EngineConfig":
+        """From the dict a Tolanex config.json holds (width, vocab, max_positions, embedding.bigram, norm.eps, residual_mult, layers) plus runtime
+        sizing."""
+        bg = model_cfg["embedding"]["bigram"]
+        return EngineConfig(num_layers=len(model_cfg["layers"]), hidden=model_cfg["width"], vocab=model_cfg["vocab"],
+                            rms_eps=model_cfg["norm"]["eps"], embed_scale=1.0, logit_scale=1.0, arch="tolanex", layers=model_cfg["layers"],
+                            tie_embeddings=False, num_q_heads=0, num_kv_heads=0, head_dim=0, intermediate=0, norm_kind=2,
+                            max_positions=int(model_cfg["max_positions"]), residual_mult=float(model_cfg.get("residual_mult", 1.0)),
+                            bigram=(int(bg["buckets"]), int(bg["mul_prev"]), int(bg["mul_cur"])), **runtime)
 
     def kv_bytes_per_token(self) -> int:
         return 2 * self.num_layers * self.num_kv_heads * self.head_dim * 2
@@ -123,7 +136,8 @@ class Engine:
         c.rope_theta = cfg.rope_theta
         c.gpu_mem_fraction = cfg.gpu_mem_fraction
         c.arch = {"qwen3": capi.ARCH_QWEN3, "phi3": capi.ARCH_PHI3, "opt": capi.ARCH_OPT, "lerasun": capi.ARCH_LERASUN,
-                  "kedasun": capi.ARCH_KEDASUN, "bumalix": capi.ARCH_BUMALIX, "tinevik": capi.ARCH_TINEVIK}[cfg.arch]
+                  "kedasun": capi.ARCH_KEDASUN, "bumalix": capi.ARCH_BUMALIX, "tinevik": capi.ARCH_TINEVIK,
+                  "tolanex": capi.ARCH_TOLANEX}[cfg.arch]
         c.norm_kind = int(cfg.norm_kind)
         c.loop_start, c.loop_stop, c.loop_times = (int(v) for v in cfg.loop)
         c.logit_softcap = float(cfg.logit_softcap)
@@ -131,11 +145,13 @@ class Engine:
         c.logit_scale = float(cfg.logit_scale)
         c.embed_scale = float(cfg.embed_scale)
         c.norm_groups = int(cfg.norm_groups)
+        c.residual_mult = float(cfg.residual_mult)
+        c.bigram_buckets, c.bigram_mul_prev, c.bigram_mul_cur = (int(v) for v in cfg.bigram)
         self._specs = None
         if cfg.layers is not None:
             self._specs = (b2_layer_spec * len(cfg.layers))()
             for sp, layer in zip(self._specs, cfg.layers):
-                _fill_layer_spec(sp, dict(layer, _tinevik=True) if cfg.arch == "tinevik" else layer)
+                _fill_layer_spec(sp, dict(layer, _family=cfg.arch))
             c.layer_specs = self._specs
         c.rotary_dim = int(cfg.rotary_dim)
         c.max_positions = int(cfg.max_positions)
@@ -162,17 +178,19 @@ class Engine:
         specs = (b2_layer_spec * 1024)()
         check(lib.b2_config_from_dir(model_dir.encode(), C.byref(c), specs, 1024), lib)
         arch = {capi.ARCH_QWEN3: "qwen3", capi.ARCH_PHI3: "phi3", capi.ARCH_OPT: "opt", capi.ARCH_LERASUN: "lerasun",
-                capi.ARCH_KEDASUN: "kedasun", capi.ARCH_BUMALIX: "bumalix", capi.ARCH_TINEVIK: "tinevik"}[c.arch]
+                capi.ARCH_KEDASUN: "kedasun", capi.ARCH_BUMALIX: "bumalix", capi.ARCH_TINEVIK: "tinevik",
+                capi.ARCH_TOLANEX: "tolanex"}[c.arch]
         layers = None
-        if arch in ("lerasun", "kedasun", "bumalix", "tinevik"):
-            layers = [_layer_dict(specs[i]) for i in range(c.num_layers)]
+        if arch in ("lerasun", "kedasun", "bumalix", "tinevik", "tolanex"):
+            layers = [_layer_dict(specs[i], arch) for i in range(c.num_layers)]
         cfg = EngineConfig(num_layers=c.num_layers, hidden=c.hidden, num_q_heads=c.num_q_heads, num_kv_heads=c.num_kv_heads,
                            head_dim=c.head_dim, intermediate=c.intermediate, vocab=c.vocab, tie_embeddings=bool(c.tie_embeddings),
                            rms_eps=c.rms_eps, rope_theta=c.rope_theta, arch=arch, rotary_dim=c.rotary_dim,
                            max_positions=c.max_positions, sliding_window=c.sliding_window, layers=layers,
                            compute_f32=(dtype == "float32"), logit_scale=c.logit_scale, embed_scale=c.embed_scale,
                            norm_groups=c.norm_groups, loop=(c.loop_start, c.loop_stop, c.loop_times), logit_softcap=c.logit_softcap,
-                           norm_kind=c.norm_kind, **runtime)
+                           norm_kind=c.norm_kind, residual_mult=c.residual_mult,
+                           bigram=(c.bigram_buckets, c.bigram_mul_prev, c.bigram_mul_cur), **runtime)
         return cls(cfg, device=device, safetensors_path=os.path.join(model_dir, "model.safetensors"))
 
     # ---- weights -----------------------------------------------------------------------
@@ -349,7 +367,9 @@ class Engine:
 
 def _fill_layer_spec(sp, layer: dict) -> None:
     """One "layers" entry of a layer-list config.json -> b2_layer_spec (the C registry does the same for a directory)."""
-    if layer["type"] == "gla" or layer["mixer"].get("q_rank") is not None or (layer["type"] == "attention" and layer.get("_tinevik")):
+    if layer.get("_family") == "tolanex":
+        return _fill_outnorm_spec(sp, layer)
+    if layer["type"] == "gla" or layer["mixer"].get("q_rank") is not None or (layer["type"] == "attention" and layer.get("_family") == "tinevik"):
         return _fill_mixed_spec(sp, layer)
     if layer["type"] in ("attention", "attention_2"):
         return _fill_heads_spec(sp, layer)
@@ -376,7 +396,7 @@ def _fill_layer_spec(sp, layer: dict) -> None:
 
 def _fill_mixed_spec(sp, layer: dict) -> None:
     """Tinevik: "gla", "attention" (scores mixed over the heads before the softmax, rotated values) and "latent_attention" (query latent,
-    window, output gate).  An "attention" entry of this family is marked with "_tinevik": True (Engine.__init__ does it for arch "tinevik")."""
+    window, output gate)."""
     m = layer["mixer"]
     sp.kv_from = -1
     sp.weights_of = int(layer["weights_of"]) if layer.get("weights_of") is not None else -1
@@ -428,10 +448,52 @@ def _mixed_layer_dict(sp) -> dict:
         mlp = {"kind": "dense", "ff": sp.ff_dim}
     elif sp.ff == capi.FF_TABLE_EXPERTS:
         mlp = {"kind": "moe", "expert": {"ff": sp.ff_dim, "limit": sp.ff_limit}, "router": {"experts": sp.experts, "top": sp.top}}
-    d = {"type": ty, "mixer": m, "mlp": mlp, "_tinevik": True}
+    d = {"type": ty, "mixer": m, "mlp": mlp}
     if sp.weights_of >= 0:
         d["weights_of"] = sp.weights_of
     return d
+
+
+def _fill_outnorm_spec(sp, layer: dict) -> None:
+    """Tolanex: "delta" (gated delta rule with a decay per head) and "latent_attention" (nothing rotated, no sink, kv_from)."""
+    m = layer["mixer"]
+    sp.kv_from = sp.weights_of = -1
+    sp.heads, sp.dim, sp.vdim = int(m["heads"]), int(m["dim"]), int(m["vdim"])
+    sp.kv_heads = int(m.get("kv_heads", m["heads"]))
+    if layer["type"] == "delta":
+        sp.mixer, sp.conv_taps = capi.MIXER_HEAD_DELTA, int(m["conv"])
+    elif layer["type"] == "latent_attention":
+        sp.mixer, sp.kv_rank, sp.scale = capi.MIXER_LATENT_ATTENTION, int(m["kv_rank"]), float(m["scale"])
+        sp.kv_from = int(m["kv_from"]) if m.get("kv_from") is not None else -1
+    else:
+        raise B2Error("mixer type %r not built" % layer["type"])
+    mlp = layer.get("mlp")
+    sp.ff = capi.FF_NONE
+    if mlp is not None:
+        if mlp["kind"] != "moe":
+            raise B2Error("feed-forward kind %r not built" % mlp["kind"])
+        r = mlp["router"]
+        g = r.get("groups") or {"count": 1, "keep": 1}
+        sp.ff, sp.ff_dim, sp.experts, sp.top = capi.FF_SOFTMAX_EXPERTS, int(mlp["expert"]["ff"]), int(r["experts"]), int(r["top"])
+        sp.groups, sp.groups_keep, sp.router_scale = int(g["count"]), int(g["keep"]), float(r.get("scale", 1.0))
+        sp.shared_ff = int(mlp["shared"]["ff"]) if mlp.get("shared") else 0
+
+
+def _outnorm_layer_dict(sp) -> dict:
+    m = {"heads": sp.heads, "dim": sp.dim, "vdim": sp.vdim}
+    if sp.mixer == capi.MIXER_HEAD_DELTA:
+        m.update(kv_heads=sp.kv_heads, conv=sp.conv_taps)
+    else:
+        m.update(kv_rank=sp.kv_rank, scale=sp.scale)
+        if sp.kv_from >= 0:
+            m["kv_from"] = sp.kv_from
+    mlp = None
+    if sp.ff == capi.FF_SOFTMAX_EXPERTS:
+        mlp = {"kind": "moe", "expert": {"ff": sp.ff_dim},
+               "router": {"experts": sp.experts, "top": sp.top, "groups": {"count": sp.groups, "keep": sp.groups_keep}, "scale": sp.router_scale}}
+        if sp.shared_ff > 0:
+            mlp["shared"] = {"ff": sp.shared_ff}
+    return {"type": "delta" if sp.mixer == capi.MIXER_HEAD_DELTA else "latent_attention", "mixer": m, "mlp": mlp}
 
 
 def _fill_state_spec(sp, layer: dict) -> None:
@@ -486,7 +548,9 @@ def _fill_heads_spec(sp, layer: dict) -> None:
         sp.ff, sp.ff_dim, sp.ff_limit = capi.FF_CLAMPED_GATED, int(mlp["ff"]), float(mlp["limit"])
 
 
-def _layer_dict(sp) -> dict:
+def _layer_dict(sp, arch: str = "") -> dict:
+    if arch == "tolanex":
+        return _outnorm_layer_dict(sp)
     if sp.mixer in (capi.MIXER_DECAY_STATE, capi.MIXER_MIXED_SCORE_ATTENTION, capi.MIXER_GATED_LATENT):
         return _mixed_layer_dict(sp)
     if sp.mixer in (capi.MIXER_WINDOW_AND_STATE, capi.MIXER_DELTA_STATE):

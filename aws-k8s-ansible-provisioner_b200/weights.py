@@ -287,6 +287,59 @@ def tinevik_random_state_dict(model_cfg: dict, seed: int = 0, rank_a: int = 16) 
     return sd
 
 
+def tolanex_tensor_shapes(model_cfg: dict) -> dict[str, tuple[int, ...]]:
+    """Tensor names and shapes of a Tolanex checkpoint for the dict its config.json holds."""
+    W, V = model_cfg["width"], model_cfg["vocab"]
+    s: dict[str, tuple[int, ...]] = {"embed": (V, W), "bigram": (model_cfg["embedding"]["bigram"]["buckets"] + 1, W), "pos": (model_cfg["max_positions"], W)}
+    for i, layer in enumerate(model_cfg["layers"]):
+        m, mlp, p = layer["mixer"], layer.get("mlp"), f"l{i}."
+        H, D, Dv, q = m["heads"], m["dim"], m["vdim"], f"l{i}.mix."
+        s[p + "norm1"] = (W,)
+        if layer["type"] == "delta":
+            G = m.get("kv_heads", H)
+            for n, c in (("q", G * D), ("k", G * D), ("v", H * Dv)):
+                s[q + n], s[q + n + ".conv"] = (c, W), (c, m["conv"])
+            s[q + "b"], s[q + "a"], s[q + "A_log"], s[q + "dt_bias"] = (H, W), (H, W), (H,), (H,)
+            s[q + "norm"], s[q + "g"] = (Dv,), (H * Dv, W)
+        else:
+            R = m["kv_rank"]
+            s[q + "q"] = (H * D, W)
+            if m.get("kv_from") is None:
+                s[q + "dkv"], s[q + "dkv.norm"] = (R, W), (R,)
+            s[q + "uk"], s[q + "uv"] = (H * D, R), (H * Dv, R)
+        s[q + "o"] = (W, H * Dv)
+        if mlp is not None:
+            F, f = mlp["expert"]["ff"], p + "mlp."
+            s[p + "norm2"], s[f + "router"] = (W,), (mlp["router"]["experts"], W)
+            for e in range(mlp["router"]["experts"]):
+                s[f"{f}e{e}.gate"], s[f"{f}e{e}.up"], s[f"{f}e{e}.down"] = (F, W), (F, W), (W, F)
+            if mlp.get("shared"):
+                Fs = mlp["shared"]["ff"]
+                s[f + "shared.gate"], s[f + "shared.up"], s[f + "shared.down"], s[f + "shared.sg"] = (Fs, W), (Fs, W), (W, Fs), (1, W)
+    s["final.norm"], s["head"] = (W,), (V, W)
+    return s
+
+
+def tolanex_random_state_dict(model_cfg: dict, seed: int = 0) -> dict[str, torch.Tensor]:
+    """Random bf16 weights scaled by 1/sqrt(fan-in), gains around one, decays that forget over tens to hundreds of tokens."""
+    g = torch.Generator().manual_seed(seed)
+    sd = {}
+    for name, shape in tolanex_tensor_shapes(model_cfg).items():
+        last = name.rsplit(".", 1)[-1]
+        if "norm" in name:
+            t = 1.0 + 0.1 * torch.randn(shape, generator=g)
+        elif last == "A_log":
+            t = torch.log(0.5 + 2.0 * torch.rand(shape, generator=g))
+        elif last == "dt_bias":
+            t = torch.randn(shape, generator=g) - 3.0
+        elif last == "conv" or name in ("embed", "bigram", "pos"):
+            t = 0.5 * torch.randn(shape, generator=g)
+        else:
+            t = torch.randn(shape, generator=g) * (shape[-1] ** -0.5)
+        sd[name] = t.to(torch.bfloat16)
+    return sd
+
+
 def write_model_dir(model_cfg: dict, sd: dict[str, torch.Tensor], path: str) -> str:
     """config.json + model.safetensors of a layer-list model, as the registry and the loader read them."""
     import os

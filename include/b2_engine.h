@@ -25,7 +25,7 @@
 extern "C" {
 #endif
 
-#define B2_ABI_VERSION 6
+#define B2_ABI_VERSION 7
 
 typedef struct b2_engine b2_engine;
 
@@ -33,7 +33,8 @@ typedef struct b2_engine b2_engine;
  * mixer's sizes and constants, and its feed-forward.  Families whose layers are all alike (Qwen3, Phi-3, OPT) leave
  * the list NULL and describe the layer through the scalar fields of b2_config. */
 enum b2_mixer_kind {
-  B2_MIXER_LATENT_ATTENTION = 1, /* one shared low-rank latent per token (Lerasun) */
+  B2_MIXER_LATENT_ATTENTION = 1, /* one shared low-rank latent per token (Lerasun; with rot_dim 0 nothing is rotated, and a family may have no
+                                    sink: Tolanex) */
   B2_MIXER_ATTENTION = 2,        /* per-head keys and values, grouped queries, rotary positions on interleaved pairs (Kedasun "attention") */
   B2_MIXER_CONV_ATTENTION = 3    /* biased projections, a short causal convolution on q / k / v, unit-RMS q and k, a linear distance penalty,
                                     a window that keeps the first tokens, mixing of the heads' softmax weights, an output gate (Kedasun
@@ -51,8 +52,10 @@ enum b2_mixer_kind {
                                     q and k heads RMS-normed with one gain per entry of a head; rotary positions on half-split pairs
                                     (i, i + rot_dims/2) with the angles divided by rot_factor; values rotated by their own position over
                                     all of vdim and the weighted sum turned back by the query's (Tinevik "attention") */
-  B2_MIXER_GATED_LATENT = 8      /* attention over a per-token latent with no rotated piece: the query itself goes through a normed latent of
+  B2_MIXER_GATED_LATENT = 8,     /* attention over a per-token latent with no rotated piece: the query itself goes through a normed latent of
                                     q_rank entries, a sliding window, a sigmoid gate on the concatenated heads (Tinevik "latent_attention") */
+  B2_MIXER_HEAD_DELTA = 9        /* gated delta rule with ONE decay per head: short causal convolutions on q / k / v, unit-vector q and k, a step size
+                                    and a decay per head straight from the layer's input, a silu gate as wide as the values (Tolanex "delta") */
 };
 enum b2_ff_kind {
   B2_FF_NONE = 0,
@@ -62,8 +65,11 @@ enum b2_ff_kind {
   B2_FF_SCALED_GATED_EXPERTS = 4,/* sigmoid router, the `top` largest scores; expert = W_d (silu(W_g y) * (W_u y)) on y = score * x (scores not
                                     renormalised); a shared expert of the same form (shared_ff) on x itself is added */
   B2_FF_XIELU = 5,               /* W_d a(W_u x), a(z) = softplus(p) z^2 + z / 2 for z > 0, (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 otherwise */
-  B2_FF_TABLE_EXPERTS = 6        /* experts of the B2_FF_CLAMPED_GATED form; an integer table row per token id names the token's `top` experts,
+  B2_FF_TABLE_EXPERTS = 6,       /* experts of the B2_FF_CLAMPED_GATED form; an integer table row per token id names the token's `top` experts,
                                     each weighted 1 / top (no router) */
+  B2_FF_SOFTMAX_EXPERTS = 7      /* softmax router over all experts, groups ranked by their best score (groups, groups_keep), the `top` largest of the kept
+                                    groups weighted by score * router_scale (not renormalised) on their OUTPUT; expert = W_d (silu(W_g x) * (W_u x)); a
+                                    shared expert of the same form (shared_ff) times sigmoid(w_sg . x) is added */
 };
 typedef struct b2_layer_spec {
   int32_t mixer;        /* b2_mixer_kind */
@@ -104,6 +110,8 @@ typedef struct b2_layer_spec {
   float   softcap;      /* scores <- softcap * tanh(scores / softcap) before the softmax (0 = none) */
   int32_t score_mix;    /* 1: the heads' capped scores are mixed by a heads x heads matrix before the softmax */
   int32_t rot_values;   /* 1: values are rotated by their position over all of vdim and the output turned back */
+  /* ABI 7 */
+  float   router_scale; /* B2_FF_SOFTMAX_EXPERTS: factor on the chosen scores (0 = 1) */
 } b2_layer_spec;
 
 /* Architecture + runtime sizing.  Field meanings follow HF Qwen3Config
@@ -149,7 +157,14 @@ typedef struct b2_config {
   float   logit_softcap;     /* logits <- cap * tanh(logits / cap) (0 = none) */
   /* ABI 6 */
   int32_t norm_kind;         /* layer-list families: 0 = RMS norms as the family defines them; 1 = layer norms with gain and bias
-                                ((x - mean) / sqrt(variance + eps) * w + b), in front of and behind every sublayer and at the end */
+                                ((x - mean) / sqrt(variance + eps) * w + b), in front of and behind every sublayer and at the end; 2 = RMS norms
+                                behind the sublayers only: the sublayers read the stream itself */
+  /* ABI 7 (Tolanex).  max_positions: rows of its learned position table */
+  float   residual_mult;     /* a sublayer's normed output is multiplied by this before it joins the stream (0 = 1) */
+  int32_t bigram_buckets;    /* > 0: row (previous token * bigram_mul_prev + token * bigram_mul_cur) mod bigram_buckets of a table of
+                                bigram_buckets + 1 rows joins the embedding; a sequence's first token takes the last row */
+  int64_t bigram_mul_prev;
+  int64_t bigram_mul_cur;
 } b2_config;
 
 /* Model families.  QWEN3: HF:models/qwen3/modeling_qwen3.py (QK-norm, separate q/k/v and gate/up
@@ -183,11 +198,18 @@ typedef struct b2_config {
  * feed-forwards: B2_FF_XIELU, B2_FF_TABLE_EXPERTS or none.  Tensor names: embed, l<i>.norm1|norm1b|norm2|norm2b (+ .b), l<i>.mix.{q,k,v,g,o,norm,a1,a2,
  * a2.b} (gla), l<i>.mix.{q,k,v,o,q.norm,k.norm,talk} (attention), l<i>.mix.{dq,dq.norm,uq,dkv,dkv.norm,uk,uv,g,o} (latent_attention),
  * l<i>.mlp.{up,down,act} or l<i>.mlp.{table (int32), e<k>.{gate,up,down}}, final.norm (+ .b).  The low-rank width (a1) is taken from the tensors. */
-enum b2_arch { B2_ARCH_QWEN3 = 0, B2_ARCH_PHI3 = 1, B2_ARCH_OPT = 2, B2_ARCH_LERASUN = 3, B2_ARCH_KEDASUN = 4, B2_ARCH_BUMALIX = 5, B2_ARCH_TINEVIK = 6 };
+/* TOLANEX: a layer list as well.  The stream starts as embed[token] + bigram[row] + pos[position] (bigram_*, max_positions); the sublayers read the
+ * stream itself and only their outputs are normed: h <- h + m rms(mixer(h)) w1, then h <- h + m rms(ff(h)) w2 with m = residual_mult on an fp32
+ * residual stream (norm_kind 2).  Mixers: B2_MIXER_HEAD_DELTA, B2_MIXER_LATENT_ATTENTION (rot_dim 0, no sink, kv_from); feed-forward:
+ * B2_FF_SOFTMAX_EXPERTS or none.  Per-sequence state: the matrix states, the convolutions' last inputs and the previous token.  Tensor names: embed,
+ * bigram, pos, l<i>.norm1|norm2, l<i>.mix.{q,k,v (+ .conv), b, a, A_log, dt_bias, norm, g, o} (delta), l<i>.mix.{q,dkv,dkv.norm,uk,uv,o}
+ * (latent_attention; no dkv with kv_from), l<i>.mlp.{router, e<k>.{gate,up,down}, shared.{gate,up,down,sg}}, final.norm, head. */
+enum b2_arch { B2_ARCH_QWEN3 = 0, B2_ARCH_PHI3 = 1, B2_ARCH_OPT = 2, B2_ARCH_LERASUN = 3, B2_ARCH_KEDASUN = 4, B2_ARCH_BUMALIX = 5, B2_ARCH_TINEVIK = 6,
+               B2_ARCH_TOLANEX = 7 };
 
 /* Model registry: reads MODEL_DIR/config.json and fills the architecture fields of *cfg (the runtime sizing fields --
  * max_model_len, block_size, num_blocks, max_seqs, max_batch_tokens, use_cuda_graphs, compute_f32 -- are left as the caller
- * set them).  HF configs are told apart by "model_type" (qwen3, phi3, opt); a config with "architecture": "Lerasun", "Kedasun", "Bumalix" or "Tinevik" fills
+ * set them).  HF configs are told apart by "model_type" (qwen3, phi3, opt); a config with "architecture": "Lerasun", "Kedasun", "Bumalix", "Tinevik" or "Tolanex" fills
  * specs[0 .. num_layers) as well and points cfg->layer_specs at it (max_specs = capacity of specs; may be 0 / NULL for the
  * HF families).  Returns 0, or a negative code with b2_last_error(). */
 int  b2_config_from_dir(const char* model_dir, b2_config* cfg, b2_layer_spec* specs, int32_t max_specs);

@@ -46,12 +46,12 @@ def test_registry_reads_the_layer_list(pkg, lib, tmp_path):
     # the Python mirror fills the same bytes from the same dict, and reads them back into an equal layer list
     mine = (capi.b2_layer_spec * 4)()
     for sp, layer in zip(mine, cfg["layers"]):
-        eng._fill_layer_spec(sp, dict(layer, _tinevik=True))
+        eng._fill_layer_spec(sp, dict(layer, _family="tinevik"))
     assert bytes(mine) == bytes(specs)[:C.sizeof(mine)]
     back = [eng._layer_dict(specs[i]) for i in range(4)]
     again = (capi.b2_layer_spec * 4)()
     for sp, layer in zip(again, back):
-        eng._fill_layer_spec(sp, layer)
+        eng._fill_layer_spec(sp, dict(layer, _family="tinevik"))
     assert bytes(again) == bytes(mine)
 
 
