@@ -496,8 +496,27 @@ def tinevik_model_cfg(width, heads, inter, vocab=32000):
     return {"architecture": "Tinevik", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "logit_scale": 1.0, "norm": {"eps": 1e-6}, "layers": ls}
 
 
+# ---- --family tolanex: width, heads (128 wide), Qwen3's feed-forward width.  Four layers: latent attention (latent 512), the gated delta rule with a decay
+#      per head (two value heads per key head), latent attention over the first layer's latents, the delta rule again; behind each 16 experts in four groups
+#      (two kept, two experts chosen) and a gated shared expert, with Qwen3's active parameter count; vocab 32000.  The closest existing families are Bumalix
+#      (delta rule, routed and shared gated experts) and Tinevik (latent attention without positions); both run beside it at the same sizes.
+def tolanex_model_cfg(width, heads, inter, vocab=32000):
+    lat = {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": 512, "scale": 128 ** -0.5}
+    dlt = {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}
+    ff = (inter // 3 + 63) // 64 * 64
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": 16, "top": 2, "groups": {"count": 4, "keep": 2}, "scale": 2.5}, "shared": {"ff": ff}}
+    ls = [{"type": "latent_attention", "mixer": lat, "mlp": moe}, {"type": "delta", "mixer": dlt, "mlp": moe},
+          {"type": "latent_attention", "mixer": dict(lat, kv_from=0), "mlp": moe}, {"type": "delta", "mixer": dlt, "mlp": moe}]
+    return {"architecture": "Tolanex", "vocab": vocab, "width": width, "max_positions": 4096, "residual_mult": 0.7, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 30011, "mul_prev": 8191, "mul_cur": 31}}, "layers": ls}
+
+
 def family_models(pkg, weights, family, tag):
     """(name, engine configuration, state-dict maker) of the family's model and of Qwen3 at the same width, depth, heads and feed-forward size."""
+    if family == "tolanex":
+        width, heads, inter = BUMALIX_SIZES[tag]
+        mc = tolanex_model_cfg(width, heads, inter)
+        return [("tolanex", pkg.EngineConfig.tolanex(mc), lambda c: weights.tolanex_random_state_dict(mc, seed=0))] + family_models(pkg, weights, "tinevik", tag)
     if family == "tinevik":
         width, heads, inter = BUMALIX_SIZES[tag]
         mc, bc = tinevik_model_cfg(width, heads, inter), bumalix_model_cfg(width, heads, inter)
@@ -526,7 +545,7 @@ def family_models(pkg, weights, family, tag):
 
 
 def run_family(args, local):
-    """Prefill and decode throughput of a layer-list family (Lerasun, Kedasun, Bumalix, Tinevik) at layer sizes of real models (random weights), and of
+    """Prefill and decode throughput of a layer-list family (Lerasun, Kedasun, Bumalix, Tinevik, Tolanex) at layer sizes of real models (random weights), and of
     Qwen3 at the same width, depth, head count and (active) feed-forward size: one JSON line per size and model, with the decode step's
     per-kernel-class times (CUDA events around every launch of an eager step)."""
     import torch
@@ -581,7 +600,7 @@ def main():
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--value-only", action="store_true", help="device-resident timing only (ablation runs)")
-    ap.add_argument("--family", default="", choices=["", "lerasun", "kedasun", "bumalix", "tinevik"],
+    ap.add_argument("--family", default="", choices=["", "lerasun", "kedasun", "bumalix", "tinevik", "tolanex"],
                     help="instead of the headline workload: the named family beside the closest GQA model at equal size (one GPU)")
     ap.add_argument("--family-sizes", default="w1024,w2048,w4096")
     ap.add_argument("--family-only", default="", help="time only the named model of the pair (the family's name, or qwen3)")
