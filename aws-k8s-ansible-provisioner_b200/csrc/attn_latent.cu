@@ -9,6 +9,10 @@
 // kv_rank + rot_dim numbers per cached token for ALL heads, which is what makes this cache small.
 // The sink is one more term of the softmax denominator with no key and no value: unscaled, counted once.
 //
+// Long prompt portions may instead attend over keys and values rebuilt from their context's latents (latent_gather, one product,
+// latent_store_pages, then attn_prefill_tc.cu): a query-key pair costs dim + vdim multiply-adds instead of 2 kv_rank, and the rebuilding is paid
+// once per context token and head.
+//
 // Everything here is fp32 arithmetic (scores, softmax, rotary angles in fp64 before the rounding, norms); the cache and
 // the operands handed on are fp32 or bf16.  Kernels:
 //   latent_finish     what follows the fused q | latent projection: rotary on the query's rotated piece, unit-RMS norm of
@@ -151,6 +155,31 @@ __global__ void __launch_bounds__(128) latent_pair_finish_kernel(const float* __
   if (slot < 0) return;
   TC* crow = cache + (size_t)slot * kv_rank;
   for (int i = threadIdx.x; i < kv_rank; i += 128) stf(crow + i, row[off_c + i] * rc * gain_c[i]);
+}
+
+// One CTA per (page, context): 16 cached rows of `rank` numbers (a multiple of 8), contiguous in the cache and in the output.
+__global__ void __launch_bounds__(256) latent_gather_kernel(const bf16* __restrict__ cache, int rank, const int32_t* __restrict__ block_table, int bt_stride,
+                                                            const LatentContext* __restrict__ ctx, bf16* __restrict__ rows) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const LatentContext c = ctx[blockIdx.y];
+  const int pg = blockIdx.x;
+  if (pg >= c.pages) return;
+  const uint4* src = reinterpret_cast<const uint4*>(cache + (size_t)block_table[(size_t)c.bt_row * bt_stride + pg] * 16 * rank);
+  uint4* dst = reinterpret_cast<uint4*>(rows + (size_t)(c.page0 + pg) * 16 * rank);
+  const int per_row = rank >> 3, valid = min(16, c.len - pg * 16) * per_row;
+  for (int i = threadIdx.x; i < 16 * per_row; i += 256) dst[i] = i < valid ? src[i] : make_uint4(0, 0, 0, 0);
+}
+
+// One CTA per (page, head): the head's 16 key rows and 16 value rows, 128 wide, into the page layout of the GQA kernels.
+__global__ void __launch_bounds__(256) latent_store_pages_kernel(const bf16* __restrict__ kv, int heads, bf16* __restrict__ k_pages, bf16* __restrict__ v_pages) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int pg = blockIdx.x, a = blockIdx.y, r = threadIdx.x >> 4, c = threadIdx.x & 15;
+  const bf16* row = kv + ((size_t)pg * 16 + r) * 2 * heads * 128;
+  const size_t at = (((size_t)pg * heads + a) * 16 + r) * 128 + kv_swizzled_chunk(r, c) * 8;
+  *reinterpret_cast<uint4*>(k_pages + at) = *reinterpret_cast<const uint4*>(row + a * 128 + c * 8);
+  *reinterpret_cast<uint4*>(v_pages + at) = *reinterpret_cast<const uint4*>(row + (heads + a) * 128 + c * 8);
 }
 
 constexpr int LA_WARPS = 8, LA_KEYS = 32;
@@ -657,6 +686,20 @@ int launch_latent_pair_finish(const float* proj, int ld, int off_q, int q_rank, 
   else
     B2_CUDA_OK(b2_launch(latent_pair_finish_kernel<bf16, bf16>, dim3(T), dim3(128), 0, s, proj, ld, off_q, q_rank, off_c, kv_rank, gain_q, gain_c, eps,
                          slots, (bf16*)xq, (bf16*)cache));
+  return 0;
+}
+
+int launch_latent_gather(const bf16* cache, int rank, const int32_t* block_table, int bt_stride, const LatentContext* ctx_dev, int nctx, int max_pages,
+                         bf16* rows, cudaStream_t s) {
+  if (nctx <= 0 || max_pages <= 0) return 0;
+  B2_REQUIRE(rank % 8 == 0, "latent_gather: rank %d is no multiple of 8", rank);
+  B2_CUDA_OK(b2_launch(latent_gather_kernel, dim3(max_pages, nctx), dim3(256), 0, s, cache, rank, block_table, bt_stride, ctx_dev, rows));
+  return 0;
+}
+
+int launch_latent_store_pages(const bf16* kv, int heads, int pages, bf16* k_pages, bf16* v_pages, cudaStream_t s) {
+  if (pages <= 0) return 0;
+  B2_CUDA_OK(b2_launch(latent_store_pages_kernel, dim3(pages, heads), dim3(256), 0, s, kv, heads, k_pages, v_pages));
   return 0;
 }
 

@@ -72,7 +72,7 @@ constexpr float PT_RESCALE = 8.0f;  // log2 units: the reference maximum is rais
 __global__ void __launch_bounds__(PT_THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, const bf16* __restrict__ q,
                        const int32_t* __restrict__ block_table, int bt_stride, const PrefillTile* __restrict__ tiles,
-                       bf16* __restrict__ out, int nq, int nkv, float scale_log2, int window, int pair_mode) {
+                       bf16* __restrict__ out, int nq, int nkv, float scale_log2, int window, int pair_mode, int head_step) {
   extern __shared__ uint8_t smem_raw[];
   __shared__ __align__(8) uint64_t k_full, v_full, s_full, p_full, o_full;
   __shared__ uint32_t tmem_slot;
@@ -88,7 +88,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
   // MMA rows are TWO consecutive 64-token tiles of one sequence x the real head, instead of one tile x (real, zero) heads --
   // half the CTAs, no MMA rows spent on zeros; the partner head's output rows are not written (the output projection's
   // columns for them are zeros, and the buffer holds finite values from its allocation).  The host pads every sequence to an
-  // even number of tiles (a tile with nrows == 0), so tiles 2i and 2i + 1 always belong together.
+  // even number of tiles (a tile with nrows == 0), so tiles 2i and 2i + 1 always belong together.  head_step 1 (pair_mode only): queries and
+  // outputs hold the real heads side by side, without partner heads between them.
   const int ti = gridDim.x - 1 - blockIdx.x;
   const PrefillTile tile = tiles[pair_mode ? 2 * ti : ti];                // rows 0..63 (and, without pair_mode, 64..127)
   const PrefillTile tile_b = pair_mode ? tiles[2 * ti + 1] : tile;        // rows 64..127 in pair_mode
@@ -191,7 +192,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
       const int rh = row >> 6, rt = row & 63;
       const PrefillTile& st = rh ? tile_b : tile;
       const bool in = rt < st.nrows;
-      const bf16* src = q + ((size_t)(st.q_row0 + (in ? rt : 0)) * nq + kvh * 2 + (pair_mode ? 0 : rh)) * PT_HD + c * 8;
+      const bf16* src = q + ((size_t)(st.q_row0 + (in ? rt : 0)) * nq + kvh * head_step + (pair_mode ? 0 : rh)) * PT_HD + c * 8;
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(q_s + (c >> 3) * PT_HALF_BYTES + row * 128 + (((c & 7) ^ (row & 7)) << 4)),
                    "l"(src), "r"(in ? 16 : 0)
                    : "memory");
@@ -310,7 +311,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
     const float inv = l_row > 0.f ? __fdiv_rn(1.0f, l_row) : 0.f;
     mbar_wait(smem_u32(&o_full), (it - 1) & 1);
     tc_fence_after();
-    bf16* dst = out + ((size_t)(mt.q_row0 + t) * nq + kvh * 2 + h) * PT_HD + kh * HALF;
+    bf16* dst = out + ((size_t)(mt.q_row0 + t) * nq + kvh * head_step + h) * PT_HD + kh * HALF;
 #pragma unroll 1
     for (int c0 = 0; c0 < HALF; c0 += 16) {
       uint32_t ov[16];
@@ -342,7 +343,8 @@ int launch_attn_prefill_tc(const bf16* q, const bf16* k_pages, const bf16* v_pag
                            int bt_stride, const PrefillTile* tiles_dev, int ntiles, bf16* out, int nq, int nkv, int hd, int block_size,
                            cudaStream_t s, float softmax_scale, int window, int pair_mode) {
   if (ntiles <= 0) return 0;
-  B2_REQUIRE(hd == PT_HD && block_size == 16 && nq == 2 * nkv, "attn_prefill_tc: built for 128-wide heads in GQA groups of two, 16-token pages");
+  const int head_step = pair_mode && nq == nkv ? 1 : 2;
+  B2_REQUIRE(hd == PT_HD && block_size == 16 && nq == head_step * nkv, "attn_prefill_tc: built for 128-wide heads in GQA groups of two, 16-token pages");
   B2_REQUIRE(num_pages >= 1, "attn_prefill_tc: the page pool's size is needed for the tensor maps");
   B2_REQUIRE(bt_stride <= PT_MAX_PAGES, "attn_prefill_tc: contexts beyond %d tokens not built (block table row of %d pages)", PT_MAX_PAGES * 16, bt_stride);
   CUtensorMap tk, tv;
@@ -357,7 +359,7 @@ int launch_attn_prefill_tc(const bf16* q, const bf16* k_pages, const bf16* v_pag
   const float scale_log2 = (float)(scale * 1.4426950408889634);
   B2_REQUIRE(!pair_mode || ntiles % 2 == 0, "attn_prefill_tc: pair mode needs an even tile list (each sequence padded to an even number of tiles)");
   B2_CUDA_OK(b2_launch(attn_prefill_tc_kernel, dim3(pair_mode ? ntiles / 2 : ntiles, nkv), dim3(PT_THREADS), (size_t)PT_SMEM, s, tk, tv, q, block_table,
-                       bt_stride, tiles_dev, out, nq, nkv, scale_log2, window, pair_mode));
+                       bt_stride, tiles_dev, out, nq, nkv, scale_log2, window, pair_mode, head_step));
   return 0;
 }
 

@@ -113,6 +113,7 @@ struct ListLayer {
   // the experts of every token id [vocab][top].
   float *bias1 = nullptr, *bias1b = nullptr, *bias2 = nullptr, *bias2b = nullptr, *latq_gain = nullptr;
   void* uq = nullptr;
+  bf16* ukv = nullptr;        // key and value up-projections as one matrix [heads (dim + vdim)][kv_rank]: layers that rebuild keys and values
   int32_t* table = nullptr;
   // Norms behind the sublayers only (Tolanex): gain1b / gain2b.  Its delta mixer projects q | k | v | beta | decay | gate in `wqd` (off_sg = the
   // gate's first column), with `a_log` and `a2_bias` per head; its latent mixer q (| the latent) in `wqd`; `router` holds the shared expert's
@@ -356,6 +357,17 @@ struct b2_engine {
   void *l_bigram = nullptr, *l_pos = nullptr;
   int32_t* l_tok_ring = nullptr;     // [sequence slots][2]: the token at a position, by the position's parity (a sequence's previous token)
   float* l_sg = nullptr;             // the shared expert's gate, one number per token row
+  // Prompt portions whose latent attention runs over rebuilt keys and values (attn_latent.cu): the step's long portions in groups whose contexts
+  // fit the scratch pools; a paired tile list, a block table of scratch pages and the contexts of each group.  d_tiles holds the short portions' tiles first.
+  struct LatentGroup { int ctx0, nctx, max_pages, pages, tile0, ntiles; };
+  int lx_pages_cap = 0;              // pages of the scratch pools (0: no layer takes this form)
+  bf16 *lx_rows = nullptr, *lx_kv = nullptr, *lx_k = nullptr, *lx_v = nullptr;
+  PrefillTile *d_xtiles = nullptr, *h_xtiles = nullptr;
+  LatentContext *d_xctx = nullptr, *h_xctx = nullptr;
+  int32_t *d_xtable = nullptr, *h_xtable = nullptr;
+  int xtiles_cap = 0;
+  std::vector<LatentGroup> lx_groups;
+  int lx_short_tiles = 0, lx_short_lo = 0, lx_short_hi = 0;   // tiles of the portions that stay in the absorbed form, and the rows they span
 };
 
 namespace {
@@ -1701,6 +1713,23 @@ int forward_mixed_list(b2_engine* e, int T, int ntiles, int nlast) {
 // rule with a decay per head (attn_state.cu over the sequence slots) and attention over a cached latent (attn_latent.cu, absorbed form; a layer
 // may read the region another layer wrote).  Feed-forward: experts chosen by a softmax router with grouped selection, weighted on their
 // output, plus a gated shared expert.  Per-sequence state besides the cache: matrix states, convolution rings, the previous token.
+constexpr int LATENT_REBUILD_ROWS = 128;    // portions of at least this many tokens attend over rebuilt keys and values
+
+// C (bf16 [M][N]) = A (bf16 [M][K]) . Wt^T on the tcgen05 projection kernel (K a multiple of 64, N at least 128)
+int list_dense_bf16(b2_engine* e, const bf16* A, const bf16* Wt, bf16* C, int M, int N, int K, cudaStream_t s) {
+  TcGemmArgs a;
+  a.bn = tc_pick_bn(M);
+  B2_TRY(b2_make_tmap_bf16(&a.tmap_w, Wt, (uint64_t)N, (uint64_t)K, (uint64_t)K, 128));
+  B2_TRY(b2_make_tmap_bf16(&a.tmap_x, A, (uint64_t)M, (uint64_t)K, (uint64_t)K, (uint32_t)a.bn));
+  a.T = M; a.N = N; a.K = K;
+  a.nsplit = 1;
+  a.out = C;
+  a.x_raw = A;
+  a.argmax_packed = nullptr;
+  a.epilogue = TC_EPI_BF16;
+  return launch_linear_tc(a, s);
+}
+
 constexpr float TOLANEX_UNIT_EPS = 1e-6f;   // q and k of the delta rule: x / sqrt(sum(x^2) + 1e-6)
 
 int forward_outnorm_list(b2_engine* e, int T, int ntiles, int nlast) {
@@ -1756,31 +1785,57 @@ int forward_outnorm_list(b2_engine* e, int T, int ntiles, int nlast) {
       const bool own = sp.kv_from < 0;
       const LatentGeom g{sp.heads, sp.dim, 0, sp.vdim, sp.kv_rank, 0, 0.f, sp.scale, c.rms_eps, 0};
       char* cache = e->regions[R.k_region].base;
+      const bool rebuild = L.ukv != nullptr && ntiles > 0 && !e->lx_groups.empty();
+      const int n_abs_tiles = rebuild ? e->lx_short_tiles : ntiles, lo = rebuild ? e->lx_short_lo : 0, rows = rebuild ? e->lx_short_hi - lo : T;
       {
         KL k(e, B2K_ROPE_KV);   // queries as operands; the token's normed latent into the cache
         if (!k.skip()) B2_TRY(launch_latent_finish(e->l_qd, L.nqd, g, own ? 1 : 0, L.lat_gain, e->d_positions, e->d_slots, e->l_qnope, f, e->l_q, cache, f, T, st));
       }
-      {
-        KL k(e, B2K_GEMM_QKV);   // the query pulled through the key up-projection, all heads in one strided batch
-        AnyGemm a;
-        a.A = e->l_qnope; a.W = L.ukT; a.C = e->l_qabs; a.M = T; a.N = sp.kv_rank; a.K = sp.dim;
-        a.lda = (long)sp.heads * sp.dim; a.ldw = sp.dim; a.ldc = (long)sp.heads * sp.kv_rank;
-        a.a_bs = sp.dim; a.w_bs = (long)sp.kv_rank * sp.dim; a.c_bs = sp.kv_rank;
-        if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, 1, sp.heads, 0, st));
+      if (rows > 0) {   // the absorbed form: decode steps and short portions (a step with long ones too: the rows the short ones span)
+        const size_t qo = (size_t)lo * sp.heads;
+        {
+          KL k(e, B2K_GEMM_QKV);   // the query pulled through the key up-projection, all heads in one strided batch
+          AnyGemm a;
+          a.A = (char*)e->l_qnope + qo * sp.dim * e->esz; a.W = L.ukT; a.C = e->l_qabs + qo * sp.kv_rank; a.M = rows; a.N = sp.kv_rank; a.K = sp.dim;
+          a.lda = (long)sp.heads * sp.dim; a.ldw = sp.dim; a.ldc = (long)sp.heads * sp.kv_rank;
+          a.a_bs = sp.dim; a.w_bs = (long)sp.kv_rank * sp.dim; a.c_bs = sp.kv_rank;
+          if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, 1, sp.heads, 0, st));
+        }
+        {
+          KL k(e, ntiles > 0 ? B2K_MISC : B2K_ATTN_DECODE);
+          if (!k.skip()) B2_TRY(launch_latent_attention(e->l_qabs, e->l_q, cache, f, g, e->d_block_table, e->bt_stride, c.block_size, tiles, n_abs_tiles, e->d_positions,
+                                                        e->d_seq_lens, nullptr, e->l_olat, f, T, st, e->l_attn_scratch, e->l_attn_scratch_floats, c.max_model_len));
+        }
+        {
+          KL k(e, B2K_GEMM_O);   // values of every head from the weighted latent
+          AnyGemm a;
+          a.A = (char*)e->l_olat + qo * sp.kv_rank * e->esz; a.W = L.uv; a.C = (char*)e->l_av + qo * sp.vdim * e->esz; a.M = rows; a.N = sp.vdim; a.K = sp.kv_rank;
+          a.lda = (long)sp.heads * sp.kv_rank; a.ldw = sp.kv_rank; a.ldc = (long)HV;
+          a.a_bs = sp.kv_rank; a.w_bs = (long)sp.vdim * sp.kv_rank; a.c_bs = sp.vdim;
+          if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, f, sp.heads, 0, st));
+        }
       }
-      {
-        KL k(e, ntiles > 0 ? B2K_MISC : B2K_ATTN_DECODE);
-        if (!k.skip()) B2_TRY(launch_latent_attention(e->l_qabs, e->l_q, cache, f, g, e->d_block_table, e->bt_stride, c.block_size, tiles, ntiles, e->d_positions,
-                                                      e->d_seq_lens, nullptr, e->l_olat, f, T, st, e->l_attn_scratch, e->l_attn_scratch_floats, c.max_model_len));
-      }
-      {
-        KL k(e, B2K_GEMM_O);   // values of every head from the weighted latent
-        AnyGemm a;
-        a.A = e->l_olat; a.W = L.uv; a.C = e->l_av; a.M = T; a.N = sp.vdim; a.K = sp.kv_rank;
-        a.lda = (long)sp.heads * sp.kv_rank; a.ldw = sp.kv_rank; a.ldc = (long)HV;
-        a.a_bs = sp.kv_rank; a.w_bs = (long)sp.vdim * sp.kv_rank; a.c_bs = sp.vdim;
-        if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, f, sp.heads, 0, st));
-      }
+      if (rebuild)   // long portions: keys and values of their contexts rebuilt, attention on tcgen05 (their rows of l_av are written last)
+        for (const b2_engine::LatentGroup& gp : e->lx_groups) {
+          {
+            KL k(e, B2K_MISC);
+            if (!k.skip()) B2_TRY(launch_latent_gather((const bf16*)cache, sp.kv_rank, e->d_block_table, e->bt_stride, e->d_xctx + gp.ctx0, gp.nctx, gp.max_pages,
+                                                       e->lx_rows, st));
+          }
+          {
+            KL k(e, B2K_GEMM_QKV);
+            if (!k.skip()) B2_TRY(list_dense_bf16(e, e->lx_rows, L.ukv, e->lx_kv, gp.pages * 16, 2 * sp.heads * 128, sp.kv_rank, st));
+          }
+          {
+            KL k(e, B2K_ROPE_KV);
+            if (!k.skip()) B2_TRY(launch_latent_store_pages(e->lx_kv, sp.heads, gp.pages, e->lx_k, e->lx_v, st));
+          }
+          {
+            KL k(e, B2K_MISC);
+            if (!k.skip()) B2_TRY(launch_attn_prefill_tc((const bf16*)e->l_qnope, e->lx_k, e->lx_v, gp.pages, e->d_xtable, e->bt_stride, e->d_xtiles + gp.tile0, gp.ntiles,
+                                                         (bf16*)e->l_av, sp.heads, sp.heads, 128, 16, st, sp.scale, 0, 1));
+          }
+        }
     }
     {
       KL k(e, B2K_GEMM_O);
@@ -2489,8 +2544,16 @@ int list_tensor(b2_engine* e, const std::string& name, const void* host, size_t 
       if (rest == "mix.q") { B2_TRY(want(H * dn * W)); return done(put_operand(e, L.wqd, 0, src, H * dn * W)); }
       if (rest == "mix.dkv" && sp.kv_from < 0) { B2_TRY(want(r * W)); return done(put_operand(e, L.wqd, H * dn * W, src, r * W)); }
       if (rest == "mix.dkv.norm" && sp.kv_from < 0) { B2_TRY(want(r)); return done(put_f32(L.lat_gain, src, r, 0.0f)); }
-      if (rest == "mix.uk") { B2_TRY(want(H * dn * r)); return done(put_key_up(e, L.ukT, src, H, dn, r)); }
-      if (rest == "mix.uv") { B2_TRY(want(HV * r)); return done(put_operand(e, L.uv, 0, src, HV * r)); }
+      if (rest == "mix.uk") {
+        B2_TRY(want(H * dn * r));
+        if (L.ukv) B2_TRY(put_operand(e, L.ukv, 0, src, H * dn * r));
+        return done(put_key_up(e, L.ukT, src, H, dn, r));
+      }
+      if (rest == "mix.uv") {
+        B2_TRY(want(HV * r));
+        if (L.ukv) B2_TRY(put_operand(e, L.ukv, H * dn * r, src, HV * r));
+        return done(put_operand(e, L.uv, 0, src, HV * r));
+      }
     }
     if (sp.ff == B2_FF_SOFTMAX_EXPERTS) {
       const size_t sf = sp.shared_ff, ne = sp.experts;
@@ -3309,7 +3372,7 @@ int outnorm_engine_alloc(b2_engine* e) {
   B2_TRY(xalloc(&e->l_pos, (size_t)c.max_positions * W));
   B2_TRY(falloc(&e->l_final_gain, W));
   e->ll.resize(c.num_layers);
-  size_t max_q = 1, max_hv = 1, max_up = 1, max_act = 1, max_hr = 1, max_hd = 1, max_sff = 0, max_nqd = 1;
+  size_t max_q = 1, max_hv = 1, max_up = 1, max_act = 1, max_hr = 1, max_hd = 1, max_sff = 0, max_nqd = 1, max_rebuild_nq = 0, max_rebuild_rank = 0;
   int max_top = 1, max_exp = 1, max_lat_heads = 1, max_rank = 1, max_state_heads = 1;
   bool any_latent = false, any_experts = false;
   for (int l = 0; l < c.num_layers; ++l) {
@@ -3356,6 +3419,16 @@ int outnorm_engine_alloc(b2_engine* e) {
       L.nqd = L.n_fixed = L.nq + (sp.kv_from < 0 ? sp.kv_rank : 0);
       B2_TRY(xalloc(&L.ukT, (size_t)sp.heads * sp.kv_rank * sp.dim));
       B2_TRY(xalloc(&L.uv, HV * sp.kv_rank));
+      static const bool use_rebuild = [] { const char* v = getenv("B2_LATENT_REBUILD"); return !(v && *v == '0'); }();   // 0: the absorbed form only (cross-check)
+      if (use_rebuild && !e->f32 && sp.dim == 128 && sp.vdim == 128 && sp.kv_rank % 64 == 0 && c.block_size == 16 && (c.max_model_len + 15) / 16 <= 1024 &&
+          c.max_batch_tokens >= LATENT_REBUILD_ROWS) {
+        char* q = nullptr;
+        B2_TRY(dalloc(&q, (size_t)2 * L.nq * sp.kv_rank * es));
+        L.ukv = reinterpret_cast<bf16*>(q);
+        e->weight_bytes += (int64_t)2 * L.nq * sp.kv_rank * es;
+        max_rebuild_nq = std::max(max_rebuild_nq, (size_t)L.nq);
+        max_rebuild_rank = std::max(max_rebuild_rank, (size_t)sp.kv_rank);
+      }
       any_latent = true;
       max_hd = std::max(max_hd, (size_t)L.nq);
       max_hr = std::max(max_hr, (size_t)sp.heads * sp.kv_rank);
@@ -3428,6 +3501,24 @@ int outnorm_engine_alloc(b2_engine* e) {
       e->l_attn_scratch_floats = latent_attention_scratch_floats(bucket_batch(c.max_seqs), max_lat_heads, max_rank);
       B2_TRY(dalloc(&e->l_attn_scratch, e->l_attn_scratch_floats));
     }
+  }
+  if (max_rebuild_nq > 0) {   // scratch for the contexts of one group: as many as a step brings at least, one full-length context at most needs
+    const size_t ctx_pages = (size_t)(c.max_model_len + 15) / 16;
+    e->lx_pages_cap = (int)std::max(ctx_pages, Tc / 16 + (size_t)c.max_seqs);
+    const size_t rows = (size_t)e->lx_pages_cap * 16;
+    B2_TRY(dalloc(&e->lx_rows, rows * max_rebuild_rank));
+    B2_TRY(dalloc(&e->lx_kv, rows * 2 * max_rebuild_nq));
+    B2_TRY(dalloc(&e->lx_k, rows * max_rebuild_nq));
+    B2_TRY(dalloc(&e->lx_v, rows * max_rebuild_nq));
+    B2_CUDA_OK(cudaMemset(e->lx_k, 0, rows * max_rebuild_nq * 2));
+    B2_CUDA_OK(cudaMemset(e->lx_v, 0, rows * max_rebuild_nq * 2));
+    e->xtiles_cap = (int)(Tc / 64 + 2 * (size_t)c.max_seqs + 2);
+    B2_TRY(dalloc(&e->d_xtiles, (size_t)e->xtiles_cap));
+    B2_TRY(dalloc(&e->d_xctx, (size_t)c.max_seqs));
+    B2_TRY(dalloc(&e->d_xtable, (size_t)c.max_seqs * ctx_pages));
+    B2_CUDA_OK(cudaMallocHost(&e->h_xtiles, (size_t)e->xtiles_cap * sizeof(PrefillTile)));
+    B2_CUDA_OK(cudaMallocHost(&e->h_xctx, (size_t)c.max_seqs * sizeof(LatentContext)));
+    B2_CUDA_OK(cudaMallocHost(&e->h_xtable, (size_t)c.max_seqs * ctx_pages * sizeof(int32_t)));
   }
   if (any_experts) {
     B2_TRY(dalloc(&e->l_ffd, Tc * W));
@@ -4356,6 +4447,10 @@ extern "C" void b2_engine_free(b2_engine* e) {
   if (e->ev_tok) cudaEventDestroy(e->ev_tok);
   F(e->partial2); F(e->attn_scratch2); F(e->ssq);
   if (e->l_head == e->l_embed) e->l_head = nullptr;   // (a tied head is the embedding table)
+  F(e->lx_rows); F(e->lx_kv); F(e->lx_k); F(e->lx_v); F(e->d_xtiles); F(e->d_xctx); F(e->d_xtable);
+  if (e->h_xtiles) cudaFreeHost(e->h_xtiles);
+  if (e->h_xctx) cudaFreeHost(e->h_xctx);
+  if (e->h_xtable) cudaFreeHost(e->h_xtable);
   F(e->l_final_bias); F(e->l_bigram); F(e->l_pos); F(e->l_tok_ring); F(e->l_sg);
   F(e->l_embed); F(e->l_head); F(e->l_embed_gain); F(e->l_final_gain); F(e->l_pool); F(e->l_h); F(e->l_qd); F(e->l_qrot); F(e->l_qabs);
   F(e->l_xperm); F(e->l_upf); if (e->h_offsets) cudaFreeHost(e->h_offsets);
@@ -4366,7 +4461,7 @@ extern "C" void b2_engine_free(b2_engine* e) {
     F(L.wqd); F(L.ukT); F(L.uv); F(L.wo); F(L.up); F(L.down); F(L.gain1); F(L.gain2); F(L.lat_gain); F(L.sink); F(L.router); F(L.corr);
     F(L.gain1b); F(L.gain2b); F(L.qkv_bias); F(L.o_bias); F(L.conv_w); F(L.talk); F(L.vmix); F(L.conv_ring);
     F(L.wo2); F(L.sh_up); F(L.sh_down); F(L.qk_gain); F(L.head_gain); F(L.a2); F(L.a2_bias); F(L.g2); F(L.a_log); F(L.out_gain_l); F(L.out_gain_r); F(L.poly);
-    F(L.bias1); F(L.bias1b); F(L.bias2); F(L.bias2b); F(L.latq_gain); F(L.uq); F(L.table);
+    F(L.bias1); F(L.bias1b); F(L.bias2); F(L.bias2b); F(L.latq_gain); F(L.uq); F(L.ukv); F(L.table);
   }
   for (auto& R : e->runs) {
     F(R.state); F(R.ring);
@@ -4525,6 +4620,30 @@ extern "C" int b2_prefill_logits(b2_engine* e, const int32_t* ids, const int32_t
   return prefill_impl(e, ids, seq_offsets, nseq, seq_ids, rows, nrows, out_logits, out_tokens);
 }
 namespace {
+// A long portion joins the step's list of rebuilt contexts: sequence row i of the block table, n tokens behind `len` cached ones, token rows from
+// row0 on.  A group's contexts lie side by side in the scratch pools; a context that does not fit any more opens the next group.
+void latent_context_add(b2_engine* e, int i, int len, int n, int row0) {
+  const int pages = (len + n + 15) / 16;
+  const b2_engine::LatentGroup* last = e->lx_groups.empty() ? nullptr : &e->lx_groups.back();
+  if (last == nullptr || last->pages + pages > e->lx_pages_cap) {
+    b2_engine::LatentGroup g{};
+    if (last) {
+      g.ctx0 = last->ctx0 + last->nctx;
+      g.tile0 = last->tile0 + last->ntiles;
+    }
+    e->lx_groups.push_back(g);
+  }
+  b2_engine::LatentGroup& g = e->lx_groups.back();
+  const int x = g.ctx0 + g.nctx++;
+  e->h_xctx[x] = LatentContext{i, len + n, g.pages, pages};
+  int32_t* bt = e->h_xtable + (size_t)x * e->bt_stride;
+  for (int p = 0; p < e->bt_stride; ++p) bt[p] = p < pages ? g.pages + p : 0;   // (past the end: the group's first page, masked)
+  for (int j = 0; j < n; j += 64) e->h_xtiles[g.tile0 + g.ntiles++] = PrefillTile{row0 + j, len + j, std::min(64, n - j), x};
+  if (g.ntiles & 1) e->h_xtiles[g.tile0 + g.ntiles++] = PrefillTile{row0, len + n, 0, x};   // tiles 2i and 2i + 1 belong to one sequence
+  g.pages += pages;
+  g.max_pages = std::max(g.max_pages, pages);
+}
+
 int prefill_impl(b2_engine* e, const int32_t* ids, const int32_t* seq_offsets, int32_t nseq, const int32_t* seq_ids, const int32_t* rows,
                  int32_t nrows, float* out_logits, int32_t* out_tokens) {
   B2_REQUIRE(e && ids && seq_offsets && seq_ids && nseq >= 1, "b2_prefill: bad arguments");
@@ -4572,9 +4691,13 @@ int prefill_impl(b2_engine* e, const int32_t* ids, const int32_t* seq_offsets, i
   int32_t* rowinfo = e->d_row_seq ? bt + (size_t)nseq * e->bt_stride : nullptr;
   B2_REQUIRE(!rowinfo || (size_t)(rowinfo - e->h_stage) + (size_t)3 * T <= e->h_stage_ints, "b2_prefill: %d tokens exceed the staging buffer", T);
   int ntiles = 0, row0 = 0;
+  e->lx_groups.clear();
+  e->lx_short_tiles = e->lx_short_lo = e->lx_short_hi = 0;
+  std::vector<PrefillTile> long_tiles;   // (behind the short portions' tiles)
   for (int i = 0; i < nseq; ++i) {
     Seq& s = e->seqs[seq_ids[i]];
     const int n = seq_offsets[i + 1] - seq_offsets[i] - skip[i];
+    const bool rebuild = e->lx_pages_cap > 0 && n >= LATENT_REBUILD_ROWS;
     const int32_t* src = ids + seq_offsets[i] + skip[i];
     for (int j = 0; j < n; ++j) {
       const int p = s.len + j;
@@ -4593,14 +4716,35 @@ int prefill_impl(b2_engine* e, const int32_t* ids, const int32_t* seq_offsets, i
     memcpy(bt + (size_t)i * e->bt_stride, s.blocks.data(), s.blocks.size() * 4);
     const int first_tile = ntiles;
     for (int j = 0; j < n; j += 64) {
+      const PrefillTile tl{row0 + j, s.len + j, std::min(64, n - j), i};
+      if (rebuild) {
+        long_tiles.push_back(tl);
+        continue;
+      }
       B2_REQUIRE(ntiles < e->tiles_cap, "b2_prefill: too many attention tiles");
-      e->h_tiles[ntiles++] = PrefillTile{row0 + j, s.len + j, std::min(64, n - j), i};
+      e->h_tiles[ntiles++] = tl;
+    }
+    if (rebuild) {
+      latent_context_add(e, i, s.len, n, row0);
+    } else {
+      if (e->lx_short_tiles == 0) e->lx_short_lo = row0;
+      e->lx_short_hi = row0 + n;
+      e->lx_short_tiles = ntiles;
     }
     if (prefill_tile_pairs(e) && ((ntiles - first_tile) & 1)) {  // attn_prefill_tc.cu, pair mode: tiles 2i and 2i + 1 belong together
       B2_REQUIRE(ntiles < e->tiles_cap, "b2_prefill: too many attention tiles");
       e->h_tiles[ntiles++] = PrefillTile{row0, s.len + n, 0, i};
     }
     row0 += n;
+  }
+  B2_REQUIRE(ntiles + (int)long_tiles.size() <= e->tiles_cap, "b2_prefill: too many attention tiles");
+  for (const PrefillTile& tl : long_tiles) e->h_tiles[ntiles++] = tl;
+  if (!e->lx_groups.empty()) {
+    const b2_engine::LatentGroup& gl = e->lx_groups.back();
+    const int nctx = gl.ctx0 + gl.nctx, nx = gl.tile0 + gl.ntiles;
+    B2_CUDA_OK(cudaMemcpyAsync(e->d_xtiles, e->h_xtiles, nx * sizeof(PrefillTile), cudaMemcpyHostToDevice, e->stream));
+    B2_CUDA_OK(cudaMemcpyAsync(e->d_xctx, e->h_xctx, nctx * sizeof(LatentContext), cudaMemcpyHostToDevice, e->stream));
+    B2_CUDA_OK(cudaMemcpyAsync(e->d_xtable, e->h_xtable, (size_t)nctx * e->bt_stride * 4, cudaMemcpyHostToDevice, e->stream));
   }
   B2_CUDA_OK(cudaMemcpyAsync(e->d_tokens, tok, T * 4, cudaMemcpyHostToDevice, e->stream));
   B2_CUDA_OK(cudaMemcpyAsync(e->d_positions, pos, T * 4, cudaMemcpyHostToDevice, e->stream));

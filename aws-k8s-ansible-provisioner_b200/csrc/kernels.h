@@ -200,6 +200,7 @@ int launch_attn_prefill(const bf16* q, const bf16* k_pages, const bf16* v_pages,
 int launch_attn_prefill_tc(const bf16* q, const bf16* k_pages, const bf16* v_pages, int64_t num_pages, const int32_t* block_table,
                            int bt_stride, const PrefillTile* tiles_dev, int ntiles, bf16* out, int nq, int nkv, int hd, int block_size,
                            cudaStream_t s, float softmax_scale = 0.f, int window = 0, int pair_mode = 0);
+// pair_mode: one query head per kv head; nq == 2 nkv with a partner head behind every real one, or nq == nkv without them
 
 // ---- sampling.cu ----
 struct SampleRow {  // one row to draw from (temperature <= 0: greedy arg-max, lowest index on ties)
@@ -434,6 +435,20 @@ int launch_latent_attention(const float* q_abs, const float* q_rot, const void* 
 // scratch: device floats for the key splits of a decode step (latent_attention_scratch_floats); without it a decode step runs
 // unsplit.  max_context: longest cache the engine can hold (bounds the number of splits).
 size_t latent_attention_scratch_floats(int max_rows, int max_heads, int max_rank);
+// Prompt portions long enough to pay for it attend over REBUILT keys and values instead: the portion's whole context of latents is gathered, one
+// product gives every head's key and value, and the GQA kernels' page layout takes them (attn_prefill_tc.cu runs over it, one query head per
+// kv head).  A context is a sequence's cached tokens and the portion's own, page by page: context i's pages become rows
+// [16 page0, 16 (page0 + pages)) of ctx and pages [page0, page0 + pages) of the rebuilt pools.
+struct LatentContext {
+  int bt_row;     // row of the block table
+  int len;        // tokens; the rest of the last page is zeros
+  int page0;
+  int pages;
+};
+int launch_latent_gather(const bf16* cache, int rank, const int32_t* block_table, int bt_stride, const LatentContext* ctx_dev, int nctx, int max_pages,
+                         bf16* rows, cudaStream_t s);
+// kv [pages * 16][2 * heads * 128] bf16 (keys of every head, then values) -> k_pages, v_pages [pages][heads][16][128] (kv_swizzled_chunk)
+int launch_latent_store_pages(const bf16* kv, int heads, int pages, bf16* k_pages, bf16* v_pages, cudaStream_t s);
 
 // ---- moe_route.cu: sigmoid or softmax router with a choice offset and grouped selection, and the token permutation by expert ----
 struct RouteGeom {

@@ -229,6 +229,37 @@ def test_bf16_close_to_the_restatement(make):
         assert np.median(rel) < BF16_BAR / 3 and np.quantile(rel, 0.95) < 2 * BF16_BAR, (np.median(rel), np.quantile(rel, 0.95))
 
 
+def test_bf16_rebuilt_keys_and_values():
+    """128-wide heads over a latent in multiples of 64: prompt portions of at least 128 tokens attend over keys and values rebuilt from their
+    context, shorter ones and decode steps stay in the absorbed form.  Long and short portions in one step, portions whose contexts do not fit the
+    scratch together, contexts that end inside a page, a reader with another head count; sharpened queries, so that a lost or doubled key shows."""
+    cfg = model([(lat(2, 128, 128, 64, 0.09), None), (delta(2, 1, 16, 16), moe(4, 2, 64, (2, 1), 1.5, 64)), (lat(3, 128, 128, 64, 0.09, kv_from=0), None)],
+                vocab=211, width=96, bigram=(53, 17, 3), positions=1024)
+    w = sharpen(cfg, random_weights(cfg, seed=33), factor=2.0)
+    prompts = [tokens(cfg, n, 34 + n) for n in (700, 655, 590, 40)]
+    refs = [ref_logits(cfg, w, p) for p in prompts]
+    scale = max(np.abs(r).max() for r in refs)
+    with engine(cfg, w, f32=False, max_model_len=720, num_blocks=190, max_seqs=4, max_batch_tokens=512) as e:
+        sids, done, rel = [e.seq_create(len(p)) for p in prompts], [0, 0, 0, 0], []
+        # (the scratch holds one context of the longest length: from the fourth step on the long portions' contexts are in groups of their own)
+        plan = [[(0, 300), (1, 130)], [(2, 200), (3, 20), (0, 128)], [(1, 2), (2, 128), (3, 17), (0, 133)], [(1, 330), (0, 1), (2, 128)],
+                [(0, 128), (1, 160), (2, 129), (3, 1)], [(1, 3), (0, 5)], [(0, 1), (1, 1), (2, 1), (3, 1)], [(2, 4), (1, 29)]]
+        for step in plan:
+            chunks = [prompts[r][done[r]:done[r] + c] for r, c in step]
+            if all(c == 1 for _, c in step):
+                e.decode_step([sids[r] for r, _ in step], in_tokens=[x[0] for x in chunks], want_output=False)
+                lg = e.get_logits(len(step))
+            else:
+                lg, _ = e.prefill_logits([sids[r] for r, _ in step], chunks, list(range(sum(c for _, c in step))))
+            base = 0
+            for r, c in step:
+                rel += list(np.abs(lg[base:base + c] - refs[r][done[r]:done[r] + c]).max(axis=1) / scale)
+                base += c
+                done[r] += c
+        rel = np.array(rel)
+        assert np.median(rel) < BF16_BAR / 3 and np.quantile(rel, 0.95) < 2 * BF16_BAR, (np.median(rel), np.quantile(rel, 0.95))
+
+
 def test_bf16_long_step_runs_the_experts_one_by_one():
     """A step with at least 2048 (token, choice) pairs takes the per-expert tensor-core products; short portions of the same prompt take
     the ragged ones: both agree with the restatement."""
