@@ -714,6 +714,8 @@ int launch_latent_attention(const float* q_abs, const float* q_rot, const void* 
                             cudaStream_t s, float* scratch, size_t scratch_floats, int max_context) {
   if (T <= 0 || (tiles != nullptr && ntiles <= 0)) return 0;
   static const bool use_mma = [] { const char* e = getenv("B2_LATENT_MMA"); return !(e && *e == '0'); }();
+  if (tiles == nullptr && !cache_f32 && !x_f32 && latent_decode_ok(g, block_size, T, max_context))
+    return launch_latent_decode(q_abs, q_rot, (const bf16*)cache, g, block_table, bt_stride, positions, seq_lens, sink, (bf16*)out_lat, T, max_context, s);
   const size_t mma_smem = mma_attn_smem(g);
   if (!cache_f32 && use_mma && g.kv_rank <= 512 && mma_smem <= 200 * 1024) {
     B2_REQUIRE(x_f32 == 0, "latent_attention: operands and cache have one element type");

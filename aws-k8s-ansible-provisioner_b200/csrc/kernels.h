@@ -435,6 +435,10 @@ int launch_latent_attention(const float* q_abs, const float* q_rot, const void* 
 // scratch: device floats for the key splits of a decode step (latent_attention_scratch_floats); without it a decode step runs
 // unsplit.  max_context: longest cache the engine can hold (bounds the number of splits).
 size_t latent_attention_scratch_floats(int max_rows, int max_heads, int max_rank);
+// ---- attn_latent_decode.cu: the decode form for a bf16 cache on clusters of eight CTAs (launch_latent_attention picks it when it fits) ----
+bool latent_decode_ok(const LatentGeom& g, int block_size, int B, int max_context);
+int launch_latent_decode(const float* q_abs, const float* q_rot, const bf16* cache, const LatentGeom& g, const int32_t* block_table, int bt_stride,
+                         const int32_t* positions, const int32_t* seq_lens, const float* sink, bf16* out_lat, int B, int max_context, cudaStream_t s);
 // Prompt portions long enough to pay for it attend over REBUILT keys and values instead: the portion's whole context of latents is gathered, one
 // product gives every head's key and value, and the GQA kernels' page layout takes them (attn_prefill_tc.cu runs over it, one query head per
 // kv head).  A context is a sequence's cached tokens and the portion's own, page by page: context i's pages become rows
