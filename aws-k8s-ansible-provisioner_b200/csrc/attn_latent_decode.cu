@@ -2,10 +2,10 @@
 // mathematics): every sequence brings one token, i.e. `heads` query rows that all read the same cached rows.
 //
 // A cluster of eight CTAs takes one sequence and sixteen heads; each CTA takes an eighth of the visible keys.  A sequence of a thousand tokens is
-// then about 128 keys per CTA -- two tiles of 64, which are both requested before the first is used, so that a CTA waits for HBM once.  Per tile:
-//   S [16 x 64]   = Q . K^T      warp w: keys 8w .. 8w + 7, mma.m16n8k16 (bf16 operands, fp32 sums)
-//   P             = exp(S - m)   sixteen threads per head, running maximum and sum in registers; bf16 P (the summed weights are the rounded ones)
-//   O [16 x rank] += P . C       warp w: an eighth of the latent, accumulators in registers; rescaled when a row's maximum moved
+// then about 128 keys per CTA -- four tiles of 32, two of them in flight; two CTAs fit on an SM.  Per tile:
+//   S [16 x 32]   = Q . K^T      warp w: keys 8w .. 8w + 7, mma.m16n8k16 (bf16 operands, fp32 sums)
+//   P             = exp(S - m)   eight threads per head, running maximum and sum in registers; bf16 P (the summed weights are the rounded ones)
+//   O [16 x rank] += P . C       warp w: a quarter of the latent, accumulators in registers; rescaled when a row's maximum moved
 // The eight partial results (maximum, sum, unnormalised latents) meet through distributed shared memory: CTA z folds its eighth of the latent for all
 // sixteen heads, with the sink as one more term of the denominator, and writes it.  No partials go through global memory and no merge launch follows.
 #include "kernels.h"
@@ -15,7 +15,7 @@ namespace b2 {
 namespace {
 
 constexpr int LD_SPLITS = 8;       // CTAs of a cluster: shares of the keys
-constexpr int LD_HEADS = 16, LD_KEYS = 64, LD_THREADS = 256;
+constexpr int LD_HEADS = 16, LD_KEYS = 32, LD_THREADS = 128, LD_WARPS = LD_THREADS / 32;
 constexpr int LD_SS = LD_KEYS + 8; // row stride of S and P
 
 __device__ __forceinline__ void ld_mma(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
@@ -64,9 +64,9 @@ inline size_t ld_smem(const LatentGeom& g, int pages_cap) {
   return (size_t)(LD_HEADS + 2 * LD_KEYS) * dp * 2 + (size_t)LD_HEADS * LD_SS * (4 + 2) + (size_t)(5 * LD_HEADS + LD_HEADS * LD_SPLITS) * 4 + (size_t)pages_cap * 4;
 }
 
-// NF: 16-wide pieces of the latent per warp (kv_rank <= 128 NF)
+// NF: 16-wide pieces of the latent per warp (kv_rank <= 64 NF)
 template <int NF>
-__global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(LatentDecodeArgs a) {
+__global__ void __launch_bounds__(LD_THREADS, 2) latent_decode_kernel(LatentDecodeArgs a) {
   extern __shared__ __align__(128) unsigned char smraw[];
   const LatentGeom& g = a.g;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -82,9 +82,13 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(LatentDeco
   float* wgt = row_f + 3 * LD_HEADS;                          // [16][8] weights of the shares
   int* pages = reinterpret_cast<int*>(wgt + LD_HEADS * LD_SPLITS);
   float* Os = reinterpret_cast<float*>(Ks);                   // after the sweep: [16][R16 + 4]
-  pdl_wait();
-  pdl_launch_dependents();
-  if (a.seq_lens[b] <= 0) return;   // (all CTAs of the cluster)
+  // Lengths, positions, the block table and the cached rows (the newest one too) are older than the kernel right before this one, which made the
+  // absorbed queries: the keys are on their way before the wait.
+  if (a.seq_lens[b] <= 0) {   // (all CTAs of the cluster)
+    pdl_wait();
+    pdl_launch_dependents();
+    return;
+  }
   const int pos = a.positions[b];
   // this CTA's keys: 16-key units [u0, u1) of the visible range
   const int lo = g.window > 0 ? max(0, pos - g.window + 1) : 0;
@@ -109,7 +113,24 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(LatentDeco
   };
   if (n_tiles > 0) issue(0);
   if (n_tiles > 1) issue(1);
+  pdl_wait();
+  pdl_launch_dependents();
   // queries, rounded to the operand type; columns past D and heads past the last one are zeros
+  if (D == D32 && R % 4 == 0) {   // eight threads per head row, four numbers at a time: independent loads, many in flight together
+    const int r = tid >> 3;
+    const size_t row = (size_t)b * g.heads + h0 + (r < nh ? r : 0);
+    const float4* qa = reinterpret_cast<const float4*>(a.q_abs + row * R);
+    const float4* qr = reinterpret_cast<const float4*>(a.q_rot + row * g.rot_dim);
+    const int r4 = R >> 2;
+#pragma unroll 9
+    for (int c = tid & 7; c < (D >> 2); c += 8) {
+      const float4 v = c < r4 ? __ldg(qa + c) : __ldg(qr + (c - r4));
+      uint2 pk;
+      pk.x = r < nh ? pack_bf16x2(v.x, v.y) : 0u;
+      pk.y = r < nh ? pack_bf16x2(v.z, v.w) : 0u;
+      *reinterpret_cast<uint2*>(Qs + r * DP + c * 4) = pk;
+    }
+  } else
   for (int i = tid; i < LD_HEADS * (D32 >> 1); i += LD_THREADS) {
     const int r = i / (D32 >> 1), d = (i - r * (D32 >> 1)) * 2;
     float v[2];
@@ -129,7 +150,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(LatentDeco
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int x = 0; x < 4; ++x) oacc[f][n][x] = 0.f;
-  const int sr = tid >> 4, sq = tid & 15;                     // softmax: head row, and which four keys
+  const int sr = tid >> 3, sq = tid & 7;                      // softmax: head row, and which four keys
   float m_run = -INFINITY, l_run = 0.f;
   const uint32_t q_addr = smem_u32(Qs) + (uint32_t)((lane & 15) * DP + (lane >> 4) * 8) * 2u;
   const uint32_t p_addr = smem_u32(Ps) + (uint32_t)((lane & 15) * LD_SS + (lane >> 4) * 8) * 2u;
@@ -171,7 +192,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(LatentDeco
         mx = fmaxf(mx, s[x]);
       }
 #pragma unroll
-      for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      for (int o = 4; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
       const float m_new = fmaxf(m_run, mx), f = m_run == -INFINITY ? 0.f : expf(m_run - m_new);
       float p[4], sum = 0.f;
 #pragma unroll
@@ -180,7 +201,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(LatentDeco
         sum += p[x];                                                                                  // that multiply the latents
       }
 #pragma unroll
-      for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      for (int o = 4; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
       l_run = l_run * f + sum;
       m_run = m_new;
       uint2 pk;
@@ -311,10 +332,11 @@ int launch_latent_decode(const float* q_abs, const float* q_rot, const bf16* cac
   const int pages_cap = ((max_context + 15) / 16 + LD_SPLITS - 1) / LD_SPLITS + 1;
   const LatentDecodeArgs a{q_abs, q_rot, cache, g, block_table, bt_stride, positions, seq_lens, sink, out_lat, pages_cap};
   const size_t smem = ld_smem(g, pages_cap);
-  const int nf = (g.kv_rank + 127) / 128;
+  const int nf = (g.kv_rank + 16 * LD_WARPS - 1) / (16 * LD_WARPS);
   if (nf <= 1) return launch_ld<1>(a, B, smem, s);
   if (nf == 2) return launch_ld<2>(a, B, smem, s);
-  return launch_ld<4>(a, B, smem, s);
+  if (nf <= 4) return launch_ld<4>(a, B, smem, s);
+  return launch_ld<8>(a, B, smem, s);
 }
 
 }  // namespace b2
