@@ -113,6 +113,7 @@ struct ListLayer {
   // the experts of every token id [vocab][top].
   float *bias1 = nullptr, *bias1b = nullptr, *bias2 = nullptr, *bias2b = nullptr, *latq_gain = nullptr;
   void* uq = nullptr;
+  bf16* router_op = nullptr;  // the router (and the gate's row) as a bf16 operand
   bf16* ukv = nullptr;        // key and value up-projections as one matrix [heads (dim + vdim)][kv_rank]: layers that rebuild keys and values
   int32_t* table = nullptr;
   // Norms behind the sublayers only (Tolanex): gain1b / gain2b.  Its delta mixer projects q | k | v | beta | decay | gate in `wqd` (off_sg = the
@@ -356,6 +357,7 @@ struct b2_engine {
   // sum of three embedding rows, output norms (Tolanex)
   void *l_bigram = nullptr, *l_pos = nullptr;
   int32_t* l_tok_ring = nullptr;     // [sequence slots][2]: the token at a position, by the position's parity (a sequence's previous token)
+  float* l_rz = nullptr;             // a prompt-sized step's router logits
   float* l_sg = nullptr;             // the shared expert's gate, one number per token row
   // Prompt portions whose latent attention runs over rebuilt keys and values (attn_latent.cu): the step's long portions in groups whose contexts
   // fit the scratch pools; a paired tile list, a block table of scratch pages and the contexts of each group.  d_tiles holds the short portions' tiles first.
@@ -953,8 +955,21 @@ int list_dense(b2_engine* e, const void* A, const void* Wt, float* C, int M, int
 // up sums (l_upf, fp32, expert order) -> act(operand is fp32?) -> l_act -> l_y (fp32, expert order).  The permutation (l_offsets,
 // l_slot_token) is in place.  Prompt-sized bf16 steps (prompt = true) run expert by expert on the tcgen05 projection kernel: rows gathered into
 // expert order, the experts' slot ranges read back (one small copy and a stream synchronisation per layer); everything else as ragged groups.
+// plain_silu: the activation is silu(gate) * up as it is, so the gate/up products that have it in their epilogue may be used.
+bool list_gate_up_fused(int M, int F, int W) {
+  static const bool on = [] { const char* v = getenv("B2_LIST_GU_FUSED"); return !(v && *v == '0'); }();
+  return on && list_use_tc() && gateup_prefill_shapes_ok(M, F, W);
+}
+// act (bf16 [M][F]) = silu(A . Wgu[0..F)^T) * (A . Wgu[F..2F)^T) for prompt-sized M (gemm_gateup.cu)
+int list_gate_up(const bf16* A, const bf16* Wgu, bf16* act, int M, int F, int W, cudaStream_t s) {
+  CUtensorMap tw, tx;
+  B2_TRY(b2_make_tmap_bf16(&tw, Wgu, (uint64_t)2 * F, (uint64_t)W, (uint64_t)W, 128));
+  B2_TRY(b2_make_tmap_bf16(&tx, A, (uint64_t)M, (uint64_t)W, (uint64_t)W, 128));
+  return launch_gateup_swiglu_prefill(tw, tx, act, M, F, W, 0, s);
+}
+
 template <typename Act>
-int list_gated_experts(b2_engine* e, const ListLayer& L, int layer, int T, bool prompt, cudaStream_t s, Act act) {
+int list_gated_experts(b2_engine* e, const ListLayer& L, int layer, int T, bool prompt, cudaStream_t s, Act act, bool plain_silu = false) {
   const b2_layer_spec& sp = L.sp;
   const int W = e->cfg.hidden, f = e->f32 ? 1 : 0, F = sp.ff_dim, pairs = T * sp.top;
   const bool tc_experts = prompt && list_use_tc() && !f && e->l_xperm != nullptr && pairs >= LIST_TC_EXPERT_ROWS && W % 64 == 0 && F % 64 == 0 && W >= 128 &&
@@ -970,12 +985,19 @@ int list_gated_experts(b2_engine* e, const ListLayer& L, int layer, int T, bool 
     B2_REQUIRE(off[0] == 0 && off[sp.experts] == pairs, "layer %d: the experts' slot ranges do not cover the step's %d pairs", layer, pairs);
     {
       KL k(e, B2K_GEMM_GATEUP);
-      for (int x = 0; x < sp.experts; ++x)
-        if (off[x + 1] > off[x])
-          B2_TRY(list_dense(e, e->l_xperm + (size_t)off[x] * W, (const bf16*)L.up + (size_t)x * 2 * F * W, e->l_upf + (size_t)off[x] * 2 * F,
-                            off[x + 1] - off[x], 2 * F, W, 1.f, s));
+      for (int x = 0; x < sp.experts; ++x) {
+        const int n = off[x + 1] - off[x];
+        const bf16 *xa = e->l_xperm + (size_t)off[x] * W, *wu = (const bf16*)L.up + (size_t)x * 2 * F * W;
+        if (n == 0) continue;
+        if (plain_silu && list_gate_up_fused(n, F, W)) {
+          B2_TRY(list_gate_up(xa, wu, (bf16*)e->l_act + (size_t)off[x] * F, n, F, W, s));
+          continue;
+        }
+        B2_TRY(list_dense(e, xa, wu, e->l_upf + (size_t)off[x] * 2 * F, n, 2 * F, W, 1.f, s));
+        if (plain_silu) B2_TRY(launch_silu_gate(e->l_upf + (size_t)off[x] * 2 * F, nullptr, nullptr, (bf16*)e->l_act + (size_t)off[x] * F, 0, n, F, s));
+      }
     }
-    {
+    if (!plain_silu) {
       KL k(e, B2K_ACT);
       B2_TRY(act(0));
     }
@@ -994,14 +1016,19 @@ int list_gated_experts(b2_engine* e, const ListLayer& L, int layer, int T, bool 
     if (!k.skip()) B2_TRY(launch_ragged_tiles(e->l_offsets, sp.experts, e->l_tile_group, e->l_tile_row0, e->l_ntiles, max_tiles, s));
   }
   AnyGemm a;
+  bool fused_act = false;
   a.tile_group = e->l_tile_group; a.tile_row0 = e->l_tile_row0; a.n_tiles = e->l_ntiles; a.group_offsets = e->l_offsets;
   {
     KL k(e, B2K_GEMM_GATEUP);  // gate | up of every (token, choice) pair in expert order, fp32 sums
     a.A = e->l_x1; a.a_rows = e->l_slot_token; a.W = L.up; a.C = e->l_upf; a.N = 2 * F; a.K = W; a.lda = W; a.ldw = W; a.ldc = 2 * F;
     a.w_bs = (long)2 * F * W; a.epilogue = ANY_EPI_STORE;
-    if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, 1, 1, max_tiles, s, pairs, sp.experts));
+    fused_act = plain_silu && !f && any_gemm_silu_pair_ok(a, pairs, 1);
+    if (fused_act) {
+      a.C = e->l_act; a.ldc = F; a.epilogue = ANY_EPI_SILU_PAIR;
+    }
+    if (!k.skip()) B2_TRY(launch_gemm_any(a, f, f, fused_act ? 0 : 1, 1, max_tiles, s, pairs, sp.experts));
   }
-  {
+  if (!fused_act) {
     KL k(e, B2K_ACT);
     if (!k.skip()) B2_TRY(act(f));
   }
@@ -1855,11 +1882,20 @@ int forward_outnorm_list(b2_engine* e, int T, int ntiles, int nlast) {
       cudaStream_t sS = multi && shared ? e->l_side[0] : st;
       auto shared_expert = [&]() -> int {   // (buffers of its own: in short steps it runs beside the routed experts)
         if (sS != st) b2_pdl_skip_next();   // behind a cross-stream edge: an ordinary, full dependency
-        {
+        AnyGemm a;
+        a.A = e->l_x1; a.W = L.sh_up; a.C = e->l_act2; a.M = T; a.N = 2 * sp.shared_ff; a.K = W; a.lda = W; a.ldw = W; a.ldc = sp.shared_ff;
+        a.epilogue = ANY_EPI_SILU_PAIR;
+        if (!f && any_gemm_silu_pair_ok(a, T, 0)) {
           KL k(e, B2K_GEMM_GATEUP);
-          if (!k.skip()) B2_TRY(dense(e->l_x1, L.sh_up, e->l_upf2, T, 2 * sp.shared_ff, W, sS));
-        }
-        {
+          if (!k.skip()) B2_TRY(launch_gemm_any(a, 0, 0, 0, 1, 0, sS));
+        } else if (!f && list_gate_up_fused(T, sp.shared_ff, W)) {
+          KL k(e, B2K_GEMM_GATEUP);
+          if (!k.skip()) B2_TRY(list_gate_up((const bf16*)e->l_x1, (const bf16*)L.sh_up, (bf16*)e->l_act2, T, sp.shared_ff, W, sS));
+        } else {
+          {
+            KL k(e, B2K_GEMM_GATEUP);
+            if (!k.skip()) B2_TRY(dense(e->l_x1, L.sh_up, e->l_upf2, T, 2 * sp.shared_ff, W, sS));
+          }
           KL k(e, B2K_ACT);
           if (!k.skip()) B2_TRY(launch_silu_gate(e->l_upf2, nullptr, nullptr, e->l_act2, f, T, sp.shared_ff, sS));
         }
@@ -1878,14 +1914,24 @@ int forward_outnorm_list(b2_engine* e, int T, int ntiles, int nlast) {
       }
       {
         KL k(e, B2K_ACT);
-        if (!k.skip()) B2_TRY(launch_route(e->l_x1, f, L.router, nullptr, rg, e->l_idx, e->l_rw, T, W, st, shared ? e->l_sg : nullptr));
+        // Prompt-sized bf16 steps form the logits as a product of bf16 operands: a checkpoint's router is bf16, so every product of two operands is
+        // exact and only the fp32 sums' order differs.
+        const int er = sp.experts + (shared ? 1 : 0);
+        if (L.router_op != nullptr && T >= 512 && !k.skip()) {
+          AnyGemm a;
+          a.A = e->l_x1; a.W = L.router_op; a.C = e->l_rz; a.M = T; a.N = er; a.K = W; a.lda = W; a.ldw = W; a.ldc = er;
+          B2_TRY(launch_gemm_any(a, 0, 0, 1, 1, 0, st));
+          B2_TRY(launch_route_select(e->l_rz, er, nullptr, rg, e->l_idx, e->l_rw, T, st, shared ? e->l_sg : nullptr));
+        } else if (!k.skip()) {
+          B2_TRY(launch_route(e->l_x1, f, L.router, nullptr, rg, e->l_idx, e->l_rw, T, W, st, shared ? e->l_sg : nullptr));
+        }
       }
       {
         KL k(e, B2K_MISC);
         if (!k.skip()) B2_TRY(launch_route_permute(e->l_idx, T, sp.top, sp.experts, e->l_offsets, e->l_offsets_stride, e->l_slot_token, e->l_pair_slot, st));
       }
       B2_TRY(list_gated_experts(e, L, l, T, ntiles > 0 && !multi, st,
-                                [&](int act_f32) { return launch_silu_gate(e->l_upf, nullptr, nullptr, e->l_act, act_f32, pairs, F, st); }));
+                                [&](int act_f32) { return launch_silu_gate(e->l_upf, nullptr, nullptr, e->l_act, act_f32, pairs, F, st); }, true));
       if (sS == st && shared) B2_TRY(shared_expert());
       if (sS != st) {
         B2_CUDA_OK(cudaStreamWaitEvent(st, e->l_ev[1], 0));
@@ -2557,8 +2603,16 @@ int list_tensor(b2_engine* e, const std::string& name, const void* host, size_t 
     }
     if (sp.ff == B2_FF_SOFTMAX_EXPERTS) {
       const size_t sf = sp.shared_ff, ne = sp.experts;
-      if (rest == "mlp.router") { B2_TRY(want(ne * W)); return done(put_f32(L.router, src, ne * W, 0.0f)); }
-      if (sf > 0 && rest == "mlp.shared.sg") { B2_TRY(want(W)); return done(put_f32(L.router + ne * W, src, W, 0.0f)); }
+      if (rest == "mlp.router") {
+        B2_TRY(want(ne * W));
+        if (L.router_op) B2_TRY(put_operand(e, L.router_op, 0, src, ne * W));
+        return done(put_f32(L.router, src, ne * W, 0.0f));
+      }
+      if (sf > 0 && rest == "mlp.shared.sg") {
+        B2_TRY(want(W));
+        if (L.router_op) B2_TRY(put_operand(e, L.router_op, ne * W, src, W));
+        return done(put_f32(L.router + ne * W, src, W, 0.0f));
+      }
       if (sf > 0 && rest == "mlp.shared.gate") { B2_TRY(want(sf * W)); return done(put_operand(e, L.sh_up, 0, src, sf * W)); }
       if (sf > 0 && rest == "mlp.shared.up") { B2_TRY(want(sf * W)); return done(put_operand(e, L.sh_up, sf * W, src, sf * W)); }
       if (sf > 0 && rest == "mlp.shared.down") { B2_TRY(want(W * sf)); return done(put_operand(e, L.sh_down, 0, src, W * sf)); }
@@ -3447,6 +3501,11 @@ int outnorm_engine_alloc(b2_engine* e) {
                  "layer %d: bad router sizes (experts %d, top %d, groups %d, keep %d, ff %d)", l, sp.experts, sp.top, sp.groups, sp.groups_keep, sp.ff_dim);
       B2_TRY(falloc(&L.gain2b, W));
       B2_TRY(falloc(&L.router, (size_t)(sp.experts + (sp.shared_ff > 0 ? 1 : 0)) * W));
+      if (!e->f32) {
+        char* q = nullptr;
+        B2_TRY(dalloc(&q, (size_t)(sp.experts + 1) * W * es));
+        L.router_op = reinterpret_cast<bf16*>(q);
+      }
       B2_TRY(xalloc(&L.up, (size_t)sp.experts * 2 * sp.ff_dim * W));
       B2_TRY(xalloc(&L.down, (size_t)sp.experts * W * sp.ff_dim));
       if (sp.shared_ff > 0) {
@@ -3531,6 +3590,7 @@ int outnorm_engine_alloc(b2_engine* e) {
     }
     B2_TRY(dalloc(&e->l_rw, Tc * max_top));
     B2_TRY(dalloc(&e->l_sg, Tc));
+    if (!e->f32) B2_TRY(dalloc(&e->l_rz, Tc * (size_t)(max_exp + 1)));
     B2_TRY(dalloc(&e->l_idx, Tc * max_top));
     e->l_offsets_stride = max_exp + 1;
     B2_TRY(dalloc(&e->l_offsets, (size_t)3 * (max_exp + 1)));
@@ -4451,7 +4511,7 @@ extern "C" void b2_engine_free(b2_engine* e) {
   if (e->h_xtiles) cudaFreeHost(e->h_xtiles);
   if (e->h_xctx) cudaFreeHost(e->h_xctx);
   if (e->h_xtable) cudaFreeHost(e->h_xtable);
-  F(e->l_final_bias); F(e->l_bigram); F(e->l_pos); F(e->l_tok_ring); F(e->l_sg);
+  F(e->l_final_bias); F(e->l_bigram); F(e->l_pos); F(e->l_tok_ring); F(e->l_sg); F(e->l_rz);
   F(e->l_embed); F(e->l_head); F(e->l_embed_gain); F(e->l_final_gain); F(e->l_pool); F(e->l_h); F(e->l_qd); F(e->l_qrot); F(e->l_qabs);
   F(e->l_xperm); F(e->l_upf); if (e->h_offsets) cudaFreeHost(e->h_offsets);
   F(e->l_q); F(e->l_vfirst); F(e->l_cross); F(e->l_qb); F(e->d_row_seq); F(e->d_row_first); F(e->d_row_end);
@@ -4461,7 +4521,7 @@ extern "C" void b2_engine_free(b2_engine* e) {
     F(L.wqd); F(L.ukT); F(L.uv); F(L.wo); F(L.up); F(L.down); F(L.gain1); F(L.gain2); F(L.lat_gain); F(L.sink); F(L.router); F(L.corr);
     F(L.gain1b); F(L.gain2b); F(L.qkv_bias); F(L.o_bias); F(L.conv_w); F(L.talk); F(L.vmix); F(L.conv_ring);
     F(L.wo2); F(L.sh_up); F(L.sh_down); F(L.qk_gain); F(L.head_gain); F(L.a2); F(L.a2_bias); F(L.g2); F(L.a_log); F(L.out_gain_l); F(L.out_gain_r); F(L.poly);
-    F(L.bias1); F(L.bias1b); F(L.bias2); F(L.bias2b); F(L.latq_gain); F(L.uq); F(L.ukv); F(L.table);
+    F(L.bias1); F(L.bias1b); F(L.bias2); F(L.bias2b); F(L.latq_gain); F(L.uq); F(L.ukv); F(L.router_op); F(L.table);
   }
   for (auto& R : e->runs) {
     F(R.state); F(R.ring);

@@ -447,29 +447,41 @@ __device__ __forceinline__ void mma_16816(float* d, unsigned a0, unsigned a1, un
 template <typename TC, int NT, int U, int NW>
 __global__ void __launch_bounds__(32 * NW) gemm_any_rows_mma_kernel(AnyGemm g) {
   __shared__ float red[NW][NT][32][4];
-  pdl_wait();
-  pdl_launch_dependents();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, c = lane & 3;
   const bf16* A = reinterpret_cast<const bf16*>(g.A);
   const bf16* W = reinterpret_cast<const bf16*>(g.W);
   TC* C = reinterpret_cast<TC*>(g.C);
+  const bool ragged = g.group_offsets != nullptr, pair = g.epilogue == ANY_EPI_SILU_PAIR;
+  const int K = g.K, n0 = blockIdx.x * (pair ? 8 : 16), N = pair ? g.N / 2 : g.N;   // pair: N gate rows, then N up rows; a CTA owns 8 of each
+  W += (size_t)(ragged ? blockIdx.y : blockIdx.z) * g.w_bs;
+  const bf16* w_lo = W + (long)min(n0 + gq, N - 1) * g.ldw + c * 8;       // rows past N are read again and dropped at the store
+  const bf16* w_hi = W + (long)(pair ? N + min(n0 + gq, N - 1) : min(n0 + gq + 8, N - 1)) * g.ldw + c * 8;
+  const int nchunk = (K + 31) >> 5;
+  uint4 wl[U], wh[U];
+  auto load_w = [&](int ch0) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int k = (ch0 + NW * u) << 5;
+      const bool in = k + c * 8 < K;   // K is a multiple of 8: a lane's eight elements are inside or outside together
+      wl[u] = in ? ld_stream(w_lo + k) : make_uint4(0, 0, 0, 0);
+      wh[u] = in ? ld_stream(w_hi + k) : make_uint4(0, 0, 0, 0);
+    }
+  };
+  bool have_w = !ragged;
+  if (have_w) load_w(warp);   // weights are constants: the first ones are on their way before the kernel in front has finished
+  pdl_wait();
+  pdl_launch_dependents();
   int row_lo, row_hi;
   if (g.group_offsets != nullptr) {   // ragged: blockIdx.y = group
     row_lo = g.group_offsets[blockIdx.y];
     row_hi = g.group_offsets[blockIdx.y + 1];
     if (row_lo >= row_hi) return;
-    W += (size_t)blockIdx.y * g.w_bs;
   } else {
     row_lo = 0;
     row_hi = g.M;
     A += (size_t)blockIdx.z * g.a_bs;
-    W += (size_t)blockIdx.z * g.w_bs;
     C += (size_t)blockIdx.z * g.c_bs;
   }
-  const int K = g.K, n0 = blockIdx.x * 16;
-  const bf16* w_lo = W + (long)min(n0 + gq, g.N - 1) * g.ldw + c * 8;       // rows past N are read again and dropped at the store
-  const bf16* w_hi = W + (long)min(n0 + gq + 8, g.N - 1) * g.ldw + c * 8;
-  const int nchunk = (K + 31) >> 5;
   for (int r0 = row_lo; r0 < row_hi; r0 += 8 * NT) {
     const bf16* tok[NT];
 #pragma unroll
@@ -483,13 +495,13 @@ __global__ void __launch_bounds__(32 * NW) gemm_any_rows_mma_kernel(AnyGemm g) {
 #pragma unroll
       for (int i = 0; i < 4; ++i) acc[t][i] = 0.f;
     for (int ch0 = warp; ch0 < nchunk; ch0 += NW * U) {
-      uint4 wl[U], wh[U], tv[U][NT];
+      uint4 tv[U][NT];
+      if (!have_w) load_w(ch0);
+      have_w = false;
 #pragma unroll
       for (int u = 0; u < U; ++u) {
         const int k = (ch0 + NW * u) << 5;
-        const bool in = k + c * 8 < K;   // K is a multiple of 8: a lane's eight elements are inside or outside together
-        wl[u] = in ? ld_stream(w_lo + k) : make_uint4(0, 0, 0, 0);
-        wh[u] = in ? ld_stream(w_hi + k) : make_uint4(0, 0, 0, 0);
+        const bool in = k + c * 8 < K;
 #pragma unroll
         for (int t = 0; t < NT; ++t)
           tv[u][t] = (in && tok[t] != nullptr) ? __ldg(reinterpret_cast<const uint4*>(tok[t] + k)) : make_uint4(0, 0, 0, 0);
@@ -508,6 +520,25 @@ __global__ void __launch_bounds__(32 * NW) gemm_any_rows_mma_kernel(AnyGemm g) {
       *reinterpret_cast<float4*>(&red[warp][t][lane][0]) = make_float4(acc[t][0], acc[t][1], acc[t][2], acc[t][3]);
     __syncthreads();
     // fragment element i of lane (g, c): weight row g + 8 * (i / 2), token row 2c + (i % 2)
+    if (pair) {   // rows 0..7 of the tile are gate rows, rows 8..15 the up rows of the same features
+      for (int idx = tid; idx < NT * 64; idx += 32 * NW) {
+        const int t = idx >> 6, rem = idx & 63, wr = rem & 7, tk = rem >> 3, ln = wr * 4 + (tk >> 1), i = tk & 1;
+        const int r = r0 + t * 8 + tk, n = n0 + wr;
+        if (r >= row_hi || n >= N) continue;
+        float gt = ((red[0][t][ln][i] + red[1][t][ln][i]) + red[2][t][ln][i]) + red[3][t][ln][i];
+        float up = ((red[0][t][ln][i + 2] + red[1][t][ln][i + 2]) + red[2][t][ln][i + 2]) + red[3][t][ln][i + 2];
+#pragma unroll
+        for (int w = 4; w < NW; ++w) {
+          gt += red[w][t][ln][i];
+          up += red[w][t][ln][i + 2];
+        }
+        const float v = gt / (1.0f + expf(-gt)) * up;
+        TC* dst = C + (size_t)r * g.ldc + n;
+        if constexpr (sizeof(TC) == 4) *dst = v;
+        else *dst = __float2bfloat16_rn(v);
+      }
+      continue;
+    }
     for (int idx = tid; idx < NT * 128; idx += 32 * NW) {
       const int t = idx >> 7, rem = idx & 127, wr = rem & 15, tk = rem >> 4;   // consecutive threads -> consecutive weight rows
       const int ln = (wr & 7) * 4 + (tk >> 1), i = (wr >> 3) * 2 + (tk & 1);
@@ -540,7 +571,7 @@ inline bool rows_mma_ok(const AnyGemm& g) {
 
 template <typename TC>
 int launch_rows_mma(const AnyGemm& g, int groups, int batch, cudaStream_t s) {
-  const dim3 grid((g.N + 15) / 16, groups > 0 ? groups : 1, groups > 0 ? 1 : (batch > 0 ? batch : 1));
+  const dim3 grid(g.epilogue == ANY_EPI_SILU_PAIR ? (g.N / 2 + 7) / 8 : (g.N + 15) / 16, groups > 0 ? groups : 1, groups > 0 ? 1 : (batch > 0 ? batch : 1));
   // rows per pass: a ragged group's count is only known on the device (16 covers the usual handful per expert; more rows
   // take more passes over weights that are then in L2)
   const int rows = groups > 0 ? 16 : g.M;
@@ -586,6 +617,18 @@ int any_gemm_ragged_rows_limit() {
   return use_rows ? 8 * RB : 0;
 }
 
+// does a launch with this many rows (of all groups together, when ragged) take the form that has the gate/up epilogue?
+bool any_gemm_silu_pair_ok(const AnyGemm& g, int rows, int ragged) {
+  static const bool on = [] {
+    for (const char* n : {"B2_ANY_ROWS", "B2_ANY_ROWS_MMA", "B2_ANY_SILU"}) {
+      const char* e = getenv(n);
+      if (e && *e == '0') return false;
+    }
+    return true;
+  }();
+  return on && rows > 0 && rows <= (ragged ? 8 : 4) * RB && g.K <= 16384 && g.N % 2 == 0 && rows_mma_ok(g);
+}
+
 int launch_ragged_tiles(const int* group_offsets, int G, int* tile_group, int* tile_row0, int* n_tiles, int cap, cudaStream_t s) {
   B2_CUDA_OK(b2_launch(ragged_tiles_kernel, dim3(1), dim3(32), 0, s, group_offsets, G, tile_group, tile_row0, n_tiles, cap));
   return 0;
@@ -593,6 +636,8 @@ int launch_ragged_tiles(const int* group_offsets, int G, int* tile_group, int* t
 
 int launch_gemm_any(const AnyGemm& g, int a_f32, int w_f32, int c_f32, int batch, int max_tiles, cudaStream_t s, int ragged_rows, int groups) {
   if (g.N <= 0 || g.K <= 0) return 0;
+  B2_REQUIRE(g.epilogue != ANY_EPI_SILU_PAIR || any_gemm_silu_pair_ok(g, g.tile_group != nullptr ? ragged_rows : g.M, g.tile_group != nullptr),
+             "gemm_any: the gate/up epilogue is built for few rows of bf16 operands");
   B2_REQUIRE(g.epilogue != ANY_EPI_ADD || c_f32, "gemm_any: the add epilogue needs an fp32 C");
   {  // few rows: stream the weights (rows of every group counted together for the ragged form: they bound the work per group)
     static const bool use_rows = [] { const char* e = getenv("B2_ANY_ROWS"); return !(e && *e == '0'); }();

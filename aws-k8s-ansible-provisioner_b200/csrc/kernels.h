@@ -216,7 +216,12 @@ int launch_sample_rows(const bf16* logits, const SampleRow* rows_host, SampleRow
 int device_num_sms();
 
 // ---- gemm_any.cu: C = A . W^T for any shape, bf16 or fp32 operands, strided batch or ragged groups ----
-enum AnyEpilogue { ANY_EPI_STORE = 0, ANY_EPI_RELU2 = 1, ANY_EPI_ADD = 2 };
+enum AnyEpilogue {
+  ANY_EPI_STORE = 0,
+  ANY_EPI_RELU2 = 1,
+  ANY_EPI_ADD = 2,
+  ANY_EPI_SILU_PAIR = 3   // W holds N/2 gate rows, then N/2 up rows: C [rows][N/2] = silu(gate) * up (few rows of bf16 operands: any_gemm_silu_pair_ok)
+};
 struct AnyGemm {
   const void* A = nullptr;   // [rows][lda]
   const void* W = nullptr;   // [N][ldw]
@@ -232,6 +237,7 @@ struct AnyGemm {
   int epilogue = ANY_EPI_STORE;
   float alpha = 1.f;
 };
+bool any_gemm_silu_pair_ok(const AnyGemm& g, int rows, int ragged);
 int any_gemm_tile_rows();
 int any_gemm_ragged_rows_limit();
 int launch_ragged_tiles(const int* group_offsets, int G, int* tile_group, int* tile_row0, int* n_tiles, int cap, cudaStream_t s);
@@ -466,6 +472,9 @@ struct RouteGeom {
 // gate_out != null: the router has one more row, and gate_out [T] = sigmoid of its product with x
 int launch_route(const void* x, int x_f32, const float* router, const float* correction, const RouteGeom& g, int32_t* idx, float* weight,
                  int T, int W, cudaStream_t s, float* gate_out = nullptr);
+// The same from logits that a product has formed already: z [T][ld] = experts' logits (and the gate's behind them when gate_out is given)
+int launch_route_select(const float* z, int ld, const float* correction, const RouteGeom& g, int32_t* idx, float* weight, int T, cudaStream_t s,
+                        float* gate_out = nullptr);
 // no router: idx[t][k] = table[ids[t]][k] (table [vocab][top] int32, entries clamped into [0, experts)), weight[t][k] = 1 / top
 int launch_route_table(const int32_t* ids, const int32_t* table, int vocab, int experts, int top, int32_t* idx, float* weight, int T, cudaStream_t s);
 // counting sort of the T*top (token, choice) pairs by expert: offsets [experts + 1] (the buffer holds 3 * stride ints,

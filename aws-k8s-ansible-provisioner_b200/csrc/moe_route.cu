@@ -19,63 +19,11 @@ namespace b2 {
 
 namespace {
 
-constexpr int RT_WARPS = 16;
-
-// A CTA takes NTOK tokens: their rows are staged once as fp32, warp w takes router rows w, w + 16, ... (a row is read once for all tokens of
-// the CTA), then one warp per token forms the scores and selects.  A token's arithmetic does not depend on NTOK.
-template <typename TX, int NTOK>
-__global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const TX* __restrict__ x, const float* __restrict__ router,
-                                                              const float* __restrict__ correction, RouteGeom g, int32_t* __restrict__ idx,
-                                                              float* __restrict__ weight, int T, int W, float* __restrict__ gate_out) {
-  extern __shared__ __align__(16) float sm[];  // x rows [NTOK][W rounded up to 4] (read as float4), then per token: s [E + 1], choice [E], group scores [groups]
-  pdl_wait();
-  pdl_launch_dependents();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t0 = blockIdx.x * NTOK, tn = min(NTOK, T - t0);
-  const int E = g.experts, ER = E + (gate_out != nullptr ? 1 : 0), Wp = (W + 3) & ~3, per_tok = 2 * E + 1 + g.groups;
-  float* xs = sm;
-  float* sc = xs + NTOK * Wp;
-  for (int i = threadIdx.x; i < NTOK * W; i += RT_WARPS * 32) {
-    const int tt = i / W, c = i - tt * W;
-    xs[tt * Wp + c] = tt < tn ? (float)x[(size_t)(t0 + tt) * W + c] : 0.f;
-  }
-  __syncthreads();
-  const bool vec = (W % 4 == 0);
-  for (int e = warp; e < ER; e += RT_WARPS) {
-    const float* rr = router + (size_t)e * W;
-    float acc[NTOK];
-#pragma unroll
-    for (int tt = 0; tt < NTOK; ++tt) acc[tt] = 0.f;
-    if (vec) {
-#pragma unroll 8
-      for (int i = lane * 4; i < W; i += 128) {
-        const float4 r4 = *reinterpret_cast<const float4*>(rr + i);
-#pragma unroll
-        for (int tt = 0; tt < NTOK; ++tt) {
-          const float4 x4 = *reinterpret_cast<const float4*>(xs + tt * Wp + i);
-          acc[tt] = fmaf(x4.x, r4.x, acc[tt]); acc[tt] = fmaf(x4.y, r4.y, acc[tt]); acc[tt] = fmaf(x4.z, r4.z, acc[tt]); acc[tt] = fmaf(x4.w, r4.w, acc[tt]);
-        }
-      }
-    } else {
-      for (int i = lane; i < W; i += 32) {
-        const float r = rr[i];
-#pragma unroll
-        for (int tt = 0; tt < NTOK; ++tt) acc[tt] = fmaf(xs[tt * Wp + i], r, acc[tt]);
-      }
-    }
-#pragma unroll
-    for (int tt = 0; tt < NTOK; ++tt) {
-      const float z = warp_sum(acc[tt]);
-      if (lane == 0) sc[tt * per_tok + e] = (g.softmax && e < E) ? z : 1.0f / (1.0f + expf(-z));   // (the extra row is a gate: always a sigmoid)
-    }
-  }
-  __syncthreads();
-  if (warp >= tn) return;
-  const int t = t0 + warp;
-  float* s = sc + warp * per_tok;
-  float* ch = s + E + 1;
-  float* gs = ch + E;
-  if (gate_out != nullptr && lane == 0) gate_out[t] = s[E];
+// One warp: a token's router products s [E] (and, with a softmax, still logits) become scores, the choices and their weights.  ch [E] and
+// gs [groups] are the warp's scratch in shared memory.
+__device__ void route_pick(float* s, float* ch, float* gs, const RouteGeom& g, const float* __restrict__ correction, int t, int32_t* __restrict__ idx,
+                           float* __restrict__ weight) {
+  const int lane = threadIdx.x & 31, E = g.experts;
   if (g.softmax) {
     float m = -INFINITY, sum = 0.f;
     for (int e = lane; e < E; e += 32) m = fmaxf(m, s[e]);
@@ -140,6 +88,80 @@ __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const TX* __restri
   const float inv = 1.0f / (sum + 1e-20f);
   if (lane == 0)
     for (int k = 0; k < g.top; ++k) weight[(size_t)t * g.top + k] *= inv;
+}
+
+// A CTA takes NTOK tokens: their rows are staged once as fp32, warp w takes router rows w, w + 16, ... (a row is read once for all tokens of
+// the CTA), then one warp per token forms the scores and selects.  A token's arithmetic does not depend on NTOK.
+template <typename TX, int NTOK, int RT_WARPS>
+__global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const TX* __restrict__ x, const float* __restrict__ router,
+                                                              const float* __restrict__ correction, RouteGeom g, int32_t* __restrict__ idx,
+                                                              float* __restrict__ weight, int T, int W, float* __restrict__ gate_out) {
+  extern __shared__ __align__(16) float sm[];  // x rows [NTOK][W rounded up to 4] (read as float4), then per token: s [E + 1], choice [E], group scores [groups]
+  pdl_wait();
+  pdl_launch_dependents();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t0 = blockIdx.x * NTOK, tn = min(NTOK, T - t0);
+  const int E = g.experts, ER = E + (gate_out != nullptr ? 1 : 0), Wp = (W + 3) & ~3, per_tok = 2 * E + 1 + g.groups;
+  float* xs = sm;
+  float* sc = xs + NTOK * Wp;
+  for (int i = threadIdx.x; i < NTOK * W; i += RT_WARPS * 32) {
+    const int tt = i / W, c = i - tt * W;
+    xs[tt * Wp + c] = tt < tn ? (float)x[(size_t)(t0 + tt) * W + c] : 0.f;
+  }
+  __syncthreads();
+  const bool vec = (W % 4 == 0);
+  for (int e = warp; e < ER; e += RT_WARPS) {
+    const float* rr = router + (size_t)e * W;
+    float acc[NTOK];
+#pragma unroll
+    for (int tt = 0; tt < NTOK; ++tt) acc[tt] = 0.f;
+    if (vec) {
+#pragma unroll 8
+      for (int i = lane * 4; i < W; i += 128) {
+        const float4 r4 = *reinterpret_cast<const float4*>(rr + i);
+#pragma unroll
+        for (int tt = 0; tt < NTOK; ++tt) {
+          const float4 x4 = *reinterpret_cast<const float4*>(xs + tt * Wp + i);
+          acc[tt] = fmaf(x4.x, r4.x, acc[tt]); acc[tt] = fmaf(x4.y, r4.y, acc[tt]); acc[tt] = fmaf(x4.z, r4.z, acc[tt]); acc[tt] = fmaf(x4.w, r4.w, acc[tt]);
+        }
+      }
+    } else {
+      for (int i = lane; i < W; i += 32) {
+        const float r = rr[i];
+#pragma unroll
+        for (int tt = 0; tt < NTOK; ++tt) acc[tt] = fmaf(xs[tt * Wp + i], r, acc[tt]);
+      }
+    }
+#pragma unroll
+    for (int tt = 0; tt < NTOK; ++tt) {
+      const float z = warp_sum(acc[tt]);
+      if (lane == 0) sc[tt * per_tok + e] = (g.softmax && e < E) ? z : 1.0f / (1.0f + expf(-z));   // (the extra row is a gate: always a sigmoid)
+    }
+  }
+  __syncthreads();
+  if (warp >= tn) return;
+  const int t = t0 + warp;
+  float* s = sc + warp * per_tok;
+  float* ch = s + E + 1;
+  float* gs = ch + E;
+  if (gate_out != nullptr && lane == 0) gate_out[t] = s[E];
+  route_pick(s, ch, gs, g, correction, t, idx, weight);
+}
+
+// The same behind a product that has formed the logits z [T][ld] already (experts, then the gate's): one warp per token.
+__global__ void __launch_bounds__(256) route_select_kernel(const float* __restrict__ z, int ld, const float* __restrict__ correction, RouteGeom g,
+                                                           int32_t* __restrict__ idx, float* __restrict__ weight, int T, float* __restrict__ gate_out) {
+  extern __shared__ __align__(16) float sm[];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 8 + warp, E = g.experts;
+  if (t >= T) return;
+  float* s = sm + warp * (2 * E + g.groups);
+  const float* zr = z + (size_t)t * ld;
+  for (int e = lane; e < E; e += 32) s[e] = g.softmax ? zr[e] : 1.0f / (1.0f + expf(-zr[e]));
+  if (gate_out != nullptr && lane == 0) gate_out[t] = 1.0f / (1.0f + expf(-zr[E]));
+  __syncwarp();
+  route_pick(s, s + E, s + 2 * E, g, correction, t, idx, weight);
 }
 
 // the permutation in three steps: histogram (any number of CTAs), scan (one thread; experts are few), placement
@@ -311,7 +333,7 @@ int launch_route(const void* x, int x_f32, const float* router, const float* cor
   // prompt-sized steps: several tokens per CTA share one pass over the router's rows
   const int ntok = T >= 1024 && bytes(4) <= 48 * 1024 ? 4 : T >= 512 && bytes(2) <= 48 * 1024 ? 2 : 1;
   const dim3 grid((T + ntok - 1) / ntok);
-#define B2_ROUTE(TX, N) B2_CUDA_OK(b2_launch(route_kernel<TX, N>, grid, dim3(RT_WARPS * 32), bytes(N), s, (const TX*)x, router, correction, g, idx, weight, T, W, gate_out))
+#define B2_ROUTE(TX, N) B2_CUDA_OK(b2_launch(route_kernel<TX, N, (N == 1 ? 32 : 16)>, grid, dim3(N == 1 ? 1024 : 512), bytes(N), s, (const TX*)x, router, correction, g, idx, weight, T, W, gate_out))
   if (x_f32) {
     if (ntok == 4) B2_ROUTE(float, 4);
     else if (ntok == 2) B2_ROUTE(float, 2);
@@ -322,6 +344,17 @@ int launch_route(const void* x, int x_f32, const float* router, const float* cor
     else B2_ROUTE(bf16, 1);
   }
 #undef B2_ROUTE
+  return 0;
+}
+
+int launch_route_select(const float* z, int ld, const float* correction, const RouteGeom& g, int32_t* idx, float* weight, int T, cudaStream_t s, float* gate_out) {
+  if (T <= 0) return 0;
+  B2_REQUIRE(g.experts >= 1 && g.groups >= 1 && g.groups <= 64 && g.experts % g.groups == 0 && g.keep >= 1 && g.keep <= g.groups && g.top >= 1 &&
+                 g.top <= g.keep * (g.experts / g.groups),
+             "route_select: bad sizes (experts %d, groups %d, keep %d, top %d)", g.experts, g.groups, g.keep, g.top);
+  const size_t smem = (size_t)8 * (2 * g.experts + g.groups) * sizeof(float);
+  B2_REQUIRE(smem <= 48 * 1024, "route_select: %d experts", g.experts);
+  B2_CUDA_OK(b2_launch(route_select_kernel, dim3((T + 7) / 8), dim3(256), smem, s, z, ld, correction, g, idx, weight, T, gate_out));
   return 0;
 }
 
