@@ -30,8 +30,9 @@
 //   lowrank_act        y = act(W2 . lr + bias) for the low-rank second stages (decays, output gates), fp32
 //   conv_unit_finish   delta rule: causal convolution + silu on q | k | v (a thread per channel), then unit vectors and the query scale
 //                      (a warp per head), beta
-//   conv_ring_store    the ring update, after every token of the step has read the ring
-//   state_scan         the recurrence
+//   conv_unit_rows     the same for prompt-sized steps (a CTA walks down sixteen rows of one head)
+//   conv_ring_store    the ring update, after every token of the step has read the ring (a decode step's tokens do it themselves)
+//   state_scan         the recurrence; state_scan_head: the delta rule with one decay per head on packed fp32 pairs
 //   state_out_gate     per-head RMS norm of the read-out with a gain, times the gate (silu or given), operand type out
 #include "kernels.h"
 
@@ -112,7 +113,7 @@ __global__ void __launch_bounds__(256) conv_unit_finish_kernel(const float* __re
                                                                const int32_t* __restrict__ positions, const int32_t* __restrict__ slots,
                                                                float unit_eps, float* __restrict__ out, float* __restrict__ beta_out, int upc,
                                                                const float* __restrict__ a_log, const float* __restrict__ dt_bias,
-                                                               float* __restrict__ decay_out) {
+                                                               float* __restrict__ decay_out, float* __restrict__ ring_store) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -149,6 +150,7 @@ __global__ void __launch_bounds__(256) conv_unit_finish_kernel(const float* __re
       }
     }
     orow[c] = silu_f(acc);
+    if (ring_store) ring_store[((size_t)row_seq[t] * taps + pos % taps) * C + c] = row[c];   // (a row of the ring that this launch does not read)
   }
   __syncthreads();   // (the CTA reads back only what it wrote itself)
   const float qscale = rsqrtf((float)g.dim);
@@ -165,6 +167,85 @@ __global__ void __launch_bounds__(256) conv_unit_finish_kernel(const float* __re
       beta_out[(size_t)t * g.heads + a] = sigmoid_f(row[C + a]);
       if (a_log) decay_out[(size_t)t * g.heads + a] = expf(-expf(a_log[a]) * softplus_f(row[C + g.heads + a] + dt_bias[a]));
     }
+}
+
+// Prompt-sized steps: a CTA takes CR_ROWS neighbouring token rows of one head unit (a query, key or value head).  A thread owns channels and walks
+// down the rows with the last inputs in registers, so a projected row is read once; query and key heads then pass through shared memory for
+// their unit vectors (a warp per row).
+constexpr int CR_ROWS = 16;
+template <int TAPS>
+__global__ void __launch_bounds__(128) conv_unit_rows_kernel(const float* __restrict__ proj, int ld, StateGeom g, const float* __restrict__ conv_w,
+                                                             const float* __restrict__ ring, const int32_t* __restrict__ row_seq,
+                                                             const int32_t* __restrict__ row_first, const int32_t* __restrict__ positions,
+                                                             const int32_t* __restrict__ slots, float unit_eps, float* __restrict__ out,
+                                                             float* __restrict__ beta_out, const float* __restrict__ a_log, const float* __restrict__ dt_bias,
+                                                             float* __restrict__ decay_out, int T) {
+  extern __shared__ float tile[];   // [CR_ROWS][dim] of a query or key head
+  __shared__ int s_first[CR_ROWS], s_pos[CR_ROWS], s_seq[CR_ROWS];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t0 = blockIdx.x * CR_ROWS, tn = min(CR_ROWS, T - t0), u = blockIdx.y;
+  const int nqk = g.kv_heads * g.dim, C = 2 * nqk + g.heads * g.vdim;
+  const bool unit = u < 2 * g.kv_heads;
+  const int width = unit ? g.dim : g.vdim, ch0 = unit ? u * g.dim : 2 * nqk + (u - 2 * g.kv_heads) * g.vdim;
+  if ((int)threadIdx.x < tn) {
+    s_first[threadIdx.x] = slots[t0 + threadIdx.x] < 0 ? -1 : row_first[t0 + threadIdx.x];
+    s_pos[threadIdx.x] = positions[t0 + threadIdx.x];
+    s_seq[threadIdx.x] = row_seq[t0 + threadIdx.x];
+  }
+  __syncthreads();
+  for (int cc = threadIdx.x; cc < width; cc += 128) {
+    const int c = ch0 + cc;
+    float w[TAPS], hist[TAPS];   // hist[d]: the input d rows back
+#pragma unroll
+    for (int d = 0; d < TAPS; ++d) w[d] = conv_w[(size_t)c * TAPS + TAPS - 1 - d];
+    for (int i = 0; i < tn;) {   // runs of rows of one portion
+      const int first = s_first[i], pos = s_pos[i], back = t0 + i - first;
+      int e = i + 1;
+      while (e < tn && s_first[e] == first) ++e;
+#pragma unroll
+      for (int d = 1; d < TAPS; ++d)
+        hist[d] = first < 0 ? 0.f
+                  : d <= back   ? proj[(size_t)(t0 + i - d) * ld + c]
+                  : pos - d >= 0 ? ring[((size_t)s_seq[i] * TAPS + (pos - d) % TAPS) * C + c]
+                                 : 0.f;
+#pragma unroll 4
+      for (; i < e; ++i) {
+        const float x = proj[(size_t)(t0 + i) * ld + c];
+        float acc = 0.f;
+#pragma unroll
+        for (int d = TAPS - 1; d >= 1; --d) acc = fmaf(w[d], hist[d], acc);
+        acc = fmaf(w[0], x, acc);
+#pragma unroll
+        for (int d = TAPS - 1; d >= 2; --d) hist[d] = hist[d - 1];
+        hist[1] = x;
+        const float y = silu_f(acc);
+        if (unit) tile[i * width + cc] = y;
+        else if (first >= 0) out[(size_t)(t0 + i) * C + c] = y;
+      }
+    }
+  }
+  if (unit) {
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const float qscale = u < g.kv_heads ? rsqrtf((float)g.dim) : 1.0f;
+    for (int i = warp; i < tn; i += 4) {
+      const float* h = tile + i * width;
+      float ss = 0.f;
+      for (int d = lane; d < width; d += 32) ss = fmaf(h[d], h[d], ss);
+      const float r = (1.0f / sqrtf(warp_sum(ss) + unit_eps)) * qscale;
+      if (s_first[i] < 0) continue;
+      for (int d = lane; d < width; d += 32) out[(size_t)(t0 + i) * C + ch0 + d] = h[d] * r;
+    }
+  }
+  if (u == 0) {
+    for (int i = threadIdx.x; i < tn * g.heads; i += 128) {
+      const int t = t0 + i / g.heads, a = i % g.heads;
+      const float* row = proj + (size_t)t * ld + C;
+      beta_out[(size_t)t * g.heads + a] = sigmoid_f(row[a]);
+      if (a_log) decay_out[(size_t)t * g.heads + a] = expf(-expf(a_log[a]) * softplus_f(row[g.heads + a] + dt_bias[a]));
+    }
+  }
 }
 
 __global__ void __launch_bounds__(128) conv_ring_store_kernel(const float* __restrict__ proj, int ld, int C, int taps, float* __restrict__ ring,
@@ -185,6 +266,9 @@ constexpr int SC_CHUNK = 8;     // tokens of one stage (two stages)
 
 __device__ __forceinline__ void cp_async_f32(float* smem_dst, const float* gsrc) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(gsrc) : "memory");
+}
+__device__ __forceinline__ void cp_async_16(float* smem_dst, const float* gsrc) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem_dst)), "l"(gsrc) : "memory");
 }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
@@ -423,6 +507,201 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
   }
 }
 
+// ---- the delta rule with one decay per head, packed: the same grid, lanes and staging as state_scan_kernel with NC = 4, the state of a lane held
+// as pairs of neighbouring channels so that every multiply-add works on two of them (fma.rn.f32x2, two independent fp32 operations).  The state is
+// kept as a factor times a matrix: a decay multiplies the factor only, u enters divided by it, and the matrix takes the factor in (and the factor
+// becomes one) before it could run out of range, so a decay of any size down to zero is exact to rounding.  The
+// keys of a token stay in registers between the two sums that read them; the read-out's sum over the eight lanes leaves each column with
+// one lane pair.
+typedef unsigned long long f32x2_t;
+__device__ __forceinline__ f32x2_t x2_pack(float a, float b) {
+  f32x2_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void x2_unpack(f32x2_t v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ f32x2_t x2_fma(f32x2_t a, f32x2_t b, f32x2_t c) {
+  f32x2_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2_t x2_mul(f32x2_t a, f32x2_t b) {
+  f32x2_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+template <int DPT>   // channels per lane: 4, 8 or 16 (dim <= 8 DPT); lane j owns channels 32 m + 4 j + (0..3): rows are staged as they are, 16 bytes a copy
+__global__ void __launch_bounds__(256) state_scan_head_kernel(const float* __restrict__ q, int ldq, const float* __restrict__ k, int ldk,
+                                                              const float* __restrict__ v, int ldv, const float* __restrict__ decay,
+                                                              const float* __restrict__ beta, StateGeom g, float qscale, float* __restrict__ state,
+                                                              const int32_t* __restrict__ last_rows, const int32_t* __restrict__ row_seq,
+                                                              const int32_t* __restrict__ row_first, const int32_t* __restrict__ row_end,
+                                                              const int32_t* __restrict__ positions, const int32_t* __restrict__ slots,
+                                                              float* __restrict__ out, int cols) {
+  constexpr int NC = 4, CH = SC_CHUNK, DP = DPT * SC_LANES, MAXC = 32 * NC, HP = DPT / 2;
+  __shared__ __align__(16) float qs[2][CH][DP], ks[2][CH][DP];
+  __shared__ __align__(16) float vs[2][CH][MAXC];
+  __shared__ float bs[2][CH], ds[2][CH];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int r_last = last_rows ? last_rows[blockIdx.x] : (int)blockIdx.x;
+  const int first = row_first[r_last], end = row_end[r_last];
+  if (slots[first] < 0) return;   // padding row of a decode bucket
+  const int a = blockIdx.y, kh = a / (g.heads / g.kv_heads);
+  const int col0 = blockIdx.z * cols;
+  const int grp = threadIdx.x / SC_LANES, j = threadIdx.x % SC_LANES, cl = grp * NC;
+  const int pos0 = positions[first], n = end - first;
+  const int nthreads = blockDim.x;
+  const size_t head_floats = (size_t)g.dim * g.vdim;
+  float* sbase = state + ((size_t)row_seq[first] * 2 * g.heads) * head_floats;
+  const float* s_in = sbase + ((size_t)((pos0 + 1) & 1) * g.heads + a) * head_floats;
+  float* s_out = sbase + ((size_t)((pos0 + n - 1) & 1) * g.heads + a) * head_floats;
+  // channels past dim and columns past vdim never change: zero keys, queries and values
+  for (int i = threadIdx.x; i < 2 * CH * (DP - g.dim); i += nthreads) {
+    const int st = i / (CH * (DP - g.dim)), rem = i % (CH * (DP - g.dim)), tt = rem / (DP - g.dim), d = g.dim + rem % (DP - g.dim);
+    qs[st][tt][d] = 0.f;
+    ks[st][tt][d] = 0.f;
+  }
+  const int vcols = min(cols, g.vdim - col0);
+  if (vcols < cols) {
+    for (int i = threadIdx.x; i < 2 * CH * (cols - vcols); i += nthreads) {
+      const int row = i / (cols - vcols), c = vcols + i % (cols - vcols);
+      vs[row / CH][row % CH][c] = 0.f;
+    }
+  }
+  __syncthreads();
+  const int dq = g.dim >> 2, vq4 = vcols >> 2;   // 16-byte pieces of a row
+  const int dsh = (dq & (dq - 1)) == 0 ? 31 - __clz(dq) : -1, vsh = (vq4 & (vq4 - 1)) == 0 ? 31 - __clz(vq4) : -1;
+  const float* qb = q + (size_t)first * ldq + kh * g.dim;
+  const float* kb = k + (size_t)first * ldk + kh * g.dim;
+  const float* vb = v + (size_t)first * ldv + a * g.vdim + col0;
+  auto issue = [&](int c0, int st) {
+    const int cn = min(CH, n - c0);
+    for (int i = threadIdx.x; i < cn * dq; i += nthreads) {
+      const int tt = dsh >= 0 ? i >> dsh : i / dq, d = (i - tt * dq) * 4;
+      cp_async_16(&qs[st][tt][d], qb + (size_t)(c0 + tt) * ldq + d);
+      cp_async_16(&ks[st][tt][d], kb + (size_t)(c0 + tt) * ldk + d);
+    }
+    for (int i = threadIdx.x; i < cn * vq4; i += nthreads) {
+      const int tt = vsh >= 0 ? i >> vsh : i / vq4, c = (i - tt * vq4) * 4;
+      cp_async_16(&vs[st][tt][c], vb + (size_t)(c0 + tt) * ldv + c);
+    }
+    for (int i = threadIdx.x; i < cn; i += nthreads) {
+      cp_async_f32(&bs[st][i], beta + (size_t)(first + c0 + i) * g.heads + a);
+      cp_async_f32(&ds[st][i], decay + (size_t)(first + c0 + i) * g.heads + a);
+    }
+  };
+  issue(0, 0);
+  const bool live = col0 + cl + NC <= g.vdim;   // this group's four columns (vdim is a multiple of four)
+  auto channel = [&](int i) { return (i >> 2) * 32 + 4 * j + (i & 3); };
+  f32x2_t s[HP][NC];
+#pragma unroll
+  for (int i = 0; i < HP; ++i) {
+    float lo[NC], hi[NC];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int d = channel(2 * i + x);
+      float* dst = x ? hi : lo;
+      float4 w = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (live && pos0 > 0 && d < g.dim) w = *reinterpret_cast<const float4*>(s_in + (size_t)d * g.vdim + col0 + cl);
+      dst[0] = w.x; dst[1] = w.y; dst[2] = w.z; dst[3] = w.w;
+    }
+#pragma unroll
+    for (int c = 0; c < NC; ++c) s[i][c] = x2_pack(lo[c], hi[c]);
+  }
+  float fac = 1.0f;   // the state is fac * s: a decay multiplies one number
+  int st = 0;
+  for (int c0 = 0; c0 < n; c0 += CH, st ^= 1) {
+    const int cn = min(CH, n - c0);
+    cp_async_wait_all();                         // this chunk's copies (the only ones in flight)
+    __syncthreads();                             // ... of every thread; and every thread has left the other stage
+    if (c0 + CH < n) issue(c0 + CH, st ^ 1);     // the next chunk's copies run beside this chunk's arithmetic
+    for (int tt = 0; tt < cn; ++tt) {
+      const float4 vq = *reinterpret_cast<const float4*>(&vs[st][tt][cl]);
+      const float vc[NC] = {vq.x, vq.y, vq.z, vq.w};
+      const float bt = bs[st][tt];
+      fac *= ds[st][tt];
+      if (fac < 1e-12f) {   // (the same in every thread of the CTA)
+        const f32x2_t f2 = x2_pack(fac, fac);
+#pragma unroll
+        for (int i = 0; i < HP; ++i)
+#pragma unroll
+          for (int c = 0; c < NC; ++c) s[i][c] = x2_mul(f2, s[i][c]);
+        fac = 1.0f;
+      }
+      const float inv = 1.0f / fac;
+      const ulonglong2* kp = reinterpret_cast<const ulonglong2*>(&ks[st][tt][4 * j]);   // (32 channels on: eight pieces of 16 bytes)
+      const ulonglong2* qp = reinterpret_cast<const ulonglong2*>(&qs[st][tt][4 * j]);
+      f32x2_t kk[HP], sum[NC];
+#pragma unroll
+      for (int i = 0; i < HP; i += 2) {
+        const ulonglong2 w = kp[(i >> 1) * 8];
+        kk[i] = w.x;
+        kk[i + 1] = w.y;
+      }
+#pragma unroll
+      for (int c = 0; c < NC; ++c) sum[c] = x2_mul(s[0][c], kk[0]);
+#pragma unroll
+      for (int i = 1; i < HP; ++i)
+#pragma unroll
+        for (int c = 0; c < NC; ++c) sum[c] = x2_fma(s[i][c], kk[i], sum[c]);
+      f32x2_t u2[NC];
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        float lo, hi;
+        x2_unpack(sum[c], lo, hi);
+        float kv = lo + hi;
+        kv += __shfl_xor_sync(0xffffffffu, kv, 1);
+        kv += __shfl_xor_sync(0xffffffffu, kv, 2);
+        kv += __shfl_xor_sync(0xffffffffu, kv, 4);
+        const float u = bt * fmaf(vc[c], inv, -kv);   // beta (v - fac S^T k) / fac
+        u2[c] = x2_pack(u, u);
+      }
+#pragma unroll
+      for (int i = 0; i < HP; i += 2) {
+        const ulonglong2 w = qp[(i >> 1) * 8];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          s[i][c] = x2_fma(kk[i], u2[c], s[i][c]);
+          s[i + 1][c] = x2_fma(kk[i + 1], u2[c], s[i + 1][c]);
+          sum[c] = i == 0 ? x2_mul(s[0][c], w.x) : x2_fma(s[i][c], w.x, sum[c]);
+          sum[c] = x2_fma(s[i + 1][c], w.y, sum[c]);
+        }
+      }
+      // sum over the eight lanes: each exchange halves the columns a lane still holds, then the last two lanes of a column add
+      float o[NC];
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        float lo, hi;
+        x2_unpack(sum[c], lo, hi);
+        o[c] = lo + hi;
+      }
+      const bool up1 = (j & 1) != 0, up2 = (j & 2) != 0;
+      const float a0 = (up1 ? o[2] : o[0]) + __shfl_xor_sync(0xffffffffu, up1 ? o[0] : o[2], 1);
+      const float a1 = (up1 ? o[3] : o[1]) + __shfl_xor_sync(0xffffffffu, up1 ? o[1] : o[3], 1);
+      float r = (up2 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, up2 ? a0 : a1, 2);
+      r += __shfl_xor_sync(0xffffffffu, r, 4);
+      const int c = (up1 ? 2 : 0) + (up2 ? 1 : 0);   // the column this lane ended with
+      if (j < 4 && live)
+        out[(size_t)(first + c0 + tt) * ((size_t)g.heads * g.vdim) + a * g.vdim + col0 + cl + c] = r * (qscale * fac);
+    }
+  }
+  const f32x2_t f2 = x2_pack(fac, fac);
+#pragma unroll
+  for (int i = 0; i < HP; ++i) {
+    float lo[NC], hi[NC];
+#pragma unroll
+    for (int c = 0; c < NC; ++c) x2_unpack(x2_mul(f2, s[i][c]), lo[c], hi[c]);
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int d = channel(2 * i + x);
+      const float* src = x ? hi : lo;
+      if (live && d < g.dim) *reinterpret_cast<float4*>(s_out + (size_t)d * g.vdim + col0 + cl) = make_float4(src[0], src[1], src[2], src[3]);
+    }
+  }
+}
+
 // One warp per (token, head): y = o / sqrt(mean(o^2) + eps) * gain * gate, gate = silu(gate_in) or gate_in as it is.
 template <typename TX>
 __global__ void __launch_bounds__(128) state_out_gate_kernel(const float* __restrict__ o, const float* __restrict__ gain,
@@ -485,7 +764,7 @@ int launch_lowrank_act(const float* lr, int ld, int lr_off, int rank, const floa
 
 int launch_conv_unit_finish(const float* proj, int ld, const StateGeom& g, int taps, const float* conv_w, float* ring, const int32_t* row_seq,
                             const int32_t* row_first, const int32_t* row_end, const int32_t* positions, const int32_t* slots, float unit_eps,
-                            float* out, float* beta_out, int T, cudaStream_t s, const float* a_log, const float* dt_bias, float* decay_out) {
+                            float* out, float* beta_out, int T, cudaStream_t s, const float* a_log, const float* dt_bias, float* decay_out, int single_rows) {
   if (T <= 0) return 0;
   B2_REQUIRE(a_log == nullptr || (dt_bias != nullptr && decay_out != nullptr), "conv_unit_finish: a decay per head needs its bias and its output");
   B2_REQUIRE(taps >= 1 && conv_w && (ring || taps == 1) && row_seq && row_first && row_end, "conv_unit_finish: the convolution needs its weights and state");
@@ -494,13 +773,21 @@ int launch_conv_unit_finish(const float* proj, int ld, const StateGeom& g, int t
   const dim3 grid(T, (units + upc - 1) / upc);
 #define B2_CONV_FINISH(TAPS)                                                                                                                      \
   B2_CUDA_OK(b2_launch(conv_unit_finish_kernel<TAPS>, grid, dim3(256), 0, s, proj, ld, g, taps, conv_w, (const float*)ring, row_seq, row_first, positions, \
-                       slots, unit_eps, out, beta_out, upc, a_log, dt_bias, decay_out))
-  if (taps == 4) B2_CONV_FINISH(4);
+                       slots, unit_eps, out, beta_out, upc, a_log, dt_bias, decay_out, single_rows && taps > 1 ? ring : (float*)nullptr))
+#define B2_CONV_ROWS(TAPS)                                                                                                                        \
+  B2_CUDA_OK(b2_launch(conv_unit_rows_kernel<TAPS>, dim3((T + CR_ROWS - 1) / CR_ROWS, units), dim3(128), (size_t)CR_ROWS * g.dim * 4, s, proj, ld, g, conv_w, \
+                       (const float*)ring, row_seq, row_first, positions, slots, unit_eps, out, beta_out, a_log, dt_bias, decay_out, T))
+  const bool rows = !single_rows && T >= 512 && taps >= 2 && taps <= 4 && g.dim <= 512;
+  if (rows && taps == 4) B2_CONV_ROWS(4);
+  else if (rows && taps == 3) B2_CONV_ROWS(3);
+  else if (rows) B2_CONV_ROWS(2);
+  else if (taps == 4) B2_CONV_FINISH(4);
   else if (taps == 3) B2_CONV_FINISH(3);
   else if (taps == 2) B2_CONV_FINISH(2);
   else B2_CONV_FINISH(0);
 #undef B2_CONV_FINISH
-  if (taps > 1)
+#undef B2_CONV_ROWS
+  if (taps > 1 && !single_rows)
     B2_CUDA_OK(b2_launch(conv_ring_store_kernel, dim3(T), dim3(128), 0, s, proj, ld, C, taps, ring, row_seq, row_end, positions, slots));
   return 0;
 }
@@ -524,6 +811,19 @@ int launch_state_scan(const float* q, int ldq, const float* k, int ldk, const fl
   if (g.rule == STATE_RULE_DECAY)
     return launch_scan_rule<STATE_RULE_DECAY>(dpt, grid, block, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,
                                               row_first, row_end, positions, slots, out, cols);
+  static const bool packed = [] { const char* e = getenv("B2_SCAN_PACKED"); return !(e && *e == '0'); }();   // 0: the generic form (cross-check)
+  const bool rows16 = g.dim % 4 == 0 && g.vdim % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ldv % 4 == 0 &&
+                      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15) == 0;
+  if (g.rule == STATE_RULE_DELTA_HEAD && packed && rows16 && dpt <= 16) {
+#define B2_SCAN_HEAD(D)                                                                                                                          \
+  B2_CUDA_OK(b2_launch(state_scan_head_kernel<D>, grid, block, 0, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,   \
+                       row_first, row_end, positions, slots, out, cols))
+    if (dpt <= 4) B2_SCAN_HEAD(4);
+    else if (dpt == 8) B2_SCAN_HEAD(8);
+    else B2_SCAN_HEAD(16);
+#undef B2_SCAN_HEAD
+    return 0;
+  }
   if (g.rule == STATE_RULE_DELTA_HEAD)
     return launch_scan_rule<STATE_RULE_DELTA_HEAD>(dpt, grid, block, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,
                                                    row_first, row_end, positions, slots, out, cols);

@@ -1797,7 +1797,7 @@ int forward_outnorm_list(b2_engine* e, int T, int ntiles, int nlast) {
       {
         KL k(e, B2K_ROPE_KV);   // convolutions, unit vectors, step sizes and decays
         if (!k.skip()) B2_TRY(launch_conv_unit_finish(e->l_qd, L.nqd, sg, sp.conv_taps, L.conv_w, R.ring, e->d_row_seq, e->d_row_first, e->d_row_end,
-                                                      e->d_positions, e->d_slots, TOLANEX_UNIT_EPS, e->l_q, e->l_beta, T, st, L.a_log, L.a2_bias, e->l_dec));
+                                                      e->d_positions, e->d_slots, TOLANEX_UNIT_EPS, e->l_q, e->l_beta, T, st, L.a_log, L.a2_bias, e->l_dec, ntiles == 0 ? 1 : 0));
       }
       {
         KL k(e, B2K_CHAIN);

@@ -401,7 +401,8 @@ int launch_lowrank_act(const float* lr, int ld, int lr_off, int rank, const floa
 int launch_conv_unit_finish(const float* proj, int ld, const StateGeom& g, int taps, const float* conv_w, float* ring, const int32_t* row_seq,
                             const int32_t* row_first, const int32_t* row_end, const int32_t* positions, const int32_t* slots, float unit_eps,
                             float* out, float* beta_out, int T, cudaStream_t s, const float* a_log = nullptr, const float* dt_bias = nullptr,
-                            float* decay_out = nullptr);
+                            float* decay_out = nullptr, int single_rows = 0);
+// single_rows: every row is a portion of its own (a decode step): the row's ring entry is written by the kernel that reads the others
 // The recurrence over every portion of the step: portion i ends at row last_rows[i] (null: row i is a portion of one token); q / k rows of
 // kv_heads*dim at strides ldq / ldk, v rows of heads*vdim at stride ldv, decay [T][heads*dim] ([T][heads] with STATE_RULE_DELTA_HEAD), beta [T][heads] (delta rule); q is multiplied
 // by qscale.  state [slots][2][heads][dim][vdim] fp32 (state_floats_per_slot); out [T][heads*vdim] fp32.  Rows whose slot is negative are skipped.

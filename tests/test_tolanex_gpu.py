@@ -171,6 +171,21 @@ def test_each_mechanism_alone(name, width):
         run_schedule(e, cfg, toks, ref, F32_BAR, [2, 31, 3, 16, 2], 54)         # portions, then 21 decode steps
 
 
+@pytest.mark.parametrize("dim,vdim", [(16, 8), (12, 6), (72, 20)])
+def test_decays_of_every_size(dim, vdim):
+    """Heads that hardly forget, that forget within a few tokens (the state's scale leaves the range of a float within a prompt) and that forget
+    everything at once (a decay that is zero in fp32), in one layer; long prompts, portions and decoding."""
+    cfg = model([(delta(6, 2, dim, vdim), None)], vocab=131, width=48)
+    w = random_weights(cfg, seed=41)
+    w["l0.mix.A_log"] = torch.tensor([-6.0, -1.0, 1.0, 2.0, 3.0, 5.0]).to(torch.bfloat16).float()
+    w["l0.mix.dt_bias"] = torch.tensor([-4.0, 0.0, 1.0, 2.0, 3.0, 3.0]).to(torch.bfloat16).float()
+    toks = tokens(cfg, 300, 42)
+    ref = ref_logits(cfg, w, toks)
+    with engine(cfg, w) as e:
+        run_schedule(e, cfg, toks, ref, F32_BAR, [300], 300)
+        run_schedule(e, cfg, toks, ref, F32_BAR, [2, 131, 40, 2, 65], 240)
+
+
 def test_the_previous_token_is_carried():
     """The bigram row of a portion's first token, of a decoded token and of a new sequence's first token in a slot that another sequence used.
     Rows are large against the token's own, so a wrong one is a gross error; portions of even and odd length end at either parity."""
