@@ -209,19 +209,27 @@ __global__ void __launch_bounds__(128) conv_unit_rows_kernel(const float* __rest
                   : d <= back   ? proj[(size_t)(t0 + i - d) * ld + c]
                   : pos - d >= 0 ? ring[((size_t)s_seq[i] * TAPS + (pos - d) % TAPS) * C + c]
                                  : 0.f;
-#pragma unroll 4
-      for (; i < e; ++i) {
-        const float x = proj[(size_t)(t0 + i) * ld + c];
-        float acc = 0.f;
+      while (i < e) {   // eight rows' loads in flight at a time
+        const int m = min(8, e - i);
+        float x[8];
 #pragma unroll
-        for (int d = TAPS - 1; d >= 1; --d) acc = fmaf(w[d], hist[d], acc);
-        acc = fmaf(w[0], x, acc);
+        for (int r = 0; r < 8; ++r) x[r] = r < m ? proj[(size_t)(t0 + i + r) * ld + c] : 0.f;
 #pragma unroll
-        for (int d = TAPS - 1; d >= 2; --d) hist[d] = hist[d - 1];
-        hist[1] = x;
-        const float y = silu_f(acc);
-        if (unit) tile[i * width + cc] = y;
-        else if (first >= 0) out[(size_t)(t0 + i) * C + c] = y;
+        for (int r = 0; r < 8; ++r) {
+          if (r < m) {
+            float acc = 0.f;
+#pragma unroll
+            for (int d = TAPS - 1; d >= 1; --d) acc = fmaf(w[d], hist[d], acc);
+            acc = fmaf(w[0], x[r], acc);
+#pragma unroll
+            for (int d = TAPS - 1; d >= 2; --d) hist[d] = hist[d - 1];
+            hist[1] = x[r];
+            const float y = silu_f(acc);
+            if (unit) tile[(i + r) * width + cc] = y;
+            else if (first >= 0) out[(size_t)(t0 + i + r) * C + c] = y;
+          }
+        }
+        i += m;
       }
     }
   }
@@ -630,7 +638,7 @@ __global__ void __launch_bounds__(256) state_scan_head_kernel(const float* __res
           for (int c = 0; c < NC; ++c) s[i][c] = x2_mul(f2, s[i][c]);
         fac = 1.0f;
       }
-      const float inv = 1.0f / fac;
+      const float inv = __fdividef(1.0f, fac);   // (1e-12 <= fac <= 1)
       const ulonglong2* kp = reinterpret_cast<const ulonglong2*>(&ks[st][tt][4 * j]);   // (32 channels on: eight pieces of 16 bytes)
       const ulonglong2* qp = reinterpret_cast<const ulonglong2*>(&qs[st][tt][4 * j]);
       f32x2_t kk[HP], sum[NC];
@@ -720,6 +728,25 @@ __global__ void __launch_bounds__(128) state_out_gate_kernel(const float* __rest
   ss = warp_sum(ss);
   const float r = 1.0f / sqrtf(ss / (float)vdim + eps);
   TX* dst = out + ((size_t)t * heads + a) * vdim;
+  if (vdim % 4 == 0 && gate_ld % 4 == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0) {   // sixteen bytes at a time
+    for (int i = lane * 4; i < vdim; i += 128) {
+      const float4 ov = *reinterpret_cast<const float4*>(orow + i), gv = *reinterpret_cast<const float4*>(grow + i);
+      const float4 nv = *reinterpret_cast<const float4*>(gain + i);
+      const float oo[4] = {ov.x, ov.y, ov.z, ov.w}, gg[4] = {gv.x, gv.y, gv.z, gv.w}, nn[4] = {nv.x, nv.y, nv.z, nv.w};
+      float y[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) y[k] = oo[k] * r * nn[k] * (gate_silu ? silu_f(gg[k]) : gg[k]);
+      if constexpr (sizeof(TX) == 4) {
+        *reinterpret_cast<float4*>(dst + i) = make_float4(y[0], y[1], y[2], y[3]);
+      } else {
+        uint2 pk;
+        pk.x = pack_bf16x2(y[0], y[1]);
+        pk.y = pack_bf16x2(y[2], y[3]);
+        *reinterpret_cast<uint2*>(dst + i) = pk;
+      }
+    }
+    return;
+  }
   for (int i = lane; i < vdim; i += 32) {
     const float gt = gate_silu ? silu_f(grow[i]) : grow[i];
     dst[i] = (TX)(orow[i] * r * gain[i] * gt);

@@ -1916,11 +1916,9 @@ int forward_outnorm_list(b2_engine* e, int T, int ntiles, int nlast) {
         KL k(e, B2K_ACT);
         // Prompt-sized bf16 steps form the logits as a product of bf16 operands: a checkpoint's router is bf16, so every product of two operands is
         // exact and only the fp32 sums' order differs.
-        const int er = sp.experts + (shared ? 1 : 0);
+        const int er = std::max(128, sp.experts + (shared ? 1 : 0));   // (zero rows fill the operand up to the tcgen05 kernel's tile)
         if (L.router_op != nullptr && T >= 512 && !k.skip()) {
-          AnyGemm a;
-          a.A = e->l_x1; a.W = L.router_op; a.C = e->l_rz; a.M = T; a.N = er; a.K = W; a.lda = W; a.ldw = W; a.ldc = er;
-          B2_TRY(launch_gemm_any(a, 0, 0, 1, 1, 0, st));
+          B2_TRY(dense(e->l_x1, L.router_op, e->l_rz, T, er, W, st));
           B2_TRY(launch_route_select(e->l_rz, er, nullptr, rg, e->l_idx, e->l_rw, T, st, shared ? e->l_sg : nullptr));
         } else if (!k.skip()) {
           B2_TRY(launch_route(e->l_x1, f, L.router, nullptr, rg, e->l_idx, e->l_rw, T, W, st, shared ? e->l_sg : nullptr));
@@ -3503,7 +3501,9 @@ int outnorm_engine_alloc(b2_engine* e) {
       B2_TRY(falloc(&L.router, (size_t)(sp.experts + (sp.shared_ff > 0 ? 1 : 0)) * W));
       if (!e->f32) {
         char* q = nullptr;
-        B2_TRY(dalloc(&q, (size_t)(sp.experts + 1) * W * es));
+        const size_t rn = (size_t)std::max(128, sp.experts + 1) * W * es;
+        B2_TRY(dalloc(&q, rn));
+        B2_CUDA_OK(cudaMemset(q, 0, rn));
         L.router_op = reinterpret_cast<bf16*>(q);
       }
       B2_TRY(xalloc(&L.up, (size_t)sp.experts * 2 * sp.ff_dim * W));
@@ -3590,7 +3590,7 @@ int outnorm_engine_alloc(b2_engine* e) {
     }
     B2_TRY(dalloc(&e->l_rw, Tc * max_top));
     B2_TRY(dalloc(&e->l_sg, Tc));
-    if (!e->f32) B2_TRY(dalloc(&e->l_rz, Tc * (size_t)(max_exp + 1)));
+    if (!e->f32) B2_TRY(dalloc(&e->l_rz, Tc * (size_t)std::max(128, max_exp + 1)));
     B2_TRY(dalloc(&e->l_idx, Tc * max_top));
     e->l_offsets_stride = max_exp + 1;
     B2_TRY(dalloc(&e->l_offsets, (size_t)3 * (max_exp + 1)));
