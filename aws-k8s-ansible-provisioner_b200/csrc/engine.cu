@@ -933,7 +933,7 @@ bool list_use_tc() {
 int list_dense(b2_engine* e, const void* A, const void* Wt, float* C, int M, int N, int K, float alpha, cudaStream_t stream = nullptr) {
   cudaStream_t ls = stream ? stream : e->stream;
   const int f = e->f32 ? 1 : 0;
-  if (list_use_tc() && !f && alpha == 1.f && M > 64 && N >= 128 && K % 64 == 0) {
+  if (list_use_tc() && !f && alpha == 1.f && (M > 64 || N >= 16384) && N >= 128 && K % 64 == 0) {
     TcGemmArgs a;
     a.bn = tc_pick_bn(M);
     B2_TRY(b2_make_tmap_bf16(&a.tmap_w, Wt, (uint64_t)N, (uint64_t)K, (uint64_t)K, 128));

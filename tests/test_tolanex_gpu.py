@@ -440,6 +440,24 @@ def test_bf16_decode_batches(nseq):
     assert np.median(rel) < BF16_BAR and np.quantile(rel, 0.9) < 3 * BF16_BAR, (np.median(rel), max(rel))
 
 
+@pytest.mark.parametrize("nseq", [1, 3])
+def test_bf16_wide_head(nseq):
+    """A vocabulary wide enough for a decode step's head to take the tcgen05 projection kernel, with fewer rows than its token tile."""
+    cfg = model([(delta(2, 1, 16, 16), moe(4, 2, 64, (2, 1), 1.5, 64))], vocab=16400, width=64, positions=64)
+    w = random_weights(cfg, seed=43)
+    prompts = [tokens(cfg, 20 + i, 44 + i) for i in range(nseq)]
+    refs = [ref_logits(cfg, w, p) for p in prompts]
+    with engine(cfg, w, f32=False, max_model_len=64, num_blocks=20, max_batch_tokens=128) as e:
+        sids = [e.seq_create(40) for _ in prompts]
+        lg, _ = e.prefill_logits(sids, [p[:-3] for p in prompts], [len(prompts[0]) - 4])
+        rel = [err(lg[0], refs[0][len(prompts[0]) - 4])]
+        for k in range(3, 0, -1):
+            e.decode_step(sids, in_tokens=[p[len(p) - k] for p in prompts], want_output=False)
+            lg = e.get_logits(nseq)
+            rel += [err(lg[i], refs[i][len(prompts[i]) - k]) for i in range(nseq)]
+    assert max(rel) < 3 * BF16_BAR and np.median(rel) < BF16_BAR / 2, rel
+
+
 def test_refusals():
     P = pkg()
     cfg = cfg_b()
