@@ -362,6 +362,36 @@ def test_mixed_batch_equals_each_alone():
                 done[r] += 1
 
 
+def test_long_portions_of_several_requests_in_one_step():
+    """A prompt-sized step of several requests: portions that start in the middle of the row blocks of the convolution and of the scan's chunks,
+    some continuing from state, one two tokens long, then decoding."""
+    cfg = model([(delta(4, 2, 12, 8, 4), moe(8, 2, 12, (4, 2), 1.3, 16)), (delta(2, 2, 8, 20, 2), None), (lat(2, 8, 8, 16, 0.35), None), (delta(3, 1, 20, 6, 3), None)],
+                vocab=151, width=56)
+    w = random_weights(cfg, seed=45)
+    prompts = [tokens(cfg, n, 46 + n) for n in (262, 290, 60, 215)]
+    refs = [ref_logits(cfg, w, p) for p in prompts]
+    with engine(cfg, w) as e:
+        sids, done = [e.seq_create(300) for _ in prompts], [0, 0, 0, 0]
+        for sizes in ([5, 3, 50, 0], [250, 280, 2, 0], [1, 2, 1, 210], [6, 5, 7, 5]):
+            live = [r for r in range(4) if sizes[r]]
+            lg, _ = e.prefill_logits([sids[r] for r in live], [prompts[r][done[r]:done[r] + sizes[r]] for r in live], list(range(sum(sizes))))
+            base = 0
+            for r in live:
+                assert err(lg[base:base + sizes[r]], refs[r][done[r]:done[r] + sizes[r]]) < F32_BAR, (sizes, r)
+                base += sizes[r]
+                done[r] += sizes[r]
+        # one more long step from fresh sequences, all of them decoding afterwards
+        for s_ in sids:
+            e.seq_free(s_)
+        sids = [e.seq_create(300) for _ in prompts]
+        e.prefill_logits(sids, [p[:-2] for p in prompts], [])
+        for k in (2, 1):
+            e.decode_step(sids, in_tokens=[p[-k] for p in prompts], want_output=False)
+            lg = e.get_logits(4)
+            for r in range(4):
+                assert err(lg[r], refs[r][len(prompts[r]) - k]) < F32_BAR, (k, r)
+
+
 def test_pages_and_slots_are_used_again():
     """Eight usable pages, two sequence slots: every round frees its request, the next one gets the same slot (and with it the matrix
     states, convolution inputs and previous token the last request left) and the same pages in another order."""
