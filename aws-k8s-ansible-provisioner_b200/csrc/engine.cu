@@ -183,7 +183,7 @@ struct b2_engine {
   // all-zero partner head.  The padding lives in the WEIGHTS (zero rows of Wqkv, zero columns of Wo,
   // scattered once at load time), so activations, KV pages and kernels need no special cases and the
   // arithmetic on the real elements is untouched; the cost is wasted bytes, which only matters for the
-  // parity configurations that use it (DESIGN.md section 4).
+  // parity configurations that use it.
   int nq = 0, nkv = 0, hd = 128;  // internal (padded) head counts / width handed to the kernels
   int qhead_step = 1;             // real query head h lives at internal head h * qhead_step
   bool native_geom = true;        // cfg geometry == internal geometry (Qwen3): weights copy straight in
@@ -4222,7 +4222,7 @@ extern "C" int b2_engine_create(const b2_config* cfg, const char* safetensors_pa
     E_TRY(dalloc(&e->attn_scratch, e->attn_scratch_floats));
     E_CUDA(cudaMemset(e->attn_scratch, 0, e->attn_scratch_floats * sizeof(float)));  // arrival counters start at zero
     // two-lane decode: B2_MB = smallest padded decode batch that is cut into two half-batch lanes (0 = off)
-    // Off by default: measured slower (C2: 2.03 against 1.90 ms/step) -- DESIGN.md section 4 has the timeline.
+    // Off by default: measured slower (C2: 2.03 against 1.90 ms/step).
     e->mb_min_batch = c.arch == B2_ARCH_OPT ? 0 : env_int("B2_MB", 0);
     if (c.arch != B2_ARCH_OPT && c.max_seqs >= 2) {
       E_CUDA(cudaStreamCreateWithFlags(&e->stream2, cudaStreamNonBlocking));
