@@ -6,11 +6,13 @@ import os
 
 # B2_LIB_PATH: an alternative build of the same library (A/B measurements of one source change); never a fallback
 LIB_PATH = os.environ.get("B2_LIB_PATH") or os.path.join(os.path.dirname(os.path.abspath(__file__)), "libb2engine.so")
-ABI_VERSION = 7
-ARCH_QWEN3, ARCH_PHI3, ARCH_OPT, ARCH_LERASUN, ARCH_KEDASUN, ARCH_BUMALIX, ARCH_TINEVIK, ARCH_TOLANEX = 0, 1, 2, 3, 4, 5, 6, 7
+ABI_VERSION = 8
+ARCH_QWEN3, ARCH_PHI3, ARCH_OPT, ARCH_LERASUN, ARCH_KEDASUN, ARCH_BUMALIX, ARCH_TINEVIK, ARCH_TOLANEX, ARCH_RESITAR = 0, 1, 2, 3, 4, 5, 6, 7, 8
 MIXER_LATENT_ATTENTION, MIXER_ATTENTION, MIXER_CONV_ATTENTION, MIXER_WINDOW_AND_STATE, MIXER_DELTA_STATE = 1, 2, 3, 4, 5
 MIXER_DECAY_STATE, MIXER_MIXED_SCORE_ATTENTION, MIXER_GATED_LATENT, MIXER_HEAD_DELTA = 6, 7, 8, 9
+MIXER_CHUNK_AND_SSM, MIXER_FULL_AND_TIMEMIX = 10, 11
 FF_NONE, FF_ROUTED_EXPERTS, FF_CLAMPED_GATED, FF_POLYNORM, FF_SCALED_GATED_EXPERTS, FF_XIELU, FF_TABLE_EXPERTS, FF_SOFTMAX_EXPERTS = 0, 1, 2, 3, 4, 5, 6, 7
+FF_SWIGLU, FF_TOP_SOFTMAX_EXPERTS = 8, 9
 NUM_KERNEL_CLASSES = 12
 
 
@@ -28,6 +30,8 @@ class b2_layer_spec(C.Structure):
         ("s_heads", C.c_int32), ("s_dim", C.c_int32), ("s_vdim", C.c_int32), ("s_tau", C.c_float), ("shared_ff", C.c_int32),
         ("weights_of", C.c_int32), ("q_rank", C.c_int32), ("rot_factor", C.c_float), ("softcap", C.c_float), ("score_mix", C.c_int32),
         ("rot_values", C.c_int32), ("router_scale", C.c_float),
+        ("mix_left", C.c_float), ("mix_right", C.c_float), ("chunk", C.c_int32), ("s_groups", C.c_int32), ("s_norm_groups", C.c_int32),
+        ("rot_halves", C.c_int32), ("rot_orig", C.c_int32), ("rot_fast", C.c_float), ("rot_slow", C.c_float),
     ]
 
 
@@ -43,7 +47,7 @@ class b2_config(C.Structure):
         ("embed_scale", C.c_float), ("norm_groups", C.c_int32),
         ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32), ("logit_softcap", C.c_float),
         ("norm_kind", C.c_int32), ("residual_mult", C.c_float), ("bigram_buckets", C.c_int32), ("bigram_mul_prev", C.c_int64),
-        ("bigram_mul_cur", C.c_int64),
+        ("bigram_mul_cur", C.c_int64), ("streams", C.c_int32),
     ]
 
 

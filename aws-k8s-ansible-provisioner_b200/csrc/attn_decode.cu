@@ -70,12 +70,13 @@ __global__ void __launch_bounds__(AD_WARPS * 32, 1)
 attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                    const int32_t* __restrict__ block_table, int bt_stride, const int32_t* __restrict__ seq_lens,
                    float* __restrict__ scratch, bf16* __restrict__ out, int B, int nq, int nkv, float scale, int early,
-                   int window, int tag) {
+                   int window, int tag, int chunk) {
   extern __shared__ __align__(128) uint8_t smem[];
   // Sliding-window attention (Phi-3, HF:models/phi3/modeling_phi3.py:265 sliding_window): a query at position
   // S-1 sees the last `window` keys only, i.e. tokens lo(S) = max(0, S - window) .. S-1.  Whole pages below lo are
   // never enumerated (first_page), the partly covered one is masked.  window == 0: everything is visible.
-  auto lo_of = [&](int S) { return (window > 0 && S > window) ? S - window : 0; };
+  // chunk > 0: tokens floor((S - 1) / chunk) * chunk .. S-1 instead.
+  auto lo_of = [&](int S) { return S > 0 ? first_seen_key(S - 1, window, chunk) : 0; };
   auto first_page_of = [&](int S) { return lo_of(S) / AD_BS; };
   auto pages_of = [&](int S) { return (S + AD_BS - 1) / AD_BS - first_page_of(S); };
   __shared__ __align__(8) uint64_t bars[AD_WARPS][AD_STAGES];
@@ -457,13 +458,13 @@ static int ad_grid() {
 template <int W, int S>
 static int launch_cfg(const bf16* q, const bf16* k_pages, const bf16* v_pages, const int32_t* block_table, int bt_stride,
                       const int32_t* seq_lens, float* scratch, bf16* out, int B, int nq, int nkv, float scale, int window,
-                      cudaStream_t s, int tag) {
+                      cudaStream_t s, int tag, int chunk) {
   constexpr int SMEM = W * S * AD_STAGE;
   static B2PerDeviceOnce attr_once, carve_once;
   if (attr_once.need()) B2_CUDA_OK(cudaFuncSetAttribute(attn_decode_kernel<W, S>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM));
   b2_prefer_max_smem(attn_decode_kernel<W, S>, carve_once);
   B2_CUDA_OK(b2_launch(attn_decode_kernel<W, S>, dim3(ad_grid()), dim3(W * 32), (size_t)SMEM, s, q, k_pages, v_pages, block_table,
-                       bt_stride, seq_lens, scratch, out, B, nq, nkv, scale, b2_pdl_early_mask() & 1, window, tag));
+                       bt_stride, seq_lens, scratch, out, B, nq, nkv, scale, b2_pdl_early_mask() & 1, window, tag, chunk));
   return 0;
 }
 
@@ -471,9 +472,9 @@ static int launch_cfg(const bf16* q, const bf16* k_pages, const bf16* v_pages, c
 // must be zero when the kernel starts -- the kernel leaves them zero again when it is done.
 int launch_attn_decode(const bf16* q, const bf16* k_pages, const bf16* v_pages, const int32_t* block_table,
                        int bt_stride, const int32_t* seq_lens, float* scratch, bf16* out, int B, int nq, int nkv,
-                       int hd, int block_size, cudaStream_t s, float softmax_scale, int window, int tag) {
+                       int hd, int block_size, cudaStream_t s, float softmax_scale, int window, int tag, int chunk) {
   if (B <= 0) return 0;
-  B2_REQUIRE(window >= 0, "attn_decode: negative window");
+  B2_REQUIRE(window >= 0 && chunk >= 0, "attn_decode: negative window or chunk");
   B2_REQUIRE(hd == AD_HD && block_size == AD_BS, "attn_decode: built for head_dim 128 / page 16 (got %d / %d)", hd, block_size);
   B2_REQUIRE(nq == 2 * nkv, "attn_decode: built for a GQA group of 2 (nq=%d nkv=%d)", nq, nkv);
   B2_REQUIRE(B <= AD_MAX_B && B * nkv <= AD_CNT, "attn_decode: batch %d x %d kv heads exceeds %d units", B, nkv, AD_CNT);
@@ -486,7 +487,7 @@ int launch_attn_decode(const bf16* q, const bf16* k_pages, const bf16* v_pages, 
     cfg = 82;
     if (e) { int w = 0, st = 0; if (sscanf(e, "%dx%d", &w, &st) == 2) cfg = w * 10 + st; }
   }
-#define AD_CASE(W, S) case (W) * 10 + (S): return launch_cfg<W, S>(q, k_pages, v_pages, block_table, bt_stride, seq_lens, scratch, out, B, nq, nkv, scale, window, s, tag)
+#define AD_CASE(W, S) case (W) * 10 + (S): return launch_cfg<W, S>(q, k_pages, v_pages, block_table, bt_stride, seq_lens, scratch, out, B, nq, nkv, scale, window, s, tag, chunk)
   switch (cfg) {
     AD_CASE(8, 3);
     AD_CASE(6, 4);

@@ -7,7 +7,8 @@
 //     that is run twice from the same bookkeeping -- the warm-up ahead of a graph capture -- leaves the same state),
 //   q and k heads divided by their root mean square,
 //   a linear distance penalty slope_a * (i - j) with slope_a = 2^(-slope_exp (a + 1) / heads),
-//   a sliding window that also keeps the first tokens of the sequence,
+//   a sliding window that also keeps the first tokens of the sequence, or chunks counted from position 0,
+//   rotary positions from a table (half-split or interleaved pairs, any frequencies), a token's value being its key before the rotation,
 //   value mixing v <- (1 - lam) v + lam v_first with the values another layer computed for the same token,
 //   mixing of the heads' softmax weights by a heads x heads matrix, and a sigmoid gate per head.
 //
@@ -20,6 +21,7 @@
 // Kernels:
 //   heads_finish      what follows the fused q | k | v (| gate) projection, one CTA per (token, head): bias, convolution, rotary or
 //                     unit-RMS norm, value mixing, cache row write, fp32 queries
+//   heads_finish_table  the same for rotary positions from a table (rot_table makes it), one CTA per token
 //   conv_tail_store   the ring update, after every token of the step has read the ring
 //   heads_attention   one warp per (query token, head) for prompt portions; for a decode step the eight warps of a CTA
 //                     split the keys of one (sequence, head) and merge.  Tiles of 32 keys: lane j scores key j, then lane
@@ -243,20 +245,78 @@ __global__ void __launch_bounds__(128) conv_tail_store_kernel(const float* __res
   for (int c = threadIdx.x; c < C; c += 128) dst[c] = row[c] + (bias ? bias[c] : 0.f);
 }
 
+// Rotary positions from a table, interleaved or half-split pairs.  A CTA takes `upc` heads of one token (query heads, key heads, value heads; without
+// v in the projection the key heads write both caches), one warp per head at a time.
+template <typename TC>
+__global__ void __launch_bounds__(256) heads_finish_table_kernel(const float* __restrict__ proj, int ld, HeadsGeom g, const float* __restrict__ bias,
+                                                                 const float* __restrict__ table, int halves, int keys_as_values,
+                                                                 const int32_t* __restrict__ positions, const int32_t* __restrict__ slots,
+                                                                 float* __restrict__ q_out, bf16* __restrict__ q_bf16, TC* __restrict__ k_cache,
+                                                                 TC* __restrict__ v_cache, int upc) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const int slot = slots[t];
+  if (slot < 0) return;   // padding row of a decode bucket
+  const int D = g.dim, half = g.rot_dims / 2, nq = g.heads * D, nk = g.kv_heads * D, nv = g.kv_heads * g.vdim;
+  const int units = g.heads + (keys_as_values ? 1 : 2) * g.kv_heads, u_lo = blockIdx.y * upc, u_hi = min(units, u_lo + upc);
+  const float* cs = table + (size_t)positions[t] * g.rot_dims;
+  const float* row = proj + (size_t)t * ld;
+  auto put = [&](TC* cache, int kvh, int width, int d, float v) {
+    if (g.swizzled) stf(cache + swizzled_index(slot, kvh, g.kv_heads, d), v);
+    else stf(cache + ((size_t)slot * g.kv_heads + kvh) * width + d, v);
+  };
+  for (int u = u_lo + warp; u < u_hi; u += nw) {
+    if (u >= g.heads + g.kv_heads) {
+      const int vh = u - g.heads - g.kv_heads, c0 = nq + nk + vh * g.vdim;
+      for (int i = lane; i < g.vdim; i += 32) put(v_cache, vh, g.vdim, i, row[c0 + i] + (bias ? bias[c0 + i] : 0.f));
+      continue;
+    }
+    const bool is_q = u < g.heads;
+    const int c0 = u * D, kh = u - g.heads;
+    auto emit = [&](int d, float v) {
+      if (!is_q) put(k_cache, kh, D, d, v);
+      else if (q_bf16 != nullptr) q_bf16[(size_t)t * nq + c0 + d] = __float2bfloat16_rn(v);
+      else q_out[(size_t)t * nq + c0 + d] = v;
+    };
+    for (int p = lane; p < half; p += 32) {
+      const int ia = halves ? p : 2 * p, ib = halves ? p + half : 2 * p + 1;
+      const float a = row[c0 + ia] + (bias ? bias[c0 + ia] : 0.f), b = row[c0 + ib] + (bias ? bias[c0 + ib] : 0.f), c = cs[p], s = cs[half + p];
+      emit(ia, a * c - b * s);
+      emit(ib, b * c + a * s);
+      if (!is_q && keys_as_values) {
+        put(v_cache, kh, D, ia, a);
+        put(v_cache, kh, D, ib, b);
+      }
+    }
+    for (int i = g.rot_dims + lane; i < D; i += 32) {
+      const float a = row[c0 + i] + (bias ? bias[c0 + i] : 0.f);
+      emit(i, a);
+      if (!is_q && keys_as_values) put(v_cache, kh, D, i, a);
+    }
+  }
+  (void)nv;
+}
+
+__global__ void __launch_bounds__(128) rot_table_kernel(const double* __restrict__ freqs, int half, double mul, float* __restrict__ table) {
+  const double p = (double)blockIdx.x;
+  for (int i = threadIdx.x; i < half; i += 128) {
+    double sd, cd;
+    sincos(p * freqs[i], &sd, &cd);
+    table[(size_t)blockIdx.x * 2 * half + i] = (float)(cd * mul);
+    table[(size_t)blockIdx.x * 2 * half + half + i] = (float)(sd * mul);
+  }
+}
+
 constexpr int HA_WARPS = 8;
 
 // Visible key tiles of query position i: tiles [0, nA) cover the kept first tokens, tiles [tB, i / 32] the window.
 struct TileRange {
   int nA, tB, total;
 };
-__device__ __forceinline__ TileRange visible_tiles(int i, int window, int keep_first) {
+__device__ __forceinline__ TileRange visible_tiles(int i, int window, int keep_first, int chunk) {
   TileRange r;
-  const int last = i >> 5;
-  if (window <= 0) {
-    r.nA = 0; r.tB = 0; r.total = last + 1;
-    return r;
-  }
-  const int lo = max(i - window + 1, 0);
+  const int last = i >> 5, lo = first_seen_key(i, window, chunk);
   const int endA = min(keep_first, lo);  // kept keys below the window
   r.nA = (endA + 31) >> 5;
   r.tB = max(lo >> 5, r.nA);
@@ -318,13 +378,13 @@ __global__ void __launch_bounds__(HA_WARPS * 32) heads_attention_kernel(const fl
 #pragma unroll
   for (int n = 0; n < NV; ++n) acc[n] = 0.f;
   if (live) {
-    const TileRange tr = visible_tiles(pos, g.window, g.keep_first);
+    const TileRange tr = visible_tiles(pos, g.window, g.keep_first, g.chunk);
     const int32_t* bt = block_table + (size_t)bt_row * bt_stride;
-    const int lo = g.window > 0 ? pos - g.window + 1 : 0;
+    const int lo = first_seen_key(pos, g.window, g.chunk);
     for (int vi = DECODE ? warp : 0; vi < tr.total; vi += DECODE ? HA_WARPS : 1) {
       const int tile = vi < tr.nA ? vi : tr.tB + (vi - tr.nA);
       const int j = (tile << 5) + lane;
-      const bool vis = j <= pos && (g.window <= 0 || j >= lo || j < g.keep_first);
+      const bool vis = j <= pos && (j >= lo || j < g.keep_first);
       float s = -INFINITY;
       size_t slot = 0;
       if (vis) {
@@ -523,12 +583,9 @@ __global__ void __launch_bounds__(128 * HPC, 2) heads_attention_mma_kernel(const
   for (int n = 0; n < NO; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
   // key tiles some row of the CTA sees
   const int last_key = tl.q_pos0 + tl.nrows - 1, last_tile = last_key / HM_KEYS;
-  int nA = 0, tB = 0;
-  if (g.window > 0) {
-    const int lo_min = max(tl.q_pos0 - g.window + 1, 0);
-    nA = (min(g.keep_first, lo_min) + HM_KEYS - 1) / HM_KEYS;
-    tB = max(lo_min / HM_KEYS, nA);
-  }
+  const int lo_min = first_seen_key(tl.q_pos0, g.window, g.chunk), lo_max = first_seen_key(last_key, g.window, g.chunk);
+  const int lo0 = first_seen_key(p0, g.window, g.chunk), lo1 = first_seen_key(p1, g.window, g.chunk);
+  const int nA = (min(g.keep_first, lo_min) + HM_KEYS - 1) / HM_KEYS, tB = max(lo_min / HM_KEYS, nA);
   const int total = nA + (last_tile - tB + 1);
   const int32_t* bt = block_table + (size_t)tl.bt_row * bt_stride;
   constexpr float LOG2E = 1.4426950408889634f;
@@ -585,7 +642,7 @@ __global__ void __launch_bounds__(128 * HPC, 2) heads_attention_mma_kernel(const
     // scale, distance penalty, mask; row maxima over the quad.  A tile that every row of the CTA sees whole needs no mask.
     float t0 = -INFINITY, t1 = -INFINITY;
     const bool whole = tl.nrows == HM_ROWS && key0 + HM_KEYS - 1 <= tl.q_pos0 &&
-                       (g.window <= 0 || last_key - key0 < g.window || key0 + HM_KEYS - 1 < g.keep_first);
+                       (lo_max <= key0 || key0 + HM_KEYS - 1 < g.keep_first);
     if (whole) {
 #pragma unroll
       for (int n = 0; n < HM_KEYS / 8; ++n) {
@@ -605,7 +662,7 @@ __global__ void __launch_bounds__(128 * HPC, 2) heads_attention_mma_kernel(const
         for (int e = 0; e < 4; ++e) {
           const int j = key0 + n * 8 + 2 * tq + (e & 1);
           const int p = (e & 2) ? p1 : p0;
-          const bool ok = ((e & 2) ? live1 : live0) && j <= p && (g.window <= 0 || p - j < g.window || j < g.keep_first);
+          const bool ok = ((e & 2) ? live1 : live0) && j <= p && (j >= ((e & 2) ? lo1 : lo0) || j < g.keep_first);
           const float v = ok ? sc[n][e] * g.scale - slope * (float)(p - j) : -INFINITY;
           sc[n][e] = v;
           if (e & 2) t1 = fmaxf(t1, v);
@@ -706,7 +763,7 @@ int launch_attention_mma(const float* q, const bf16* k, const bf16* v, const Hea
     *rc = launch_attention_mma_t<DD / 16, VV / 8, TO>(q, k, v, g, bt, bt_stride, block_size, tiles, ntiles, out, s);                 \
     return 1;                                                                                                                      \
   }
-  HM_CASE(32, 32) HM_CASE(64, 32) HM_CASE(64, 64) HM_CASE(96, 64) HM_CASE(96, 96) HM_CASE(128, 64) HM_CASE(128, 128) HM_CASE(192, 128) HM_CASE(256, 128)
+  HM_CASE(32, 32) HM_CASE(64, 32) HM_CASE(64, 64) HM_CASE(64, 128) HM_CASE(96, 64) HM_CASE(96, 96) HM_CASE(128, 64) HM_CASE(128, 128) HM_CASE(192, 128) HM_CASE(256, 128)
 #undef HM_CASE
   return 0;
 }
@@ -1679,6 +1736,31 @@ int launch_heads_finish_rownorm(const float* proj, int ld, const HeadsGeom& g, c
     else B2_ROWNORM(bf16, 128, q_bf16);
   }
 #undef B2_ROWNORM
+  return 0;
+}
+
+int launch_heads_finish_table(const float* proj, int ld, const HeadsGeom& g, const float* bias, const float* table, int halves, int keys_as_values,
+                              const int32_t* positions, const int32_t* slots, float* q_out, bf16* q_bf16, void* k_cache, void* v_cache, int cache_f32,
+                              int T, cudaStream_t s) {
+  if (T <= 0) return 0;
+  B2_REQUIRE(g.rot_dims == 0 || table != nullptr, "heads_finish_table: rotary positions need their table");
+  B2_REQUIRE(!keys_as_values || g.dim == g.vdim, "heads_finish_table: keys that serve as values need dim == vdim (%d, %d)", g.dim, g.vdim);
+  B2_REQUIRE(!g.swizzled || (!cache_f32 && q_bf16 != nullptr && g.dim == 128 && g.vdim == 128), "heads_finish_table: the GQA page layout holds 128-wide bf16 heads");
+  const int units = g.heads + (keys_as_values ? 1 : 2) * g.kv_heads, upc = T >= 256 ? units : 8;   // few tokens: several CTAs each
+  const dim3 grid(T, (units + upc - 1) / upc);
+  if (cache_f32)
+    B2_CUDA_OK(b2_launch(heads_finish_table_kernel<float>, grid, dim3(256), 0, s, proj, ld, g, bias, table, halves, keys_as_values, positions, slots, q_out, q_bf16,
+                         (float*)k_cache, (float*)v_cache, upc));
+  else
+    B2_CUDA_OK(b2_launch(heads_finish_table_kernel<bf16>, grid, dim3(256), 0, s, proj, ld, g, bias, table, halves, keys_as_values, positions, slots, q_out, q_bf16,
+                         (bf16*)k_cache, (bf16*)v_cache, upc));
+  return 0;
+}
+
+int launch_rot_table(const double* freqs, int half, double mul, float* table, int npos, cudaStream_t s) {
+  if (half <= 0 || npos <= 0) return 0;
+  rot_table_kernel<<<npos, 128, 0, s>>>(freqs, half, mul, table);
+  B2_CUDA_OK(cudaGetLastError());
   return 0;
 }
 

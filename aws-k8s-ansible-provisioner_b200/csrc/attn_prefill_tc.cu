@@ -72,7 +72,7 @@ constexpr float PT_RESCALE = 8.0f;  // log2 units: the reference maximum is rais
 __global__ void __launch_bounds__(PT_THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, const bf16* __restrict__ q,
                        const int32_t* __restrict__ block_table, int bt_stride, const PrefillTile* __restrict__ tiles,
-                       bf16* __restrict__ out, int nq, int nkv, float scale_log2, int window, int pair_mode, int head_step) {
+                       bf16* __restrict__ out, int nq, int nkv, float scale_log2, int window, int pair_mode, int head_step, int chunk) {
   extern __shared__ uint8_t smem_raw[];
   __shared__ __align__(8) uint64_t k_full, v_full, s_full, p_full, o_full;
   __shared__ uint32_t tmem_slot;
@@ -96,7 +96,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
   const int kvh = blockIdx.y;
   const int kv_len = (pair_mode && tile_b.nrows > 0) ? tile_b.q_pos0 + tile_b.nrows : tile.q_pos0 + tile.nrows;
   const int n_kt = (kv_len + PT_BN - 1) / PT_BN;
-  const int kt0 = (window > 0 && tile.q_pos0 - window + 1 > 0) ? (tile.q_pos0 - window + 1) / PT_BN : 0;
+  const int kt0 = first_seen_key(tile.q_pos0, window, chunk) / PT_BN;
   const int32_t* bt = block_table + (size_t)tile.bt_row * bt_stride;
 
   if (threadIdx.x == 0) {
@@ -220,9 +220,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
       // A tile that lies wholly inside the range of EVERY row of the CTA (all but the last one or two tiles of a row
       // block) takes the branch without per-element masks; the test is uniform over the CTA.
       const int hi_col = row_ok ? min(qpos, row_kv_len - 1) : -1;
-      const int lo_col = (window > 0 && qpos - window + 1 > 0) ? qpos - window + 1 : 0;
+      const int lo_col = first_seen_key(qpos, window, chunk);
       const bool full_tile = key0 + PT_BN - 1 <= tile.q_pos0 && tile.nrows == PT_TQ && tile_b.nrows == PT_TQ &&
-                             (window <= 0 || tile_b.q_pos0 + PT_TQ - 1 - key0 < window);
+                             first_seen_key(tile_b.q_pos0 + PT_TQ - 1, window, chunk) <= key0;
       // pass 1: the row maximum (the scale is positive: max(s * c) = c * max(s)); four chains instead of one
       float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll 1
@@ -341,7 +341,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
 // num_pages: pages in the pool k_pages / v_pages point to (the TMA maps cover exactly the pool).
 int launch_attn_prefill_tc(const bf16* q, const bf16* k_pages, const bf16* v_pages, int64_t num_pages, const int32_t* block_table,
                            int bt_stride, const PrefillTile* tiles_dev, int ntiles, bf16* out, int nq, int nkv, int hd, int block_size,
-                           cudaStream_t s, float softmax_scale, int window, int pair_mode) {
+                           cudaStream_t s, float softmax_scale, int window, int pair_mode, int chunk) {
   if (ntiles <= 0) return 0;
   const int head_step = pair_mode && nq == nkv ? 1 : 2;
   B2_REQUIRE(hd == PT_HD && block_size == 16 && nq == head_step * nkv, "attn_prefill_tc: built for 128-wide heads in GQA groups of two, 16-token pages");
@@ -359,7 +359,7 @@ int launch_attn_prefill_tc(const bf16* q, const bf16* k_pages, const bf16* v_pag
   const float scale_log2 = (float)(scale * 1.4426950408889634);
   B2_REQUIRE(!pair_mode || ntiles % 2 == 0, "attn_prefill_tc: pair mode needs an even tile list (each sequence padded to an even number of tiles)");
   B2_CUDA_OK(b2_launch(attn_prefill_tc_kernel, dim3(pair_mode ? ntiles / 2 : ntiles, nkv), dim3(PT_THREADS), (size_t)PT_SMEM, s, tk, tv, q, block_table,
-                       bt_stride, tiles_dev, out, nq, nkv, scale_log2, window, pair_mode, head_step));
+                       bt_stride, tiles_dev, out, nq, nkv, scale_log2, window, pair_mode, head_step, chunk));
   return 0;
 }
 

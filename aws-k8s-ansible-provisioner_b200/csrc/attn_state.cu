@@ -6,6 +6,8 @@
 //   STATE_RULE_DELTA   S <- diag(a_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t     (gated delta rule)
 //
 //   STATE_RULE_DELTA_HEAD   the same with ONE decay per head, S <- a_t S
+//   STATE_RULE_DECAY_HEAD   S <- a_t S + d_t k_t v_t^T;  o_t = S^T q_t + D v_t                          (state-space recurrence, d_t the step size)
+//   STATE_RULE_BONUS   o_t = (S + diag(u) k_t v_t^T)^T q_t;  S <- diag(a_t) S + k_t v_t^T               (time mixing with a bonus for the current token)
 //
 // a_t is a decay per head and key channel (or per head) in (0, 1); it scales the rows of S.  Query/key head of state head a is
 // a / (heads / kv_heads).
@@ -32,8 +34,10 @@
 //                      (a warp per head), beta
 //   conv_unit_rows     the same for prompt-sized steps (a CTA walks down sixteen rows of one head)
 //   conv_ring_store    the ring update, after every token of the step has read the ring (a decode step's tokens do it themselves)
+//   conv_act           state-space mixer: causal convolution with bias + silu on x | B | C, step sizes and decays
 //   state_scan         the recurrence; state_scan_head: the delta rule with one decay per head on packed fp32 pairs
 //   state_out_gate     per-head RMS norm of the read-out with a gain, times the gate (silu or given), operand type out
+//   gate_part_norm     the read-out times silu(gate), RMS-normed in equal parts, operand type out
 #include "kernels.h"
 
 namespace b2 {
@@ -54,7 +58,10 @@ __global__ void __launch_bounds__(256) lowrank_act_kernel(const float* __restric
   pdl_wait();
   pdl_launch_dependents();
   const int t0 = blockIdx.x * LR_TOKENS, tn = min(LR_TOKENS, T - t0);
-  for (int i = threadIdx.x; i < tn * rank; i += 256) lrs[i] = lr[(size_t)(t0 + i / rank) * ld + lr_off + i % rank];
+  for (int i = threadIdx.x; i < tn * rank; i += 256) {
+    const float v = lr[(size_t)(t0 + i / rank) * ld + lr_off + i % rank];
+    lrs[i] = mode == LOWRANK_DECAY_EXP ? tanhf(v) : v;
+  }
   __syncthreads();
   const int c = blockIdx.y * 256 + threadIdx.x;
   if (c >= C) return;
@@ -97,6 +104,7 @@ __global__ void __launch_bounds__(256) lowrank_act_kernel(const float* __restric
     float y;
     if (mode == LOWRANK_SIGMOID) y = sigmoid_f(zz);
     else if (mode == LOWRANK_DECAY_SIGMOID_POW) y = expf(-rt * softplus_f(-zz));               // sigmoid(z)^rate
+    else if (mode == LOWRANK_DECAY_EXP) y = expf(-expf(zz));
     else y = expf(-rt * softplus_f(zz));                                                       // exp(-exp(A) softplus(z))
     out[(size_t)(t0 + tt) * C + c] = y;
   }
@@ -256,6 +264,89 @@ __global__ void __launch_bounds__(128) conv_unit_rows_kernel(const float* __rest
   }
 }
 
+// A thread owns a channel of x | B | C and walks down `rows` neighbouring token rows with the last inputs in registers (rows = 1 in short steps).  proj
+// [T][ld] fp32 = x | B | C | step logits.  The first CTA column also forms the step sizes and decays.
+template <int TAPS>   // 0: any number of taps
+__global__ void __launch_bounds__(128) conv_act_kernel(const float* __restrict__ proj, int ld, int C, int heads, int taps_any, const float* __restrict__ conv_w,
+                                                       const float* __restrict__ conv_b, const float* __restrict__ a_log, const float* __restrict__ dt_bias,
+                                                       const float* __restrict__ ring, float* __restrict__ ring_store, const int32_t* __restrict__ row_seq,
+                                                       const int32_t* __restrict__ row_first, const int32_t* __restrict__ positions,
+                                                       const int32_t* __restrict__ slots, float* __restrict__ out, float* __restrict__ step,
+                                                       float* __restrict__ decay, int rows, int T) {
+  const int t0 = blockIdx.x * rows, tn = min(rows, T - t0), c = blockIdx.y * 128 + threadIdx.x;
+  const int taps = TAPS > 0 ? TAPS : taps_any;
+  float w[TAPS > 0 ? TAPS : 1], bias = 0.f;   // constants of the model: readable before the kernel in front is done
+  if (c < C) {
+    bias = conv_b[c];
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int d = 0; d < TAPS; ++d) w[d] = conv_w[(size_t)c * TAPS + TAPS - 1 - d];
+    }
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  if (c < C) {
+    for (int i = 0; i < tn;) {   // runs of rows of one portion
+      const int t = t0 + i, first = row_first[t], pos = positions[t], back = t - first;
+      const bool live = slots[t] >= 0;
+      const float* rg = ring + (size_t)row_seq[t] * taps * C + c;
+      int e = i + 1;
+      while (e < tn && row_first[t0 + e] == first) ++e;
+      if constexpr (TAPS > 0) {
+        float hist[TAPS];   // hist[d]: the input d rows back
+#pragma unroll
+        for (int d = 1; d < TAPS; ++d)
+          hist[d] = !live       ? 0.f
+                    : d <= back ? proj[(size_t)(t - d) * ld + c]
+                    : pos >= d  ? rg[(size_t)((pos - d) % TAPS) * C]
+                                : 0.f;
+        while (i < e) {   // eight rows' loads in flight at a time
+          const int m = min(8, e - i);
+          float x[8];
+#pragma unroll
+          for (int r = 0; r < 8; ++r) x[r] = r < m ? proj[(size_t)(t0 + i + r) * ld + c] : 0.f;
+#pragma unroll
+          for (int r = 0; r < 8; ++r) {
+            if (r < m) {
+              float acc = bias;
+#pragma unroll
+              for (int d = TAPS - 1; d >= 1; --d) acc = fmaf(w[d], hist[d], acc);
+              acc = fmaf(w[0], x[r], acc);
+#pragma unroll
+              for (int d = TAPS - 1; d >= 2; --d) hist[d] = hist[d - 1];
+              if (TAPS > 1) hist[TAPS > 1 ? 1 : 0] = x[r];
+              if (live) {
+                out[(size_t)(t0 + i + r) * C + c] = silu_f(acc);
+                if (ring_store) ring_store[((size_t)row_seq[t] * TAPS + pos % TAPS) * C + c] = x[r];   // (steps of single rows: an entry that no row reads)
+              }
+            }
+          }
+          i += m;
+        }
+      } else {
+        for (; i < e; ++i) {
+          const int tt = t0 + i, pp = positions[tt], bb = tt - first;
+          if (!live) continue;
+          float acc = bias;
+          for (int d = taps - 1; d >= 0; --d) {
+            const float xx = d <= bb ? proj[(size_t)(tt - d) * ld + c] : (pp >= d ? rg[(size_t)((pp - d) % taps) * C] : 0.f);
+            acc = fmaf(conv_w[(size_t)c * taps + taps - 1 - d], xx, acc);
+          }
+          out[(size_t)tt * C + c] = silu_f(acc);
+          if (ring_store) ring_store[((size_t)row_seq[tt] * taps + pp % taps) * C + c] = proj[(size_t)tt * ld + c];
+        }
+      }
+    }
+  }
+  if (blockIdx.y == 0)
+    for (int i = threadIdx.x; i < tn * heads; i += 128) {
+      const int t = t0 + i / heads, a = i % heads;
+      const float d = softplus_f(proj[(size_t)t * ld + C + a] + dt_bias[a]);
+      step[(size_t)t * heads + a] = d;
+      decay[(size_t)t * heads + a] = expf(-expf(a_log[a]) * d);
+    }
+}
+
 __global__ void __launch_bounds__(128) conv_ring_store_kernel(const float* __restrict__ proj, int ld, int C, int taps, float* __restrict__ ring,
                                                               const int32_t* __restrict__ row_seq, const int32_t* __restrict__ row_end,
                                                               const int32_t* __restrict__ positions, const int32_t* __restrict__ slots) {
@@ -299,7 +390,8 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
   constexpr int VW = DPT >= 4 ? 4 : DPT;    // channels per shared-memory load
   constexpr int DP = DPT * SC_LANES;
   constexpr int MAXC = 32 * NC;             // columns of a CTA at most
-  constexpr bool HEAD = RULE == STATE_RULE_DELTA_HEAD;   // one decay per head and token: nothing staged per channel
+  constexpr bool HEAD = RULE == STATE_RULE_DELTA_HEAD || RULE == STATE_RULE_DECAY_HEAD;   // one decay per head and token: nothing staged per channel
+  constexpr bool BETA = RULE != STATE_RULE_DECAY && RULE != STATE_RULE_BONUS;
   __shared__ __align__(16) float qs[2][CH][RS], ks[2][CH][RS], as[HEAD ? 1 : 2][HEAD ? 1 : CH][HEAD ? 4 : RS];
   __shared__ float ds[2][HEAD ? CH : 1];
   __shared__ __align__(16) float vs[2][CH][MAXC];
@@ -359,7 +451,7 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
       const int tt = vsh >= 0 ? i >> vsh : i / vcols, c = vsh >= 0 ? i & (vcols - 1) : i % vcols;
       cp_async_f32(&vs[st][tt][c], vb + (size_t)(c0 + tt) * ldv + c);
     }
-    if (RULE != STATE_RULE_DECAY) {   // (a plain `if`: a discarded loop without braces took the statement behind it along)
+    if (BETA) {   // (a plain `if`: a discarded loop without braces took the statement behind it along)
       for (int i = threadIdx.x; i < cn; i += nthreads) {
         cp_async_f32(&bs[st][i], beta + (size_t)(first + c0 + i) * g.heads + a);
         if (HEAD) {
@@ -376,6 +468,15 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
 #pragma unroll
     for (int c = 0; c < NC; ++c) s[i][c] = (pos0 > 0 && d < g.dim && col0 + cl + c < g.vdim) ? s_in[(size_t)d * g.vdim + col0 + cl + c] : 0.f;
   }
+  float bonus[RULE == STATE_RULE_BONUS ? DPT : 1];   // this lane's channels
+  if constexpr (RULE == STATE_RULE_BONUS) {
+#pragma unroll
+    for (int i = 0; i < DPT; ++i) {
+      const int d = i * SC_LANES + j;
+      bonus[i] = d < g.dim ? g.bonus[a * g.dim + d] : 0.f;
+    }
+  }
+  const float skip = RULE == STATE_RULE_DECAY_HEAD ? g.skip[a] : 0.f;
   auto load = [&](const float* p, int i, float* dst) {
     if constexpr (VW == 4) {
       const float4 x = *reinterpret_cast<const float4*>(p + i);
@@ -422,6 +523,42 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
               acc[c] = fmaf(s[i + x][c], qv[x], acc[c]);
             }
         }
+      } else if constexpr (RULE == STATE_RULE_DECAY_HEAD) {
+        const float gd = ds[st][tt], bt = bs[st][tt];
+        float wv[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) wv[c] = bt * vc[c];
+#pragma unroll
+        for (int i = 0; i < DPT; i += VW) {
+          load(kp, i, kw);
+          load(qp, i, qv);
+#pragma unroll
+          for (int x = 0; x < VW; ++x)
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+              s[i + x][c] = fmaf(kw[x], wv[c], gd * s[i + x][c]);
+              acc[c] = fmaf(s[i + x][c], qv[x], acc[c]);
+            }
+        }
+      } else if constexpr (RULE == STATE_RULE_BONUS) {
+        float ruk = 0.f;   // sum of q u k over this lane's channels: every column's bonus is that times its v
+#pragma unroll
+        for (int i = 0; i < DPT; i += VW) {
+          load(ap, i, av);
+          load(kp, i, kw);
+          load(qp, i, qv);
+#pragma unroll
+          for (int x = 0; x < VW; ++x) {
+            ruk = fmaf(qv[x] * bonus[i + x], kw[x], ruk);
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+              acc[c] = fmaf(s[i + x][c], qv[x], acc[c]);
+              s[i + x][c] = fmaf(av[x], s[i + x][c], kw[x] * vc[c]);
+            }
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) acc[c] = fmaf(ruk, vc[c], acc[c]);
       } else if constexpr (HEAD) {
         // S' = g S + k u^T with u = beta (v - g S^T k): the decay is a number, so it leaves the sum over the key channels and joins the update
         const float gd = ds[st][tt], bt = bs[st][tt];
@@ -502,7 +639,7 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
         float* orow = out + (size_t)(first + c0 + tt) * ((size_t)g.heads * g.vdim) + a * g.vdim + col0 + cl;
 #pragma unroll
         for (int c = 0; c < NC; ++c)
-          if (col0 + cl + c < g.vdim) orow[c] = acc[c] * qscale;
+          if (col0 + cl + c < g.vdim) orow[c] = RULE == STATE_RULE_DECAY_HEAD ? fmaf(skip, vc[c], acc[c] * qscale) : acc[c] * qscale;
       }
     }
   }
@@ -714,7 +851,7 @@ __global__ void __launch_bounds__(256) state_scan_head_kernel(const float* __res
 template <typename TX>
 __global__ void __launch_bounds__(128) state_out_gate_kernel(const float* __restrict__ o, const float* __restrict__ gain,
                                                              const float* __restrict__ gate, int gate_ld, int gate_silu, TX* __restrict__ out,
-                                                             int heads, int vdim, float eps, int T) {
+                                                             int heads, int vdim, float eps, int T, int gain_per_head, float scale, int out_ld) {
   pdl_wait();
   pdl_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -726,9 +863,10 @@ __global__ void __launch_bounds__(128) state_out_gate_kernel(const float* __rest
   float ss = 0.f;
   for (int i = lane; i < vdim; i += 32) ss = fmaf(orow[i], orow[i], ss);
   ss = warp_sum(ss);
-  const float r = 1.0f / sqrtf(ss / (float)vdim + eps);
-  TX* dst = out + ((size_t)t * heads + a) * vdim;
-  if (vdim % 4 == 0 && gate_ld % 4 == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0) {   // sixteen bytes at a time
+  const float r = scale / sqrtf(ss / (float)vdim + eps);
+  TX* dst = out + (size_t)t * out_ld + (size_t)a * vdim;
+  if (gain_per_head) gain += (size_t)a * vdim;
+  if (vdim % 4 == 0 && gate_ld % 4 == 0 && out_ld % 4 == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0) {   // sixteen bytes at a time
     for (int i = lane * 4; i < vdim; i += 128) {
       const float4 ov = *reinterpret_cast<const float4*>(orow + i), gv = *reinterpret_cast<const float4*>(grow + i);
       const float4 nv = *reinterpret_cast<const float4*>(gain + i);
@@ -751,6 +889,95 @@ __global__ void __launch_bounds__(128) state_out_gate_kernel(const float* __rest
     const float gt = gate_silu ? silu_f(grow[i]) : grow[i];
     dst[i] = (TX)(orow[i] * r * gain[i] * gt);
   }
+}
+
+// One CTA of NT threads per (token, part): v = o * silu(gate) is formed once and kept in registers (R groups of four numbers a thread) or, for other
+// sizes (R = 0), in shared memory.
+template <typename TX, int NT, int R>
+__global__ void __launch_bounds__(NT) gate_part_norm_kernel(const float* __restrict__ o, const float* __restrict__ gate, int gate_ld,
+                                                            const float* __restrict__ gain, float scale, TX* __restrict__ out, int out_ld, int N, int part,
+                                                            float eps) {
+  extern __shared__ float vrow[];
+  __shared__ float red[NT / 32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, c0 = blockIdx.y * part;
+  const float* orow = o + (size_t)t * N + c0;
+  const float* grow = gate + (size_t)t * gate_ld + c0;
+  TX* dst = out + (size_t)t * out_ld + c0;
+  float ss = 0.f;
+  float4 v[R > 0 ? R : 1];
+  if constexpr (R > 0) {
+    float4 gv[R];
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int i = threadIdx.x + r * NT;
+      const bool in = 4 * i < part;
+      v[r] = in ? reinterpret_cast<const float4*>(orow)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+      gv[r] = in ? reinterpret_cast<const float4*>(grow)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      v[r].x *= silu_f(gv[r].x); v[r].y *= silu_f(gv[r].y); v[r].z *= silu_f(gv[r].z); v[r].w *= silu_f(gv[r].w);
+      ss += (v[r].x * v[r].x + v[r].y * v[r].y) + (v[r].z * v[r].z + v[r].w * v[r].w);
+    }
+  } else {
+    for (int i = threadIdx.x; i < part; i += NT) {
+      const float x = orow[i] * silu_f(grow[i]);
+      vrow[i] = x;
+      ss = fmaf(x, x, ss);
+    }
+  }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int w = 0; w < NT / 32; ++w) tot += red[w];
+  const float rn = scale / sqrtf(tot / (float)part + eps);
+  if constexpr (R > 0) {
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int i = threadIdx.x + r * NT;
+      if (4 * i >= part) continue;
+      const float4 gn = reinterpret_cast<const float4*>(gain + c0)[i];
+      const float y[4] = {v[r].x * rn * gn.x, v[r].y * rn * gn.y, v[r].z * rn * gn.z, v[r].w * rn * gn.w};
+      if constexpr (sizeof(TX) == 4) {
+        *reinterpret_cast<float4*>(dst + 4 * i) = make_float4(y[0], y[1], y[2], y[3]);
+      } else {
+        uint2 pk;
+        pk.x = pack_bf16x2(y[0], y[1]);
+        pk.y = pack_bf16x2(y[2], y[3]);
+        *reinterpret_cast<uint2*>(dst + 4 * i) = pk;
+      }
+    }
+  } else {
+    for (int i = threadIdx.x; i < part; i += NT) dst[i] = (TX)(vrow[i] * rn * gain[c0 + i]);   // (a thread's own columns)
+  }
+}
+
+template <typename TX>
+int gate_part_norm_typed(const float* o, const float* gate, int gate_ld, const float* gain, int parts, float scale, TX* out, int out_ld, int N, float eps,
+                         int T, cudaStream_t s) {
+  const int part = N / parts;
+  const dim3 grid(T, parts);
+#define B2_GPN(NT, R)                                                                                                                              \
+  do {                                                                                                                                             \
+    B2_CUDA_OK(b2_launch(gate_part_norm_kernel<TX, NT, R>, grid, dim3(NT), 0, s, o, gate, gate_ld, gain, scale, out, out_ld, N, part, eps));        \
+    return 0;                                                                                                                                      \
+  } while (0)
+  const bool vec = part % 4 == 0 && gate_ld % 4 == 0 && out_ld % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  if (vec && part <= 512) B2_GPN(128, 1);
+  if (vec && part <= 2048) B2_GPN(256, 2);
+  if (vec && part <= 4096) B2_GPN(512, 2);
+  if (vec && part <= 8192) B2_GPN(512, 4);
+#undef B2_GPN
+  B2_REQUIRE((size_t)part * 4 <= 160 * 1024, "gate_part_norm: a part of %d numbers does not fit in shared memory", part);
+  static B2PerDeviceOnce once;
+  if ((size_t)part * 4 > 48 * 1024) b2_prefer_max_smem(gate_part_norm_kernel<TX, 256, 0>, once);
+  B2_CUDA_OK(b2_launch(gate_part_norm_kernel<TX, 256, 0>, grid, dim3(256), (size_t)part * 4, s, o, gate, gate_ld, gain, scale, out, out_ld, N, part, eps));
+  return 0;
 }
 
 template <int RULE>
@@ -825,7 +1052,8 @@ int launch_state_scan(const float* q, int ldq, const float* k, int ldk, const fl
                       cudaStream_t s) {
   if (portions <= 0) return 0;
   B2_REQUIRE(g.heads >= 1 && g.kv_heads >= 1 && g.heads % g.kv_heads == 0 && g.dim >= 1 && g.vdim >= 1, "state_scan: bad sizes");
-  B2_REQUIRE(g.rule == STATE_RULE_DECAY || ((g.rule == STATE_RULE_DELTA || g.rule == STATE_RULE_DELTA_HEAD) && beta != nullptr), "state_scan: rule %d", g.rule);
+  B2_REQUIRE(g.rule == STATE_RULE_DECAY || (g.rule == STATE_RULE_BONUS && g.bonus != nullptr) ||
+                 (g.rule == STATE_RULE_DECAY_HEAD && g.skip != nullptr && beta != nullptr) || ((g.rule == STATE_RULE_DELTA || g.rule == STATE_RULE_DELTA_HEAD) && beta != nullptr), "state_scan: rule %d", g.rule);
   int dpt = 1;
   while (dpt * SC_LANES < g.dim) dpt *= 2;
   B2_REQUIRE(dpt <= 32, "state_scan: key width %d not built (at most 256)", g.dim);
@@ -837,6 +1065,12 @@ int launch_state_scan(const float* q, int ldq, const float* k, int ldk, const fl
   const dim3 grid(portions, g.heads, (g.vdim + cols - 1) / cols), block(cols / nc * SC_LANES);
   if (g.rule == STATE_RULE_DECAY)
     return launch_scan_rule<STATE_RULE_DECAY>(dpt, grid, block, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,
+                                              row_first, row_end, positions, slots, out, cols);
+  if (g.rule == STATE_RULE_DECAY_HEAD)
+    return launch_scan_rule<STATE_RULE_DECAY_HEAD>(dpt, grid, block, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,
+                                                   row_first, row_end, positions, slots, out, cols);
+  if (g.rule == STATE_RULE_BONUS)
+    return launch_scan_rule<STATE_RULE_BONUS>(dpt, grid, block, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,
                                               row_first, row_end, positions, slots, out, cols);
   static const bool packed = [] { const char* e = getenv("B2_SCAN_PACKED"); return !(e && *e == '0'); }();   // 0: the generic form (cross-check)
   const bool rows16 = g.dim % 4 == 0 && g.vdim % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ldv % 4 == 0 &&
@@ -861,13 +1095,47 @@ int launch_state_scan(const float* q, int ldq, const float* k, int ldk, const fl
 size_t state_floats_per_slot(const StateGeom& g) { return (size_t)2 * g.heads * g.dim * g.vdim; }
 
 int launch_state_out_gate(const float* o, const float* gain, const float* gate, int gate_ld, int gate_silu, void* out, int out_f32,
-                          int heads, int vdim, float eps, int T, cudaStream_t s) {
+                          int heads, int vdim, float eps, int T, cudaStream_t s, int gain_per_head, float scale, int out_ld) {
   if (T <= 0) return 0;
+  if (out_ld <= 0) out_ld = heads * vdim;
   const long units = (long)T * heads;
   const dim3 grid((unsigned)((units + 3) / 4));
-  if (out_f32) B2_CUDA_OK(b2_launch(state_out_gate_kernel<float>, grid, dim3(128), 0, s, o, gain, gate, gate_ld, gate_silu, (float*)out, heads, vdim, eps, T));
-  else B2_CUDA_OK(b2_launch(state_out_gate_kernel<bf16>, grid, dim3(128), 0, s, o, gain, gate, gate_ld, gate_silu, (bf16*)out, heads, vdim, eps, T));
+  if (out_f32)
+    B2_CUDA_OK(b2_launch(state_out_gate_kernel<float>, grid, dim3(128), 0, s, o, gain, gate, gate_ld, gate_silu, (float*)out, heads, vdim, eps, T, gain_per_head,
+                         scale, out_ld));
+  else
+    B2_CUDA_OK(b2_launch(state_out_gate_kernel<bf16>, grid, dim3(128), 0, s, o, gain, gate, gate_ld, gate_silu, (bf16*)out, heads, vdim, eps, T, gain_per_head,
+                         scale, out_ld));
   return 0;
+}
+
+int launch_conv_act_finish(const float* proj, int ld, int channels, int heads, int taps, const float* conv_w, const float* conv_b, const float* a_log,
+                           const float* dt_bias, float* ring, const int32_t* row_seq, const int32_t* row_first, const int32_t* row_end,
+                           const int32_t* positions, const int32_t* slots, float* out, float* step, float* decay, int T, int single_rows, cudaStream_t s) {
+  if (T <= 0) return 0;
+  B2_REQUIRE(taps >= 1 && (ring != nullptr || taps == 1), "conv_act_finish: a convolution of %d taps needs its ring", taps);
+  const int rows = single_rows || T < 512 ? 1 : CR_ROWS;
+  const dim3 grid((T + rows - 1) / rows, (channels + 127) / 128);
+  float* store = single_rows && taps > 1 ? ring : nullptr;
+#define B2_CONV_ACT(TAPS)                                                                                                                        \
+  B2_CUDA_OK(b2_launch(conv_act_kernel<TAPS>, grid, dim3(128), 0, s, proj, ld, channels, heads, taps, conv_w, conv_b, a_log, dt_bias, (const float*)ring, store, \
+                       row_seq, row_first, positions, slots, out, step, decay, rows, T))
+  if (taps == 4) B2_CONV_ACT(4);
+  else if (taps == 3) B2_CONV_ACT(3);
+  else if (taps == 2) B2_CONV_ACT(2);
+  else B2_CONV_ACT(0);
+#undef B2_CONV_ACT
+  if (taps > 1 && !single_rows)
+    B2_CUDA_OK(b2_launch(conv_ring_store_kernel, dim3(T), dim3(128), 0, s, proj, ld, channels, taps, ring, row_seq, row_end, positions, slots));
+  return 0;
+}
+
+int launch_gate_part_norm(const float* o, const float* gate, int gate_ld, const float* gain, int parts, float scale, void* out, int out_f32, int out_ld,
+                          int N, float eps, int T, cudaStream_t s) {
+  if (T <= 0) return 0;
+  B2_REQUIRE(parts >= 1 && N % parts == 0, "gate_part_norm: %d numbers in %d parts", N, parts);
+  return out_f32 ? gate_part_norm_typed<float>(o, gate, gate_ld, gain, parts, scale, (float*)out, out_ld, N, eps, T, s)
+                 : gate_part_norm_typed<bf16>(o, gate, gate_ld, gain, parts, scale, (bf16*)out, out_ld, N, eps, T, s);
 }
 
 }  // namespace b2

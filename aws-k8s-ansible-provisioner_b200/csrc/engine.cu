@@ -119,6 +119,14 @@ struct ListLayer {
   // Norms behind the sublayers only (Tolanex): gain1b / gain2b.  Its delta mixer projects q | k | v | beta | decay | gate in `wqd` (off_sg = the
   // gate's first column), with `a_log` and `a2_bias` per head; its latent mixer q (| the latent) in `wqd`; `router` holds the shared expert's
   // gate row behind the experts' rows.
+  // Two mixers side by side on several residual streams (Resitar).  hc[0 / 1]: the mixer's / feed-forward's stream numbers in | out | mix.  `wqd` = left
+  // q | k (| v) | gate (off_sg), then the state-space mixer's z (off_sq) | x | B | C (off_sk) | step logits; the time mixing has `wshift` = r | k | v | g one
+  // behind the other (each reads a blend of its own), the low-rank stage w1 with zero rows up to rank_pad, `a2` = w2, `a2_bias` = w0 (or dt_bias), `mu`,
+  // `bonus`.  `wo` = both output projections side by side, [W][left heads | right heads]: the two scales are applied to their inputs.
+  float *hc[2] = {nullptr, nullptr}, *mu = nullptr, *bonus = nullptr, *skip = nullptr, *conv_b = nullptr;
+  void *wshift = nullptr, *w1 = nullptr;
+  int rank_pad = 0;
+  const float* rot_table = nullptr;   // [max_model_len][rot_dims] (owned by the engine: layers with equal rotary settings share it)
 };
 // One run of a layer.  A looped layer runs once per pass with the same weights (ListLayer) but a cache and state of its own.
 struct ListRun {
@@ -127,9 +135,12 @@ struct ListRun {
   int k_region = -1, v_region = -1;
   float* state = nullptr;      // [sequence slots][2][heads][dim][vdim] fp32 (attn_state.cu)
   float* ring = nullptr;       // [sequence slots][taps][channels] fp32: the convolutions' last inputs
+  void* shift_ring = nullptr;  // [sequence slots][2][W] operand type: the last mixer input (index = position mod 2)
 };
 inline bool list_arch(int arch) { return arch == B2_ARCH_LERASUN || arch == B2_ARCH_KEDASUN || arch == B2_ARCH_BUMALIX || arch == B2_ARCH_TINEVIK ||
-                                        arch == B2_ARCH_TOLANEX; }
+                                        arch == B2_ARCH_TOLANEX || arch == B2_ARCH_RESITAR; }
+// mixers that keep keys and values per head in a region pair per run
+inline bool keeps_kv(int mixer) { return mixer == B2_MIXER_WINDOW_AND_STATE || mixer == B2_MIXER_CHUNK_AND_SSM || mixer == B2_MIXER_FULL_AND_TIMEMIX; }
 
 struct Seq {
   bool active = false;
@@ -359,6 +370,13 @@ struct b2_engine {
   int32_t* l_tok_ring = nullptr;     // [sequence slots][2]: the token at a position, by the position's parity (a sequence's previous token)
   float* l_rz = nullptr;             // a prompt-sized step's router logits
   float* l_sg = nullptr;             // the shared expert's gate, one number per token row
+  // several residual streams (Resitar; l_h is then [T][streams][W])
+  int n_streams = 1;
+  struct RotTable { b2_layer_spec key; float* table; };
+  std::vector<RotTable> rot_tables;
+  void *l_shift = nullptr, *l_ao = nullptr;      // the five blends [5][T][W]; the attention's output before the gate
+  float *l_rkvg = nullptr, *l_lr = nullptr, *l_cv = nullptr;   // the time mixing's projections [4][T][heads * dim]; its low-rank values; convolved x | B | C
+  size_t l_lr_cols = 0;
   // Prompt portions whose latent attention runs over rebuilt keys and values (attn_latent.cu): the step's long portions in groups whose contexts
   // fit the scratch pools; a paired tile list, a block table of scratch pages and the contexts of each group.  d_tiles holds the short portions' tiles first.
   struct LatentGroup { int ctx0, nctx, max_pages, pages, tile0, ntiles; };
@@ -930,10 +948,11 @@ bool list_use_tc() {
   static const bool use_tc = [] { const char* v = getenv("B2_LIST_TC"); return !(v && *v == '0'); }();
   return use_tc;
 }
+bool list_dense_tc(const b2_engine* e, int M, int N, int K) { return list_use_tc() && !e->f32 && (M > 64 || N >= 16384) && N >= 128 && K % 64 == 0; }
 int list_dense(b2_engine* e, const void* A, const void* Wt, float* C, int M, int N, int K, float alpha, cudaStream_t stream = nullptr) {
   cudaStream_t ls = stream ? stream : e->stream;
   const int f = e->f32 ? 1 : 0;
-  if (list_use_tc() && !f && alpha == 1.f && (M > 64 || N >= 16384) && N >= 128 && K % 64 == 0) {
+  if (alpha == 1.f && list_dense_tc(e, M, N, K)) {
     TcGemmArgs a;
     a.bn = tc_pick_bn(M);
     B2_TRY(b2_make_tmap_bf16(&a.tmap_w, Wt, (uint64_t)N, (uint64_t)K, (uint64_t)K, 128));
@@ -966,6 +985,31 @@ int list_gate_up(const bf16* A, const bf16* Wgu, bf16* act, int M, int F, int W,
   B2_TRY(b2_make_tmap_bf16(&tw, Wgu, (uint64_t)2 * F, (uint64_t)W, (uint64_t)W, 128));
   B2_TRY(b2_make_tmap_bf16(&tx, A, (uint64_t)M, (uint64_t)W, (uint64_t)W, 128));
   return launch_gateup_swiglu_prefill(tw, tx, act, M, F, W, 0, s);
+}
+
+// out (fp32 [T][W]) = W_down (silu(W_gate x) * (W_up x)), x operand rows [T][W], wup = gate rows, then up rows; upf fp32 [T][2F] and act [T][F] are scratch.
+int list_gated_dense(b2_engine* e, const void* x, const void* wup, const void* wdown, float* upf, void* act, float* out, int T, int F, cudaStream_t s) {
+  const int W = e->cfg.hidden, f = e->f32 ? 1 : 0;
+  AnyGemm a;
+  a.A = x; a.W = wup; a.C = act; a.M = T; a.N = 2 * F; a.K = W; a.lda = W; a.ldw = W; a.ldc = F;
+  a.epilogue = ANY_EPI_SILU_PAIR;
+  if (!f && any_gemm_silu_pair_ok(a, T, 0)) {
+    KL k(e, B2K_GEMM_GATEUP);
+    if (!k.skip()) B2_TRY(launch_gemm_any(a, 0, 0, 0, 1, 0, s));
+  } else if (!f && list_gate_up_fused(T, F, W)) {
+    KL k(e, B2K_GEMM_GATEUP);
+    if (!k.skip()) B2_TRY(list_gate_up((const bf16*)x, (const bf16*)wup, (bf16*)act, T, F, W, s));
+  } else {
+    {
+      KL k(e, B2K_GEMM_GATEUP);
+      if (!k.skip()) B2_TRY(list_dense(e, x, wup, upf, T, 2 * F, W, 1.f, s));
+    }
+    KL k(e, B2K_ACT);
+    if (!k.skip()) B2_TRY(launch_silu_gate(upf, nullptr, nullptr, act, f, T, F, s));
+  }
+  KL k(e, B2K_GEMM_DOWN);
+  if (!k.skip()) B2_TRY(list_dense(e, act, wdown, out, T, W, F, 1.f, s));
+  return 0;
 }
 
 template <typename Act>
@@ -1882,28 +1926,7 @@ int forward_outnorm_list(b2_engine* e, int T, int ntiles, int nlast) {
       cudaStream_t sS = multi && shared ? e->l_side[0] : st;
       auto shared_expert = [&]() -> int {   // (buffers of its own: in short steps it runs beside the routed experts)
         if (sS != st) b2_pdl_skip_next();   // behind a cross-stream edge: an ordinary, full dependency
-        AnyGemm a;
-        a.A = e->l_x1; a.W = L.sh_up; a.C = e->l_act2; a.M = T; a.N = 2 * sp.shared_ff; a.K = W; a.lda = W; a.ldw = W; a.ldc = sp.shared_ff;
-        a.epilogue = ANY_EPI_SILU_PAIR;
-        if (!f && any_gemm_silu_pair_ok(a, T, 0)) {
-          KL k(e, B2K_GEMM_GATEUP);
-          if (!k.skip()) B2_TRY(launch_gemm_any(a, 0, 0, 0, 1, 0, sS));
-        } else if (!f && list_gate_up_fused(T, sp.shared_ff, W)) {
-          KL k(e, B2K_GEMM_GATEUP);
-          if (!k.skip()) B2_TRY(list_gate_up((const bf16*)e->l_x1, (const bf16*)L.sh_up, (bf16*)e->l_act2, T, sp.shared_ff, W, sS));
-        } else {
-          {
-            KL k(e, B2K_GEMM_GATEUP);
-            if (!k.skip()) B2_TRY(dense(e->l_x1, L.sh_up, e->l_upf2, T, 2 * sp.shared_ff, W, sS));
-          }
-          KL k(e, B2K_ACT);
-          if (!k.skip()) B2_TRY(launch_silu_gate(e->l_upf2, nullptr, nullptr, e->l_act2, f, T, sp.shared_ff, sS));
-        }
-        {
-          KL k(e, B2K_GEMM_DOWN);
-          if (!k.skip()) B2_TRY(dense(e->l_act2, L.sh_down, e->l_ffd, T, W, sp.shared_ff, sS));
-        }
-        return 0;
+        return list_gated_dense(e, e->l_x1, L.sh_up, L.sh_down, e->l_upf2, e->l_act2, e->l_ffd, T, sp.shared_ff, sS);
       };
       if (sS != st) {
         B2_CUDA_OK(cudaEventRecord(e->l_ev[0], st));
@@ -1959,6 +1982,232 @@ int forward_outnorm_list(b2_engine* e, int T, int ntiles, int nlast) {
   return 0;
 }
 
+// Resitar: n residual streams h [T][n][W] in fp32.  A sublayer reads rms(sum_s in[s] h_s) and all streams follow from the old ones and its output in ONE
+// kernel with the next sublayer's mixed and normed input (streams_step).  The layers run in the order of e->runs: a looped layer appears once per pass with
+// cache regions and state of its own.  A mixer is two mixers on the same input: softmax attention with an output gate (attn_heads.cu, or the GQA kernels
+// when the sizes are theirs) beside a matrix-state mixer (attn_state.cu over the sequence slots); their gated read-outs, scaled, sit side by side in one
+// operand row and ONE product with both output projections gives the mixer's output.
+int forward_streams_list(b2_engine* e, int T, int ntiles, int nlast) {
+  const b2_config& c = e->cfg;
+  const int W = c.hidden, f = e->f32 ? 1 : 0, n = e->n_streams;
+  const size_t es = e->esz;
+  cudaStream_t st = e->stream;
+  auto dbg = [&](int slot) -> int {
+    if ((e->debug_flags & 1) && e->dbg_hidden_f32 != nullptr && T <= e->dbg_cap_tokens && slot < e->dbg_slots)
+      return launch_streams_sum(e->l_h, n, e->dbg_hidden_f32 + (size_t)slot * e->dbg_cap_tokens * W, T, W, st);
+    return 0;
+  };
+  // Short steps are chains of small launches: the state mixer then runs on a stream of its own beside the attention (parallel branches of a captured
+  // step), its low-rank stage on a third.  Profiled and debugged steps stay on one stream.
+  const bool multi = T <= 256 && !e->profiling && !(e->debug_flags & 1) && e->skip_mask == 0 && e->l_side[0] != nullptr;
+  cudaStream_t sB = multi ? e->l_side[0] : st, sC = multi ? e->l_side[1] : st;
+  auto edge = [&](cudaEvent_t ev, cudaStream_t from, cudaStream_t to) -> int {   // `to` continues behind what `from` has been given
+    if (from == to) return 0;
+    B2_CUDA_OK(cudaEventRecord(ev, from));
+    B2_CUDA_OK(cudaStreamWaitEvent(to, ev, 0));
+    return 0;
+  };
+  auto full_edge = [&]() { if (multi) b2_pdl_skip_next(); };   // behind a cross-stream edge: an ordinary, full dependency
+  auto dense = [&](const void* A, const void* Wt, float* C, int M, int N, int K, cudaStream_t s_) -> int { return list_dense(e, A, Wt, C, M, N, K, 1.f, s_); };
+  const PrefillTile* tiles = ntiles > 0 ? e->d_tiles : nullptr;
+  const int portions = ntiles > 0 ? e->step_portions : T;
+  const int32_t* last_rows = ntiles > 0 ? e->d_last_rows : nullptr;
+  {
+    KL k(e, B2K_EMBED);
+    if (!k.skip()) B2_TRY(launch_embed_streams(e->d_tokens, e->l_embed, f, e->l_embed_gain, e->l_h, n, T, W, c.vocab, c.rms_eps, st));
+  }
+  B2_TRY(dbg(0));
+  {
+    const ListLayer& L0 = e->ll[e->runs[0].layer];
+    KL k(e, B2K_NORM);
+    if (!k.skip()) B2_TRY(launch_streams_step(e->l_h, n, nullptr, StreamBranch(), L0.hc[0], L0.gain1, e->l_x1, f, T, W, c.rms_eps, nullptr, st));
+  }
+  for (size_t r = 0; r < e->runs.size(); ++r) {
+    const ListRun& R = e->runs[r];
+    ListLayer& L = e->ll[R.layer];
+    const b2_layer_spec& sp = L.sp;
+    const bool ssm = sp.mixer == B2_MIXER_CHUNK_AND_SSM;
+    const int HV = sp.heads * sp.vdim, HR = sp.s_heads * sp.s_vdim, OC = HV + HR;
+    const ListLayer* NL = r + 1 < e->runs.size() ? &e->ll[e->runs[r + 1].layer] : nullptr;
+    auto boundary = [&](int q, const StreamBranch& br) -> int {   // streams take up sublayer q's output; the next sublayer's input in the same pass
+      const StreamMix cur{L.hc[q], L.hc[q] + n, L.hc[q] + 2 * n};
+      const bool ff_next = q == 0 && sp.ff != B2_FF_NONE;
+      const float* in = ff_next ? L.hc[1] : NL ? NL->hc[0] : nullptr;
+      const float* gain = ff_next ? L.gain2 : NL ? NL->gain1 : nullptr;
+      KL k(e, B2K_NORM);
+      if (k.skip()) return 0;
+      return launch_streams_step(e->l_h, n, &cur, br, in, gain, gain ? e->l_x1 : nullptr, f, T, W, c.rms_eps, nullptr, st);
+    };
+    if (!ssm) {   // (the blends need the mixer's input only: the time mixing starts beside the attention's projection)
+      B2_TRY(edge(e->l_ev[0], st, sB));
+      full_edge();
+      {
+        KL k(e, B2K_ACT);
+        if (!k.skip()) B2_TRY(launch_token_shift(e->l_x1, f, L.mu, R.shift_ring, e->l_shift, T, W, e->d_row_seq, e->d_row_first, e->d_row_end, e->d_positions, e->d_slots, sB));
+      }
+    }
+    {
+      KL k(e, B2K_GEMM_QKV);   // q | k (| v) | gate, and the state-space mixer's z | x | B | C | step logits: one projection
+      if (multi && !ssm) b2_pdl_skip_next();   // (its predecessor on this stream is in front of the fork's record)
+      if (!k.skip()) B2_TRY(dense(e->l_x1, L.wqd, e->l_qd, T, L.nqd, W, st));
+    }
+    // ---- the state mixer ----
+    if (ssm) {
+      const int C = HR + 2 * sp.s_groups * sp.s_dim, gn = sp.s_groups * sp.s_dim;
+      StateGeom sg{sp.s_heads, sp.s_groups, sp.s_dim, sp.s_vdim, STATE_RULE_DECAY_HEAD};
+      sg.skip = L.skip;
+      B2_TRY(edge(e->l_ev[0], st, sB));
+      full_edge();
+      {
+        KL k(e, B2K_ROPE_KV);   // convolutions, step sizes, decays
+        if (!k.skip()) B2_TRY(launch_conv_act_finish(e->l_qd + L.off_sk, L.nqd, C, sp.s_heads, sp.conv_taps, L.conv_w, L.conv_b, L.a_log, L.a2_bias, R.ring, e->d_row_seq,
+                                                     e->d_row_first, e->d_row_end, e->d_positions, e->d_slots, e->l_cv, e->l_beta, e->l_dec, T, ntiles == 0 ? 1 : 0, sB));
+      }
+      {
+        KL k(e, B2K_CHAIN);
+        if (!k.skip()) B2_TRY(launch_state_scan(e->l_cv + HR + gn, C, e->l_cv + HR, C, e->l_cv, C, e->l_dec, e->l_beta, sg, 1.0f, R.state, portions, last_rows, e->d_row_seq,
+                                                e->d_row_first, e->d_row_end, e->d_positions, e->d_slots, e->l_so, sB));
+      }
+      {
+        KL k(e, B2K_ACT);
+        if (!k.skip()) B2_TRY(launch_gate_part_norm(e->l_so, e->l_qd + L.off_sq, L.nqd, L.head_gain, sp.s_norm_groups, sp.mix_right, (char*)e->l_av + (size_t)HV * es, f, OC, HR,
+                                                    c.rms_eps, T, sB));
+      }
+    } else {
+      StateGeom sg{sp.s_heads, sp.s_heads, sp.s_dim, sp.s_vdim, STATE_RULE_BONUS};
+      sg.bonus = L.bonus;
+      const size_t TH = (size_t)T * HR;
+      auto blend = [&](int m) { return (const char*)e->l_shift + (size_t)m * T * W * es; };   // r, k, v, g, w
+      B2_TRY(edge(e->l_ev[1], sB, sC));
+      full_edge();
+      {
+        KL k(e, B2K_GEMM_QKV);   // the low-rank stage of the decays (zero rows fill it up to the tcgen05 kernel's tile)
+        const int rn = list_dense_tc(e, T, L.rank_pad, W) ? L.rank_pad : L.rank_a;
+        if (!k.skip()) {
+          B2_TRY(dense(blend(4), L.w1, e->l_lr, T, rn, W, sC));
+          B2_TRY(launch_lowrank_act(e->l_lr, rn, 0, L.rank_a, L.a2, L.a2_bias, LOWRANK_DECAY_EXP, 0.f, nullptr, 0, e->l_dec, T, HR, sC));
+        }
+      }
+      full_edge();
+      {
+        KL k(e, B2K_GEMM_QKV);   // r, k, v and the gate, each from its own blend
+        if (!k.skip()) {
+          if (list_dense_tc(e, T, HR, W)) {
+            for (int m = 0; m < 4; ++m) B2_TRY(dense(blend(m), (const char*)L.wshift + (size_t)m * HR * W * es, e->l_rkvg + m * TH, T, HR, W, sB));
+          } else {
+            AnyGemm a;
+            a.A = e->l_shift; a.W = L.wshift; a.C = e->l_rkvg; a.M = T; a.N = HR; a.K = W; a.lda = W; a.ldw = W; a.ldc = HR;
+            a.a_bs = (long)T * W; a.w_bs = (long)HR * W; a.c_bs = (long)TH;
+            B2_TRY(launch_gemm_any(a, f, f, 1, 4, 0, sB));
+          }
+        }
+      }
+      B2_TRY(edge(e->l_ev[2], sC, sB));
+      full_edge();
+      {
+        KL k(e, B2K_CHAIN);
+        if (!k.skip()) B2_TRY(launch_state_scan(e->l_rkvg, HR, e->l_rkvg + TH, HR, e->l_rkvg + 2 * TH, HR, e->l_dec, nullptr, sg, 1.0f, R.state, portions, last_rows,
+                                                e->d_row_seq, e->d_row_first, e->d_row_end, e->d_positions, e->d_slots, e->l_so, sB));
+      }
+      {
+        KL k(e, B2K_ACT);
+        if (!k.skip()) B2_TRY(launch_state_out_gate(e->l_so, L.head_gain, e->l_rkvg + 3 * TH, HR, 1, (char*)e->l_av + (size_t)HV * es, f, sp.s_heads, sp.s_vdim, c.rms_eps, T, sB, 1,
+                                                    sp.mix_right, OC));
+      }
+    }
+    // ---- the attention ----
+    {
+      HeadsGeom g{sp.heads, sp.kv_heads, sp.dim, sp.vdim, sp.rot_dims, sp.rot_base, sp.scale, c.rms_eps, 0, 0, 0, 0.f, 0, 0, 0, L.gqa_tc ? 1 : 0};
+      g.chunk = sp.chunk;
+      char* kc = e->regions[R.k_region].base;
+      char* vc = e->regions[R.v_region].base;
+      if (multi && ssm) b2_pdl_skip_next();
+      {
+        KL k(e, B2K_ROPE_KV);
+        if (!k.skip()) B2_TRY(launch_heads_finish_table(e->l_qd, L.nqd, g, L.qkv_bias, L.rot_table, sp.rot_halves, ssm ? 1 : 0, e->d_positions, e->d_slots, e->l_q,
+                                                        L.gqa_tc ? e->l_qb : nullptr, kc, vc, f, T, st));
+      }
+      if (L.gqa_tc) {   // the framework's GQA kernels: tcgen05 for prompt portions, the page-balanced stream for decode steps
+        KL k(e, ntiles > 0 ? B2K_MISC : B2K_ATTN_DECODE);
+        if (!k.skip()) {
+          if (ntiles > 0)
+            B2_TRY(launch_attn_prefill_tc(e->l_qb, (const bf16*)kc, (const bf16*)vc, e->num_blocks, e->d_block_table, e->bt_stride, e->d_tiles, ntiles, (bf16*)e->l_ao, sp.heads,
+                                          sp.kv_heads, 128, c.block_size, st, sp.scale, 0, 0, sp.chunk));
+          else
+            B2_TRY(launch_attn_decode(e->l_qb, (const bf16*)kc, (const bf16*)vc, e->d_block_table, e->bt_stride, e->d_seq_lens, e->attn_scratch, (bf16*)e->l_ao, T, sp.heads,
+                                      sp.kv_heads, 128, c.block_size, st, sp.scale, 0, 0, sp.chunk));
+        }
+      } else {
+        KL k(e, ntiles > 0 ? B2K_MISC : B2K_ATTN_DECODE);
+        if (!k.skip()) B2_TRY(launch_heads_attention(e->l_q, kc, vc, f, g, e->d_block_table, e->bt_stride, c.block_size, tiles, ntiles, e->d_positions, e->d_seq_lens, e->l_ao, 1, T, st));
+      }
+      KL k(e, B2K_ACT);
+      if (!k.skip()) B2_TRY(launch_sigmoid_gate(e->l_ao, e->l_qd + L.off_sg, L.nqd, e->l_av, f, T, HV, st, L.gqa_tc ? 1 : 0, sp.mix_left, OC));
+    }
+    B2_TRY(edge(e->l_ev[3], sB, st));
+    full_edge();
+    {
+      KL k(e, B2K_GEMM_O);   // both output projections
+      if (!k.skip()) B2_TRY(dense(e->l_av, L.wo, e->l_mix, T, W, OC, st));
+    }
+    {
+      StreamBranch br;
+      br.a = e->l_mix;
+      br.bias = L.o_bias;
+      br.bias_scale = sp.mix_left;
+      B2_TRY(boundary(0, br));
+    }
+    if (sp.ff == B2_FF_SWIGLU) {
+      B2_TRY(list_gated_dense(e, e->l_x1, L.up, L.down, e->l_upf, e->l_act, e->l_mix, T, sp.ff_dim, st));
+      StreamBranch br;
+      br.a = e->l_mix;
+      B2_TRY(boundary(1, br));
+    } else if (sp.ff == B2_FF_TOP_SOFTMAX_EXPERTS) {
+      RouteGeom rg{sp.experts, sp.top, 1, 1, 0};
+      rg.softmax = 1;
+      rg.logit_bias = L.corr;
+      const int F = sp.ff_dim, pairs = T * sp.top;
+      {
+        KL k(e, B2K_ACT);
+        const int er = std::max(128, sp.experts);   // (zero rows fill the operand up to the tcgen05 kernel's tile)
+        if (L.router_op != nullptr && T >= 512 && !k.skip()) {
+          B2_TRY(dense(e->l_x1, L.router_op, e->l_rz, T, er, W, st));
+          B2_TRY(launch_route_select(e->l_rz, er, nullptr, rg, e->l_idx, e->l_rw, T, st));
+        } else if (!k.skip()) {
+          B2_TRY(launch_route(e->l_x1, f, L.router, nullptr, rg, e->l_idx, e->l_rw, T, W, st));
+        }
+      }
+      {
+        KL k(e, B2K_MISC);
+        if (!k.skip()) B2_TRY(launch_route_permute(e->l_idx, T, sp.top, sp.experts, e->l_offsets, e->l_offsets_stride, e->l_slot_token, e->l_pair_slot, st));
+      }
+      B2_TRY(list_gated_experts(e, L, R.layer, T, ntiles > 0 && !multi, st,
+                                [&](int act_f32) { return launch_silu_gate(e->l_upf, nullptr, nullptr, e->l_act, act_f32, pairs, F, st); }, true));
+      StreamBranch br;
+      br.y = e->l_y;
+      br.weight = e->l_rw;
+      br.pair_slot = e->l_pair_slot;
+      br.top = sp.top;
+      B2_TRY(boundary(1, br));
+    }
+    B2_TRY(dbg((int)r + 1));
+  }
+  {
+    KL k(e, B2K_NORM);
+    if (!k.skip()) B2_TRY(launch_streams_step(e->l_h, n, nullptr, StreamBranch(), nullptr, e->l_final_gain, e->l_xl, f, nlast, W, c.rms_eps, ntiles > 0 ? e->d_last_rows : nullptr, st));
+  }
+  {
+    KL k(e, B2K_LMHEAD);
+    if (!k.skip()) B2_TRY(dense(e->l_xl, e->l_head, e->l_logits, nlast, c.vocab, W, st));
+  }
+  {
+    KL k(e, B2K_MISC);
+    bf16* lb = (e->debug_flags & 2) ? e->logits : nullptr;
+    if (!k.skip()) B2_TRY(launch_logits_finish(e->l_logits, e->d_out_tokens, lb, bucket_batch(std::max(c.max_seqs, 1)), nlast, c.vocab, e->v_pad, st));
+  }
+  return 0;
+}
+
 // Two-lane decode.  At batch 64 a decode step is two things that do not overlap when they depend on each other: the
 // attention pass of a layer (HBM-bound, about half the step) and the eight small kernels between two attention
 // passes (a chain of dependent launches that moves 31 MB of weights in ~30 us: latency-bound, HBM nearly idle).
@@ -1982,6 +2231,7 @@ int forward(b2_engine* e, int T, int ntiles, int nlast, int attn_split) {
   if (c.arch == B2_ARCH_BUMALIX) return forward_state_list(e, T, ntiles, nlast);
   if (c.arch == B2_ARCH_TINEVIK) return forward_mixed_list(e, T, ntiles, nlast);
   if (c.arch == B2_ARCH_TOLANEX) return forward_outnorm_list(e, T, ntiles, nlast);
+  if (c.arch == B2_ARCH_RESITAR) return forward_streams_list(e, T, ntiles, nlast);
   if (c.arch == B2_ARCH_OPT) return forward_opt(e, T, ntiles, nlast);
   if (ntiles == 0 && e->use_chain == 2 && e->fused_ok && c.arch == B2_ARCH_QWEN3 && !(e->debug_flags & 1) &&
       e->force_gemm_impl != 0 && T > e->simt_max_tokens && T <= 64 && e->skip_mask == 0)
@@ -2357,6 +2607,19 @@ int put_key_up(b2_engine* e, void* dst, const uint16_t* src, size_t heads, size_
   return put_operand(e, dst, 0, tr.data(), tr.size());
 }
 
+// src [rows][cols] into columns [col0, col0 + cols) of an operand matrix with ld columns
+int put_operand_cols(b2_engine* e, void* dst, size_t ld, size_t col0, const uint16_t* src, size_t rows, size_t cols) {
+  char* d = reinterpret_cast<char*>(dst) + col0 * e->esz;
+  if (!e->f32) {
+    B2_CUDA_OK(cudaMemcpy2D(d, ld * 2, src, cols * 2, cols * 2, rows, cudaMemcpyHostToDevice));
+    return 0;
+  }
+  std::vector<uint32_t> wide(rows * cols);
+  for (size_t i = 0; i < wide.size(); ++i) wide[i] = (uint32_t)src[i] << 16;
+  B2_CUDA_OK(cudaMemcpy2D(d, ld * 4, wide.data(), cols * 4, cols * 4, rows, cudaMemcpyHostToDevice));
+  return 0;
+}
+
 int list_tensor(b2_engine* e, const std::string& name, const void* host, size_t nbytes) {
   const b2_config& c = e->cfg;
   const size_t W = c.hidden;
@@ -2374,7 +2637,7 @@ int list_tensor(b2_engine* e, const std::string& name, const void* host, size_t 
   };
   if (name == "embed") { B2_TRY(want((size_t)c.vocab * W)); return done(put_operand(e, e->l_embed, 0, src, (size_t)c.vocab * W)); }
   if (name == "head" && e->l_head != e->l_embed) { B2_TRY(want((size_t)c.vocab * W)); return done(put_operand(e, e->l_head, 0, src, (size_t)c.vocab * W)); }
-  if (name == "embed.norm") { B2_TRY(want(W)); return done(put_f32(e->l_embed_gain, src, W, 1.0f)); }
+  if (name == "embed.norm" && e->l_embed_gain) { B2_TRY(want(W)); return done(put_f32(e->l_embed_gain, src, W, c.arch == B2_ARCH_LERASUN ? 1.0f : 0.0f)); }
   if (name == "final.norm") { B2_TRY(want(W)); return done(put_f32(e->l_final_gain, src, W, c.arch == B2_ARCH_LERASUN ? 1.0f : 0.0f)); }
   if (name == "final.norm.b" && e->l_final_bias) { B2_TRY(want(W)); return done(put_f32(e->l_final_bias, src, W, 0.0f)); }
   if (name == "bigram" && e->l_bigram) {
@@ -2614,6 +2877,95 @@ int list_tensor(b2_engine* e, const std::string& name, const void* host, size_t 
       if (sf > 0 && rest == "mlp.shared.gate") { B2_TRY(want(sf * W)); return done(put_operand(e, L.sh_up, 0, src, sf * W)); }
       if (sf > 0 && rest == "mlp.shared.up") { B2_TRY(want(sf * W)); return done(put_operand(e, L.sh_up, sf * W, src, sf * W)); }
       if (sf > 0 && rest == "mlp.shared.down") { B2_TRY(want(W * sf)); return done(put_operand(e, L.sh_down, 0, src, W * sf)); }
+      if (rest.compare(0, 5, "mlp.e") == 0) {
+        size_t d2 = rest.find('.', 5);
+        if (d2 != std::string::npos) {
+          const int ex = atoi(rest.substr(5, d2 - 5).c_str());
+          const std::string which = rest.substr(d2 + 1);
+          if (ex >= 0 && ex < sp.experts) {   // gate rows, then up rows, expert by expert: one product gives both
+            if (which == "gate") { B2_TRY(want(ff * W)); return done(put_operand(e, L.up, (size_t)ex * 2 * ff * W, src, ff * W)); }
+            if (which == "up") { B2_TRY(want(ff * W)); return done(put_operand(e, L.up, ((size_t)ex * 2 + 1) * ff * W, src, ff * W)); }
+            if (which == "down") { B2_TRY(want(W * ff)); return done(put_operand(e, L.down, (size_t)ex * W * ff, src, W * ff)); }
+          }
+        }
+      }
+    }
+    b2_set_error("unknown tensor name %s", name.c_str());
+    return -22;
+  }
+  if (c.arch == B2_ARCH_RESITAR) {
+    const size_t n = e->n_streams, nq = L.nq, nk = L.nk, nv = L.nv, HV = H * dv, sh = sp.s_heads, HR = sh * sp.s_vdim, OC = HV + HR;
+    const bool ssm = sp.mixer == B2_MIXER_CHUNK_AND_SSM;
+    if (rest == "norm1") { B2_TRY(want(W)); return done(put_f32(L.gain1, src, W, 0.0f)); }
+    if (rest == "norm2" && L.gain2) { B2_TRY(want(W)); return done(put_f32(L.gain2, src, W, 0.0f)); }
+    for (int q = 0; q < 2; ++q) {
+      const std::string hp = q == 0 ? "hc1." : "hc2.";
+      if (rest == hp + "in") { B2_TRY(want(n)); return done(put_f32(L.hc[q], src, n, 0.0f)); }
+      if (rest == hp + "out") { B2_TRY(want(n)); return done(put_f32(L.hc[q] + n, src, n, 0.0f)); }
+      if (rest == hp + "mix") { B2_TRY(want(n * n)); return done(put_f32(L.hc[q] + 2 * n, src, n * n, 0.0f)); }
+    }
+    if (rest == "mix.left.q") { B2_TRY(want(nq * W)); return done(put_operand(e, L.wqd, 0, src, nq * W)); }
+    if (rest == "mix.left.k") { B2_TRY(want(nk * W)); return done(put_operand(e, L.wqd, nq * W, src, nk * W)); }
+    if (rest == "mix.left.v" && !ssm) { B2_TRY(want(nv * W)); return done(put_operand(e, L.wqd, (nq + nk) * W, src, nv * W)); }
+    if (rest == "mix.left.g") { B2_TRY(want(HV * W)); return done(put_operand(e, L.wqd, (size_t)L.off_sg * W, src, HV * W)); }
+    if (rest == "mix.left.q.b") { B2_TRY(want(nq)); return done(put_f32(L.qkv_bias, src, nq, 0.0f)); }
+    if (rest == "mix.left.k.b") { B2_TRY(want(nk)); return done(put_f32(L.qkv_bias + nq, src, nk, 0.0f)); }
+    if (rest == "mix.left.v.b" && !ssm) { B2_TRY(want(nv)); return done(put_f32(L.qkv_bias + nq + nk, src, nv, 0.0f)); }
+    if (rest == "mix.left.o.b" && ssm) { B2_TRY(want(W)); return done(put_f32(L.o_bias, src, W, 0.0f)); }
+    if (rest == "mix.left.o") { B2_TRY(want(W * HV)); return done(put_operand_cols(e, L.wo, OC, 0, src, W, HV)); }
+    if (rest == "mix.right.o") { B2_TRY(want(W * HR)); return done(put_operand_cols(e, L.wo, OC, HV, src, W, HR)); }
+    if (rest == "mix.right.norm") { B2_TRY(want(HR)); return done(put_f32(L.head_gain, src, HR, 0.0f)); }
+    if (ssm) {
+      const size_t C = HR + 2 * (size_t)sp.s_groups * sp.s_dim, taps = sp.conv_taps;
+      if (rest == "mix.right.in") { B2_TRY(want((HR + C + sh) * W)); return done(put_operand(e, L.wqd, (size_t)L.off_sq * W, src, (HR + C + sh) * W)); }
+      if (rest == "mix.right.conv") { B2_TRY(want(C * taps)); return done(put_f32(L.conv_w, src, C * taps, 0.0f)); }
+      if (rest == "mix.right.conv.b") { B2_TRY(want(C)); return done(put_f32(L.conv_b, src, C, 0.0f)); }
+      if (rest == "mix.right.dt_bias") { B2_TRY(want(sh)); return done(put_f32(L.a2_bias, src, sh, 0.0f)); }
+      if (rest == "mix.right.A_log") { B2_TRY(want(sh)); return done(put_f32(L.a_log, src, sh, 0.0f)); }
+      if (rest == "mix.right.D") { B2_TRY(want(sh)); return done(put_f32(L.skip, src, sh, 0.0f)); }
+    } else {
+      static const char* const blends[5] = {"r", "k", "v", "g", "w"};
+      for (size_t m = 0; m < 5; ++m) {
+        if (rest == std::string("mix.right.mu.") + blends[m]) { B2_TRY(want(W)); return done(put_f32(L.mu + m * W, src, W, 0.0f)); }
+        if (m < 4 && rest == std::string("mix.right.") + blends[m]) { B2_TRY(want(HR * W)); return done(put_operand(e, L.wshift, m * HR * W, src, HR * W)); }
+      }
+      if (rest == "mix.right.w0") { B2_TRY(want(HR)); return done(put_f32(L.a2_bias, src, HR, 0.0f)); }
+      if (rest == "mix.right.u") { B2_TRY(want(HR)); return done(put_f32(L.bonus, src, HR, 0.0f)); }
+      if (rest == "mix.right.w1") {   // [rank][W], the rank from the size; zero rows up to the tcgen05 projection's tile
+        B2_REQUIRE(nbytes >= 2 * W && nbytes % (2 * W) == 0, "tensor %s: %zu bytes are not rows of %zu values", name.c_str(), nbytes, W);
+        if (L.w1) cudaFree(L.w1);
+        L.w1 = nullptr;
+        L.rank_a = (int)(nbytes / (2 * W));
+        L.rank_pad = std::max(128, L.rank_a);
+        char* q = nullptr;
+        B2_TRY(dalloc(&q, (size_t)L.rank_pad * W * e->esz));
+        L.w1 = q;
+        B2_CUDA_OK(cudaMemset(q, 0, (size_t)L.rank_pad * W * e->esz));
+        e->weight_bytes += (int64_t)((size_t)L.rank_a * W * e->esz);
+        return done(put_operand(e, L.w1, 0, src, (size_t)L.rank_a * W));
+      }
+      if (rest == "mix.right.w2") {
+        B2_REQUIRE(nbytes >= 2 && nbytes % 2 == 0, "tensor %s: %zu bytes", name.c_str(), nbytes);
+        if (L.a2) cudaFree(L.a2);
+        L.a2 = nullptr;
+        B2_TRY(dalloc(&L.a2, nbytes / 2));
+        L.a2_floats = nbytes / 2;
+        e->weight_bytes += (int64_t)(nbytes * 2);
+        return done(put_f32(L.a2, src, nbytes / 2, 0.0f));
+      }
+    }
+    if (sp.ff == B2_FF_SWIGLU) {
+      if (rest == "mlp.gate") { B2_TRY(want(ff * W)); return done(put_operand(e, L.up, 0, src, ff * W)); }
+      if (rest == "mlp.up") { B2_TRY(want(ff * W)); return done(put_operand(e, L.up, ff * W, src, ff * W)); }
+      if (rest == "mlp.down") { B2_TRY(want(W * ff)); return done(put_operand(e, L.down, 0, src, W * ff)); }
+    } else if (sp.ff == B2_FF_TOP_SOFTMAX_EXPERTS) {
+      const size_t ne = sp.experts;
+      if (rest == "mlp.router") {
+        B2_TRY(want(ne * W));
+        if (L.router_op) B2_TRY(put_operand(e, L.router_op, 0, src, ne * W));
+        return done(put_f32(L.router, src, ne * W, 0.0f));
+      }
+      if (rest == "mlp.router.b") { B2_TRY(want(ne)); return done(put_f32(L.corr, src, ne, 0.0f)); }
       if (rest.compare(0, 5, "mlp.e") == 0) {
         size_t d2 = rest.find('.', 5);
         if (d2 != std::string::npos) {
@@ -3645,8 +3997,335 @@ int outnorm_finalize(b2_engine* e) {
   return 0;
 }
 
+// The rotary table of a layer's settings (layers with equal settings share one).  Pairs whose frequency turns more than rot_fast times over rot_orig positions
+// keep it, pairs that turn less than rot_slow times are divided by rot_factor, the ones between are blended along a ramp over the pair index.
+int rot_table_for(b2_engine* e, const b2_layer_spec& sp, const float** out) {
+  *out = nullptr;
+  if (sp.rot_dims <= 0) return 0;
+  for (const auto& t : e->rot_tables)
+    if (t.key.rot_dims == sp.rot_dims && t.key.rot_base == sp.rot_base && t.key.rot_factor == sp.rot_factor && t.key.rot_orig == sp.rot_orig &&
+        t.key.rot_fast == sp.rot_fast && t.key.rot_slow == sp.rot_slow) {
+      *out = t.table;
+      return 0;
+    }
+  const int half = sp.rot_dims / 2;
+  const double dims = sp.rot_dims, base = sp.rot_base, factor = sp.rot_factor > 0.f ? sp.rot_factor : 1.0;
+  std::vector<double> freq(half);
+  double mul = 1.0, lo = 0.0, hi = 0.0;
+  if (sp.rot_orig > 0) {
+    const double pi = 3.14159265358979323846;
+    auto index_of = [&](double turns) { return dims * log((double)sp.rot_orig / (2.0 * pi * turns)) / (2.0 * log(base)); };
+    lo = std::max(floor(index_of(sp.rot_fast)), 0.0);
+    hi = std::min(ceil(index_of(sp.rot_slow)), dims - 1.0);
+    mul = 0.1 * log(factor) + 1.0;
+  }
+  for (int i = 0; i < half; ++i) {
+    const double fi = pow(base, -2.0 * i / dims);
+    const double ramp = sp.rot_orig > 0 ? std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0) : 0.0;
+    freq[i] = fi / factor * ramp + fi * (1.0 - ramp);
+  }
+  double* d = nullptr;
+  float* table = nullptr;
+  B2_TRY(dalloc(&d, (size_t)half));
+  B2_TRY(dalloc(&table, (size_t)e->cfg.max_model_len * sp.rot_dims));
+  e->rot_tables.push_back({sp, table});
+  B2_CUDA_OK(cudaMemcpy(d, freq.data(), (size_t)half * sizeof(double), cudaMemcpyHostToDevice));
+  B2_TRY(launch_rot_table(d, half, mul, table, e->cfg.max_model_len, e->stream));
+  B2_CUDA_OK(cudaStreamSynchronize(e->stream));
+  cudaFree(d);
+  *out = table;
+  return 0;
+}
+
+// The same for the family with several residual streams and two mixers side by side in every layer (Resitar).
+int streams_engine_alloc(b2_engine* e) {
+  const b2_config& c = e->cfg;
+  const size_t W = c.hidden, es = e->esz;
+  B2_REQUIRE(!e->specs.empty() && (int)e->specs.size() == c.num_layers, "Resitar: layer_specs missing");
+  B2_REQUIRE(c.hidden >= 1 && c.vocab >= 1 && c.num_layers >= 1, "Resitar: bad sizes");
+  B2_REQUIRE(c.loop_times >= 0 && (c.loop_times == 0 || (c.loop_start >= 0 && c.loop_start <= c.loop_stop && c.loop_stop <= c.num_layers)),
+             "Resitar: loop [%d, %d) x %d outside the %d layers", c.loop_start, c.loop_stop, c.loop_times, c.num_layers);
+  e->n_streams = c.streams > 0 ? c.streams : 1;
+  B2_REQUIRE(e->n_streams <= STREAMS_MAX, "Resitar: %d residual streams (at most %d)", e->n_streams, STREAMS_MAX);
+  const size_t n = e->n_streams;
+  auto xalloc = [&](void** p, size_t elems) -> int {
+    char* q = nullptr;
+    B2_TRY(dalloc(&q, std::max<size_t>(elems, 1) * es));
+    *p = q;
+    e->weight_bytes += (int64_t)(elems * es);
+    return 0;
+  };
+  auto falloc = [&](float** p, size_t m) -> int {
+    B2_TRY(dalloc(p, std::max<size_t>(m, 1)));
+    B2_CUDA_OK(cudaMemset(*p, 0, std::max<size_t>(m, 1) * 4));
+    e->weight_bytes += (int64_t)(m * 4);
+    return 0;
+  };
+  e->weight_bytes = 0;
+  B2_TRY(xalloc(&e->l_embed, (size_t)c.vocab * W));
+  if (c.tie_embeddings) e->l_head = e->l_embed;   // the embedding table itself is the head
+  else B2_TRY(xalloc(&e->l_head, (size_t)c.vocab * W));
+  B2_TRY(falloc(&e->l_embed_gain, W));
+  B2_TRY(falloc(&e->l_final_gain, W));
+  e->ll.resize(c.num_layers);
+  size_t max_q = 1, max_hv = 1, max_oc = 1, max_so = 1, max_hr = 0, max_cv = 0, max_dec = 1, max_heads = 1, max_nqd = 1, max_up = 0, max_act = 0, gqa_scratch = 0;
+  int max_top = 1, max_exp = 1;
+  bool any_experts = false;
+  for (int l = 0; l < c.num_layers; ++l) {
+    ListLayer& L = e->ll[l];
+    L.sp = e->specs[l];
+    const b2_layer_spec& sp = L.sp;
+    const bool ssm = sp.mixer == B2_MIXER_CHUNK_AND_SSM;
+    B2_REQUIRE(ssm || sp.mixer == B2_MIXER_FULL_AND_TIMEMIX, "layer %d: mixer kind %d not built for this family", l, sp.mixer);
+    B2_REQUIRE(sp.heads >= 1 && sp.kv_heads >= 1 && sp.heads % sp.kv_heads == 0 && sp.dim >= 1 && sp.vdim >= 1 && sp.chunk >= 0,
+               "layer %d: bad attention sizes (heads %d, kv_heads %d, dim %d, vdim %d, chunk %d)", l, sp.heads, sp.kv_heads, sp.dim, sp.vdim, sp.chunk);
+    B2_REQUIRE(!ssm || sp.vdim == sp.dim, "layer %d: keys that serve as values need vdim %d == dim %d", l, sp.vdim, sp.dim);
+    B2_REQUIRE(sp.rot_dims >= 0 && sp.rot_dims <= sp.dim && sp.rot_dims % 2 == 0, "layer %d: rot dims %d must be even and <= dim %d", l, sp.rot_dims, sp.dim);
+    B2_REQUIRE(sp.rot_orig <= 0 || (sp.rot_factor > 0.f && sp.rot_fast > 0.f && sp.rot_slow > 0.f && sp.rot_base > 1.f), "layer %d: bad rotary scaling", l);
+    B2_REQUIRE(sp.s_heads >= 1 && sp.s_dim >= 1 && sp.s_dim <= 256 && sp.s_vdim >= 1, "layer %d: bad state-mixer sizes (heads %d, state width %d (at most 256), vdim %d)", l,
+               sp.s_heads, sp.s_dim, sp.s_vdim);
+    const size_t HV = (size_t)sp.heads * sp.vdim, HR = (size_t)sp.s_heads * sp.s_vdim;
+    L.nq = sp.heads * sp.dim;
+    L.nk = sp.kv_heads * sp.dim;
+    L.nv = sp.kv_heads * sp.vdim;
+    L.off_sg = L.nq + L.nk + (ssm ? 0 : L.nv);
+    L.off_sq = L.off_sg + (int)HV;
+    L.n_fixed = L.off_sq;
+    B2_TRY(falloc(&L.gain1, W));
+    B2_TRY(falloc(&L.qkv_bias, (size_t)L.off_sg));
+    B2_TRY(falloc(&L.head_gain, HR));
+    if (ssm) {
+      B2_REQUIRE(sp.s_groups >= 1 && sp.s_heads % sp.s_groups == 0 && sp.conv_taps >= 1 && sp.s_norm_groups >= 1 && HR % sp.s_norm_groups == 0,
+                 "layer %d: bad state-space sizes (heads %d, groups %d, taps %d, norm groups %d)", l, sp.s_heads, sp.s_groups, sp.conv_taps, sp.s_norm_groups);
+      const size_t C = HR + 2 * (size_t)sp.s_groups * sp.s_dim;
+      L.off_sk = L.off_sq + (int)HR;
+      L.n_fixed = L.off_sk + (int)C + sp.s_heads;
+      B2_TRY(falloc(&L.o_bias, W));
+      B2_TRY(falloc(&L.conv_w, C * sp.conv_taps));
+      B2_TRY(falloc(&L.conv_b, C));
+      B2_TRY(falloc(&L.a_log, sp.s_heads));
+      B2_TRY(falloc(&L.a2_bias, sp.s_heads));
+      B2_TRY(falloc(&L.skip, sp.s_heads));
+      max_cv = std::max(max_cv, C);
+      max_dec = std::max(max_dec, (size_t)sp.s_heads);
+      max_heads = std::max(max_heads, (size_t)sp.s_heads);
+    } else {
+      B2_TRY(falloc(&L.mu, 5 * W));
+      B2_TRY(falloc(&L.bonus, HR));
+      B2_TRY(falloc(&L.a2_bias, HR));
+      B2_TRY(xalloc(&L.wshift, 4 * HR * W));
+      max_hr = std::max(max_hr, HR);
+      max_dec = std::max(max_dec, HR);
+    }
+    L.nqd = L.n_fixed;
+    B2_TRY(xalloc(&L.wqd, (size_t)L.nqd * W));
+    B2_TRY(xalloc(&L.wo, W * (HV + HR)));
+    B2_TRY(rot_table_for(e, sp, &L.rot_table));
+    for (int q = 0; q < 2; ++q) {   // a checkpoint's numbers replace these (one plain stream)
+      B2_TRY(falloc(&L.hc[q], 2 * n + n * n));
+      std::vector<float> plain(2 * n + n * n, 0.f);
+      for (size_t i = 0; i < 2 * n; ++i) plain[i] = 1.f;
+      for (size_t i = 0; i < n; ++i) plain[2 * n + i * n + i] = 1.f;
+      B2_CUDA_OK(cudaMemcpy(L.hc[q], plain.data(), plain.size() * 4, cudaMemcpyHostToDevice));
+    }
+    static const bool use_gqa_tc = [] { const char* v = getenv("B2_HEADS_GQA_TC"); return !(v && *v == '0'); }();
+    L.gqa_tc = use_gqa_tc && !e->f32 && sp.dim == 128 && sp.vdim == 128 && sp.heads == 2 * sp.kv_heads && c.block_size == 16 && (c.max_model_len + 15) / 16 <= 1024 &&
+               (long)bucket_batch(c.max_seqs) * sp.kv_heads <= 4096;
+    if (L.gqa_tc) gqa_scratch = std::max(gqa_scratch, attn_decode_scratch_floats(bucket_batch(c.max_seqs), sp.heads, sp.kv_heads, 128));
+    max_q = std::max(max_q, (size_t)L.nq);
+    max_hv = std::max(max_hv, HV);
+    max_so = std::max(max_so, HR);
+    max_oc = std::max(max_oc, HV + HR);
+    max_nqd = std::max(max_nqd, (size_t)L.nqd);
+    if (sp.ff == B2_FF_SWIGLU) {
+      B2_REQUIRE(sp.ff_dim >= 1, "layer %d: bad feed-forward width", l);
+      B2_TRY(falloc(&L.gain2, W));
+      B2_TRY(xalloc(&L.up, (size_t)2 * sp.ff_dim * W));
+      B2_TRY(xalloc(&L.down, W * sp.ff_dim));
+      max_up = std::max(max_up, (size_t)2 * sp.ff_dim);
+      max_act = std::max(max_act, (size_t)sp.ff_dim);
+    } else if (sp.ff == B2_FF_TOP_SOFTMAX_EXPERTS) {
+      B2_REQUIRE(sp.experts >= 1 && sp.top >= 1 && sp.top <= sp.experts && sp.ff_dim >= 1, "layer %d: bad router sizes (experts %d, top %d, ff %d)", l, sp.experts, sp.top, sp.ff_dim);
+      B2_TRY(falloc(&L.gain2, W));
+      B2_TRY(falloc(&L.router, (size_t)sp.experts * W));
+      B2_TRY(falloc(&L.corr, sp.experts));
+      if (!e->f32 && W % 64 == 0) {
+        char* q = nullptr;
+        const size_t rn = (size_t)std::max(128, sp.experts) * W * es;
+        B2_TRY(dalloc(&q, rn));
+        B2_CUDA_OK(cudaMemset(q, 0, rn));
+        L.router_op = reinterpret_cast<bf16*>(q);
+      }
+      B2_TRY(xalloc(&L.up, (size_t)sp.experts * 2 * sp.ff_dim * W));
+      B2_TRY(xalloc(&L.down, (size_t)sp.experts * W * sp.ff_dim));
+      any_experts = true;
+      max_top = std::max(max_top, sp.top);
+      max_exp = std::max(max_exp, sp.experts);
+      max_up = std::max(max_up, (size_t)sp.top * 2 * sp.ff_dim);
+      max_act = std::max(max_act, (size_t)sp.top * sp.ff_dim);
+    } else {
+      B2_REQUIRE(sp.ff == B2_FF_NONE, "layer %d: feed-forward kind %d not built for this family", l, sp.ff);
+    }
+  }
+  // ---- the order the layers run in, and the state of every run ----
+  auto add_run = [&](int layer) -> int {
+    ListRun R;
+    R.layer = layer;
+    const b2_layer_spec& sp = e->ll[layer].sp;
+    const bool ssm = sp.mixer == B2_MIXER_CHUNK_AND_SSM;
+    const size_t sf = (size_t)c.max_seqs * state_floats_per_slot(StateGeom{sp.s_heads, ssm ? sp.s_groups : sp.s_heads, sp.s_dim, sp.s_vdim, 0});
+    B2_TRY(dalloc(&R.state, sf));
+    B2_CUDA_OK(cudaMemset(R.state, 0, sf * 4));
+    if (ssm && sp.conv_taps > 1) {
+      const size_t rf = (size_t)c.max_seqs * sp.conv_taps * ((size_t)sp.s_heads * sp.s_vdim + 2 * (size_t)sp.s_groups * sp.s_dim);
+      B2_TRY(dalloc(&R.ring, rf));
+      B2_CUDA_OK(cudaMemset(R.ring, 0, rf * 4));
+    }
+    if (!ssm) {
+      char* q = nullptr;
+      B2_TRY(dalloc(&q, (size_t)c.max_seqs * 2 * W * es));
+      B2_CUDA_OK(cudaMemset(q, 0, (size_t)c.max_seqs * 2 * W * es));
+      R.shift_ring = q;
+    }
+    e->runs.push_back(R);
+    return 0;
+  };
+  const bool looped = c.loop_times > 0 && c.loop_stop > c.loop_start;
+  for (int l = 0; l < (looped ? c.loop_start : c.num_layers); ++l) B2_TRY(add_run(l));
+  if (looped) {
+    for (int t = 0; t < c.loop_times; ++t)
+      for (int l = c.loop_start; l < c.loop_stop; ++l) B2_TRY(add_run(l));
+    for (int l = c.loop_stop; l < c.num_layers; ++l) B2_TRY(add_run(l));
+  }
+  e->l_has_state = true;
+  e->dbg_slots = (int)e->runs.size() + 1;
+  for (int i = 0; i < 2; ++i) B2_CUDA_OK(cudaStreamCreateWithFlags(&e->l_side[i], cudaStreamNonBlocking));
+  for (int i = 0; i < 4; ++i) B2_CUDA_OK(cudaEventCreateWithFlags(&e->l_ev[i], cudaEventDisableTiming));
+  // ---- activations ----
+  e->cap_tokens = ((std::max(c.max_batch_tokens, c.max_seqs) + 255) / 256) * 256;
+  const size_t Tc = e->cap_tokens;
+  e->l_rows_cap = (int)(Tc + bucket_batch(c.max_seqs));
+  e->l_max_top = max_top;
+  e->v_pad = (c.vocab + 7) / 8 * 8;
+  auto aalloc = [&](void** p, size_t elems) -> int {
+    char* q = nullptr;
+    B2_TRY(dalloc(&q, elems * es));
+    *p = q;
+    return 0;
+  };
+  B2_TRY(dalloc(&e->l_h, Tc * n * W));
+  B2_TRY(dalloc(&e->l_qd, Tc * max_nqd));
+  e->l_qd_cols = max_nqd;
+  B2_TRY(dalloc(&e->l_q, Tc * max_q));
+  if (gqa_scratch > 0) {
+    B2_TRY(dalloc(&e->l_qb, Tc * max_q));
+    e->attn_scratch_floats = gqa_scratch;
+    B2_TRY(dalloc(&e->attn_scratch, gqa_scratch));
+    B2_CUDA_OK(cudaMemset(e->attn_scratch, 0, gqa_scratch * sizeof(float)));   // arrival counters start at zero
+  }
+  {
+    float* q = nullptr;   // (fp32 rows, or bf16 rows of the GQA kernels)
+    B2_TRY(dalloc(&q, Tc * max_hv));
+    e->l_ao = q;
+  }
+  B2_TRY(dalloc(&e->l_dec, Tc * max_dec));
+  B2_TRY(dalloc(&e->l_beta, Tc * max_heads));
+  B2_TRY(dalloc(&e->l_so, Tc * max_so));
+  if (max_cv > 0) B2_TRY(dalloc(&e->l_cv, Tc * max_cv));
+  if (max_hr > 0) {
+    B2_TRY(dalloc(&e->l_rkvg, 4 * Tc * max_hr));
+    B2_TRY(aalloc(&e->l_shift, 5 * Tc * W));
+  }
+  B2_TRY(dalloc(&e->l_mix, Tc * W));
+  B2_TRY(dalloc(&e->l_logits, (size_t)e->l_rows_cap * c.vocab));
+  B2_TRY(aalloc(&e->l_x1, Tc * W));
+  B2_TRY(aalloc(&e->l_av, Tc * max_oc));
+  B2_TRY(aalloc(&e->l_xl, (size_t)e->l_rows_cap * W));
+  if (max_up > 0) {
+    B2_TRY(dalloc(&e->l_upf, Tc * max_up));
+    B2_TRY(aalloc(&e->l_act, Tc * max_act));
+  }
+  if (any_experts) {
+    B2_TRY(dalloc(&e->l_y, Tc * max_top * W));
+    B2_TRY(dalloc(&e->l_rw, Tc * max_top));
+    if (!e->f32) B2_TRY(dalloc(&e->l_rz, Tc * (size_t)std::max(128, max_exp)));
+    B2_TRY(dalloc(&e->l_idx, Tc * max_top));
+    e->l_offsets_stride = max_exp + 1;
+    B2_TRY(dalloc(&e->l_offsets, (size_t)3 * (max_exp + 1)));
+    B2_CUDA_OK(cudaMemset(e->l_offsets, 0, (size_t)3 * (max_exp + 1) * 4));
+    B2_TRY(dalloc(&e->l_slot_token, Tc * max_top));
+    B2_TRY(dalloc(&e->l_pair_slot, Tc * max_top));
+    B2_CUDA_OK(cudaMemset(e->l_pair_slot, 0, Tc * max_top * 4));
+    e->l_tiles_cap = (int)(Tc * max_top / any_gemm_tile_rows() + max_exp + 1);
+    B2_TRY(dalloc(&e->l_tile_group, (size_t)e->l_tiles_cap));
+    B2_TRY(dalloc(&e->l_tile_row0, (size_t)e->l_tiles_cap));
+    B2_TRY(dalloc(&e->l_ntiles, (size_t)1));
+    B2_CUDA_OK(cudaMemset(e->l_ntiles, 0, 4));
+    if (!e->f32 && Tc * max_top >= (size_t)LIST_TC_EXPERT_ROWS && max_exp > 1) {   // prompt-sized expert products on the tcgen05 projection kernel
+      B2_TRY(dalloc(&e->l_xperm, Tc * max_top * W));
+      B2_CUDA_OK(cudaMallocHost(&e->h_offsets, (size_t)(max_exp + 1) * sizeof(int32_t)));
+    }
+  }
+  for (int32_t** p : {&e->d_row_seq, &e->d_row_first, &e->d_row_end}) {
+    B2_TRY(dalloc(p, Tc));
+    B2_CUDA_OK(cudaMemset(*p, 0, Tc * 4));
+  }
+  return 0;
+}
+
+// Names of the tensors a Resitar checkpoint must hold.
+std::vector<std::string> streams_tensor_names(const b2_engine* e) {
+  std::vector<std::string> n = {"embed", "embed.norm", "final.norm"};
+  if (e->l_head != e->l_embed) n.push_back("head");
+  for (size_t l = 0; l < e->ll.size(); ++l) {
+    const b2_layer_spec& sp = e->ll[l].sp;
+    const std::string p = "l" + std::to_string(l) + ".";
+    const bool ssm = sp.mixer == B2_MIXER_CHUNK_AND_SSM, has_ff = sp.ff != B2_FF_NONE;
+    n.push_back(p + "norm1");
+    if (has_ff) n.push_back(p + "norm2");
+    for (int q = 1; q <= (has_ff ? 2 : 1); ++q)
+      for (const char* t : {"in", "out", "mix"}) n.push_back(p + "hc" + std::to_string(q) + "." + t);
+    for (const char* t : {"q", "q.b", "k", "k.b", "g", "o"}) n.push_back(p + "mix.left." + t);
+    if (ssm) {
+      n.push_back(p + "mix.left.o.b");
+      for (const char* t : {"in", "conv", "conv.b", "dt_bias", "A_log", "D", "norm", "o"}) n.push_back(p + "mix.right." + t);
+    } else {
+      for (const char* t : {"v", "v.b"}) n.push_back(p + "mix.left." + t);
+      for (const char* t : {"mu.r", "mu.k", "mu.v", "mu.g", "mu.w", "r", "k", "v", "g", "w1", "w2", "w0", "u", "norm", "o"}) n.push_back(p + "mix.right." + t);
+    }
+    if (sp.ff == B2_FF_SWIGLU) {
+      for (const char* t : {"gate", "up", "down"}) n.push_back(p + "mlp." + t);
+    } else if (sp.ff == B2_FF_TOP_SOFTMAX_EXPERTS) {
+      for (const char* t : {"router", "router.b"}) n.push_back(p + "mlp." + t);
+      for (int x = 0; x < sp.experts; ++x)
+        for (const char* t : {"gate", "up", "down"}) n.push_back(p + "mlp.e" + std::to_string(x) + "." + t);
+    }
+  }
+  return n;
+}
+// Every tensor is in: the low-rank stages' widths are known, and their buffer is sized.
+int streams_finalize(b2_engine* e) {
+  for (const std::string& name : streams_tensor_names(e)) B2_REQUIRE(e->loaded.count(name), "weights incomplete: %s missing", name.c_str());
+  size_t cols = 0;
+  for (size_t l = 0; l < e->ll.size(); ++l) {
+    const ListLayer& L = e->ll[l];
+    if (L.sp.mixer != B2_MIXER_FULL_AND_TIMEMIX) continue;
+    B2_REQUIRE(L.rank_a >= 1 && L.rank_a <= 1024 && L.a2_floats == (size_t)L.sp.s_heads * L.sp.s_dim * L.rank_a, "layer %zu: w1 has %d rows (at most 1024), w2 %zu numbers", l, L.rank_a,
+               L.a2_floats);
+    cols = std::max(cols, (size_t)L.rank_pad);
+  }
+  if (cols > e->l_lr_cols) {
+    if (e->l_lr) cudaFree(e->l_lr);
+    e->l_lr = nullptr;
+    B2_TRY(dalloc(&e->l_lr, (size_t)e->cap_tokens * cols));
+    e->l_lr_cols = cols;
+  }
+  return 0;
+}
+
 // Validates the layer list and allocates weights, activations and scratch of a layer-list engine.
 int list_engine_alloc(b2_engine* e) {
+  if (e->cfg.arch == B2_ARCH_RESITAR) return streams_engine_alloc(e);
   if (e->cfg.arch == B2_ARCH_TOLANEX) return outnorm_engine_alloc(e);
   if (e->cfg.arch == B2_ARCH_TINEVIK) return mixed_engine_alloc(e);
   if (e->cfg.arch == B2_ARCH_BUMALIX) return state_engine_alloc(e);
@@ -4033,7 +4712,7 @@ extern "C" int b2_engine_create(const b2_config* cfg, const char* safetensors_pa
   B2_REQUIRE(cfg != nullptr && out != nullptr, "b2_engine_create: null argument");
   B2_REQUIRE(cfg->abi_version == B2_ABI_VERSION, "b2_engine_create: abi_version %d != %d", cfg->abi_version, B2_ABI_VERSION);
   B2_REQUIRE(cfg->arch == B2_ARCH_QWEN3 || cfg->arch == B2_ARCH_PHI3 || cfg->arch == B2_ARCH_OPT || list_arch(cfg->arch),
-             "arch %d not built (0 = Qwen3, 1 = Phi-3, 2 = OPT, 3 = Lerasun, 4 = Kedasun, 5 = Bumalix, 6 = Tinevik, 7 = Tolanex)", cfg->arch);
+             "arch %d not built (0 = Qwen3, 1 = Phi-3, 2 = OPT, 3 = Lerasun, 4 = Kedasun, 5 = Bumalix, 6 = Tinevik, 7 = Tolanex, 8 = Resitar)", cfg->arch);
   const bool ls = list_arch(cfg->arch);  // a layer-list family: its sizes live in layer_specs and are checked in list_engine_alloc
   B2_REQUIRE(ls || !cfg->compute_f32, "compute_f32: only the layer-list families have an fp32 path");
   B2_REQUIRE(!ls || cfg->layer_specs != nullptr, "layer-list family: layer_specs is NULL");
@@ -4298,14 +4977,14 @@ extern "C" int b2_engine_create(const b2_config* cfg, const char* safetensors_pa
       // bytes one page takes in all regions together
       size_t page_bytes_all = blk_elems * 2 * 2 * c.num_layers;
       const bool heads_cache = c.arch == B2_ARCH_KEDASUN;  // a K region and a V region per layer, rows of kv_heads * dim / kv_heads * vdim
-      const bool state_arch = c.arch == B2_ARCH_BUMALIX;   // a K and a V region per RUN of a layer that has a softmax mixer
+      const bool state_arch = c.arch == B2_ARCH_BUMALIX || c.arch == B2_ARCH_RESITAR;   // a K and a V region per RUN of a layer that has a softmax mixer
       // per RUN: a K and a V region for a softmax mixer, one region of latents for a latent mixer that stores its own (kv_from: the named run's)
       const bool mixed_arch = c.arch == B2_ARCH_TINEVIK || c.arch == B2_ARCH_TOLANEX;
       auto own_latent = [](const b2_layer_spec& sp) { return sp.mixer == B2_MIXER_GATED_LATENT || (sp.mixer == B2_MIXER_LATENT_ATTENTION && sp.kv_from < 0); };
       if (state_arch) {
         page_bytes_all = 0;
         for (const ListRun& R : e->runs)
-          if (e->ll[R.layer].sp.mixer == B2_MIXER_WINDOW_AND_STATE) page_bytes_all += (size_t)c.block_size * (e->ll[R.layer].nk + e->ll[R.layer].nv) * e->esz;
+          if (keeps_kv(e->ll[R.layer].sp.mixer)) page_bytes_all += (size_t)c.block_size * (e->ll[R.layer].nk + e->ll[R.layer].nv) * e->esz;
         page_bytes_all = std::max<size_t>(page_bytes_all, 16);
       } else if (mixed_arch) {
         page_bytes_all = 0;
@@ -4344,7 +5023,7 @@ extern "C" int b2_engine_create(const b2_config* cfg, const char* safetensors_pa
         if (state_arch) {
           for (ListRun& R : e->runs) {
             const ListLayer& L = e->ll[R.layer];
-            if (L.sp.mixer != B2_MIXER_WINDOW_AND_STATE) continue;
+            if (!keeps_kv(L.sp.mixer)) continue;
             const size_t kb = (size_t)c.block_size * L.nk * e->esz, vb = (size_t)c.block_size * L.nv * e->esz;
             R.k_region = (int)e->regions.size();
             e->regions.push_back({e->l_pool + off, kb});
@@ -4450,9 +5129,9 @@ extern "C" int b2_engine_load_safetensors(b2_engine* e, const char* path) {
 extern "C" int b2_engine_finalize(b2_engine* e) {
   B2_REQUIRE(e, "b2_engine_finalize: null engine");
   const int arch = e->cfg.arch;
-  if (arch == B2_ARCH_BUMALIX || arch == B2_ARCH_TINEVIK || arch == B2_ARCH_TOLANEX) {
+  if (arch == B2_ARCH_BUMALIX || arch == B2_ARCH_TINEVIK || arch == B2_ARCH_TOLANEX || arch == B2_ARCH_RESITAR) {
     B2_CUDA_OK(cudaSetDevice(e->device));
-    B2_TRY(arch == B2_ARCH_BUMALIX ? state_finalize(e) : arch == B2_ARCH_TINEVIK ? mixed_finalize(e) : outnorm_finalize(e));
+    B2_TRY(arch == B2_ARCH_RESITAR ? streams_finalize(e) : arch == B2_ARCH_BUMALIX ? state_finalize(e) : arch == B2_ARCH_TINEVIK ? mixed_finalize(e) : outnorm_finalize(e));
     e->finalized = true;
     return 0;
   }
@@ -4511,6 +5190,8 @@ extern "C" void b2_engine_free(b2_engine* e) {
   if (e->h_xtiles) cudaFreeHost(e->h_xtiles);
   if (e->h_xctx) cudaFreeHost(e->h_xctx);
   if (e->h_xtable) cudaFreeHost(e->h_xtable);
+  for (auto& t : e->rot_tables) F(t.table);
+  F(e->l_shift); F(e->l_ao); F(e->l_rkvg); F(e->l_lr); F(e->l_cv);
   F(e->l_final_bias); F(e->l_bigram); F(e->l_pos); F(e->l_tok_ring); F(e->l_sg); F(e->l_rz);
   F(e->l_embed); F(e->l_head); F(e->l_embed_gain); F(e->l_final_gain); F(e->l_pool); F(e->l_h); F(e->l_qd); F(e->l_qrot); F(e->l_qabs);
   F(e->l_xperm); F(e->l_upf); if (e->h_offsets) cudaFreeHost(e->h_offsets);
@@ -4522,9 +5203,10 @@ extern "C" void b2_engine_free(b2_engine* e) {
     F(L.gain1b); F(L.gain2b); F(L.qkv_bias); F(L.o_bias); F(L.conv_w); F(L.talk); F(L.vmix); F(L.conv_ring);
     F(L.wo2); F(L.sh_up); F(L.sh_down); F(L.qk_gain); F(L.head_gain); F(L.a2); F(L.a2_bias); F(L.g2); F(L.a_log); F(L.out_gain_l); F(L.out_gain_r); F(L.poly);
     F(L.bias1); F(L.bias1b); F(L.bias2); F(L.bias2b); F(L.latq_gain); F(L.uq); F(L.ukv); F(L.router_op); F(L.table);
+    F(L.hc[0]); F(L.hc[1]); F(L.mu); F(L.bonus); F(L.skip); F(L.conv_b); F(L.wshift); F(L.w1);
   }
   for (auto& R : e->runs) {
-    F(R.state); F(R.ring);
+    F(R.state); F(R.ring); F(R.shift_ring);
   }
   for (auto& ev : e->l_ev)
     if (ev) cudaEventDestroy(ev);

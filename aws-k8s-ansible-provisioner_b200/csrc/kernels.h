@@ -181,8 +181,8 @@ size_t attn_decode_scratch_floats(int B, int nq, int nkv, int hd);
 int attn_decode_zero_counters(float* scratch, cudaStream_t s);
 int launch_attn_decode(const bf16* q, const bf16* k_pages, const bf16* v_pages, const int32_t* block_table,
                        int bt_stride, const int32_t* seq_lens, float* scratch, bf16* out, int B, int nq, int nkv,
-                       int hd, int block_size, cudaStream_t s, float softmax_scale = 0.f, int window = 0, int tag = 0);
-// softmax_scale 0 = hd^-0.5; a padded head passes the scale of its real width.  window > 0: sliding-window attention,
+                       int hd, int block_size, cudaStream_t s, float softmax_scale = 0.f, int window = 0, int tag = 0, int chunk = 0);
+// chunk > 0: a query sees its own chunk only (positions floor(i / chunk) * chunk .. i).  softmax_scale 0 = hd^-0.5; a padded head passes the scale of its real width.  window > 0: sliding-window attention,
 // each query sees its last `window` keys (itself included).
 
 // ---- attn_prefill.cu ----
@@ -199,7 +199,7 @@ int launch_attn_prefill(const bf16* q, const bf16* k_pages, const bf16* v_pages,
 // ---- attn_prefill_tc.cu: the same pass on tcgen05 (S and P.V in TMEM, K/V pages through TMA); num_pages = size of the pool ----
 int launch_attn_prefill_tc(const bf16* q, const bf16* k_pages, const bf16* v_pages, int64_t num_pages, const int32_t* block_table,
                            int bt_stride, const PrefillTile* tiles_dev, int ntiles, bf16* out, int nq, int nkv, int hd, int block_size,
-                           cudaStream_t s, float softmax_scale = 0.f, int window = 0, int pair_mode = 0);
+                           cudaStream_t s, float softmax_scale = 0.f, int window = 0, int pair_mode = 0, int chunk = 0);
 // pair_mode: one query head per kv head; nq == 2 nkv with a partner head behind every real one, or nq == nkv without them
 
 // ---- sampling.cu ----
@@ -311,10 +311,39 @@ int launch_embed_sum(const int32_t* ids, const void* table, const BigramTable& b
 // taken in choice order); x_next = h in the operand type (null = not wanted)
 int launch_out_norm_add(float* h, const float* a, const float* a_scale, const float* y, const float* weight, const int32_t* pair_slot, int top,
                         const float* gain, float mult, int T, int W, float eps, cudaStream_t s, void* x_next, int x_f32);
+// Several residual streams h [T][n][W] fp32 that every sublayer reads and writes by learned mixes (Resitar).  n at most STREAMS_MAX.
+constexpr int STREAMS_MAX = 16;
+// every stream of token t = table[ids[t]] / rms * gain
+int launch_embed_streams(const int32_t* ids, const void* table, int table_f32, const float* gain, float* h, int n, int T, int W, int vocab, float eps,
+                         cudaStream_t s);
+struct StreamMix {           // one sublayer's numbers (device fp32): u = sum_s in[s] h_s; h_t <- sum_s mix[s][t] h_s + out[t] y
+  const float *in, *out, *mix;
+};
+struct StreamBranch {        // a sublayer's output y[t] = a[t] + bias_scale * bias + sum_k weight[t][k] * y[pair_slot[t * top + k]] (null parts are left out)
+  const float* a = nullptr;
+  const float* bias = nullptr;
+  float bias_scale = 1.f;
+  const float* y = nullptr;
+  const float* weight = nullptr;
+  const int32_t* pair_slot = nullptr;
+  int top = 0;
+};
+// The boundary between two sublayers in one pass: the streams take up `br` by `cur` (null: they stay as they are), then x[t] = rms(u) * gain with
+// u mixed by next_in (null: the plain sum), x fp32 or bf16 (null: not wanted).  rows (only without cur): x[i] is formed from row rows[i].
+int launch_streams_step(float* h, int n, const StreamMix* cur, const StreamBranch& br, const float* next_in, const float* gain, void* x, int x_f32, int T,
+                        int W, float eps, const int32_t* rows, cudaStream_t s);
+// out[t] = sum of the streams
+int launch_streams_sum(const float* h, int n, float* out, int T, int W, cudaStream_t s);
+// out[m][t] = x[t] + (x_prev - x[t]) * mu[m] for m = 0 .. 4, operand type; mu [5][W] fp32.  x_prev is the row above, or at the start of a portion the
+// sequence's entry of ring [sequence slots][2][W] (operand type, index = position mod 2; zeros before position 0), which the same launch updates with the
+// portion's last row.
+int launch_token_shift(const void* x, int x_f32, const float* mu, void* ring, void* out, int T, int W, const int32_t* row_seq, const int32_t* row_first,
+                       const int32_t* row_end, const int32_t* positions, const int32_t* slots, cudaStream_t s);
 // act[i] = softplus(p) z^2 + z / 2 for z > 0, (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 otherwise; pq (device) = p, q
 int launch_xielu(const float* z, const float* pq, void* act, int act_f32, size_t n, cudaStream_t s);
-// out[t][i] = a[t][i] * sigmoid(gate[t * gate_ld + i]), out fp32 or bf16 [T][N]
-int launch_sigmoid_gate(const float* a, const float* gate, int gate_ld, void* out, int out_f32, int T, int N, cudaStream_t s);
+// out[t * out_ld + i] = scale * a[t][i] * sigmoid(gate[t * gate_ld + i]), a fp32 (or bf16: a_bf16) [T][N], out fp32 or bf16 (out_ld 0 = N)
+int launch_sigmoid_gate(const void* a, const float* gate, int gate_ld, void* out, int out_f32, int T, int N, cudaStream_t s, int a_bf16 = 0,
+                        float scale = 1.f, int out_ld = 0);
 
 // ---- attn_heads.cu: softmax attention with per-head keys and values, any head width, fp32 or bf16 cache ----
 struct HeadsGeom {
@@ -335,7 +364,13 @@ struct HeadsGeom {
   int rot_values;                   // 1: the value of position j is rotated by j over all of vdim (pairs (m, m + vdim/2), angle j * rot_base^(-2m/vdim))
                                     //    before it is cached, and a query's weighted sum is turned back by its own position
   float softcap;                    // scores <- softcap * tanh(scores / softcap) (0 = none)
+  int chunk;                        // > 0: key j is seen from i only when i / chunk == j / chunk (whole numbers); window and keep_first are then 0
 };
+// First position a query at position i sees (the kept first tokens aside).
+__host__ __device__ inline int first_seen_key(int i, int window, int chunk) {
+  if (chunk > 0) return i / chunk * chunk;
+  return window > 0 && i >= window ? i - window + 1 : 0;
+}
 // proj [T][ld] fp32 = q | k | v (| more) of the fused projection.  bias [heads*dim + kv_heads*(dim+vdim)] or null; conv_w [channels][taps];
 // ring [sequence slots][taps][channels] fp32 (row = position mod taps); row_seq / row_first / row_end [T]: the token's sequence slot and the first row / one past
 // the last row of its portion in this step.  vmix_mode 0 none, 1 the layer supplies v_first [T][kv_heads*vdim], 2 it blends with it by
@@ -362,6 +397,15 @@ int launch_heads_finish_rownorm(const float* proj, int ld, const HeadsGeom& g, c
 // Writes q_out [T][heads*dim] fp32 and the token's K and V cache rows (plain layout).
 int launch_heads_finish_halves(const float* proj, int ld, const HeadsGeom& g, const float* q_gain, const float* k_gain, const int32_t* positions,
                                const int32_t* slots, float* q_out, void* k_cache, void* v_cache, int cache_f32, int T, cudaStream_t s);
+// What follows a fused, biased q | k (| v) projection when q and k heads are rotated by a table: table [positions][rot_dims] fp32 = the cosines of
+// every pair, then the sines (launch_rot_table).  halves: pairs (i, i + rot_dims/2), else (2i, 2i + 1).  keys_as_values: there is no v in proj and a
+// token's value is its key before the rotation (vdim == dim).  bias [all projected rows] or null.  Writes the queries (q_out fp32, or q_bf16) and the
+// token's K and V cache rows (g.swizzled: the GQA kernels' page layout).
+int launch_heads_finish_table(const float* proj, int ld, const HeadsGeom& g, const float* bias, const float* table, int halves, int keys_as_values,
+                              const int32_t* positions, const int32_t* slots, float* q_out, bf16* q_bf16, void* k_cache, void* v_cache, int cache_f32,
+                              int T, cudaStream_t s);
+// freqs [rot_dims / 2] (device, fp64) -> table [npos][rot_dims]: mul * cos(p f_i) | mul * sin(p f_i), angles in fp64
+int launch_rot_table(const double* freqs, int half, double mul, float* table, int npos, cudaStream_t s);
 // Softmax attention whose scaled scores pass the cap and are mixed over the heads, s'_a = sum_b mix[a][b] s_b (mix [heads][heads], null =
 // none), BEFORE the softmax; causal, with g.window; with g.rot_values the weighted sum is turned back by the query's position.  All heads of
 // a query token are formed together.  tiles == null: decode form.  out [T][heads*vdim] (fp32 or bf16).
@@ -379,16 +423,22 @@ int launch_talk_gate(const float* cross, const float* talk, const float* gate, i
 enum StateRule {
   STATE_RULE_DECAY = 0,
   STATE_RULE_DELTA = 1,
-  STATE_RULE_DELTA_HEAD = 2         // the delta rule with one decay per head: `decay` is [T][heads]
+  STATE_RULE_DELTA_HEAD = 2,        // the delta rule with one decay per head: `decay` is [T][heads]
+  STATE_RULE_DECAY_HEAD = 3,        // a state-space recurrence: `decay` is [T][heads], the write is scaled by beta [T][heads], and the read-out gets
+                                    // skip[head] * v on top
+  STATE_RULE_BONUS = 4              // time mixing: the read-out sees the state BEFORE the token's write, plus the write scaled by bonus per key channel
 };
 struct StateGeom {
   int heads, kv_heads, dim, vdim;   // state head a reads query/key head a / (heads / kv_heads); S is [dim][vdim] per head
   int rule;                         // StateRule
+  const float* skip = nullptr;      // STATE_RULE_DECAY_HEAD: [heads]
+  const float* bonus = nullptr;     // STATE_RULE_BONUS: [heads][dim]
 };
 enum LowRankMode {
   LOWRANK_SIGMOID = 0,              // y = sigmoid(z)
   LOWRANK_DECAY_SIGMOID_POW = 1,    // y = sigmoid(z)^rate, formed as exp(-rate * softplus(-z))
-  LOWRANK_DECAY_SOFTPLUS = 2        // y = exp(-exp(rate_log[c / per_head]) * softplus(z))
+  LOWRANK_DECAY_SOFTPLUS = 2,       // y = exp(-exp(rate_log[c / per_head]) * softplus(z))
+  LOWRANK_DECAY_EXP = 3             // y = exp(-exp(z)), and the low-rank inputs pass tanh first
 };
 // out [T][C] fp32 = act(w2 [C][rank] . lr[t][lr_off .. lr_off + rank) + bias [C] (or null))
 int launch_lowrank_act(const float* lr, int ld, int lr_off, int rank, const float* w2, const float* bias, int mode, float rate,
@@ -412,8 +462,18 @@ int launch_state_scan(const float* q, int ldq, const float* k, int ldk, const fl
                       cudaStream_t s);
 size_t state_floats_per_slot(const StateGeom& g);
 // out[t][a][:] = o[t][a][:] / sqrt(mean(o[t][a]^2) + eps) * gain[:] * (gate_silu ? silu(gate) : gate), gate at gate[t * gate_ld + a * vdim + :]
+// gain_per_head: gain is [heads][vdim]; the result is multiplied by scale and goes to rows of out_ld (0 = heads * vdim)
 int launch_state_out_gate(const float* o, const float* gain, const float* gate, int gate_ld, int gate_silu, void* out, int out_f32,
-                          int heads, int vdim, float eps, int T, cudaStream_t s);
+                          int heads, int vdim, float eps, int T, cudaStream_t s, int gain_per_head = 0, float scale = 1.f, int out_ld = 0);
+// The state-space mixer's inputs, behind the fused projection: proj [T][ld] fp32 = x | B | C (channels of them) | step logits (heads).  Every channel
+// passes a causal convolution with bias (ring as above) and silu -> out [T][channels]; step [T][heads] = softplus(logit + dt_bias), decay [T][heads] =
+// exp(-exp(a_log) * step).  single_rows as above.
+int launch_conv_act_finish(const float* proj, int ld, int channels, int heads, int taps, const float* conv_w, const float* conv_b, const float* a_log,
+                           const float* dt_bias, float* ring, const int32_t* row_seq, const int32_t* row_first, const int32_t* row_end,
+                           const int32_t* positions, const int32_t* slots, float* out, float* step, float* decay, int T, int single_rows, cudaStream_t s);
+// v = o * silu(gate) cut into `parts` equal pieces, each divided by its own root mean square, times gain [N] and scale -> out (rows of out_ld)
+int launch_gate_part_norm(const float* o, const float* gate, int gate_ld, const float* gain, int parts, float scale, void* out, int out_f32, int out_ld,
+                          int N, float eps, int T, cudaStream_t s);
 
 // ---- attn_latent.cu: attention over a shared per-token latent (absorbed form) ----
 // The cache holds, per token, the normalised latent c [kv_rank] and the rotated key piece [rot_dim] side by side
@@ -468,6 +528,8 @@ struct RouteGeom {
   int softmax;       // 1: scores are a softmax over all experts; 0: a sigmoid per expert
   int group_best;    // 1: a group's score is its best choice score; 0: the sum of its two best
   float scale;       // raw_weights: the weights are multiplied by this (0 = 1)
+  const float* logit_bias;   // added to the experts' logits before the softmax or sigmoid (null = none); with `softmax` and not raw_weights the weights are the
+                             // softmax over the chosen logits
 };
 // x [T][W] (operand type), router [experts][W] fp32, correction [experts] fp32 (null = none) -> idx [T][top], weight [T][top].
 // gate_out != null: the router has one more row, and gate_out [T] = sigmoid of its product with x

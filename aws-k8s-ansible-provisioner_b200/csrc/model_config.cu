@@ -2,7 +2,8 @@
 // one).  b2serve, the Python mirror and bin/trace_run all choose the model class through this one function, so a family
 // is added to the framework here, in b2_engine_create and nowhere else.  Host code only.
 //
-// The fourth and fifth layer-list families, Tinevik and Tolanex, are described above their readers (tinevik_config, tolanex_config).
+// The fourth, fifth and sixth layer-list families, Tinevik, Tolanex and Resitar, are described above their readers (tinevik_config, tolanex_config,
+// resitar_config).
 // HF families are told apart by "model_type" (the keys follow HF's Qwen3Config / Phi3Config / OPTConfig); Lerasun by
 // "architecture": "Lerasun", whose config lists its layers one by one:
 //   {"architecture": "Lerasun", "vocab": V, "width": W, "logit_scale": s, "norm": {"eps": e},
@@ -625,6 +626,149 @@ int tolanex_config(const Value& j, b2_config* c, b2_layer_spec* specs, int max_s
   return 0;
 }
 
+// Resitar: {"architecture": "Resitar", "vocab": V, "width": W, "streams": n, "norm": {"eps": e}, "loop": {"start", "stop", "times"}?,
+//   "layers": [{"type": "parallel", "mixer": {"left": {"heads", "kv_heads"?, "dim", "vdim"?, "scale", "mask": {"size"}?, "rot": {"base", "dims"}?},
+//                                             "right": {"heads", "vdim", "state", "groups"?, "conv", "norm_groups"?}, "left_scale"?, "right_scale"?}, "mlp": ...},
+//              {"type": "parallel_2", "mixer": {"left": {"heads", "kv_heads"?, "dim", "vdim", "scale",
+//                                                        "rot": {"base", "dims", "scaling": {"factor", "original", "fast", "slow"}?}?},
+//                                               "right": {"heads", "dim"}, "left_scale"?, "right_scale"?},
+//               "mlp": null | {"kind": "dense", "ff"} | {"kind": "moe", "expert": {"ff"}, "router": {"experts", "top"}}}, ...]}
+int opt_int(const Value& o, const char* key, int dflt) {
+  const Value* v = o.find(key);
+  return v && v->is_number() ? (int)v->as_int() : dflt;
+}
+float opt_float(const Value& o, const char* key, float dflt) {
+  const Value* v = o.find(key);
+  return v && v->is_number() ? (float)v->as_double() : dflt;
+}
+const Value* object_at(const Value& o, const char* key) {
+  const Value* v = o.find(key);
+  return v && v->is_object() ? v : nullptr;
+}
+int resitar_config(const Value& j, b2_config* c, b2_layer_spec* specs, int max_specs) {
+  c->arch = B2_ARCH_RESITAR;
+  CFG_TRY(need_int(j, "vocab", "config", &c->vocab));
+  CFG_TRY(need_int(j, "width", "config", &c->hidden));
+  CFG_TRY(need_int(j, "streams", "config", &c->streams));
+  const Value* norm = object_at(j, "norm");
+  if (!norm) {
+    b2_set_error("config.json: norm missing");
+    return -22;
+  }
+  CFG_TRY(need_float(*norm, "eps", "norm", &c->rms_eps));
+  c->norm_groups = 1;
+  c->embed_scale = 1.0f;
+  c->logit_scale = 1.0f;
+  if (const Value* loop = object_at(j, "loop")) {
+    CFG_TRY(need_int(*loop, "start", "loop", &c->loop_start));
+    CFG_TRY(need_int(*loop, "stop", "loop", &c->loop_stop));
+    CFG_TRY(need_int(*loop, "times", "loop", &c->loop_times));
+  }
+  const Value* layers = j.find("layers");
+  if (!layers || !layers->is_array() || layers->size() == 0) {
+    b2_set_error("config.json: layers missing or empty");
+    return -22;
+  }
+  c->num_layers = (int)layers->size();
+  if (c->num_layers > max_specs || specs == nullptr) {
+    b2_set_error("config.json: %d layers, room for %d layer specs", c->num_layers, max_specs);
+    return -22;
+  }
+  if (c->loop_times > 0 && !(c->loop_start >= 0 && c->loop_start <= c->loop_stop && c->loop_stop <= c->num_layers)) {
+    b2_set_error("config.json: loop [%d, %d) outside the %d layers", c->loop_start, c->loop_stop, c->num_layers);
+    return -22;
+  }
+  for (int i = 0; i < c->num_layers; ++i) {
+    const Value& L = layers->at(i);
+    b2_layer_spec& s = specs[i];
+    memset(&s, 0, sizeof s);
+    s.kv_from = -1;
+    s.weights_of = -1;
+    char where[64];
+    snprintf(where, sizeof where, "layers[%d].mixer", i);
+    const Value* type = L.find("type");
+    const Value* m = object_at(L, "mixer");
+    if (!type || !type->is_string() || !m) {
+      b2_set_error("config.json: layers[%d] needs type and mixer", i);
+      return -22;
+    }
+    const std::string ty = type->as_string();
+    if (ty != "parallel" && ty != "parallel_2") {
+      b2_set_error("config.json: layers[%d]: mixer type '%s' not built (parallel, parallel_2)", i, ty.c_str());
+      return -22;
+    }
+    const bool ssm = ty == "parallel";
+    s.mixer = ssm ? B2_MIXER_CHUNK_AND_SSM : B2_MIXER_FULL_AND_TIMEMIX;
+    const Value *a = object_at(*m, "left"), *b = object_at(*m, "right");
+    if (!a || !b) {
+      b2_set_error("config.json: %s needs left and right", where);
+      return -22;
+    }
+    s.mix_left = opt_float(*m, "left_scale", 1.0f);
+    s.mix_right = opt_float(*m, "right_scale", 1.0f);
+    snprintf(where, sizeof where, "layers[%d].mixer.left", i);
+    CFG_TRY(need_int(*a, "heads", where, &s.heads));
+    s.kv_heads = opt_int(*a, "kv_heads", s.heads);
+    CFG_TRY(need_int(*a, "dim", where, &s.dim));
+    s.vdim = opt_int(*a, "vdim", s.dim);
+    CFG_TRY(need_float(*a, "scale", where, &s.scale));
+    s.rot_halves = ssm ? 1 : 0;
+    s.rot_factor = 1.0f;
+    if (const Value* rot = object_at(*a, "rot")) {   // no "rot": nothing is rotated
+      CFG_TRY(need_float(*rot, "base", where, &s.rot_base));
+      CFG_TRY(need_int(*rot, "dims", where, &s.rot_dims));
+      if (const Value* sc = object_at(*rot, "scaling")) {
+        CFG_TRY(need_float(*sc, "factor", where, &s.rot_factor));
+        CFG_TRY(need_int(*sc, "original", where, &s.rot_orig));
+        CFG_TRY(need_float(*sc, "fast", where, &s.rot_fast));
+        CFG_TRY(need_float(*sc, "slow", where, &s.rot_slow));
+      }
+    }
+    if (const Value* mask = object_at(*a, "mask")) CFG_TRY(need_int(*mask, "size", where, &s.chunk));   // no "mask": every earlier key is seen
+    snprintf(where, sizeof where, "layers[%d].mixer.right", i);
+    CFG_TRY(need_int(*b, "heads", where, &s.s_heads));
+    if (ssm) {
+      CFG_TRY(need_int(*b, "vdim", where, &s.s_vdim));
+      CFG_TRY(need_int(*b, "state", where, &s.s_dim));
+      CFG_TRY(need_int(*b, "conv", where, &s.conv_taps));
+      s.s_groups = opt_int(*b, "groups", 1);
+      s.s_norm_groups = opt_int(*b, "norm_groups", 1);
+    } else {
+      CFG_TRY(need_int(*b, "dim", where, &s.s_dim));
+      s.s_vdim = s.s_dim;
+    }
+    s.ff = B2_FF_NONE;
+    if (const Value* mlp = object_at(L, "mlp")) {
+      snprintf(where, sizeof where, "layers[%d].mlp", i);
+      const Value* kind = mlp->find("kind");
+      const std::string kd = kind && kind->is_string() ? kind->as_string() : "?";
+      if (kd == "dense") {
+        s.ff = B2_FF_SWIGLU;
+        CFG_TRY(need_int(*mlp, "ff", where, &s.ff_dim));
+      } else if (kd == "moe") {
+        s.ff = B2_FF_TOP_SOFTMAX_EXPERTS;
+        const Value *ex = object_at(*mlp, "expert"), *ro = object_at(*mlp, "router");
+        if (!ex || !ro) {
+          b2_set_error("config.json: %s needs expert and router", where);
+          return -22;
+        }
+        CFG_TRY(need_int(*ex, "ff", where, &s.ff_dim));
+        CFG_TRY(need_int(*ro, "experts", where, &s.experts));
+        CFG_TRY(need_int(*ro, "top", where, &s.top));
+        s.groups = s.groups_keep = 1;
+      } else {
+        b2_set_error("config.json: %s.kind '%s' not built (dense, moe)", where, kd.c_str());
+        return -22;
+      }
+    }
+  }
+  c->layer_specs = specs;
+  c->tie_embeddings = 1;
+  c->num_q_heads = c->num_kv_heads = 0;
+  c->head_dim = c->intermediate = 0;
+  return 0;
+}
+
 }  // namespace
 
 extern "C" int b2_config_from_dir(const char* model_dir, b2_config* c, b2_layer_spec* specs, int32_t max_specs) {
@@ -655,6 +799,7 @@ extern "C" int b2_config_from_dir(const char* model_dir, b2_config* c, b2_layer_
   c->residual_mult = 0.f;
   c->bigram_buckets = 0;
   c->bigram_mul_prev = c->bigram_mul_cur = 0;
+  c->streams = 0;
   const Value* archv = j.find("architecture");
   if (archv && archv->is_string()) {
     if (archv->as_string() == "Lerasun") return lerasun_config(j, c, specs, max_specs);
@@ -662,6 +807,7 @@ extern "C" int b2_config_from_dir(const char* model_dir, b2_config* c, b2_layer_
     if (archv->as_string() == "Bumalix") return bumalix_config(j, c, specs, max_specs);
     if (archv->as_string() == "Tinevik") return tinevik_config(j, c, specs, max_specs);
     if (archv->as_string() == "Tolanex") return tolanex_config(j, c, specs, max_specs);
+    if (archv->as_string() == "Resitar") return resitar_config(j, c, specs, max_specs);
     b2_set_error("%s: architecture '%s' not built", path.c_str(), archv->as_string().c_str());
     return -22;
   }

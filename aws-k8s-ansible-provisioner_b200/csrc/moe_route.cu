@@ -1,7 +1,7 @@
 // moe_route.cu -- the router of a routed-experts feed-forward, and the bookkeeping that turns its choices into ragged
 // groups for gemm_any.cu.
 //
-// Router (all fp32): z = R x, s = sigmoid(z) or a softmax of z over all experts (RouteGeom.softmax).  The CHOICE uses s + correction (an
+// Router (all fp32): z = R x (+ a bias), s = sigmoid(z) or a softmax of z over all experts (RouteGeom.softmax).  The CHOICE uses s + correction (an
 // optional per-expert offset that steers load and may make a choice score negative); the mixing WEIGHTS use s alone.  Experts are
 // `groups` equal runs of neighbours; a group's score is the sum of its two best choice scores (or its best one, group_best) and only the
 // `keep` best groups may supply experts (the others are out, not zero).  Of the allowed experts the `top` with the best choice scores
@@ -135,7 +135,10 @@ __global__ void __launch_bounds__(RT_WARPS * 32) route_kernel(const TX* __restri
 #pragma unroll
     for (int tt = 0; tt < NTOK; ++tt) {
       const float z = warp_sum(acc[tt]);
-      if (lane == 0) sc[tt * per_tok + e] = (g.softmax && e < E) ? z : 1.0f / (1.0f + expf(-z));   // (the extra row is a gate: always a sigmoid)
+      if (lane == 0) {
+        const float zb = z + (g.logit_bias && e < E ? g.logit_bias[e] : 0.f);
+        sc[tt * per_tok + e] = (g.softmax && e < E) ? zb : 1.0f / (1.0f + expf(-zb));   // (the extra row is a gate: always a sigmoid)
+      }
     }
   }
   __syncthreads();
@@ -158,7 +161,10 @@ __global__ void __launch_bounds__(256) route_select_kernel(const float* __restri
   if (t >= T) return;
   float* s = sm + warp * (2 * E + g.groups);
   const float* zr = z + (size_t)t * ld;
-  for (int e = lane; e < E; e += 32) s[e] = g.softmax ? zr[e] : 1.0f / (1.0f + expf(-zr[e]));
+  for (int e = lane; e < E; e += 32) {
+    const float zb = zr[e] + (g.logit_bias ? g.logit_bias[e] : 0.f);
+    s[e] = g.softmax ? zb : 1.0f / (1.0f + expf(-zb));
+  }
   if (gate_out != nullptr && lane == 0) gate_out[t] = 1.0f / (1.0f + expf(-zr[E]));
   __syncwarp();
   route_pick(s, s + E, s + 2 * E, g, correction, t, idx, weight);

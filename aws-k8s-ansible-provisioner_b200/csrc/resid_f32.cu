@@ -484,15 +484,311 @@ __global__ void __launch_bounds__(256) xielu_kernel(const float* __restrict__ z,
   }
 }
 
-// out[t][i] = a[t][i] * sigmoid(gate[t * gate_ld + i])
-template <typename TX>
-__global__ void __launch_bounds__(256) sigmoid_gate_kernel(const float* __restrict__ a, const float* __restrict__ gate, int gate_ld, TX* __restrict__ out,
-                                                           int N) {
+// out[t * out_ld + i] = scale * a[t][i] * sigmoid(gate[t * gate_ld + i]); VEC: four numbers at a time (rows and bases on 16-byte boundaries)
+__device__ __forceinline__ void load4(const float* p, float* v) {
+  const float4 x = *reinterpret_cast<const float4*>(p);
+  v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+}
+__device__ __forceinline__ void load4(const bf16* p, float* v) {
+  const uint2 x = *reinterpret_cast<const uint2*>(p);
+  v[0] = bf16lo(x.x); v[1] = bf16hi(x.x); v[2] = bf16lo(x.y); v[3] = bf16hi(x.y);
+}
+__device__ __forceinline__ void store4(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(bf16* p, const float* v) {
+  uint2 pk;
+  pk.x = pack_bf16x2(v[0], v[1]);
+  pk.y = pack_bf16x2(v[2], v[3]);
+  *reinterpret_cast<uint2*>(p) = pk;
+}
+template <typename TA, typename TX, bool VEC>
+__global__ void __launch_bounds__(256) sigmoid_gate_kernel(const TA* __restrict__ a, const float* __restrict__ gate, int gate_ld, TX* __restrict__ out,
+                                                           int out_ld, float scale, int N) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x;
-  for (int i = blockIdx.y * 256 + threadIdx.x; i < N; i += 256 * gridDim.y)
-    out[(size_t)t * N + i] = (TX)(a[(size_t)t * N + i] / (1.0f + expf(-gate[(size_t)t * gate_ld + i])));
+  const TA* ar = a + (size_t)t * N;
+  const float* gr = gate + (size_t)t * gate_ld;
+  TX* dst = out + (size_t)t * out_ld;
+  if constexpr (VEC) {
+    for (int i = 4 * (blockIdx.y * 256 + threadIdx.x); i < N; i += 1024 * gridDim.y) {
+      float av[4], gv[4];
+      load4(ar + i, av);
+      load4(gr + i, gv);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) av[k] = scale * (av[k] / (1.0f + expf(-gv[k])));
+      store4(dst + i, av);
+    }
+  } else {
+    for (int i = blockIdx.y * 256 + threadIdx.x; i < N; i += 256 * gridDim.y) dst[i] = (TX)(scale * ((float)ar[i] / (1.0f + expf(-gr[i]))));
+  }
+}
+
+// ---- several residual streams with learned mixes (Resitar): h [T][n][W] ----
+template <typename TT>
+__global__ void __launch_bounds__(256) embed_streams_kernel(const int32_t* __restrict__ ids, const TT* __restrict__ table, const float* __restrict__ gain,
+                                                            float* __restrict__ h, int n, int W, int vocab, float eps) {
+  __shared__ float red[8];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  int id = ids[t];
+  id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+  const TT* row = table + (size_t)id * W;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < W; i += 256) {
+    const float v = (float)row[i];
+    ss = fmaf(v, v, ss);
+  }
+  const float r = 1.0f / sqrtf(block_sum_n<256>(ss, red) / (float)W + eps);
+  float* hr = h + (size_t)t * n * W;
+  for (int i = threadIdx.x; i < W; i += 256) {
+    const float v = (float)row[i] * r * gain[i];
+    for (int s = 0; s < n; ++s) hr[(size_t)s * W + i] = v;
+  }
+}
+
+// The boundary between two sublayers: the new streams from the old ones and the sublayer's output, the next sublayer's mixed and normed input.  One CTA of
+// NT threads per row; a thread keeps R groups of four neighbouring columns of all N streams in registers, every load in flight before the sums.
+constexpr int SS_MAX_TOP = 16;
+struct StreamsArgs {
+  float* h;
+  const float *c_out, *c_mix, *next_in;   // the sublayer's numbers (c_mix null: the streams stay), the next one's input mix (null: the plain sum)
+  StreamBranch br;
+  const float* gain;
+  int W;
+  float eps;
+  const int32_t* rows;
+};
+template <typename TX, int N, int NT, int R>
+__global__ void __launch_bounds__(NT) streams_step_kernel(StreamsArgs p, TX* __restrict__ x) {
+  __shared__ float red[NT / 32];
+  __shared__ float w_s[SS_MAX_TOP];
+  __shared__ int slot_s[SS_MAX_TOP];
+  // constants of the model: readable before the kernel in front is done
+  float c_mix[N][N], c_out[N], c_in[N];
+  const bool update = p.c_mix != nullptr;
+#pragma unroll
+  for (int s = 0; s < N; ++s) {
+    c_out[s] = update ? p.c_out[s] : 0.f;
+    c_in[s] = p.next_in ? p.next_in[s] : 1.0f;
+#pragma unroll
+    for (int d = 0; d < N; ++d) c_mix[s][d] = update ? p.c_mix[s * N + d] : 0.f;
+  }
+  const int t = blockIdx.x, W4 = p.W >> 2;
+  float4 gv[R], bv[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int i = threadIdx.x + r * NT;
+    gv[r] = x != nullptr && i < W4 ? reinterpret_cast<const float4*>(p.gain)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    bv[r] = p.br.bias != nullptr && i < W4 ? reinterpret_cast<const float4*>(p.br.bias)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  const StreamBranch& br = p.br;
+  if (br.y != nullptr) {
+    if ((int)threadIdx.x < br.top) {
+      w_s[threadIdx.x] = br.weight[(size_t)t * br.top + threadIdx.x];
+      slot_s[threadIdx.x] = br.pair_slot[(size_t)t * br.top + threadIdx.x];
+    }
+    __syncthreads();
+  }
+  float4* hr = reinterpret_cast<float4*>(p.h + (size_t)(p.rows ? p.rows[t] : t) * N * p.W);
+  float4 hv[R][N], y[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int i = threadIdx.x + r * NT;
+    const bool in = i < W4;
+#pragma unroll
+    for (int s = 0; s < N; ++s) hv[r][s] = in ? hr[(size_t)s * W4 + i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    y[r] = in && br.a != nullptr ? reinterpret_cast<const float4*>(br.a + (size_t)t * p.W)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    y[r].x = fmaf(br.bias_scale, bv[r].x, y[r].x); y[r].y = fmaf(br.bias_scale, bv[r].y, y[r].y);
+    y[r].z = fmaf(br.bias_scale, bv[r].z, y[r].z); y[r].w = fmaf(br.bias_scale, bv[r].w, y[r].w);
+  }
+  if (br.y != nullptr)
+    for (int k = 0; k < br.top; ++k) {   // choice order
+      const float w = w_s[k];
+      const float4* yr = reinterpret_cast<const float4*>(br.y + (size_t)slot_s[k] * p.W);
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        const int i = threadIdx.x + r * NT;
+        if (i < W4) {
+          const float4 q = yr[i];
+          y[r].x = fmaf(w, q.x, y[r].x); y[r].y = fmaf(w, q.y, y[r].y); y[r].z = fmaf(w, q.z, y[r].z); y[r].w = fmaf(w, q.w, y[r].w);
+        }
+      }
+    }
+  float ss = 0.f;
+  float4 u[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int i = threadIdx.x + r * NT;
+    u[r] = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int d = 0; d < N; ++d) {
+      float4 o;
+      if (update) {
+        o = make_float4(c_out[d] * y[r].x, c_out[d] * y[r].y, c_out[d] * y[r].z, c_out[d] * y[r].w);
+#pragma unroll
+        for (int s = 0; s < N; ++s) {
+          const float m = c_mix[s][d];
+          o.x = fmaf(m, hv[r][s].x, o.x); o.y = fmaf(m, hv[r][s].y, o.y); o.z = fmaf(m, hv[r][s].z, o.z); o.w = fmaf(m, hv[r][s].w, o.w);
+        }
+        if (i < W4) hr[(size_t)d * W4 + i] = o;
+      } else {
+        o = hv[r][d];
+      }
+      const float c = c_in[d];
+      u[r].x = fmaf(c, o.x, u[r].x); u[r].y = fmaf(c, o.y, u[r].y); u[r].z = fmaf(c, o.z, u[r].z); u[r].w = fmaf(c, o.w, u[r].w);
+    }
+    ss += (u[r].x * u[r].x + u[r].y * u[r].y) + (u[r].z * u[r].z + u[r].w * u[r].w);
+  }
+  if (x == nullptr) return;
+  const float rn = 1.0f / sqrtf(block_sum_n<NT>(ss, red) / (float)p.W + p.eps);
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int i = threadIdx.x + r * NT;
+    if (i >= W4) continue;
+    const float o[4] = {u[r].x * rn * gv[r].x, u[r].y * rn * gv[r].y, u[r].z * rn * gv[r].z, u[r].w * rn * gv[r].w};
+    store4(x + (size_t)t * p.W + 4 * i, o);
+  }
+}
+
+// the same for any width, any number of streams up to STREAMS_MAX and any number of choices: u staged in shared memory, one column at a time
+template <typename TX>
+__global__ void __launch_bounds__(256) streams_step_any_kernel(StreamsArgs p, int n, TX* __restrict__ x) {
+  extern __shared__ float us[];
+  __shared__ float red[8];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  const StreamBranch& br = p.br;
+  float* hr = p.h + (size_t)(p.rows ? p.rows[t] : t) * n * p.W;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < p.W; i += 256) {
+    float hv[STREAMS_MAX], u = 0.f;
+    for (int s = 0; s < n; ++s) hv[s] = hr[(size_t)s * p.W + i];
+    float y = br.a ? br.a[(size_t)t * p.W + i] : 0.f;
+    if (br.bias) y = fmaf(br.bias_scale, br.bias[i], y);
+    if (br.y != nullptr)
+      for (int k = 0; k < br.top; ++k) y = fmaf(br.weight[(size_t)t * br.top + k], br.y[(size_t)br.pair_slot[(size_t)t * br.top + k] * p.W + i], y);
+    for (int d = 0; d < n; ++d) {
+      float o = hv[d];
+      if (p.c_mix != nullptr) {
+        o = p.c_out[d] * y;
+        for (int s = 0; s < n; ++s) o = fmaf(p.c_mix[s * n + d], hv[s], o);
+        hr[(size_t)d * p.W + i] = o;
+      }
+      u = fmaf(p.next_in ? p.next_in[d] : 1.0f, o, u);
+    }
+    us[i] = u;
+    ss = fmaf(u, u, ss);
+  }
+  if (x == nullptr) return;
+  const float rn = 1.0f / sqrtf(block_sum_n<256>(ss, red) / (float)p.W + p.eps);
+  for (int i = threadIdx.x; i < p.W; i += 256) x[(size_t)t * p.W + i] = (TX)(us[i] * rn * p.gain[i]);   // (a thread's own columns)
+}
+
+template <typename TX>
+int streams_step_typed(const StreamsArgs& p, int n, TX* x, int T, cudaStream_t s) {
+#define B2_STREAMS(NN, NT, R)                                                                        \
+  do {                                                                                               \
+    B2_CUDA_OK(b2_launch(streams_step_kernel<TX, NN, NT, R>, dim3(T), dim3(NT), 0, s, p, x));        \
+    return 0;                                                                                        \
+  } while (0)
+#define B2_STREAMS_N(NN)                                                                             \
+  do {                                                                                               \
+    if (p.W <= 512) B2_STREAMS(NN, 128, 1);                                                          \
+    if (T < 1024) {   /* few tokens: wide CTAs, a row is one or two rounds of loads */               \
+      if (p.W <= 2048) B2_STREAMS(NN, 512, 1);                                                       \
+      if (p.W <= 4096) B2_STREAMS(NN, 512, 2);                                                       \
+      B2_STREAMS(NN, 512, 4);                                                                        \
+    }                                                                                                \
+    if (p.W <= 1024) B2_STREAMS(NN, 256, 1);                                                         \
+    if (p.W <= 2048) B2_STREAMS(NN, 256, 2);                                                         \
+    if (p.W <= 4096) B2_STREAMS(NN, 512, 2);                                                         \
+    B2_STREAMS(NN, 512, 4);                                                                          \
+  } while (0)
+  if (p.W % 4 == 0 && p.W <= 8192 && (p.br.y == nullptr || p.br.top <= SS_MAX_TOP)) {
+    if (n == 1) B2_STREAMS_N(1);
+    if (n == 2) B2_STREAMS_N(2);
+    if (n == 3) B2_STREAMS_N(3);
+    if (n == 4) B2_STREAMS_N(4);
+  }
+#undef B2_STREAMS_N
+#undef B2_STREAMS
+  const size_t smem = (size_t)p.W * 4;
+  B2_REQUIRE(smem <= 160 * 1024, "streams_step: a row of %d numbers does not fit in shared memory", p.W);
+  static B2PerDeviceOnce once;
+  if (smem > 48 * 1024) b2_prefer_max_smem(streams_step_any_kernel<TX>, once);
+  B2_CUDA_OK(b2_launch(streams_step_any_kernel<TX>, dim3(T), dim3(256), smem, s, p, n, x));
+  return 0;
+}
+
+__global__ void __launch_bounds__(256) streams_sum_kernel(const float* __restrict__ h, int n, float* __restrict__ out, int W) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const float* hr = h + (size_t)blockIdx.x * n * W;
+  for (int i = threadIdx.x; i < W; i += 256) {
+    float v = 0.f;
+    for (int s = 0; s < n; ++s) v += hr[(size_t)s * W + i];
+    out[(size_t)blockIdx.x * W + i] = v;
+  }
+}
+
+// Blends of a row with the row before it.  A thread owns columns; in a portion's first row it reads the sequence's ring entry and then leaves the
+// portion's last row there, read and write in one thread: the two may be the same entry.
+template <typename TX, bool VEC>
+__global__ void __launch_bounds__(256) token_shift_kernel(const TX* __restrict__ x, const float* __restrict__ mu, TX* __restrict__ ring, TX* __restrict__ out,
+                                                          int T, int W, const int32_t* __restrict__ row_seq, const int32_t* __restrict__ row_first,
+                                                          const int32_t* __restrict__ row_end, const int32_t* __restrict__ positions,
+                                                          const int32_t* __restrict__ slots) {
+  constexpr int V = VEC ? 4 : 1;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, pos = positions[t], first = row_first[t];
+  const bool live = slots[t] >= 0;   // (padding rows of a decode bucket touch nothing)
+  TX* rg = ring + (size_t)row_seq[t] * 2 * W;
+  for (int i = V * (blockIdx.y * 256 + threadIdx.x); i < W; i += V * 256 * gridDim.y) {
+    float xv[V], pv[V];
+    if constexpr (VEC) load4(x + (size_t)t * W + i, xv);
+    else xv[0] = (float)x[(size_t)t * W + i];
+#pragma unroll
+    for (int k = 0; k < V; ++k) pv[k] = 0.f;
+    if (live) {
+      if (t > first) {
+        if constexpr (VEC) load4(x + (size_t)(t - 1) * W + i, pv);
+        else pv[0] = (float)x[(size_t)(t - 1) * W + i];
+      } else {
+        if (pos > 0) {
+          if constexpr (VEC) load4(rg + (size_t)((pos - 1) & 1) * W + i, pv);
+          else pv[0] = (float)rg[(size_t)((pos - 1) & 1) * W + i];
+        }
+        const int last = row_end[t] - 1;
+        TX* dst = rg + (size_t)((pos + last - t) & 1) * W + i;
+        const TX* src = x + (size_t)last * W + i;
+        if constexpr (VEC) {
+          float lv[V];
+          load4(src, lv);
+          store4(dst, lv);
+        } else {
+          *dst = *src;
+        }
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < 5; ++m) {
+      float o[V];
+      if constexpr (VEC) {
+        float mv[4];
+        load4(mu + (size_t)m * W + i, mv);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) o[k] = fmaf(pv[k] - xv[k], mv[k], xv[k]);
+        store4(out + ((size_t)m * T + t) * W + i, o);
+      } else {
+        out[((size_t)m * T + t) * W + i] = (TX)fmaf(pv[0] - xv[0], mu[(size_t)m * W + i], xv[0]);
+      }
+    }
+  }
 }
 
 // ---- sublayers that read the stream itself; only their outputs are normed (Tolanex) ----
@@ -860,11 +1156,66 @@ int launch_xielu(const float* z, const float* pq, void* act, int act_f32, size_t
   return 0;
 }
 
-int launch_sigmoid_gate(const float* a, const float* gate, int gate_ld, void* out, int out_f32, int T, int N, cudaStream_t s) {
+int launch_sigmoid_gate(const void* a, const float* gate, int gate_ld, void* out, int out_f32, int T, int N, cudaStream_t s, int a_bf16, float scale,
+                        int out_ld) {
   if (T <= 0) return 0;
-  const dim3 grid(T, T >= 1024 ? 1 : std::max(1, std::min((N + 255) / 256, 1024 / T)));
-  if (out_f32) B2_CUDA_OK(b2_launch(sigmoid_gate_kernel<float>, grid, dim3(256), 0, s, a, gate, gate_ld, (float*)out, N));
-  else B2_CUDA_OK(b2_launch(sigmoid_gate_kernel<bf16>, grid, dim3(256), 0, s, a, gate, gate_ld, (bf16*)out, N));
+  if (out_ld <= 0) out_ld = N;
+  const bool vec = N % 4 == 0 && gate_ld % 4 == 0 && out_ld % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  const int per = vec ? 1024 : 256;
+  const dim3 grid(T, T >= 1024 ? 1 : std::max(1, std::min((N + per - 1) / per, 1024 / T)));
+  B2_REQUIRE(!(a_bf16 && out_f32), "sigmoid_gate: a bf16 input goes with bf16 operands");
+#define B2_SIGMOID_GATE(TA, TX)                                                                                                                            \
+  do {                                                                                                                                                     \
+    if (vec) B2_CUDA_OK(b2_launch(sigmoid_gate_kernel<TA, TX, true>, grid, dim3(256), 0, s, (const TA*)a, gate, gate_ld, (TX*)out, out_ld, scale, N));      \
+    else B2_CUDA_OK(b2_launch(sigmoid_gate_kernel<TA, TX, false>, grid, dim3(256), 0, s, (const TA*)a, gate, gate_ld, (TX*)out, out_ld, scale, N));         \
+  } while (0)
+  if (out_f32) B2_SIGMOID_GATE(float, float);
+  else if (a_bf16) B2_SIGMOID_GATE(bf16, bf16);
+  else B2_SIGMOID_GATE(float, bf16);
+#undef B2_SIGMOID_GATE
+  return 0;
+}
+
+int launch_embed_streams(const int32_t* ids, const void* table, int table_f32, const float* gain, float* h, int n, int T, int W, int vocab, float eps,
+                         cudaStream_t s) {
+  if (T <= 0) return 0;
+  if (table_f32) B2_CUDA_OK(b2_launch(embed_streams_kernel<float>, dim3(T), dim3(256), 0, s, ids, (const float*)table, gain, h, n, W, vocab, eps));
+  else B2_CUDA_OK(b2_launch(embed_streams_kernel<bf16>, dim3(T), dim3(256), 0, s, ids, (const bf16*)table, gain, h, n, W, vocab, eps));
+  return 0;
+}
+
+int launch_streams_step(float* h, int n, const StreamMix* cur, const StreamBranch& br, const float* next_in, const float* gain, void* x, int x_f32, int T,
+                        int W, float eps, const int32_t* rows, cudaStream_t s) {
+  if (T <= 0) return 0;
+  B2_REQUIRE(n >= 1 && n <= STREAMS_MAX, "streams_step: %d streams (1 to %d)", n, STREAMS_MAX);
+  B2_REQUIRE(br.y == nullptr || (br.weight != nullptr && br.pair_slot != nullptr && br.top >= 1), "streams_step: routed rows need their weights and slots");
+  B2_REQUIRE(x == nullptr || gain != nullptr, "streams_step: the norm needs its gain");
+  B2_REQUIRE(rows == nullptr || cur == nullptr, "streams_step: selected rows are only read");
+  const StreamsArgs p{h, cur ? cur->out : nullptr, cur ? cur->mix : nullptr, next_in, br, gain, W, eps, rows};
+  return x_f32 ? streams_step_typed<float>(p, n, (float*)x, T, s) : streams_step_typed<bf16>(p, n, (bf16*)x, T, s);
+}
+
+int launch_streams_sum(const float* h, int n, float* out, int T, int W, cudaStream_t s) {
+  if (T <= 0) return 0;
+  B2_CUDA_OK(b2_launch(streams_sum_kernel, dim3(T), dim3(256), 0, s, h, n, out, W));
+  return 0;
+}
+
+int launch_token_shift(const void* x, int x_f32, const float* mu, void* ring, void* out, int T, int W, const int32_t* row_seq, const int32_t* row_first,
+                       const int32_t* row_end, const int32_t* positions, const int32_t* slots, cudaStream_t s) {
+  if (T <= 0) return 0;
+  const bool vec = W % 4 == 0;
+  const int per = vec ? 1024 : 256;
+  const dim3 grid(T, T >= 1024 ? 1 : std::max(1, std::min((W + per - 1) / per, 1024 / T)));
+#define B2_TOKEN_SHIFT(TX, V)                                                                                                                            \
+  B2_CUDA_OK(b2_launch(token_shift_kernel<TX, V>, grid, dim3(256), 0, s, (const TX*)x, mu, (TX*)ring, (TX*)out, T, W, row_seq, row_first, row_end, positions, \
+                       slots))
+  if (x_f32 && vec) B2_TOKEN_SHIFT(float, true);
+  else if (x_f32) B2_TOKEN_SHIFT(float, false);
+  else if (vec) B2_TOKEN_SHIFT(bf16, true);
+  else B2_TOKEN_SHIFT(bf16, false);
+#undef B2_TOKEN_SHIFT
   return 0;
 }
 

@@ -133,7 +133,8 @@ static bool is_file(const std::string& p) { struct stat st; return stat(p.c_str(
 
 // families whose config lists the layers one by one (they have an fp32 path)
 static bool has_layer_list(const b2_config& c) {
-  return c.arch == B2_ARCH_LERASUN || c.arch == B2_ARCH_KEDASUN || c.arch == B2_ARCH_BUMALIX || c.arch == B2_ARCH_TINEVIK || c.arch == B2_ARCH_TOLANEX;
+  return c.arch == B2_ARCH_LERASUN || c.arch == B2_ARCH_KEDASUN || c.arch == B2_ARCH_BUMALIX || c.arch == B2_ARCH_TINEVIK || c.arch == B2_ARCH_TOLANEX ||
+         c.arch == B2_ARCH_RESITAR;
 }
 
 static void fill_config(const Options& o, b2_config& c) {

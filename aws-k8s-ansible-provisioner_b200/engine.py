@@ -37,7 +37,7 @@ class EngineConfig:
     max_seqs: int = 64
     max_batch_tokens: int = 8192
     use_cuda_graphs: bool = True
-    arch: str = "qwen3"          # "qwen3" | "phi3" | "opt" | "lerasun" | "kedasun" | "bumalix" | "tinevik" | "tolanex" (include/b2_engine.h, enum b2_arch)
+    arch: str = "qwen3"          # "qwen3" | "phi3" | "opt" | "lerasun" | "kedasun" | "bumalix" | "tinevik" | "tolanex" | "resitar" (include/b2_engine.h, enum b2_arch)
     rotary_dim: int = 0          # 0 = head_dim
     max_positions: int = 0       # OPT: learned position table rows - 2 (0 = max_model_len); Tolanex: rows
     sliding_window: int = 0      # Phi-3: attend to the last N keys only (0 = all)
@@ -51,6 +51,7 @@ class EngineConfig:
     norm_kind: int = 0           # 1: layer norms with gain and bias around every sublayer (Tinevik); 2: RMS norms behind the sublayers only (Tolanex)
     residual_mult: float = 0.0   # Tolanex: factor on a sublayer's normed output (0 = 1)
     bigram: tuple = (0, 0, 0)    # Tolanex: (buckets, mul_prev, mul_cur) of the bigram table
+    streams: int = 0             # Resitar: residual streams (0 = one plain stream)
 
     @staticmethod
     def lerasun(model_cfg: dict, **runtime) -> "EngineConfig":
@@ -98,6 +99,15 @@ class EngineConfig:
                             max_positions=int(model_cfg["max_positions"]), residual_mult=float(model_cfg.get("residual_mult", 1.0)),
                             bigram=(int(bg["buckets"]), int(bg["mul_prev"]), int(bg["mul_cur"])), **runtime)
 
+    @staticmethod
+    def resitar(model_cfg: dict, **runtime) -> "EngineConfig":
+        """From the dict a Resitar config.json holds (width, vocab, streams, norm.eps, loop, layers) plus runtime sizing."""
+        lp = model_cfg.get("loop") or {}
+        return EngineConfig(num_layers=len(model_cfg["layers"]), hidden=model_cfg["width"], vocab=model_cfg["vocab"],
+                            rms_eps=model_cfg["norm"]["eps"], embed_scale=1.0, logit_scale=1.0, arch="resitar", layers=model_cfg["layers"],
+                            tie_embeddings=True, num_q_heads=0, num_kv_heads=0, head_dim=0, intermediate=0, streams=int(model_cfg["streams"]),
+                            loop=(int(lp.get("start", 0)), int(lp.get("stop", 0)), int(lp.get("times", 0))), **runtime)
+
     def kv_bytes_per_token(self) -> int:
         return 2 * self.num_layers * self.num_kv_heads * self.head_dim * 2
 
@@ -137,7 +147,8 @@ class Engine:
         c.gpu_mem_fraction = cfg.gpu_mem_fraction
         c.arch = {"qwen3": capi.ARCH_QWEN3, "phi3": capi.ARCH_PHI3, "opt": capi.ARCH_OPT, "lerasun": capi.ARCH_LERASUN,
                   "kedasun": capi.ARCH_KEDASUN, "bumalix": capi.ARCH_BUMALIX, "tinevik": capi.ARCH_TINEVIK,
-                  "tolanex": capi.ARCH_TOLANEX}[cfg.arch]
+                  "tolanex": capi.ARCH_TOLANEX, "resitar": capi.ARCH_RESITAR}[cfg.arch]
+        c.streams = int(cfg.streams)
         c.norm_kind = int(cfg.norm_kind)
         c.loop_start, c.loop_stop, c.loop_times = (int(v) for v in cfg.loop)
         c.logit_softcap = float(cfg.logit_softcap)
@@ -179,9 +190,9 @@ class Engine:
         check(lib.b2_config_from_dir(model_dir.encode(), C.byref(c), specs, 1024), lib)
         arch = {capi.ARCH_QWEN3: "qwen3", capi.ARCH_PHI3: "phi3", capi.ARCH_OPT: "opt", capi.ARCH_LERASUN: "lerasun",
                 capi.ARCH_KEDASUN: "kedasun", capi.ARCH_BUMALIX: "bumalix", capi.ARCH_TINEVIK: "tinevik",
-                capi.ARCH_TOLANEX: "tolanex"}[c.arch]
+                capi.ARCH_TOLANEX: "tolanex", capi.ARCH_RESITAR: "resitar"}[c.arch]
         layers = None
-        if arch in ("lerasun", "kedasun", "bumalix", "tinevik", "tolanex"):
+        if arch in ("lerasun", "kedasun", "bumalix", "tinevik", "tolanex", "resitar"):
             layers = [_layer_dict(specs[i], arch) for i in range(c.num_layers)]
         cfg = EngineConfig(num_layers=c.num_layers, hidden=c.hidden, num_q_heads=c.num_q_heads, num_kv_heads=c.num_kv_heads,
                            head_dim=c.head_dim, intermediate=c.intermediate, vocab=c.vocab, tie_embeddings=bool(c.tie_embeddings),
@@ -190,7 +201,7 @@ class Engine:
                            compute_f32=(dtype == "float32"), logit_scale=c.logit_scale, embed_scale=c.embed_scale,
                            norm_groups=c.norm_groups, loop=(c.loop_start, c.loop_stop, c.loop_times), logit_softcap=c.logit_softcap,
                            norm_kind=c.norm_kind, residual_mult=c.residual_mult,
-                           bigram=(c.bigram_buckets, c.bigram_mul_prev, c.bigram_mul_cur), **runtime)
+                           bigram=(c.bigram_buckets, c.bigram_mul_prev, c.bigram_mul_cur), streams=c.streams, **runtime)
         return cls(cfg, device=device, safetensors_path=os.path.join(model_dir, "model.safetensors"))
 
     # ---- weights -----------------------------------------------------------------------
@@ -369,6 +380,8 @@ def _fill_layer_spec(sp, layer: dict) -> None:
     """One "layers" entry of a layer-list config.json -> b2_layer_spec (the C registry does the same for a directory)."""
     if layer.get("_family") == "tolanex":
         return _fill_outnorm_spec(sp, layer)
+    if layer.get("_family") == "resitar":
+        return _fill_streams_spec(sp, layer)
     if layer["type"] == "gla" or layer["mixer"].get("q_rank") is not None or (layer["type"] == "attention" and layer.get("_family") == "tinevik"):
         return _fill_mixed_spec(sp, layer)
     if layer["type"] in ("attention", "attention_2"):
@@ -496,6 +509,67 @@ def _outnorm_layer_dict(sp) -> dict:
     return {"type": "delta" if sp.mixer == capi.MIXER_HEAD_DELTA else "latent_attention", "mixer": m, "mlp": mlp}
 
 
+def _fill_streams_spec(sp, layer: dict) -> None:
+    """Resitar: "parallel" (chunked attention whose values are its keys, beside a state-space recurrence) and "parallel_2" (full attention
+    beside time mixing)."""
+    m = layer["mixer"]
+    a, b = m["left"], m["right"]
+    if layer["type"] not in ("parallel", "parallel_2"):
+        raise B2Error("mixer type %r not built" % layer["type"])
+    ssm = layer["type"] == "parallel"
+    sp.kv_from = sp.weights_of = -1
+    sp.mixer = capi.MIXER_CHUNK_AND_SSM if ssm else capi.MIXER_FULL_AND_TIMEMIX
+    sp.mix_left, sp.mix_right = float(m.get("left_scale", 1.0)), float(m.get("right_scale", 1.0))
+    sp.heads, sp.kv_heads = int(a["heads"]), int(a.get("kv_heads", a["heads"]))
+    sp.dim, sp.vdim, sp.scale = int(a["dim"]), int(a.get("vdim", a["dim"])), float(a["scale"])
+    sp.rot_halves, sp.rot_factor = int(ssm), 1.0
+    rot = a.get("rot")
+    if rot:
+        sp.rot_base, sp.rot_dims = float(rot["base"]), int(rot["dims"])
+        sc = rot.get("scaling")
+        if sc:
+            sp.rot_factor, sp.rot_orig, sp.rot_fast, sp.rot_slow = float(sc["factor"]), int(sc["original"]), float(sc["fast"]), float(sc["slow"])
+    sp.chunk = int(a["mask"]["size"]) if a.get("mask") else 0
+    sp.s_heads = int(b["heads"])
+    if ssm:
+        sp.s_vdim, sp.s_dim, sp.conv_taps = int(b["vdim"]), int(b["state"]), int(b["conv"])
+        sp.s_groups, sp.s_norm_groups = int(b.get("groups", 1)), int(b.get("norm_groups", 1))
+    else:
+        sp.s_dim = sp.s_vdim = int(b["dim"])
+    mlp = layer.get("mlp")
+    sp.ff = capi.FF_NONE
+    if mlp is not None:
+        if mlp["kind"] == "dense":
+            sp.ff, sp.ff_dim = capi.FF_SWIGLU, int(mlp["ff"])
+        elif mlp["kind"] == "moe":
+            sp.ff, sp.ff_dim = capi.FF_TOP_SOFTMAX_EXPERTS, int(mlp["expert"]["ff"])
+            sp.experts, sp.top, sp.groups, sp.groups_keep = int(mlp["router"]["experts"]), int(mlp["router"]["top"]), 1, 1
+        else:
+            raise B2Error("feed-forward kind %r not built" % mlp["kind"])
+
+
+def _streams_layer_dict(sp) -> dict:
+    ssm = sp.mixer == capi.MIXER_CHUNK_AND_SSM
+    left = {"heads": sp.heads, "kv_heads": sp.kv_heads, "dim": sp.dim, "vdim": sp.vdim, "scale": sp.scale}
+    if sp.rot_dims > 0:
+        left["rot"] = {"base": sp.rot_base, "dims": sp.rot_dims}
+        if sp.rot_orig > 0:
+            left["rot"]["scaling"] = {"factor": sp.rot_factor, "original": sp.rot_orig, "fast": sp.rot_fast, "slow": sp.rot_slow}
+    if sp.chunk > 0:
+        left["mask"] = {"size": sp.chunk}
+    if ssm:
+        right = {"heads": sp.s_heads, "vdim": sp.s_vdim, "state": sp.s_dim, "conv": sp.conv_taps, "groups": sp.s_groups, "norm_groups": sp.s_norm_groups}
+    else:
+        right = {"heads": sp.s_heads, "dim": sp.s_dim}
+    mlp = None
+    if sp.ff == capi.FF_SWIGLU:
+        mlp = {"kind": "dense", "ff": sp.ff_dim}
+    elif sp.ff == capi.FF_TOP_SOFTMAX_EXPERTS:
+        mlp = {"kind": "moe", "expert": {"ff": sp.ff_dim}, "router": {"experts": sp.experts, "top": sp.top}}
+    return {"type": "parallel" if ssm else "parallel_2", "mixer": {"left": left, "right": right, "left_scale": sp.mix_left, "right_scale": sp.mix_right},
+            "mlp": mlp}
+
+
 def _fill_state_spec(sp, layer: dict) -> None:
     """Bumalix: "parallel" (windowed softmax attention beside gated linear attention) and "channel_delta" (gated delta rule)."""
     m = layer["mixer"]
@@ -551,6 +625,8 @@ def _fill_heads_spec(sp, layer: dict) -> None:
 def _layer_dict(sp, arch: str = "") -> dict:
     if arch == "tolanex":
         return _outnorm_layer_dict(sp)
+    if arch == "resitar":
+        return _streams_layer_dict(sp)
     if sp.mixer in (capi.MIXER_DECAY_STATE, capi.MIXER_MIXED_SCORE_ATTENTION, capi.MIXER_GATED_LATENT):
         return _mixed_layer_dict(sp)
     if sp.mixer in (capi.MIXER_WINDOW_AND_STATE, capi.MIXER_DELTA_STATE):

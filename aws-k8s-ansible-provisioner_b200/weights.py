@@ -340,6 +340,78 @@ def tolanex_random_state_dict(model_cfg: dict, seed: int = 0) -> dict[str, torch
     return sd
 
 
+def resitar_tensor_shapes(model_cfg: dict, rank: int = 32) -> dict[str, tuple[int, ...]]:
+    """Tensor names and shapes of a Resitar checkpoint for the dict its config.json holds.  The width of the time mixing's low-rank stage (w1) is
+    not in the config -- a checkpoint's tensors carry it -- so it is an argument here."""
+    W, V, n = model_cfg["width"], model_cfg["vocab"], model_cfg["streams"]
+    s: dict[str, tuple[int, ...]] = {"embed": (V, W), "embed.norm": (W,)}
+    for i, layer in enumerate(model_cfg["layers"]):
+        a, b, mlp, p = layer["mixer"]["left"], layer["mixer"]["right"], layer.get("mlp"), f"l{i}."
+        l, r, ssm = p + "mix.left.", p + "mix.right.", layer["type"] == "parallel"
+        H, G, D = a["heads"], a.get("kv_heads", a["heads"]), a["dim"]
+        Dv = a.get("vdim", D)
+        s[p + "norm1"] = (W,)
+        for nm, c in (("q", H * D), ("k", G * D)) + (() if ssm else (("v", G * Dv),)):
+            s[l + nm], s[l + nm + ".b"] = (c, W), (c,)
+        s[l + "g"], s[l + "o"] = (H * Dv, W), (W, H * Dv)
+        if ssm:
+            s[l + "o.b"] = (W,)
+            inner, bc = b["heads"] * b["vdim"], b.get("groups", 1) * b["state"]
+            s[r + "in"], s[r + "conv"], s[r + "conv.b"] = (2 * inner + 2 * bc + b["heads"], W), (inner + 2 * bc, b["conv"]), (inner + 2 * bc,)
+            s[r + "dt_bias"], s[r + "A_log"], s[r + "D"] = (b["heads"],), (b["heads"],), (b["heads"],)
+            s[r + "norm"], s[r + "o"] = (inner,), (W, inner)
+        else:
+            HD = b["heads"] * b["dim"]
+            for nm in "rkvgw":
+                s[r + "mu." + nm] = (W,)
+            for nm in "rkvg":
+                s[r + nm] = (HD, W)
+            s[r + "w1"], s[r + "w2"], s[r + "w0"], s[r + "u"] = (rank, W), (HD, rank), (HD,), (b["heads"], b["dim"])
+            s[r + "norm"], s[r + "o"] = (HD,), (W, HD)
+        if mlp is not None:
+            f = p + "mlp."
+            s[p + "norm2"] = (W,)
+            if mlp["kind"] == "dense":
+                s[f + "gate"], s[f + "up"], s[f + "down"] = (mlp["ff"], W), (mlp["ff"], W), (W, mlp["ff"])
+            else:
+                F, E = mlp["expert"]["ff"], mlp["router"]["experts"]
+                s[f + "router"], s[f + "router.b"] = (E, W), (E,)
+                for e in range(E):
+                    s[f"{f}e{e}.gate"], s[f"{f}e{e}.up"], s[f"{f}e{e}.down"] = (F, W), (F, W), (W, F)
+        for q in ("hc1.", "hc2.") if mlp is not None else ("hc1.",):
+            s[p + q + "in"], s[p + q + "out"], s[p + q + "mix"] = (n,), (n,), (n, n)
+    s["final.norm"] = (W,)
+    return s
+
+
+def resitar_random_state_dict(model_cfg: dict, seed: int = 0, rank: int = 32) -> dict[str, torch.Tensor]:
+    """Random bf16 weights scaled by 1/sqrt(fan-in), gains around one, stream mixes near the identity, decays that forget over tens to hundreds of
+    tokens."""
+    g = torch.Generator().manual_seed(seed)
+    sd, n = {}, model_cfg["streams"]
+    for name, shape in resitar_tensor_shapes(model_cfg, rank).items():
+        last = name.rsplit(".", 1)[-1]
+        t = torch.randn(shape, generator=g)
+        if "norm" in name:
+            t = 1.0 + 0.1 * t
+        elif ".hc" in name:
+            t = 0.1 * t + (1.0 / n if last == "in" else 1.0 if last == "out" else 0.9 * torch.eye(n))
+        elif ".mu." in name:
+            t = torch.rand(shape, generator=g)
+        elif last == "A_log":
+            t = torch.log(0.5 + 2.0 * torch.rand(shape, generator=g))
+        elif last in ("dt_bias", "w0"):
+            t = t - 3.0
+        elif last == "b":
+            t = 0.1 * t
+        elif last in ("conv", "u"):
+            t = 0.5 * t
+        elif last != "D":
+            t = t * (shape[-1] ** -0.5)
+        sd[name] = t.to(torch.bfloat16)
+    return sd
+
+
 def write_model_dir(model_cfg: dict, sd: dict[str, torch.Tensor], path: str) -> str:
     """config.json + model.safetensors of a layer-list model, as the registry and the loader read them."""
     import os

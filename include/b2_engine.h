@@ -25,7 +25,7 @@
 extern "C" {
 #endif
 
-#define B2_ABI_VERSION 7
+#define B2_ABI_VERSION 8
 
 typedef struct b2_engine b2_engine;
 
@@ -54,8 +54,17 @@ enum b2_mixer_kind {
                                     all of vdim and the weighted sum turned back by the query's (Tinevik "attention") */
   B2_MIXER_GATED_LATENT = 8,     /* attention over a per-token latent with no rotated piece: the query itself goes through a normed latent of
                                     q_rank entries, a sliding window, a sigmoid gate on the concatenated heads (Tinevik "latent_attention") */
-  B2_MIXER_HEAD_DELTA = 9        /* gated delta rule with ONE decay per head: short causal convolutions on q / k / v, unit-vector q and k, a step size
+  B2_MIXER_HEAD_DELTA = 9,       /* gated delta rule with ONE decay per head: short causal convolutions on q / k / v, unit-vector q and k, a step size
                                     and a decay per head straight from the layer's input, a silu gate as wide as the values (Tolanex "delta") */
+  B2_MIXER_CHUNK_AND_SSM = 10,   /* two mixers side by side on the same input, mix_left * left + mix_right * right (Resitar "parallel").  Left: grouped-query
+                                    softmax attention inside chunks counted from position 0 (chunk), biased q and k, rotary positions on half-split pairs,
+                                    a token's value is its key before the rotation, a sigmoid gate as wide as the concatenated heads, a biased output
+                                    projection.  Right: a state-space recurrence with one decay per head (s_heads, s_dim = state size, s_vdim, s_groups
+                                    input / read-out vectors, conv_taps, s_norm_groups pieces of its gated norm) */
+  B2_MIXER_FULL_AND_TIMEMIX = 11 /* the same around other halves (Resitar "parallel_2").  Left: grouped-query causal softmax attention, biased q, k and v,
+                                    rotary positions on interleaved pairs with wavelength-dependent scaling of the frequencies (rot_orig, rot_fast,
+                                    rot_slow, rot_factor), the same gate, no output bias.  Right: time mixing: five blends of the input with the previous
+                                    token's, a matrix state per head (s_heads, s_dim) with a decay per key channel and a bonus for the current token */
 };
 enum b2_ff_kind {
   B2_FF_NONE = 0,
@@ -67,9 +76,11 @@ enum b2_ff_kind {
   B2_FF_XIELU = 5,               /* W_d a(W_u x), a(z) = softplus(p) z^2 + z / 2 for z > 0, (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 otherwise */
   B2_FF_TABLE_EXPERTS = 6,       /* experts of the B2_FF_CLAMPED_GATED form; an integer table row per token id names the token's `top` experts,
                                     each weighted 1 / top (no router) */
-  B2_FF_SOFTMAX_EXPERTS = 7      /* softmax router over all experts, groups ranked by their best score (groups, groups_keep), the `top` largest of the kept
+  B2_FF_SOFTMAX_EXPERTS = 7,     /* softmax router over all experts, groups ranked by their best score (groups, groups_keep), the `top` largest of the kept
                                     groups weighted by score * router_scale (not renormalised) on their OUTPUT; expert = W_d (silu(W_g x) * (W_u x)); a
                                     shared expert of the same form (shared_ff) times sigmoid(w_sg . x) is added */
+  B2_FF_SWIGLU = 8,              /* W_d (silu(W_g x) * (W_u x)) */
+  B2_FF_TOP_SOFTMAX_EXPERTS = 9  /* experts of that form: the `top` largest biased router logits, weighted by the softmax over the chosen logits */
 };
 typedef struct b2_layer_spec {
   int32_t mixer;        /* b2_mixer_kind */
@@ -112,6 +123,18 @@ typedef struct b2_layer_spec {
   int32_t rot_values;   /* 1: values are rotated by their position over all of vdim and the output turned back */
   /* ABI 7 */
   float   router_scale; /* B2_FF_SOFTMAX_EXPERTS: factor on the chosen scores (0 = 1) */
+  /* ABI 8: two mixers side by side (B2_MIXER_CHUNK_AND_SSM, B2_MIXER_FULL_AND_TIMEMIX) */
+  float   mix_left;     /* factors of the two mixers' outputs */
+  float   mix_right;
+  int32_t chunk;        /* > 0: query i sees key j only when floor(i / chunk) = floor(j / chunk) */
+  int32_t s_groups;     /* groups of heads that share the recurrence's input and read-out vectors */
+  int32_t s_norm_groups;/* equal pieces of the gated norm behind the recurrence */
+  int32_t rot_halves;   /* 1: rotary pairs (i, i + rot_dims/2); 0: (2i, 2i + 1) */
+  int32_t rot_orig;     /* > 0: wavelength-dependent scaling of the rotary frequencies by rot_factor: pairs that turn more than rot_fast times over
+                           rot_orig positions keep theirs, pairs that turn less than rot_slow times are divided, a ramp between; cosines and sines
+                           are multiplied by 0.1 ln(rot_factor) + 1 */
+  float   rot_fast;
+  float   rot_slow;
 } b2_layer_spec;
 
 /* Architecture + runtime sizing.  Field meanings follow HF Qwen3Config
@@ -165,6 +188,8 @@ typedef struct b2_config {
                                 bigram_buckets + 1 rows joins the embedding; a sequence's first token takes the last row */
   int64_t bigram_mul_prev;
   int64_t bigram_mul_cur;
+  /* ABI 8 (Resitar) */
+  int32_t streams;           /* residual streams that every sublayer reads from and writes to by learned mixes (0 = one plain stream) */
 } b2_config;
 
 /* Model families.  QWEN3: HF:models/qwen3/modeling_qwen3.py (QK-norm, separate q/k/v and gate/up
@@ -204,12 +229,20 @@ typedef struct b2_config {
  * B2_FF_SOFTMAX_EXPERTS or none.  Per-sequence state: the matrix states, the convolutions' last inputs and the previous token.  Tensor names: embed,
  * bigram, pos, l<i>.norm1|norm2, l<i>.mix.{q,k,v (+ .conv), b, a, A_log, dt_bias, norm, g, o} (delta), l<i>.mix.{q,dkv,dkv.norm,uk,uv,o}
  * (latent_attention; no dkv with kv_from), l<i>.mlp.{router, e<k>.{gate,up,down}, shared.{gate,up,down,sg}}, final.norm, head. */
+/* RESITAR: a layer list as well.  The embedding row is RMS-normed with a gain; `streams` copies of the residual stream start as it.  A sublayer
+ * (mixer, then feed-forward) reads u = sum_s in[s] x_s through a plain-gain RMS norm, and all streams follow at once from the old ones,
+ * x_t <- sum_s mix[s][t] x_s + out[t] y; at the end x is their sum, and the embedding table is the head (tie_embeddings).  An optional loop over a
+ * run of layers (loop_*, no input mix).  Mixers: B2_MIXER_CHUNK_AND_SSM, B2_MIXER_FULL_AND_TIMEMIX; feed-forwards: B2_FF_SWIGLU,
+ * B2_FF_TOP_SOFTMAX_EXPERTS or none.  Per-sequence state: matrix states, convolution inputs, the previous token's mixer input.  Tensor names: embed,
+ * embed.norm, l<i>.norm1|norm2, l<i>.hc1|hc2.{in,out,mix}, l<i>.mix.left.{q,k,v (+ .b), g, o (+ .b)}, l<i>.mix.right.{in, conv (+ .b), dt_bias, A_log, D,
+ * norm, o} (parallel) or l<i>.mix.right.{mu.{r,k,v,g,w}, r, k, v, g, w1, w2, w0, u, norm, o} (parallel_2), l<i>.mlp.{gate,up,down} or l<i>.mlp.{router (+
+ * .b), e<k>.{gate,up,down}}, final.norm.  The width of the decay's low-rank stage (w1) is taken from the tensors. */
 enum b2_arch { B2_ARCH_QWEN3 = 0, B2_ARCH_PHI3 = 1, B2_ARCH_OPT = 2, B2_ARCH_LERASUN = 3, B2_ARCH_KEDASUN = 4, B2_ARCH_BUMALIX = 5, B2_ARCH_TINEVIK = 6,
-               B2_ARCH_TOLANEX = 7 };
+               B2_ARCH_TOLANEX = 7, B2_ARCH_RESITAR = 8 };
 
 /* Model registry: reads MODEL_DIR/config.json and fills the architecture fields of *cfg (the runtime sizing fields --
  * max_model_len, block_size, num_blocks, max_seqs, max_batch_tokens, use_cuda_graphs, compute_f32 -- are left as the caller
- * set them).  HF configs are told apart by "model_type" (qwen3, phi3, opt); a config with "architecture": "Lerasun", "Kedasun", "Bumalix", "Tinevik" or "Tolanex" fills
+ * set them).  HF configs are told apart by "model_type" (qwen3, phi3, opt); a config with "architecture": "Lerasun", "Kedasun", "Bumalix", "Tinevik", "Tolanex" or "Resitar" fills
  * specs[0 .. num_layers) as well and points cfg->layer_specs at it (max_specs = capacity of specs; may be 0 / NULL for the
  * HF families).  Returns 0, or a negative code with b2_last_error(). */
 int  b2_config_from_dir(const char* model_dir, b2_config* cfg, b2_layer_spec* specs, int32_t max_specs);
