@@ -511,8 +511,32 @@ def tolanex_model_cfg(width, heads, inter, vocab=32000):
             "embedding": {"bigram": {"buckets": 30011, "mul_prev": 8191, "mul_cur": 31}}, "layers": ls}
 
 
+# ---- --family resitar: width, heads (128 wide, two per kv head), Qwen3's feed-forward width.  Four layers on two residual streams: full attention with scaled
+#      rotary frequencies beside time mixing (heads of 64), attention in chunks of 512 on its own keys beside a state-space recurrence (inner width = width,
+#      heads of 64, state 128, two groups), and both again; a dense feed-forward of Qwen3's width behind the first and last, 16 experts (two per token, Qwen3's
+#      active count) behind the others; vocab 32000.  The closest existing families are Bumalix (two mixers side by side, matrix states) and Tolanex (softmax
+#      router, gated experts); both run beside it at the same sizes.
+def resitar_model_cfg(width, heads, inter, vocab=32000):
+    full = {"left": {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                     "rot": {"base": 10000.0, "dims": 128, "scaling": {"factor": 8.0, "original": 512, "fast": 32.0, "slow": 1.0}}},
+            "right": {"heads": width // 64, "dim": 64}, "left_scale": 0.7, "right_scale": 0.6}
+    chunk = {"left": {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 512}, "rot": {"base": 10000.0, "dims": 64}},
+             "right": {"heads": width // 64, "vdim": 64, "state": 128, "groups": 2, "conv": 4, "norm_groups": 2}, "left_scale": 0.7, "right_scale": 0.6}
+    dense = {"kind": "dense", "ff": inter}
+    moe = {"kind": "moe", "expert": {"ff": (inter // 2 + 63) // 64 * 64}, "router": {"experts": 16, "top": 2}}
+    ls = [{"type": "parallel_2", "mixer": full, "mlp": dense}, {"type": "parallel", "mixer": chunk, "mlp": moe},
+          {"type": "parallel_2", "mixer": full, "mlp": moe}, {"type": "parallel", "mixer": chunk, "mlp": dense}]
+    return {"architecture": "Resitar", "vocab": vocab, "width": width, "streams": 2, "norm": {"eps": 1e-6}, "layers": ls}
+
+
 def family_models(pkg, weights, family, tag):
     """(name, engine configuration, state-dict maker) of the family's model and of Qwen3 at the same width, depth, heads and feed-forward size."""
+    if family == "resitar":
+        width, heads, inter = BUMALIX_SIZES[tag]
+        mc = resitar_model_cfg(width, heads, inter)
+        beside = {m[0]: m for m in family_models(pkg, weights, "tolanex", tag)}
+        return [("resitar", pkg.EngineConfig.resitar(mc), lambda c: weights.resitar_random_state_dict(mc, seed=0, rank=64))] + [
+            beside[k] for k in ("bumalix", "tolanex", "qwen3")]
     if family == "tolanex":
         width, heads, inter = BUMALIX_SIZES[tag]
         mc = tolanex_model_cfg(width, heads, inter)
@@ -545,7 +569,7 @@ def family_models(pkg, weights, family, tag):
 
 
 def run_family(args, local):
-    """Prefill and decode throughput of a layer-list family (Lerasun, Kedasun, Bumalix, Tinevik, Tolanex) at layer sizes of real models (random weights), and of
+    """Prefill and decode throughput of a layer-list family (Lerasun, Kedasun, Bumalix, Tinevik, Tolanex, Resitar) at layer sizes of real models (random weights), and of
     Qwen3 at the same width, depth, head count and (active) feed-forward size: one JSON line per size and model, with the decode step's
     per-kernel-class times (CUDA events around every launch of an eager step)."""
     import torch
@@ -600,7 +624,7 @@ def main():
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--value-only", action="store_true", help="device-resident timing only (ablation runs)")
-    ap.add_argument("--family", default="", choices=["", "lerasun", "kedasun", "bumalix", "tinevik", "tolanex"],
+    ap.add_argument("--family", default="", choices=["", "lerasun", "kedasun", "bumalix", "tinevik", "tolanex", "resitar"],
                     help="instead of the headline workload: the named family beside the closest GQA model at equal size (one GPU)")
     ap.add_argument("--family-sizes", default="w1024,w2048,w4096")
     ap.add_argument("--family-only", default="", help="time only the named model of the pair (the family's name, or qwen3)")

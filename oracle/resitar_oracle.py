@@ -78,13 +78,13 @@ def frequencies(rot: dict):
 
 
 def rotate(x: torch.Tensor, pos: int, rot: dict, halves: bool) -> torch.Tensor:
-    """x [dim]; the first rot["dims"] entries turn, half-split or interleaved pairs."""
+    """x [heads, dim]; the first rot["dims"] entries of every head turn, half-split or interleaved pairs."""
     f, mul = frequencies(rot)
+    ang = torch.tensor([pos * fi for fi in f], dtype=torch.float64)
+    c, s = (torch.cos(ang) * mul).to(x.dtype), (torch.sin(ang) * mul).to(x.dtype)
     half, y = len(f), x.clone()
-    for i in range(half):
-        a, b = (i, i + half) if halves else (2 * i, 2 * i + 1)
-        c, s = math.cos(pos * f[i]) * mul, math.sin(pos * f[i]) * mul
-        y[a], y[b] = x[a] * c - x[b] * s, x[b] * c + x[a] * s
+    ia, ib = (slice(0, half), slice(half, 2 * half)) if halves else (slice(0, 2 * half, 2), slice(1, 2 * half, 2))
+    y[:, ia], y[:, ib] = x[:, ia] * c - x[:, ib] * s, x[:, ib] * c + x[:, ia] * s
     return y
 
 
@@ -158,8 +158,7 @@ class Stepper:
         k = (w[p + "k"] @ h + w[p + "k.b"]).reshape(G, D)
         v = k if halves else (w[p + "v"] @ h + w[p + "v.b"]).reshape(G, m["vdim"])
         if m.get("rot"):
-            q = torch.stack([rotate(x, self.pos, m["rot"], halves) for x in q])
-            k = torch.stack([rotate(x, self.pos, m["rot"], halves) for x in k])
+            q, k = rotate(q, self.pos, m["rot"], halves), rotate(k, self.pos, m["rot"], halves)
         st["k"] = torch.cat([st["k"], k[None]]) if "k" in st else k[None]
         st["v"] = torch.cat([st["v"], v[None]]) if "v" in st else v[None]
         size = (m.get("mask") or {}).get("size", 0)
