@@ -21,7 +21,7 @@
 // Kernels:
 //   heads_finish      what follows the fused q | k | v (| gate) projection, one CTA per (token, head): bias, convolution, rotary or
 //                     unit-RMS norm, value mixing, cache row write, fp32 queries
-//   heads_finish_table  the same for rotary positions from a table (rot_table makes it), one CTA per token
+//   heads_finish_table  (heads_finish_table4: four numbers at a time) the same for rotary positions from a table (rot_table makes it), one CTA per token
 //   conv_tail_store   the ring update, after every token of the step has read the ring
 //   heads_attention   one warp per (query token, head) for prompt portions; for a decode step the eight warps of a CTA
 //                     split the keys of one (sequence, head) and merge.  Tiles of 32 keys: lane j scores key j, then lane
@@ -258,7 +258,7 @@ __global__ void __launch_bounds__(256) heads_finish_table_kernel(const float* __
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int slot = slots[t];
   if (slot < 0) return;   // padding row of a decode bucket
-  const int D = g.dim, half = g.rot_dims / 2, nq = g.heads * D, nk = g.kv_heads * D, nv = g.kv_heads * g.vdim;
+  const int D = g.dim, half = g.rot_dims / 2, nq = g.heads * D, nk = g.kv_heads * D;
   const int units = g.heads + (keys_as_values ? 1 : 2) * g.kv_heads, u_lo = blockIdx.y * upc, u_hi = min(units, u_lo + upc);
   const float* cs = table + (size_t)positions[t] * g.rot_dims;
   const float* row = proj + (size_t)t * ld;
@@ -295,7 +295,96 @@ __global__ void __launch_bounds__(256) heads_finish_table_kernel(const float* __
       if (!is_q && keys_as_values) put(v_cache, kh, D, i, a);
     }
   }
-  (void)nv;
+}
+
+// The same four numbers at a time: head widths and value widths in multiples of four, rot_dims in multiples of eight, rows on 16-byte boundaries.  blockIdx.y
+// splits a token's groups in short steps.
+__device__ __forceinline__ void put4(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void put4(bf16* p, const float* v) {
+  uint2 pk;
+  pk.x = pack_bf16x2(v[0], v[1]);
+  pk.y = pack_bf16x2(v[2], v[3]);
+  *reinterpret_cast<uint2*>(p) = pk;
+}
+template <typename TC>
+__global__ void __launch_bounds__(256) heads_finish_table4_kernel(const float* __restrict__ proj, int ld, HeadsGeom g, const float* __restrict__ bias,
+                                                                  const float* __restrict__ table, int halves, int keys_as_values,
+                                                                  const int32_t* __restrict__ positions, const int32_t* __restrict__ slots,
+                                                                  float* __restrict__ q_out, bf16* __restrict__ q_bf16, TC* __restrict__ k_cache,
+                                                                  TC* __restrict__ v_cache) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, slot = slots[t];
+  if (slot < 0) return;   // padding row of a decode bucket
+  const int D = g.dim, half = g.rot_dims / 2, nq = g.heads * D, nk = g.kv_heads * D;
+  const float* cs = table + (size_t)positions[t] * g.rot_dims;
+  const float* row = proj + (size_t)t * ld;
+  auto in4 = [&](int c, float* v) {
+    const float4 x = *reinterpret_cast<const float4*>(row + c);
+    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+    if (bias) {
+      const float4 b = *reinterpret_cast<const float4*>(bias + c);
+      v[0] += b.x; v[1] += b.y; v[2] += b.z; v[3] += b.w;
+    }
+  };
+  auto cache4 = [&](TC* cache, int kvh, int width, int d, const float* v) {
+    put4(g.swizzled ? cache + swizzled_index(slot, kvh, g.kv_heads, d) : cache + ((size_t)slot * g.kv_heads + kvh) * width + d, v);
+  };
+  // groups of a q or k head: half-split, the rotated ones hold four pairs (eight numbers); interleaved, two pairs
+  const int grot = halves ? half / 4 : half / 2, gh = grot + (D - g.rot_dims) / 4, nqk = (g.heads + g.kv_heads) * gh;
+  const int nvg = keys_as_values ? 0 : g.kv_heads * (g.vdim / 4), total = nqk + nvg;
+  for (int i = blockIdx.y * 256 + threadIdx.x; i < total; i += 256 * gridDim.y) {
+    if (i >= nqk) {
+      const int c = (i - nqk) * 4, vh = c / g.vdim;
+      float v[4];
+      in4(nq + nk + c, v);
+      cache4(v_cache, vh, g.vdim, c - vh * g.vdim, v);
+      continue;
+    }
+    const int u = i / gh, gi = i - u * gh, kh = u - g.heads;
+    const bool is_q = u < g.heads;
+    auto emit = [&](int d, const float* v) {
+      if (!is_q) cache4(k_cache, kh, D, d, v);
+      else if (q_bf16 != nullptr) put4(q_bf16 + (size_t)t * nq + u * D + d, v);
+      else put4(q_out + (size_t)t * nq + u * D + d, v);
+    };
+    if (gi >= grot) {
+      const int d = g.rot_dims + (gi - grot) * 4;
+      float v[4];
+      in4(u * D + d, v);
+      emit(d, v);
+      if (!is_q && keys_as_values) cache4(v_cache, kh, D, d, v);
+    } else if (halves) {
+      const int d = gi * 4;
+      float a[4], b[4], ra[4], rb[4];
+      in4(u * D + d, a);
+      in4(u * D + half + d, b);
+      const float4 c4 = *reinterpret_cast<const float4*>(cs + d), s4 = *reinterpret_cast<const float4*>(cs + half + d);
+      const float c[4] = {c4.x, c4.y, c4.z, c4.w}, s[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        ra[x] = a[x] * c[x] - b[x] * s[x];
+        rb[x] = b[x] * c[x] + a[x] * s[x];
+      }
+      emit(d, ra);
+      emit(half + d, rb);
+      if (!is_q && keys_as_values) {
+        cache4(v_cache, kh, D, d, a);
+        cache4(v_cache, kh, D, half + d, b);
+      }
+    } else {
+      const int d = gi * 4;
+      float v[4], r[4];
+      in4(u * D + d, v);
+      const float2 c2 = *reinterpret_cast<const float2*>(cs + gi * 2), s2 = *reinterpret_cast<const float2*>(cs + half + gi * 2);
+      r[0] = v[0] * c2.x - v[1] * s2.x;
+      r[1] = v[1] * c2.x + v[0] * s2.x;
+      r[2] = v[2] * c2.y - v[3] * s2.y;
+      r[3] = v[3] * c2.y + v[2] * s2.y;
+      emit(d, r);
+      if (!is_q && keys_as_values) cache4(v_cache, kh, D, d, v);
+    }
+  }
 }
 
 __global__ void __launch_bounds__(128) rot_table_kernel(const double* __restrict__ freqs, int half, double mul, float* __restrict__ table) {
@@ -1746,6 +1835,18 @@ int launch_heads_finish_table(const float* proj, int ld, const HeadsGeom& g, con
   B2_REQUIRE(g.rot_dims == 0 || table != nullptr, "heads_finish_table: rotary positions need their table");
   B2_REQUIRE(!keys_as_values || g.dim == g.vdim, "heads_finish_table: keys that serve as values need dim == vdim (%d, %d)", g.dim, g.vdim);
   B2_REQUIRE(!g.swizzled || (!cache_f32 && q_bf16 != nullptr && g.dim == 128 && g.vdim == 128), "heads_finish_table: the GQA page layout holds 128-wide bf16 heads");
+  if (g.dim % 4 == 0 && g.vdim % 4 == 0 && g.rot_dims % 8 == 0 && ld % 4 == 0 &&
+      ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(bias) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15) == 0) {
+    const int groups = ((g.heads + g.kv_heads) * g.dim + g.kv_heads * g.vdim) / 4;
+    const dim3 grid4(T, T >= 256 ? 1 : std::max(1, (groups + 255) / 256));
+    if (cache_f32)
+      B2_CUDA_OK(b2_launch(heads_finish_table4_kernel<float>, grid4, dim3(256), 0, s, proj, ld, g, bias, table, halves, keys_as_values, positions, slots, q_out, q_bf16,
+                           (float*)k_cache, (float*)v_cache));
+    else
+      B2_CUDA_OK(b2_launch(heads_finish_table4_kernel<bf16>, grid4, dim3(256), 0, s, proj, ld, g, bias, table, halves, keys_as_values, positions, slots, q_out, q_bf16,
+                           (bf16*)k_cache, (bf16*)v_cache));
+    return 0;
+  }
   const int units = g.heads + (keys_as_values ? 1 : 2) * g.kv_heads, upc = T >= 256 ? units : 8;   // few tokens: several CTAs each
   const dim3 grid(T, (units + upc - 1) / upc);
   if (cache_f32)

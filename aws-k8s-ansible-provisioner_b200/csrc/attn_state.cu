@@ -29,13 +29,14 @@
 // not depend on where the portion was cut, so prefill, chunked prefill and token-by-token decoding give the same bits.
 //
 // Kernels:
-//   lowrank_act        y = act(W2 . lr + bias) for the low-rank second stages (decays, output gates), fp32
+//   lowrank_act        y = act(W2 . lr + bias) for the low-rank second stages (decays, output gates), fp32; lowrank_act_tile: prompt-sized steps
 //   conv_unit_finish   delta rule: causal convolution + silu on q | k | v (a thread per channel), then unit vectors and the query scale
 //                      (a warp per head), beta
 //   conv_unit_rows     the same for prompt-sized steps (a CTA walks down sixteen rows of one head)
 //   conv_ring_store    the ring update, after every token of the step has read the ring (a decode step's tokens do it themselves)
 //   conv_act           state-space mixer: causal convolution with bias + silu on x | B | C, step sizes and decays
 //   state_scan         the recurrence; state_scan_head: the delta rule with one decay per head on packed fp32 pairs
+//   state_scan_sum     the state-space and time-mixing rules on packed fp32 pairs
 //   state_out_gate     per-head RMS norm of the read-out with a gain, times the gate (silu or given), operand type out
 //   gate_part_norm     the read-out times silu(gate), RMS-normed in equal parts, operand type out
 #include "kernels.h"
@@ -48,31 +49,66 @@ __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 
-// A CTA takes LR_TOKENS tokens and 256 output channels; a thread owns one channel, reads its row of w2 once (sixteen numbers at a
+typedef unsigned long long f32x2_t;
+__device__ __forceinline__ f32x2_t x2_pack(float a, float b) {
+  f32x2_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void x2_unpack(f32x2_t v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ f32x2_t x2_fma(f32x2_t a, f32x2_t b, f32x2_t c) {
+  f32x2_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2_t x2_mul(f32x2_t a, f32x2_t b) {
+  f32x2_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+__device__ __forceinline__ float lowrank_value(float z, int mode, float rate) {
+  if (mode == LOWRANK_SIGMOID) return sigmoid_f(z);
+  if (mode == LOWRANK_DECAY_SIGMOID_POW) return expf(-rate * softplus_f(-z));   // sigmoid(z)^rate
+  if (mode == LOWRANK_DECAY_EXP) return expf(-expf(z));
+  return expf(-rate * softplus_f(z));                                           // exp(-exp(A) softplus(z))
+}
+
+// A CTA takes LR_TOKENS tokens and NT output channels; a thread owns one channel, reads its row of w2 once (sixteen numbers at a
 // time) and applies it to every token of the tile.  lr [T][ld] fp32 (rank numbers per token at column lr_off), staged in shared memory.
 constexpr int LR_TOKENS = 8;
-__global__ void __launch_bounds__(256) lowrank_act_kernel(const float* __restrict__ lr, int ld, int lr_off, int rank, const float* __restrict__ w2,
+template <int NT>
+__global__ void __launch_bounds__(NT) lowrank_act_kernel(const float* __restrict__ lr, int ld, int lr_off, int rank, const float* __restrict__ w2,
                                                           const float* __restrict__ bias, const float* __restrict__ rate_log, float rate,
                                                           int per_head, int mode, float* __restrict__ out, int C, int T) {
   extern __shared__ __align__(16) float lrs[];   // [LR_TOKENS][rank]
   pdl_wait();
   pdl_launch_dependents();
   const int t0 = blockIdx.x * LR_TOKENS, tn = min(LR_TOKENS, T - t0);
-  for (int i = threadIdx.x; i < tn * rank; i += 256) {
+  for (int i = threadIdx.x; i < tn * rank; i += NT) {
     const float v = lr[(size_t)(t0 + i / rank) * ld + lr_off + i % rank];
     lrs[i] = mode == LOWRANK_DECAY_EXP ? tanhf(v) : v;
   }
   __syncthreads();
-  const int c = blockIdx.y * 256 + threadIdx.x;
+  const int c = blockIdx.y * NT + threadIdx.x;
   if (c >= C) return;
   const float* wr = w2 + (size_t)c * rank;
+  const bool row16 = (rank & 3) == 0 && (reinterpret_cast<uintptr_t>(w2) & 15) == 0;
   float z[LR_TOKENS];
 #pragma unroll
   for (int tt = 0; tt < LR_TOKENS; ++tt) z[tt] = 0.f;
   for (int r0 = 0; r0 < rank; r0 += 16) {
     float w[16];
 #pragma unroll
-    for (int x = 0; x < 16; ++x) w[x] = r0 + x < rank ? wr[r0 + x] : 0.f;
+    for (int x = 0; x < 16; x += 4) {
+      if (row16) {
+        const float4 v = r0 + x < rank ? *reinterpret_cast<const float4*>(wr + r0 + x) : make_float4(0.f, 0.f, 0.f, 0.f);
+        w[x] = v.x; w[x + 1] = v.y; w[x + 2] = v.z; w[x + 3] = v.w;
+      } else {
+#pragma unroll
+        for (int y = 0; y < 4; ++y) w[x + y] = r0 + x + y < rank ? wr[r0 + x + y] : 0.f;
+      }
+    }
 #pragma unroll
     for (int tt = 0; tt < LR_TOKENS; ++tt) {
       if (tt < tn) {
@@ -101,12 +137,99 @@ __global__ void __launch_bounds__(256) lowrank_act_kernel(const float* __restric
   for (int tt = 0; tt < LR_TOKENS; ++tt) {
     if (tt >= tn) break;
     const float zz = z[tt] + b;
-    float y;
-    if (mode == LOWRANK_SIGMOID) y = sigmoid_f(zz);
-    else if (mode == LOWRANK_DECAY_SIGMOID_POW) y = expf(-rt * softplus_f(-zz));               // sigmoid(z)^rate
-    else if (mode == LOWRANK_DECAY_EXP) y = expf(-expf(zz));
-    else y = expf(-rt * softplus_f(zz));                                                       // exp(-exp(A) softplus(z))
-    out[(size_t)(t0 + tt) * C + c] = y;
+    out[(size_t)(t0 + tt) * C + c] = lowrank_value(zz, mode, rt);
+  }
+}
+
+// Prompt-sized steps: a register-tiled product, 64 tokens x 128 channels at a time, a thread owns eight tokens (packed in pairs) of four channels.  The
+// tokens' values are staged once (tanh applied there), then the CTA walks over its share of the channel tiles.  A channel's sum runs over the rank in
+// order, as above.
+constexpr int LT_T = 64, LT_C = 128, LT_K = 32, LT_MAX_RANK = 128;
+__global__ void __launch_bounds__(256) lowrank_act_tile_kernel(const float* __restrict__ lr, int ld, int lr_off, int rank, const float* __restrict__ w2,
+                                                               const float* __restrict__ bias, const float* __restrict__ rate_log, float rate, int per_head,
+                                                               int mode, float* __restrict__ out, int C, int T, int tiles_per_cta) {
+  extern __shared__ __align__(16) float lt_smem[];
+  float(*As)[LT_T + 4] = reinterpret_cast<float(*)[LT_T + 4]>(lt_smem);                              // [rank][64 tokens]
+  float(*Ws)[LT_C + 4] = reinterpret_cast<float(*)[LT_C + 4]>(lt_smem + (size_t)rank * (LT_T + 4));   // [LT_K][128 channels]
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t0 = blockIdx.x * LT_T, tid = threadIdx.x, tx = tid & 31, ty = tid >> 5;
+  for (int i = tid; i < LT_T * rank; i += 256) {   // a warp takes 32 tokens of one column: the stores do not collide
+    const int t = i % LT_T, r = i / LT_T;
+    float v = t0 + t < T ? lr[(size_t)(t0 + t) * ld + lr_off + r] : 0.f;
+    if (mode == LOWRANK_DECAY_EXP) v = tanhf(v);
+    As[r][t] = v;
+  }
+  const bool row16 = (rank & 3) == 0 && (reinterpret_cast<uintptr_t>(w2) & 15) == 0;
+  for (int ct = 0; ct < tiles_per_cta; ++ct) {
+    const int c0 = (blockIdx.y * tiles_per_cta + ct) * LT_C;
+    if (c0 >= C) return;
+    f32x2_t acc[4][4];   // [token pair][channel]
+#pragma unroll
+    for (int a = 0; a < 4; ++a)
+#pragma unroll
+      for (int b = 0; b < 4; ++b) acc[a][b] = 0ull;
+    for (int k0 = 0; k0 < rank; k0 += LT_K) {
+      const int kn = min(LT_K, rank - k0);
+      __syncthreads();   // As is staged / the slab before this one is used up
+      if (row16) {
+        for (int i = tid; i < LT_C * (LT_K / 4); i += 256) {
+          const int c = i % LT_C, r = (i / LT_C) * 4;
+          const float4 v = r < kn && c0 + c < C ? *reinterpret_cast<const float4*>(w2 + (size_t)(c0 + c) * rank + k0 + r) : make_float4(0.f, 0.f, 0.f, 0.f);
+          Ws[r][c] = v.x; Ws[r + 1][c] = v.y; Ws[r + 2][c] = v.z; Ws[r + 3][c] = v.w;
+        }
+      } else {
+        for (int i = tid; i < LT_C * LT_K; i += 256) {
+          const int c = i % LT_C, r = i / LT_C;
+          Ws[r][c] = r < kn && c0 + c < C ? w2[(size_t)(c0 + c) * rank + k0 + r] : 0.f;
+        }
+      }
+      __syncthreads();
+#pragma unroll 4
+      for (int r = 0; r < kn; ++r) {
+        const ulonglong2 a0 = *reinterpret_cast<const ulonglong2*>(&As[k0 + r][ty * 8]), a1 = *reinterpret_cast<const ulonglong2*>(&As[k0 + r][ty * 8 + 4]);
+        const float4 w = *reinterpret_cast<const float4*>(&Ws[r][tx * 4]);
+        const f32x2_t av[4] = {a0.x, a0.y, a1.x, a1.y}, wv[4] = {x2_pack(w.x, w.x), x2_pack(w.y, w.y), x2_pack(w.z, w.z), x2_pack(w.w, w.w)};
+#pragma unroll
+        for (int a = 0; a < 4; ++a)
+#pragma unroll
+          for (int b = 0; b < 4; ++b) acc[a][b] = x2_fma(av[a], wv[b], acc[a][b]);
+      }
+    }
+    const int c = c0 + tx * 4;
+    if (c >= C) continue;
+    float bs[4], rt[4];
+#pragma unroll
+    for (int b = 0; b < 4; ++b) {
+      const int cc = min(c + b, C - 1);
+      bs[b] = bias ? bias[cc] : 0.f;
+      rt[b] = mode == LOWRANK_DECAY_SOFTPLUS ? expf(rate_log[cc / per_head]) : rate;
+    }
+    const bool vec = c + 3 < C && C % 4 == 0;
+#pragma unroll
+    for (int a = 0; a < 4; ++a) {
+      float lo[4], hi[4];
+#pragma unroll
+      for (int b = 0; b < 4; ++b) {
+        x2_unpack(acc[a][b], lo[b], hi[b]);
+        lo[b] = lowrank_value(lo[b] + bs[b], mode, rt[b]);
+        hi[b] = lowrank_value(hi[b] + bs[b], mode, rt[b]);
+      }
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int t = t0 + ty * 8 + 2 * a + h;
+        if (t >= T) continue;
+        const float* y = h ? hi : lo;
+        float* dst = out + (size_t)t * C + c;
+        if (vec) {
+          *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+        } else {
+#pragma unroll
+          for (int b = 0; b < 4; ++b)
+            if (c + b < C) dst[b] = y[b];
+        }
+      }
+    }
   }
 }
 
@@ -347,17 +470,90 @@ __global__ void __launch_bounds__(128) conv_act_kernel(const float* __restrict__
     }
 }
 
-__global__ void __launch_bounds__(128) conv_ring_store_kernel(const float* __restrict__ proj, int ld, int C, int taps, float* __restrict__ ring,
-                                                              const int32_t* __restrict__ row_seq, const int32_t* __restrict__ row_end,
-                                                              const int32_t* __restrict__ positions, const int32_t* __restrict__ slots) {
+// The same with four neighbouring channels per thread (prompt-sized steps; channels in multiples of four, rows on 16-byte boundaries).
+template <int TAPS>
+__global__ void __launch_bounds__(128) conv_act4_kernel(const float* __restrict__ proj, int ld, int C, int heads, const float* __restrict__ conv_w,
+                                                        const float* __restrict__ conv_b, const float* __restrict__ a_log, const float* __restrict__ dt_bias,
+                                                        const float* __restrict__ ring, const int32_t* __restrict__ row_seq, const int32_t* __restrict__ row_first,
+                                                        const int32_t* __restrict__ positions, const int32_t* __restrict__ slots, float* __restrict__ out,
+                                                        float* __restrict__ step, float* __restrict__ decay, int rows, int T) {
+  const int t0 = blockIdx.x * rows, tn = min(rows, T - t0), c = (blockIdx.y * 128 + threadIdx.x) * 4;
+  float4 w[TAPS], bias = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (c < C) {
+    bias = *reinterpret_cast<const float4*>(conv_b + c);
+#pragma unroll
+    for (int d = 0; d < TAPS; ++d) {
+      const int k = TAPS - 1 - d;
+      w[d] = make_float4(conv_w[(size_t)c * TAPS + k], conv_w[(size_t)(c + 1) * TAPS + k], conv_w[(size_t)(c + 2) * TAPS + k], conv_w[(size_t)(c + 3) * TAPS + k]);
+    }
+  }
   pdl_wait();
   pdl_launch_dependents();
-  const int t = blockIdx.x;
-  if (slots[t] < 0) return;
-  if (row_end[t] - 1 - t >= taps) return;  // a later token of the same portion owns this ring row
-  float* dst = ring + ((size_t)row_seq[t] * taps + positions[t] % taps) * C;
-  const float* row = proj + (size_t)t * ld;
-  for (int c = threadIdx.x; c < C; c += 128) dst[c] = row[c];
+  if (c < C) {
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < tn;) {   // runs of rows of one portion
+      const int t = t0 + i, first = row_first[t], pos = positions[t], back = t - first;
+      const bool live = slots[t] >= 0;
+      const float* rg = ring + (size_t)row_seq[t] * TAPS * C + c;
+      int e = i + 1;
+      while (e < tn && row_first[t0 + e] == first) ++e;
+      float4 hist[TAPS];   // hist[d]: the inputs d rows back
+#pragma unroll
+      for (int d = 1; d < TAPS; ++d)
+        hist[d] = !live       ? zero
+                  : d <= back ? *reinterpret_cast<const float4*>(proj + (size_t)(t - d) * ld + c)
+                  : pos >= d  ? *reinterpret_cast<const float4*>(rg + (size_t)((pos - d) % TAPS) * C)
+                              : zero;
+      while (i < e) {   // four rows' loads in flight at a time
+        const int m = min(4, e - i);
+        float4 x[4];
+#pragma unroll
+        for (int r = 0; r < 4; ++r) x[r] = r < m ? *reinterpret_cast<const float4*>(proj + (size_t)(t0 + i + r) * ld + c) : zero;
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+          if (r < m) {
+            float4 acc = bias;
+#pragma unroll
+            for (int d = TAPS - 1; d >= 1; --d) {
+              acc.x = fmaf(w[d].x, hist[d].x, acc.x); acc.y = fmaf(w[d].y, hist[d].y, acc.y);
+              acc.z = fmaf(w[d].z, hist[d].z, acc.z); acc.w = fmaf(w[d].w, hist[d].w, acc.w);
+            }
+            acc.x = fmaf(w[0].x, x[r].x, acc.x); acc.y = fmaf(w[0].y, x[r].y, acc.y);
+            acc.z = fmaf(w[0].z, x[r].z, acc.z); acc.w = fmaf(w[0].w, x[r].w, acc.w);
+#pragma unroll
+            for (int d = TAPS - 1; d >= 2; --d) hist[d] = hist[d - 1];
+            if (TAPS > 1) hist[TAPS > 1 ? 1 : 0] = x[r];
+            if (live) *reinterpret_cast<float4*>(out + (size_t)(t0 + i + r) * C + c) = make_float4(silu_f(acc.x), silu_f(acc.y), silu_f(acc.z), silu_f(acc.w));
+          }
+        }
+        i += m;
+      }
+    }
+  }
+  if (blockIdx.y == 0)
+    for (int i = threadIdx.x; i < tn * heads; i += 128) {
+      const int t = t0 + i / heads, a = i % heads;
+      const float d = softplus_f(proj[(size_t)t * ld + C + a] + dt_bias[a]);
+      step[(size_t)t * heads + a] = d;
+      decay[(size_t)t * heads + a] = expf(-expf(a_log[a]) * d);
+    }
+}
+
+__global__ void __launch_bounds__(128) conv_ring_store_kernel(const float* __restrict__ proj, int ld, int C, int taps, float* __restrict__ ring,
+                                                              const int32_t* __restrict__ row_seq, const int32_t* __restrict__ row_end,
+                                                              const int32_t* __restrict__ positions, const int32_t* __restrict__ slots, int T) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int mine = blockIdx.x * 32 + (threadIdx.x & 31), at = mine < T ? mine : 0;
+  // every warp finds the block's rows to store: the last `taps` of a portion (a later token of the portion owns the others' entries)
+  unsigned todo = __ballot_sync(0xffffffffu, mine < T && slots[at] >= 0 && row_end[at] - 1 - mine < taps);
+  while (todo) {
+    const int t = blockIdx.x * 32 + __ffs(todo) - 1;
+    todo &= todo - 1;
+    float* dst = ring + ((size_t)row_seq[t] * taps + positions[t] % taps) * C;
+    const float* row = proj + (size_t)t * ld;
+    for (int c = threadIdx.x; c < C; c += 128) dst[c] = row[c];
+  }
 }
 
 constexpr int SC_LANES = 8;     // lanes that share a group of state columns and split the key channels
@@ -658,24 +854,6 @@ __global__ void __launch_bounds__(256) state_scan_kernel(const float* __restrict
 // becomes one) before it could run out of range, so a decay of any size down to zero is exact to rounding.  The
 // keys of a token stay in registers between the two sums that read them; the read-out's sum over the eight lanes leaves each column with
 // one lane pair.
-typedef unsigned long long f32x2_t;
-__device__ __forceinline__ f32x2_t x2_pack(float a, float b) {
-  f32x2_t r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-  return r;
-}
-__device__ __forceinline__ void x2_unpack(f32x2_t v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
-__device__ __forceinline__ f32x2_t x2_fma(f32x2_t a, f32x2_t b, f32x2_t c) {
-  f32x2_t r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-  return r;
-}
-__device__ __forceinline__ f32x2_t x2_mul(f32x2_t a, f32x2_t b) {
-  f32x2_t r;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-  return r;
-}
-
 template <int DPT>   // channels per lane: 4, 8 or 16 (dim <= 8 DPT); lane j owns channels 32 m + 4 j + (0..3): rows are staged as they are, 16 bytes a copy
 __global__ void __launch_bounds__(256) state_scan_head_kernel(const float* __restrict__ q, int ldq, const float* __restrict__ k, int ldk,
                                                               const float* __restrict__ v, int ldv, const float* __restrict__ decay,
@@ -847,6 +1025,217 @@ __global__ void __launch_bounds__(256) state_scan_head_kernel(const float* __res
   }
 }
 
+// ---- the rules whose write does not read the state (DECAY_HEAD, BONUS), packed the same way.  DECAY_HEAD: the state is a factor times a matrix, as above.
+// BONUS: decays per channel are staged beside the keys; the read-out sees the state before the write, and the bonus of a token is the number
+// sum_d q_d u_d k_d times its value.
+template <int DPT, int RULE>
+__global__ void __launch_bounds__(256) state_scan_sum_kernel(const float* __restrict__ q, int ldq, const float* __restrict__ k, int ldk,
+                                                             const float* __restrict__ v, int ldv, const float* __restrict__ decay,
+                                                             const float* __restrict__ beta, StateGeom g, float qscale, float* __restrict__ state,
+                                                             const int32_t* __restrict__ last_rows, const int32_t* __restrict__ row_seq,
+                                                             const int32_t* __restrict__ row_first, const int32_t* __restrict__ row_end,
+                                                             const int32_t* __restrict__ positions, const int32_t* __restrict__ slots,
+                                                             float* __restrict__ out, int cols) {
+  constexpr int NC = 4, CH = SC_CHUNK, DP = DPT * SC_LANES, MAXC = 32 * NC, HP = DPT / 2;
+  constexpr bool HEAD = RULE == STATE_RULE_DECAY_HEAD;
+  __shared__ __align__(16) float qs[2][CH][DP], ks[2][CH][DP], as[HEAD ? 1 : 2][HEAD ? 1 : CH][HEAD ? 4 : DP];
+  __shared__ __align__(16) float vs[2][CH][MAXC];
+  __shared__ float bs[2][CH], ds[2][CH];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int r_last = last_rows ? last_rows[blockIdx.x] : (int)blockIdx.x;
+  const int first = row_first[r_last], end = row_end[r_last];
+  if (slots[first] < 0) return;   // padding row of a decode bucket
+  const int a = blockIdx.y, kh = a / (g.heads / g.kv_heads);
+  const int col0 = blockIdx.z * cols;
+  const int grp = threadIdx.x / SC_LANES, j = threadIdx.x % SC_LANES, cl = grp * NC;
+  const int pos0 = positions[first], n = end - first;
+  const int nthreads = blockDim.x;
+  const size_t head_floats = (size_t)g.dim * g.vdim;
+  float* sbase = state + ((size_t)row_seq[first] * 2 * g.heads) * head_floats;
+  const float* s_in = sbase + ((size_t)((pos0 + 1) & 1) * g.heads + a) * head_floats;
+  float* s_out = sbase + ((size_t)((pos0 + n - 1) & 1) * g.heads + a) * head_floats;
+  // channels past dim and columns past vdim never change: zero keys, queries, decays and values
+  for (int i = threadIdx.x; i < 2 * CH * (DP - g.dim); i += nthreads) {
+    const int st = i / (CH * (DP - g.dim)), rem = i % (CH * (DP - g.dim)), tt = rem / (DP - g.dim), d = g.dim + rem % (DP - g.dim);
+    qs[st][tt][d] = 0.f;
+    ks[st][tt][d] = 0.f;
+    if (!HEAD) {
+      as[HEAD ? 0 : st][HEAD ? 0 : tt][HEAD ? 0 : d] = 0.f;
+    }
+  }
+  const int vcols = min(cols, g.vdim - col0);
+  if (vcols < cols) {
+    for (int i = threadIdx.x; i < 2 * CH * (cols - vcols); i += nthreads) {
+      const int row = i / (cols - vcols), c = vcols + i % (cols - vcols);
+      vs[row / CH][row % CH][c] = 0.f;
+    }
+  }
+  __syncthreads();
+  const int dq = g.dim >> 2, vq4 = vcols >> 2;   // 16-byte pieces of a row
+  const int dsh = (dq & (dq - 1)) == 0 ? 31 - __clz(dq) : -1, vsh = (vq4 & (vq4 - 1)) == 0 ? 31 - __clz(vq4) : -1;
+  const int lda = g.heads * g.dim;
+  const float* qb = q + (size_t)first * ldq + kh * g.dim;
+  const float* kb = k + (size_t)first * ldk + kh * g.dim;
+  const float* ab = HEAD ? decay : decay + (size_t)first * lda + a * g.dim;
+  const float* vb = v + (size_t)first * ldv + a * g.vdim + col0;
+  auto issue = [&](int c0, int st) {
+    const int cn = min(CH, n - c0);
+    for (int i = threadIdx.x; i < cn * dq; i += nthreads) {
+      const int tt = dsh >= 0 ? i >> dsh : i / dq, d = (i - tt * dq) * 4;
+      cp_async_16(&qs[st][tt][d], qb + (size_t)(c0 + tt) * ldq + d);
+      cp_async_16(&ks[st][tt][d], kb + (size_t)(c0 + tt) * ldk + d);
+      if (!HEAD) {
+        cp_async_16(&as[HEAD ? 0 : st][HEAD ? 0 : tt][HEAD ? 0 : d], ab + (size_t)(c0 + tt) * lda + d);
+      }
+    }
+    for (int i = threadIdx.x; i < cn * vq4; i += nthreads) {
+      const int tt = vsh >= 0 ? i >> vsh : i / vq4, c = (i - tt * vq4) * 4;
+      cp_async_16(&vs[st][tt][c], vb + (size_t)(c0 + tt) * ldv + c);
+    }
+    if (HEAD) {
+      for (int i = threadIdx.x; i < cn; i += nthreads) {
+        cp_async_f32(&bs[st][i], beta + (size_t)(first + c0 + i) * g.heads + a);
+        cp_async_f32(&ds[st][i], decay + (size_t)(first + c0 + i) * g.heads + a);
+      }
+    }
+  };
+  issue(0, 0);
+  const bool live = col0 + cl + NC <= g.vdim;   // this group's four columns (vdim is a multiple of four)
+  auto channel = [&](int i) { return (i >> 2) * 32 + 4 * j + (i & 3); };
+  f32x2_t s[HP][NC], bonus[HEAD ? 1 : HP];
+#pragma unroll
+  for (int i = 0; i < HP; ++i) {
+    float lo[NC], hi[NC];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int d = channel(2 * i + x);
+      float* dst = x ? hi : lo;
+      float4 w = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (live && pos0 > 0 && d < g.dim) w = *reinterpret_cast<const float4*>(s_in + (size_t)d * g.vdim + col0 + cl);
+      dst[0] = w.x; dst[1] = w.y; dst[2] = w.z; dst[3] = w.w;
+    }
+#pragma unroll
+    for (int c = 0; c < NC; ++c) s[i][c] = x2_pack(lo[c], hi[c]);
+    if (!HEAD) {
+      const int d0 = channel(2 * i), d1 = channel(2 * i + 1);
+      bonus[HEAD ? 0 : i] = x2_pack(d0 < g.dim ? g.bonus[a * g.dim + d0] : 0.f, d1 < g.dim ? g.bonus[a * g.dim + d1] : 0.f);
+    }
+  }
+  const float skip = HEAD ? g.skip[a] : 0.f;
+  const bool up1 = (j & 1) != 0, up2 = (j & 2) != 0;
+  const int ccol = (up1 ? 2 : 0) + (up2 ? 1 : 0);   // the column this lane ends a token with
+  const size_t ostep = (size_t)g.heads * g.vdim;
+  float* optr = out + (size_t)first * ostep + a * g.vdim + col0 + cl + ccol;
+  float fac = 1.0f;
+  int st = 0;
+  for (int c0 = 0; c0 < n; c0 += CH, st ^= 1) {
+    const int cn = min(CH, n - c0);
+    cp_async_wait_all();                         // this chunk's copies (the only ones in flight)
+    __syncthreads();                             // ... of every thread; and every thread has left the other stage
+    if (c0 + CH < n) issue(c0 + CH, st ^ 1);     // the next chunk's copies run beside this chunk's arithmetic
+    // one token: wr is the write's factor (DECAY_HEAD), ofac the read-out's
+    auto token = [&](int tt, float wr, float ofac) {
+      const float4 vq = *reinterpret_cast<const float4*>(&vs[st][tt][cl]);
+      const float vc[NC] = {vq.x, vq.y, vq.z, vq.w};
+      const ulonglong2* kp = reinterpret_cast<const ulonglong2*>(&ks[st][tt][4 * j]);   // (32 channels on: eight pieces of 16 bytes)
+      const ulonglong2* qp = reinterpret_cast<const ulonglong2*>(&qs[st][tt][4 * j]);
+      f32x2_t sum[NC], w2[NC];
+      float o[NC];
+      if constexpr (HEAD) {
+#pragma unroll
+        for (int c = 0; c < NC; ++c) w2[c] = x2_pack(vc[c] * wr, vc[c] * wr);
+#pragma unroll
+        for (int i = 0; i < HP; i += 2) {
+          const ulonglong2 kw = kp[(i >> 1) * 8], qw = qp[(i >> 1) * 8];
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            s[i][c] = x2_fma(kw.x, w2[c], s[i][c]);
+            s[i + 1][c] = x2_fma(kw.y, w2[c], s[i + 1][c]);
+            sum[c] = i == 0 ? x2_mul(s[0][c], qw.x) : x2_fma(s[i][c], qw.x, sum[c]);
+            sum[c] = x2_fma(s[i + 1][c], qw.y, sum[c]);
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          float lo, hi;
+          x2_unpack(sum[c], lo, hi);
+          o[c] = lo + hi;
+        }
+      } else {
+        const ulonglong2* ap = reinterpret_cast<const ulonglong2*>(&as[HEAD ? 0 : st][HEAD ? 0 : tt][HEAD ? 0 : 4 * j]);
+        f32x2_t ruk = 0ull;
+#pragma unroll
+        for (int c = 0; c < NC; ++c) w2[c] = x2_pack(vc[c], vc[c]);
+#pragma unroll
+        for (int i = 0; i < HP; i += 2) {
+          const ulonglong2 kw = kp[(i >> 1) * 8], qw = qp[(i >> 1) * 8], aw = ap[(i >> 1) * 8];
+          ruk = x2_fma(x2_mul(qw.x, bonus[HEAD ? 0 : i]), kw.x, ruk);
+          ruk = x2_fma(x2_mul(qw.y, bonus[HEAD ? 0 : i + 1]), kw.y, ruk);
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            sum[c] = i == 0 ? x2_mul(s[0][c], qw.x) : x2_fma(s[i][c], qw.x, sum[c]);
+            sum[c] = x2_fma(s[i + 1][c], qw.y, sum[c]);
+            s[i][c] = x2_fma(aw.x, s[i][c], x2_mul(kw.x, w2[c]));
+            s[i + 1][c] = x2_fma(aw.y, s[i + 1][c], x2_mul(kw.y, w2[c]));
+          }
+        }
+        float rl, rh;
+        x2_unpack(ruk, rl, rh);
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          float lo, hi;
+          x2_unpack(sum[c], lo, hi);
+          o[c] = fmaf(rl + rh, vc[c], lo + hi);
+        }
+      }
+      // sum over the eight lanes: each exchange halves the columns a lane still holds, then the last two lanes of a column add
+      const float a0 = (up1 ? o[2] : o[0]) + __shfl_xor_sync(0xffffffffu, up1 ? o[0] : o[2], 1);
+      const float a1 = (up1 ? o[3] : o[1]) + __shfl_xor_sync(0xffffffffu, up1 ? o[1] : o[3], 1);
+      float r = (up2 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, up2 ? a0 : a1, 2);
+      r += __shfl_xor_sync(0xffffffffu, r, 4);
+      r *= ofac;
+      if (HEAD) r = fmaf(skip, up1 ? (up2 ? vc[3] : vc[2]) : (up2 ? vc[1] : vc[0]), r);
+      if (j < 4 && live) *optr = r;
+      optr += ostep;
+    };
+    if constexpr (HEAD) {
+#pragma unroll 1
+      for (int tt = 0; tt < cn; ++tt) {
+        fac *= ds[st][tt];
+        if (fac < 1e-12f) {   // (the same in every thread of the CTA)
+          const f32x2_t f2 = x2_pack(fac, fac);
+#pragma unroll
+          for (int i = 0; i < HP; ++i)
+#pragma unroll
+            for (int c = 0; c < NC; ++c) s[i][c] = x2_mul(f2, s[i][c]);
+          fac = 1.0f;
+        }
+        token(tt, bs[st][tt] * __fdividef(1.0f, fac), qscale * fac);   // (1e-12 <= fac <= 1)
+      }
+    } else if (cn == CH) {
+#pragma unroll 2
+      for (int tt = 0; tt < CH; ++tt) token(tt, 0.f, qscale);
+    } else {
+#pragma unroll 1
+      for (int tt = 0; tt < cn; ++tt) token(tt, 0.f, qscale);
+    }
+  }
+  const f32x2_t f2 = x2_pack(fac, fac);
+#pragma unroll
+  for (int i = 0; i < HP; ++i) {
+    float lo[NC], hi[NC];
+#pragma unroll
+    for (int c = 0; c < NC; ++c) x2_unpack(x2_mul(f2, s[i][c]), lo[c], hi[c]);
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int d = channel(2 * i + x);
+      const float* src = x ? hi : lo;
+      if (live && d < g.dim) *reinterpret_cast<float4*>(s_out + (size_t)d * g.vdim + col0 + cl) = make_float4(src[0], src[1], src[2], src[3]);
+    }
+  }
+}
+
 // One warp per (token, head): y = o / sqrt(mean(o^2) + eps) * gain * gate, gate = silu(gate_in) or gate_in as it is.
 template <typename TX>
 __global__ void __launch_bounds__(128) state_out_gate_kernel(const float* __restrict__ o, const float* __restrict__ gain,
@@ -969,6 +1358,7 @@ int gate_part_norm_typed(const float* o, const float* gate, int gate_ld, const f
   const bool vec = part % 4 == 0 && gate_ld % 4 == 0 && out_ld % 4 == 0 &&
                    ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
   if (vec && part <= 512) B2_GPN(128, 1);
+  if (vec && part <= 1024) B2_GPN(128, 2);
   if (vec && part <= 2048) B2_GPN(256, 2);
   if (vec && part <= 4096) B2_GPN(512, 2);
   if (vec && part <= 8192) B2_GPN(512, 4);
@@ -977,6 +1367,59 @@ int gate_part_norm_typed(const float* o, const float* gate, int gate_ld, const f
   static B2PerDeviceOnce once;
   if ((size_t)part * 4 > 48 * 1024) b2_prefer_max_smem(gate_part_norm_kernel<TX, 256, 0>, once);
   B2_CUDA_OK(b2_launch(gate_part_norm_kernel<TX, 256, 0>, grid, dim3(256), (size_t)part * 4, s, o, gate, gate_ld, gain, scale, out, out_ld, N, part, eps));
+  return 0;
+}
+
+// The same for heads of 4 L numbers (L = 4 .. 32 lanes per head): a lane keeps its four numbers in registers.
+template <typename TX, int L>
+__global__ void __launch_bounds__(256) state_out_gate_lanes_kernel(const float* __restrict__ o, const float* __restrict__ gain,
+                                                                   const float* __restrict__ gate, int gate_ld, int gate_silu, TX* __restrict__ out,
+                                                                   int heads, float eps, int T, int gain_per_head, float scale, int out_ld) {
+  constexpr int V = 4 * L;
+  pdl_wait();
+  pdl_launch_dependents();
+  const long unit = ((long)blockIdx.x * 256 + threadIdx.x) / L;
+  const bool in = unit < (long)T * heads;
+  const int t = in ? (int)(unit / heads) : 0, a = in ? (int)(unit - (long)t * heads) : 0, i = (threadIdx.x % L) * 4;
+  const float4 ov = *reinterpret_cast<const float4*>(o + ((size_t)t * heads + a) * V + i);
+  const float4 gv = *reinterpret_cast<const float4*>(gate + (size_t)t * gate_ld + (size_t)a * V + i);
+  const float4 nv = *reinterpret_cast<const float4*>(gain + (gain_per_head ? (size_t)a * V : 0) + i);
+  float ss = (ov.x * ov.x + ov.y * ov.y) + (ov.z * ov.z + ov.w * ov.w);
+#pragma unroll
+  for (int m = L / 2; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+  if (!in) return;
+  const float r = scale / sqrtf(ss / (float)V + eps);
+  const float oo[4] = {ov.x, ov.y, ov.z, ov.w}, gg[4] = {gv.x, gv.y, gv.z, gv.w}, nn[4] = {nv.x, nv.y, nv.z, nv.w};
+  float y[4];
+#pragma unroll
+  for (int k = 0; k < 4; ++k) y[k] = oo[k] * r * nn[k] * (gate_silu ? silu_f(gg[k]) : gg[k]);
+  TX* dst = out + (size_t)t * out_ld + (size_t)a * V + i;
+  if constexpr (sizeof(TX) == 4) {
+    *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+  } else {
+    uint2 pk;
+    pk.x = pack_bf16x2(y[0], y[1]);
+    pk.y = pack_bf16x2(y[2], y[3]);
+    *reinterpret_cast<uint2*>(dst) = pk;
+  }
+}
+
+template <typename TX>
+int state_out_gate_typed(const float* o, const float* gain, const float* gate, int gate_ld, int gate_silu, TX* out, int heads, int vdim, float eps, int T,
+                         int gain_per_head, float scale, int out_ld, cudaStream_t s) {
+  const long units = (long)T * heads;
+  const bool vec = gate_ld % 4 == 0 && out_ld % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(gain) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+#define B2_OUT_GATE(L)                                                                                                                                     \
+  if (vec && vdim == 4 * (L)) {                                                                                                                            \
+    B2_CUDA_OK(b2_launch(state_out_gate_lanes_kernel<TX, L>, dim3((unsigned)((units * (L) + 255) / 256)), dim3(256), 0, s, o, gain, gate, gate_ld, gate_silu, out, \
+                         heads, eps, T, gain_per_head, scale, out_ld));                                                                                    \
+    return 0;                                                                                                                                              \
+  }
+  B2_OUT_GATE(4) B2_OUT_GATE(8) B2_OUT_GATE(16) B2_OUT_GATE(32)
+#undef B2_OUT_GATE
+  B2_CUDA_OK(b2_launch(state_out_gate_kernel<TX>, dim3((unsigned)((units + 3) / 4)), dim3(128), 0, s, o, gain, gate, gate_ld, gate_silu, out, heads, vdim, eps, T,
+                       gain_per_head, scale, out_ld));
   return 0;
 }
 
@@ -1010,8 +1453,22 @@ int launch_lowrank_act(const float* lr, int ld, int lr_off, int rank, const floa
   if (T <= 0 || C <= 0) return 0;
   B2_REQUIRE(rank >= 1 && rank <= 1024, "lowrank_act: rank %d (at most 1024)", rank);
   B2_REQUIRE(mode != LOWRANK_DECAY_SOFTPLUS || (rate_log != nullptr && per_head >= 1), "lowrank_act: the softplus decay needs a rate per head");
-  const dim3 grid((T + LR_TOKENS - 1) / LR_TOKENS, (C + 255) / 256);
-  B2_CUDA_OK(b2_launch(lowrank_act_kernel, grid, dim3(256), (size_t)LR_TOKENS * rank * 4, s, lr, ld, lr_off, rank, w2, bias, rate_log, rate,
+  if (T >= 256 && rank <= LT_MAX_RANK) {
+    const int tb = (T + LT_T - 1) / LT_T, tiles = (C + LT_C - 1) / LT_C;
+    int ys = 1;   // as few shares of the channel tiles as still give every SM several CTAs
+    while (ys < tiles && tb * ys < 4 * device_num_sms()) ys *= 2;
+    const int per = (tiles + ys - 1) / ys;
+    const size_t smem = ((size_t)rank * (LT_T + 4) + (size_t)LT_K * (LT_C + 4)) * 4;
+    static B2PerDeviceOnce attr_once;
+    if (attr_once.need())
+      B2_CUDA_OK(cudaFuncSetAttribute(lowrank_act_tile_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                      (int)(((size_t)LT_MAX_RANK * (LT_T + 4) + (size_t)LT_K * (LT_C + 4)) * 4)));
+    B2_CUDA_OK(b2_launch(lowrank_act_tile_kernel, dim3(tb, (tiles + per - 1) / per), dim3(256), smem, s, lr, ld, lr_off, rank, w2, bias, rate_log, rate,
+                         per_head > 0 ? per_head : 1, mode, out, C, T, per));
+    return 0;
+  }
+  const dim3 grid((T + LR_TOKENS - 1) / LR_TOKENS, (C + 63) / 64);
+  B2_CUDA_OK(b2_launch(lowrank_act_kernel<64>, grid, dim3(64), (size_t)LR_TOKENS * rank * 4, s, lr, ld, lr_off, rank, w2, bias, rate_log, rate,
                        per_head > 0 ? per_head : 1, mode, out, C, T));
   return 0;
 }
@@ -1042,7 +1499,7 @@ int launch_conv_unit_finish(const float* proj, int ld, const StateGeom& g, int t
 #undef B2_CONV_FINISH
 #undef B2_CONV_ROWS
   if (taps > 1 && !single_rows)
-    B2_CUDA_OK(b2_launch(conv_ring_store_kernel, dim3(T), dim3(128), 0, s, proj, ld, C, taps, ring, row_seq, row_end, positions, slots));
+    B2_CUDA_OK(b2_launch(conv_ring_store_kernel, dim3((T + 31) / 32), dim3(128), 0, s, proj, ld, C, taps, ring, row_seq, row_end, positions, slots, T));
   return 0;
 }
 
@@ -1066,15 +1523,31 @@ int launch_state_scan(const float* q, int ldq, const float* k, int ldk, const fl
   if (g.rule == STATE_RULE_DECAY)
     return launch_scan_rule<STATE_RULE_DECAY>(dpt, grid, block, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,
                                               row_first, row_end, positions, slots, out, cols);
+  static const bool packed = [] { const char* e = getenv("B2_SCAN_PACKED"); return !(e && *e == '0'); }();   // 0: the generic form (cross-check)
+  const bool rows16 = g.dim % 4 == 0 && g.vdim % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ldv % 4 == 0 &&
+                      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15) == 0;
+  if ((g.rule == STATE_RULE_DECAY_HEAD || g.rule == STATE_RULE_BONUS) && packed && rows16 && dpt <= 16 && (reinterpret_cast<uintptr_t>(decay) & 15) == 0) {
+#define B2_SCAN_SUM(D, R)                                                                                                                          \
+  B2_CUDA_OK(b2_launch(state_scan_sum_kernel<D, R>, grid, block, 0, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,   \
+                       row_first, row_end, positions, slots, out, cols))
+    if (g.rule == STATE_RULE_DECAY_HEAD) {
+      if (dpt <= 4) B2_SCAN_SUM(4, STATE_RULE_DECAY_HEAD);
+      else if (dpt == 8) B2_SCAN_SUM(8, STATE_RULE_DECAY_HEAD);
+      else B2_SCAN_SUM(16, STATE_RULE_DECAY_HEAD);
+    } else {
+      if (dpt <= 4) B2_SCAN_SUM(4, STATE_RULE_BONUS);
+      else if (dpt == 8) B2_SCAN_SUM(8, STATE_RULE_BONUS);
+      else B2_SCAN_SUM(16, STATE_RULE_BONUS);
+    }
+#undef B2_SCAN_SUM
+    return 0;
+  }
   if (g.rule == STATE_RULE_DECAY_HEAD)
     return launch_scan_rule<STATE_RULE_DECAY_HEAD>(dpt, grid, block, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,
                                                    row_first, row_end, positions, slots, out, cols);
   if (g.rule == STATE_RULE_BONUS)
     return launch_scan_rule<STATE_RULE_BONUS>(dpt, grid, block, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,
                                               row_first, row_end, positions, slots, out, cols);
-  static const bool packed = [] { const char* e = getenv("B2_SCAN_PACKED"); return !(e && *e == '0'); }();   // 0: the generic form (cross-check)
-  const bool rows16 = g.dim % 4 == 0 && g.vdim % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ldv % 4 == 0 &&
-                      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15) == 0;
   if (g.rule == STATE_RULE_DELTA_HEAD && packed && rows16 && dpt <= 16) {
 #define B2_SCAN_HEAD(D)                                                                                                                          \
   B2_CUDA_OK(b2_launch(state_scan_head_kernel<D>, grid, block, 0, s, q, ldq, k, ldk, v, ldv, decay, beta, g, qscale, state, last_rows, row_seq,   \
@@ -1098,15 +1571,8 @@ int launch_state_out_gate(const float* o, const float* gain, const float* gate, 
                           int heads, int vdim, float eps, int T, cudaStream_t s, int gain_per_head, float scale, int out_ld) {
   if (T <= 0) return 0;
   if (out_ld <= 0) out_ld = heads * vdim;
-  const long units = (long)T * heads;
-  const dim3 grid((unsigned)((units + 3) / 4));
-  if (out_f32)
-    B2_CUDA_OK(b2_launch(state_out_gate_kernel<float>, grid, dim3(128), 0, s, o, gain, gate, gate_ld, gate_silu, (float*)out, heads, vdim, eps, T, gain_per_head,
-                         scale, out_ld));
-  else
-    B2_CUDA_OK(b2_launch(state_out_gate_kernel<bf16>, grid, dim3(128), 0, s, o, gain, gate, gate_ld, gate_silu, (bf16*)out, heads, vdim, eps, T, gain_per_head,
-                         scale, out_ld));
-  return 0;
+  return out_f32 ? state_out_gate_typed<float>(o, gain, gate, gate_ld, gate_silu, (float*)out, heads, vdim, eps, T, gain_per_head, scale, out_ld, s)
+                 : state_out_gate_typed<bf16>(o, gain, gate, gate_ld, gate_silu, (bf16*)out, heads, vdim, eps, T, gain_per_head, scale, out_ld, s);
 }
 
 int launch_conv_act_finish(const float* proj, int ld, int channels, int heads, int taps, const float* conv_w, const float* conv_b, const float* a_log,
@@ -1120,13 +1586,21 @@ int launch_conv_act_finish(const float* proj, int ld, int channels, int heads, i
 #define B2_CONV_ACT(TAPS)                                                                                                                        \
   B2_CUDA_OK(b2_launch(conv_act_kernel<TAPS>, grid, dim3(128), 0, s, proj, ld, channels, heads, taps, conv_w, conv_b, a_log, dt_bias, (const float*)ring, store, \
                        row_seq, row_first, positions, slots, out, step, decay, rows, T))
-  if (taps == 4) B2_CONV_ACT(4);
+#define B2_CONV_ACT4(TAPS)                                                                                                                       \
+  B2_CUDA_OK(b2_launch(conv_act4_kernel<TAPS>, dim3((T + rows - 1) / rows, (channels / 4 + 127) / 128), dim3(128), 0, s, proj, ld, channels, heads, conv_w, conv_b, \
+                       a_log, dt_bias, (const float*)ring, row_seq, row_first, positions, slots, out, step, decay, rows, T))
+  const bool four = rows > 1 && taps >= 2 && taps <= 4 && channels % 4 == 0 && ld % 4 == 0 && ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(conv_b)) & 15) == 0;
+  if (four && taps == 4) B2_CONV_ACT4(4);
+  else if (four && taps == 3) B2_CONV_ACT4(3);
+  else if (four) B2_CONV_ACT4(2);
+  else if (taps == 4) B2_CONV_ACT(4);
   else if (taps == 3) B2_CONV_ACT(3);
   else if (taps == 2) B2_CONV_ACT(2);
   else B2_CONV_ACT(0);
 #undef B2_CONV_ACT
+#undef B2_CONV_ACT4
   if (taps > 1 && !single_rows)
-    B2_CUDA_OK(b2_launch(conv_ring_store_kernel, dim3(T), dim3(128), 0, s, proj, ld, channels, taps, ring, row_seq, row_end, positions, slots));
+    B2_CUDA_OK(b2_launch(conv_ring_store_kernel, dim3((T + 31) / 32), dim3(128), 0, s, proj, ld, channels, taps, ring, row_seq, row_end, positions, slots, T));
   return 0;
 }
 

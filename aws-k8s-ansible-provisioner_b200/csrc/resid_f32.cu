@@ -541,6 +541,17 @@ __global__ void __launch_bounds__(256) embed_streams_kernel(const int32_t* __res
   }
   const float r = 1.0f / sqrtf(block_sum_n<256>(ss, red) / (float)W + eps);
   float* hr = h + (size_t)t * n * W;
+  if (W % 4 == 0) {
+    for (int i = 4 * threadIdx.x; i < W; i += 1024) {
+      float v[4], gn[4];
+      load4(row + i, v);
+      load4(gain + i, gn);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v[k] = v[k] * r * gn[k];
+      for (int s = 0; s < n; ++s) store4(hr + (size_t)s * W + i, v);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < W; i += 256) {
     const float v = (float)row[i] * r * gain[i];
     for (int s = 0; s < n; ++s) hr[(size_t)s * W + i] = v;
