@@ -2,7 +2,7 @@
 
     python -m importlib ...  (see __graft_entry__.build) or:  python aws-k8s-ansible-provisioner_b200/build.py
 
-Outputs (git-ignored, shipped to the GPU box by gpurun):
+Outputs (git-ignored):
     aws-k8s-ansible-provisioner_b200/libb2engine.so     C ABI of include/b2_engine.h
     aws-k8s-ansible-provisioner_b200/b2serve            HTTP model server (when csrc/server/ exists)
 Objects are cached under build/ and rebuilt when a source or header is newer.

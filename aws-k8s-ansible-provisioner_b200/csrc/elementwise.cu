@@ -359,7 +359,7 @@ __global__ void qknorm_rope_kv_prefill_kernel(const bf16* __restrict__ qkv, cons
   }
 }
 
-// Same contract, 16 lanes per head (16 bytes each), the bf16 x bf16 products as packed HMUL2 (one rounding, identical to
+// Same contract, 16 lanes per head (16 bytes each), the bf16 x bf16 products as packed two-element multiplies (one rounding, identical to
 // rounding the exact fp32 product).  The four-byte-lane kernel above issued ~120 instructions per head per lane and ran
 // at a third of the HBM rate (61 us for 8192 tokens x 32 heads); this one is bound by the 134 MB it moves.
 // A half-warp walks four heads of one token; rot16 = rotary_dim / 16 lanes hold each half of the rotated span.
